@@ -26,6 +26,7 @@ enum StatusSite : uint32_t {
   kSiteCluster = 0x600,      // cluster partner did not arrive
   kSiteRendezvous = 0x700,   // small-message rendezvous
   kSiteGrid = 0x800,         // grid barrier
+  kSiteState = 0x900,        // no recurrent state for the position a step starts at
 };
 
 __device__ __forceinline__ void report(uint32_t* status, uint32_t site) {

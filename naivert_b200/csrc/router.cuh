@@ -70,6 +70,10 @@ __device__ __forceinline__ uint32_t router_order_key(float f) {
   return (u & 0x80000000u) ? ~u : (u | 0x80000000u);
 }
 
+__device__ __forceinline__ float router_key_value(uint32_t k) {
+  return __uint_as_float((k & 0x80000000u) ? (k ^ 0x80000000u) : ~k);
+}
+
 // 256 threads.  Waits for the upstream grid itself (after the loads that do not depend on it).
 __device__ __forceinline__ void router_scores(const RouterArgs& a, int cta, int n_ctas, RouterSmem& sm, unsigned long long* stamp = nullptr) {
   constexpr int kMaxRows = kRouterRows;
@@ -246,11 +250,51 @@ __device__ __forceinline__ void router_packet(const RouterArgs& a, int cta, int 
   }
 }
 
+// Group-limited choice: the experts form `groups` equal runs of neighbours; a run's score is the sum of its two largest
+// choice scores, and only experts of the `keep` best runs (lowest run on ties) stay eligible.  One warp per row, `ch` holds
+// the choice scores of experts lane, lane + 32, ...; groups <= 32.
+__device__ __forceinline__ void router_limit_groups(float (&ch)[8], int experts, int groups, int keep) {
+  const int lane = threadIdx.x & 31, per = experts / groups;
+  uint32_t mine = 0u;                               // lane g: ordered score of group g
+#pragma unroll 1
+  for (int g = 0; g < groups; ++g) {
+    uint32_t k1 = 0u, k2 = 0u;                      // this lane's two largest keys of the group
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int e = lane + 32 * j;
+      if (e < experts && e / per == g) {
+        const uint32_t k = router_order_key(ch[j]);
+        if (k > k1) { k2 = k1; k1 = k; } else if (k > k2) k2 = k;
+      }
+    }
+    const uint32_t b1 = __reduce_max_sync(0xffffffffu, k1);
+    const int owner = __ffs(__ballot_sync(0xffffffffu, k1 == b1)) - 1;
+    const uint32_t b2 = __reduce_max_sync(0xffffffffu, lane == owner ? k2 : k1);
+    const float f1 = router_key_value(b1), f2 = b2 ? router_key_value(b2) : 0.f;
+    if (lane == g) mine = router_order_key(f1 + f2);
+  }
+  uint32_t kept = 0u;
+#pragma unroll 1
+  for (int t = 0; t < keep; ++t) {
+    const uint32_t best = __reduce_max_sync(0xffffffffu, mine);
+    const int g = __ffs(__ballot_sync(0xffffffffu, mine == best)) - 1;
+    kept |= 1u << g;
+    if (lane == g) mine = 0u;
+  }
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int e = lane + 32 * j;
+    if (e < experts && !((kept >> (e / per)) & 1u)) ch[j] = -FLT_MAX;
+  }
+}
+
 // 256 threads; every score must be visible (the caller has synchronised the CTAs).  Results: sm.used / sm.slot_of /
 // sm.n_active, and - when `publish` - the global outputs of RouterArgs.  `probs_s` / `active_s` (shared memory,
 // may be null) receive the slot table for a consumer in the same CTA.
+// GROUPED: the choice is limited to the best `keep` of `groups` expert groups.
+template <bool GROUPED = false>
 __device__ __forceinline__ void router_select(const RouterArgs& a, RouterSmem& sm, bool publish, float* probs_s, int* active_s,
-                                              unsigned long long* stamp = nullptr) {
+                                              unsigned long long* stamp = nullptr, int groups = 1, int keep = 1) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   unsigned int* used = sm.used;
   int* slot_of = sm.slot_of;
@@ -295,6 +339,7 @@ __device__ __forceinline__ void router_select(const RouterArgs& a, RouterSmem& s
 #pragma unroll
       for (int j = 0; j < 8; ++j) { sc[j] /= sum; ch[j] = (lane + 32 * j) < a.experts ? sc[j] : -FLT_MAX; }
     }
+    if (GROUPED && keep < groups) router_limit_groups(ch, a.experts, groups, keep);
     // Every lane sorts its eight candidates once (descending key, lower expert first among equals - the experts of
     // a lane ascend with j, and the network below never swaps equal keys out of order); a selection step is then
     // two warp reductions over the lanes' heads and a pop on the winning lane.

@@ -1,0 +1,283 @@
+// Argument structs and small device helpers of the layer-stack kernels: the mechanisms from which models of
+// freely ordered layers (latent attention, gated linear recurrence, dense and expert feed-forwards, sandwich norms,
+// looped layers) are put together.  Every size and constant is a field; nothing here belongs to one model.
+//
+// Activation buffers come in two forms: bf16 (`f32` = 0: tensor-core products) and float (`f32` = 1: everything in
+// true 32-bit on the CUDA cores).  Weights are bf16 in both.  The residual stream, norms, routers, attention scores,
+// recurrent state and recurrence gates are float in both.
+#pragma once
+#include "ptx.cuh"
+
+#include <float.h>
+
+namespace nrt {
+
+// ------------------------------------------------------------------------------------ chunk (prefill) products
+enum StackEpi : int {
+  kSEpiStore = 0,      // acc * scale
+  kSEpiBias = 1,       // acc + bias; features below `act_cols` go through the tanh form of GELU
+  kSEpiTranspose = 2,  // acc stored feature-major: out[feature][token] (bf16)
+  kSEpiClampedGlu = 3, // two products g, u: g = min(g, limit), u = clamp(u), g * sigmoid(alpha g) * (u + 1)
+  kSEpiSiluGlu = 4,    // two products g, u: silu(g) * u
+};
+
+struct StackGemmArgs {
+  const void* act;              // float form: activations, element (row, z, k) at row * act_ld + z * act_zstride + k
+  const __nv_bfloat16* w;       // float form: weights, element (z, n, k) at z * w_zstride + n * w_ld + k
+  const __nv_bfloat16* w2;      // second matrix of the two-product epilogues
+  long long act_ld, act_zstride, w_ld, w_zstride;
+  int n, k, rows;               // features per group, inner size, token rows
+  int zcount;                   // independent groups (plain form): heads or blocks with their own weights and columns
+  const int* n_items;           // item form (routed experts): number of row segments, else null
+  const int* item_z;            // weight group of a segment
+  const int* item_row;          // its first row
+  int max_items;
+  int item_rows;                // rows of a segment
+  void* out;
+  int out_f32;                  // element type of `out`
+  long long out_ld, out_zstride;
+  const __nv_bfloat16* bias;    // [zcount][n]
+  int act_cols;
+  float scale, limit, alpha;
+  uint32_t* status;
+};
+
+// ------------------------------------------------------------------------------------ rows
+struct StackRowArgs {
+  // where the stream comes from: an embedding gather (tokens != null), else x as it stands
+  const int* tokens;
+  const __nv_bfloat16* table;
+  int vocab;
+  float embed_scale;
+  // sublayer output added through its own norm (null: none); with `slot_of` the row is the weighted sum of top_k rows
+  const float* y;
+  long long y_ld;
+  const int* slot_of;           // [rows][top_k]
+  const float* probs;           // [rows][top_k]
+  int top_k;
+  const __nv_bfloat16* post_w;
+  const __nv_bfloat16* add;     // vector added to the stream afterwards (null: none)
+  float* x;                     // [rows][width] in / out
+  const __nv_bfloat16* pre_w;   // norm of the next sublayer (null: none)
+  void* h;
+  int h_f32;
+  long long h_ld;
+  int width, rows;
+  float eps;
+};
+
+// ------------------------------------------------------------------------------------ latent attention
+struct LatentPrepArgs {
+  const float* proj;            // [rows][ld]: query latent | key/value latent | output gate (raw)
+  long long ld;
+  int rows, q_rank, kv_rank;
+  const __nv_bfloat16* q_w;
+  const __nv_bfloat16* kv_w;
+  float eps;
+  void* cq;                     // [rows][cq_ld]
+  long long cq_ld;
+  void* cache;                  // [capacity][cache_ld], row = position
+  long long cache_ld;
+  int f32;
+  const int* pos0;
+  int capacity;
+};
+
+struct LatentAttnArgs {
+  const void* q;                // [rows][heads * dim]
+  const void* k;                // keys of the block [kv_rows][heads * dim]
+  const void* v;                // simple form: [kv_rows][heads * vdim]; tensor-core form: feature-major [heads * vdim][v_ld]
+  long long v_ld;
+  const float* gate;            // raw output gate, element (row, head * vdim + j) at row * gate_ld + ...
+  long long gate_ld;
+  void* out;                    // [rows][heads * vdim]
+  int f32;
+  int rows, heads, dim, vdim;   // storage sizes (padded)
+  float scale;
+  const int* pos0;              // position of row 0
+  int kv0, kv_rows;             // positions covered by k / v
+  int first, last;              // first: no carried state; last: normalise, gate and store
+  float* state;                 // carried softmax state [rows][heads][vdim + 2] (max, sum, unnormalised output)
+  uint32_t* status;
+};
+
+struct LatentDecodeArgs {
+  const float* q;               // [heads][rank] queries taken into the latent space
+  const void* cache;            // [capacity][cache_ld]
+  long long cache_ld;
+  int f32;
+  int heads, rank;
+  float scale;
+  const int* pos0;
+  float* part;                  // [splits][heads][rank + 2]: max, sum, unnormalised latent output
+  int splits;
+};
+
+// ------------------------------------------------------------------------------------ gated linear recurrence
+struct RecurrenceArgs {
+  // short convolution
+  const void* xy;               // [rows][xy_ld]: gate branch | recurrence branch
+  long long xy_ld;
+  const __nv_bfloat16* conv;    // [width][taps]
+  const __nv_bfloat16* conv_b;
+  int taps;
+  float* history;               // [hist_rows][width] inputs of earlier positions, slot = position % hist_rows
+  int hist_rows;
+  void* u;                      // [rows][blocks][block_pad]
+  // recurrence
+  const float* gates;           // [rows][blocks][2 * block]: pre-activation r | i of every block
+  const float* softplus_lam;    // [width]
+  float decay;                  // log a = -decay * r * softplus(lam)
+  float* state;                 // [2][width] state after a position
+  int* tags;                    // [2]: number of tokens each state slot has seen
+  float* agg;                   // [chunks][2][width] scratch: decay product, local end state
+  void* out;                    // [rows][out_ld]
+  long long out_ld;
+  int f32;
+  int rows, width, blocks, block, block_pad;
+  const int* pos0;
+  uint32_t* status;
+};
+
+struct MoeGatherArgs {
+  const void* h;                // [rows][h_ld]
+  long long h_ld;
+  void* sorted;                 // [cap][h_ld]
+  const int* slot_of;           // [rows][top_k]
+  int rows, top_k, row_bytes;   // bytes of a row to copy (a multiple of 16)
+  int cap;
+};
+
+// ------------------------------------------------------------------------------------ one-token step
+enum StepPro : int {
+  kProResidual = 0,    // stream update + norm: x_out = x + rms(y) * post_w + add; input = rms(x_out) * in_w
+  kProNorm = 1,        // input = rms(in) * in_w
+  kProLoad = 2,        // input = in + group * in_gstride
+  kProMerge = 3,       // input = softmax-merged latent output of head `group` from the attention partials
+};
+enum StepEpi : int {
+  kTEpiStore = 0,      // acc * scale; rows from `sig_from` on through a sigmoid
+  kTEpiConv = 1,       // + bias; rows < width: GELU (tanh form); others: convolution input -> u, history
+  kTEpiGate = 2,       // acc * gate[row]
+  kTEpiGlu = 3,        // two products: clamped GLU (glu_kind 0) or SiLU GLU (1)
+  kTEpiRecur = 4,      // two products (r, i) + biases: recurrence step, times the gate branch
+};
+
+struct StepArgs {
+  // input
+  const int* tokens;
+  const __nv_bfloat16* table;
+  int vocab;
+  float embed_scale;
+  const float* x;
+  const float* y;
+  const __nv_bfloat16* post_w;
+  const __nv_bfloat16* add;
+  float* x_out;
+  const float* in_;
+  long long in_gstride;
+  const __nv_bfloat16* in_w;
+  float eps;
+  int k;
+  // attention partials
+  const float* part;
+  int splits;
+  // weights
+  const __nv_bfloat16* w;
+  const __nv_bfloat16* w2;
+  long long w_ld, w_gstride, w2_gstride;
+  int groups, n;                // groups x n output rows
+  const int* group_ids;         // weight group of each output group (routed experts), null: identity
+  // output
+  float* out;                   // [groups][n]
+  float scale;
+  int sig_from;
+  const __nv_bfloat16* bias;
+  const __nv_bfloat16* bias2;
+  const float* gate;
+  int glu_kind;
+  float limit, alpha;
+  // latent key/value row appended by this launch (kProNorm of the query latent)
+  const float* lat_in;
+  const __nv_bfloat16* lat_w;
+  int lat_rank;
+  void* lat_cache;
+  long long lat_ld;
+  int f32;                      // caches and rounding of the float form
+  // recurrence
+  const __nv_bfloat16* conv;
+  const __nv_bfloat16* conv_b;
+  int taps;
+  float* history;
+  int hist_rows;
+  float* u;
+  const float* softplus_lam;
+  float decay;
+  float* state;
+  int* tags;
+  const int* pos0;
+  int capacity;
+  uint32_t* status;
+};
+
+struct StepDownArgs {            // routed experts, second product: out[n] = sum_j p[j] * (W[id_j] act_j)[n]
+  const float* act;             // [top_k][k]
+  const __nv_bfloat16* w;       // [experts][n][w_ld]
+  long long w_ld, w_gstride;
+  const int* ids;
+  const float* probs;
+  int top_k, k, n;
+  float* out;
+};
+
+// ------------------------------------------------------------------------------------ math
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g * sigmoid_f(alpha * g) * (u + 1.0f);
+}
+__device__ __forceinline__ float silu_glu(float g, float u) { return g * sigmoid_f(g) * u; }
+
+__device__ __forceinline__ float lane_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+// Sum over the block (blockDim a multiple of 32, at most 1024); every thread gets it.  `red`: 33 floats of shared memory.
+__device__ __forceinline__ float block_sum_f(float v, float* red) {
+  v = lane_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  __syncthreads();
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float s = 0.f;
+#pragma unroll 1
+  for (int i = 0; i < nw; ++i) s += red[i];
+  return s;
+}
+__device__ __forceinline__ float bf(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+
+__device__ __forceinline__ void store_act(void* base, long long i, float v, int f32) {
+  if (f32) reinterpret_cast<float*>(base)[i] = v;
+  else reinterpret_cast<__nv_bfloat16*>(base)[i] = __float2bfloat16_rn(v);
+}
+__device__ __forceinline__ float load_act(const void* base, long long i, int f32) {
+  return f32 ? reinterpret_cast<const float*>(base)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(base)[i]);
+}
+
+// State slot that holds the recurrence after `pos` tokens; -1: none (recorded as a broken hand-over).  Position 0
+// starts from zero and writes slot 0.
+__device__ __forceinline__ int state_slot(const int* tags, int pos, uint32_t* status) {
+  if (pos == 0) return 1;
+  const int t0 = *reinterpret_cast<const volatile int*>(tags), t1 = *reinterpret_cast<const volatile int*>(tags + 1);
+  if (t0 == pos) return 0;
+  if (t1 == pos) return 1;
+  report(status, kSiteState);
+  return -1;
+}
+
+}  // namespace nrt

@@ -1,0 +1,266 @@
+// Row kernels of layer stacks (chunk path): stream update + norms, latent preparation, short convolution, the gated
+// linear recurrence as a chunked scan, and the expert row permutation.
+#include "stack.cuh"
+#include "launch.hpp"
+#include "router.cuh"
+
+#include <string.h>
+
+using namespace nrt;
+
+namespace {
+
+// ------------------------------------------------------------------------------------ stream update + norms
+// One CTA per row.  x (+ embedding) -> x += rms(y) * post_w + add -> h = rms(x) * pre_w, all in float.
+__global__ void __launch_bounds__(256) stack_rows_kernel(const StackRowArgs a) {
+  extern __shared__ float buf[];                 // [2][width]: sublayer row, stream row
+  __shared__ float red[33];
+  griddep_wait();
+  griddep_launch();
+  const int r = blockIdx.x, W = a.width;
+  float* sy = buf;
+  float* sx = buf + W;
+  float ss = 0.f;
+  if (a.y) {
+    if (a.slot_of) {
+      for (int c = threadIdx.x; c < W; c += 256) {
+        float v = 0.f;
+        for (int j = 0; j < a.top_k; ++j)
+          v = fmaf(a.probs[(size_t)r * a.top_k + j], a.y[(long long)a.slot_of[(size_t)r * a.top_k + j] * a.y_ld + c], v);
+        sy[c] = v;
+        ss = fmaf(v, v, ss);
+      }
+    } else {
+      for (int c = threadIdx.x; c < W; c += 256) {
+        const float v = a.y[(long long)r * a.y_ld + c];
+        sy[c] = v;
+        ss = fmaf(v, v, ss);
+      }
+    }
+    ss = block_sum_f(ss, red);
+  }
+  const float ry = a.y ? 1.0f / sqrtf(ss / (float)W + a.eps) : 0.f;
+  const __nv_bfloat16* emb = nullptr;
+  if (a.tokens) {
+    int t = a.tokens[r];
+    t = t < 0 ? 0 : t >= a.vocab ? a.vocab - 1 : t;
+    emb = a.table + (size_t)t * W;
+  }
+  float sq = 0.f;
+  for (int c = threadIdx.x; c < W; c += 256) {
+    float v = emb ? bf(emb + c) * a.embed_scale : a.x[(size_t)r * W + c];
+    if (a.y) v += sy[c] * ry * bf(a.post_w + c);
+    if (a.add) v += bf(a.add + c);
+    a.x[(size_t)r * W + c] = v;
+    sx[c] = v;
+    sq = fmaf(v, v, sq);
+  }
+  if (!a.pre_w) return;
+  sq = block_sum_f(sq, red);
+  const float rx = 1.0f / sqrtf(sq / (float)W + a.eps);
+  for (int c = threadIdx.x; c < W; c += 256) store_act(a.h, (long long)r * a.h_ld + c, sx[c] * rx * bf(a.pre_w + c), a.h_f32);
+}
+
+// ------------------------------------------------------------------------------------ latent preparation
+// grid (rows, 2): y = 0 normalises the query latent, y = 1 the key/value latent into its cache row.
+__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepArgs a) {
+  __shared__ float red[33];
+  griddep_wait();
+  griddep_launch();
+  const int r = blockIdx.x, which = blockIdx.y;
+  const int n = which ? a.kv_rank : a.q_rank;
+  const float* src = a.proj + (long long)r * a.ld + (which ? a.q_rank : 0);
+  const __nv_bfloat16* w = which ? a.kv_w : a.q_w;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < n; c += 256) ss = fmaf(src[c], src[c], ss);
+  const float rs = 1.0f / sqrtf(block_sum_f(ss, red) / (float)n + a.eps);
+  void* dst = which ? a.cache : a.cq;
+  const int row = which ? *a.pos0 + r : r;
+  if (which && (row < 0 || row >= a.capacity)) return;
+  const long long base = (long long)row * (which ? a.cache_ld : a.cq_ld);
+  for (int c = threadIdx.x; c < n; c += 256) store_act(dst, base + c, src[c] * rs * bf(w + c), a.f32);
+}
+
+// ------------------------------------------------------------------------------------ short convolution
+// grid (rows, channel blocks): u[r][c] = b[c] + sum_j k[c][j] x[position of tap j], zeros before the sequence.
+__global__ void __launch_bounds__(256) stack_conv_kernel(const RecurrenceArgs a) {
+  griddep_wait();
+  griddep_launch();
+  const int r = blockIdx.x, c = blockIdx.y * 256 + threadIdx.x;
+  if (c >= a.width) return;
+  const int pos = *a.pos0 + r;
+  float v = bf(a.conv_b + c);
+  for (int j = 0; j < a.taps; ++j) {
+    const int back = a.taps - 1 - j;              // tokens before the current one
+    if (back > pos) continue;
+    const float x = back <= r ? load_act(a.xy, (long long)(r - back) * a.xy_ld + a.width + c, a.f32)
+                              : a.history[(long long)((pos - back) % a.hist_rows) * a.width + c];
+    v = fmaf(bf(a.conv + (size_t)c * a.taps + j), x, v);
+  }
+  const int b = c / a.block;
+  store_act(a.u, ((long long)r * a.blocks + b) * a.block_pad + (c - b * a.block), v, a.f32);
+}
+
+// ------------------------------------------------------------------------------------ gated linear recurrence
+constexpr int kScanTokens = 64;               // tokens per CTA of the scan
+
+struct Gate { float a, drive; };
+__device__ __forceinline__ Gate gate_of(const RecurrenceArgs& p, int r, int c, int b, int cb, float sp) {
+  const float* g = p.gates + ((long long)r * p.blocks + b) * 2 * p.block;
+  const float rg = sigmoid_f(g[cb]), ig = sigmoid_f(g[p.block + cb]);
+  const float la = -p.decay * rg * sp;
+  const float u = load_act(p.u, ((long long)r * p.blocks + b) * p.block_pad + cb, p.f32);
+  Gate o;
+  o.a = expf(la);
+  o.drive = sqrtf(-expm1f(2.0f * la)) * ig * u;
+  return o;
+}
+
+// pass 1: decay product and end state (from zero) of every 64-token piece
+__global__ void __launch_bounds__(128) stack_scan_pieces_kernel(const RecurrenceArgs p) {
+  griddep_wait();
+  griddep_launch();
+  const int c = blockIdx.y * 128 + threadIdx.x;
+  if (c >= p.width) return;
+  const int b = c / p.block, cb = c - b * p.block;
+  const float sp = p.softplus_lam[c];
+  const int r0 = blockIdx.x * kScanTokens, r1 = min(p.rows, r0 + kScanTokens);
+  float prod = 1.f, s = 0.f;
+  for (int r = r0; r < r1; ++r) {
+    const Gate g = gate_of(p, r, c, b, cb, sp);
+    prod *= g.a;
+    s = fmaf(g.a, s, g.drive);
+  }
+  float* o = p.agg + (size_t)blockIdx.x * 2 * p.width;
+  o[c] = prod;
+  o[p.width + c] = s;
+}
+
+// pass 2: state at the piece's start from the carried state and the earlier pieces, then the piece itself; the last
+// piece leaves the state behind and appends the convolution history.
+__global__ void __launch_bounds__(128) stack_scan_kernel(const RecurrenceArgs p) {
+  griddep_wait();
+  griddep_launch();
+  const int c = blockIdx.y * 128 + threadIdx.x;
+  const int pos0 = *p.pos0;
+  const int slot = state_slot(p.tags, pos0, p.status);
+  const bool last = blockIdx.x == gridDim.x - 1;
+  if (slot < 0) return;
+  if (c < p.width) {
+    const int b = c / p.block, cb = c - b * p.block;
+    const float sp = p.softplus_lam[c];
+    float s = pos0 == 0 ? 0.f : p.state[(size_t)slot * p.width + c];
+    for (int q = 0; q < (int)blockIdx.x; ++q) {
+      const float* g = p.agg + (size_t)q * 2 * p.width;
+      s = fmaf(g[c], s, g[p.width + c]);
+    }
+    const int r0 = blockIdx.x * kScanTokens, r1 = min(p.rows, r0 + kScanTokens);
+    for (int r = r0; r < r1; ++r) {
+      const Gate g = gate_of(p, r, c, b, cb, sp);
+      s = fmaf(g.a, s, g.drive);
+      store_act(p.out, (long long)r * p.out_ld + c, s * load_act(p.xy, (long long)r * p.xy_ld + c, p.f32), p.f32);
+    }
+    if (last) {
+      p.state[(size_t)(1 - slot) * p.width + c] = s;
+      const int keep = min(p.taps - 1, p.rows);
+      for (int j = p.rows - keep; j < p.rows; ++j)
+        p.history[(long long)((pos0 + j) % p.hist_rows) * p.width + c] = load_act(p.xy, (long long)j * p.xy_ld + p.width + c, p.f32);
+    }
+  }
+  // A CTA that starts after this store still finds `pos0` in its own slot: only the other slot's tag changes.
+  if (last && blockIdx.y == 0 && threadIdx.x == 0) {
+    p.tags[1 - slot] = pos0 + p.rows;
+    if (pos0 == 0) p.tags[1] = -1;
+  }
+}
+
+// ------------------------------------------------------------------------------------ expert rows
+// Selection for chunk rows from a filled score matrix, experts limited to the best groups; one CTA per 16 rows.
+__global__ void __launch_bounds__(256) stack_route_kernel(const RouterArgs a_in, const int groups, const int keep) {
+  __shared__ RouterSmem sm;
+  griddep_wait();
+  griddep_launch();
+  RouterArgs a = a_in;
+  const int r0 = blockIdx.x * kRouterRows;
+  a.rows = min(kRouterRows, a_in.rows - r0);
+  a.scores += (size_t)r0 * a.experts;
+  a.topk_ids += (size_t)r0 * a.top_k;
+  a.topk_p += (size_t)r0 * a.top_k;
+  router_select<true>(a, sm, true, nullptr, nullptr, nullptr, groups, keep);
+}
+
+__global__ void __launch_bounds__(128) moe_gather_kernel(const MoeGatherArgs a) {
+  griddep_wait();
+  griddep_launch();
+  const int r = blockIdx.x, j = blockIdx.y;
+  const int slot = a.slot_of[(size_t)r * a.top_k + j];
+  if (!NRT_INDEX_OK(slot, a.cap, kBoundsExpert)) return;
+  const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const char*>(a.h) + (size_t)r * a.h_ld);
+  uint4* dst = reinterpret_cast<uint4*>(reinterpret_cast<char*>(a.sorted) + (size_t)slot * a.h_ld);
+  for (int i = threadIdx.x; i < a.row_bytes / 16; i += 128) dst[i] = src[i];
+}
+
+}  // namespace
+
+#define S(stream) reinterpret_cast<cudaStream_t>(stream)
+
+extern "C" int nrt_stack_row_args_size() { return (int)sizeof(StackRowArgs); }
+extern "C" int nrt_latent_prep_args_size() { return (int)sizeof(LatentPrepArgs); }
+extern "C" int nrt_recurrence_args_size() { return (int)sizeof(RecurrenceArgs); }
+extern "C" int nrt_moe_gather_args_size() { return (int)sizeof(MoeGatherArgs); }
+extern "C" int nrt_stack_scan_tokens() { return kScanTokens; }
+
+extern "C" int nrt_stack_rows(const void* args, void* stream) {
+  StackRowArgs a;
+  memcpy(&a, args, sizeof(a));
+  if (a.rows < 1 || a.width < 1 || (a.y && !a.post_w)) return -3;
+  const size_t smem = (size_t)a.width * 8;
+  if (smem > 200 * 1024) return -7;
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(stack_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  return launch_pdl(stack_rows_kernel, dim3(a.rows), dim3(256), smem, S(stream), false, a);
+}
+
+extern "C" int nrt_latent_prep(const void* args, void* stream) {
+  LatentPrepArgs a;
+  memcpy(&a, args, sizeof(a));
+  if (a.rows < 1 || a.q_rank < 1 || a.kv_rank < 1) return -3;
+  return launch_pdl(latent_prep_kernel, dim3(a.rows, 2), dim3(256), 0, S(stream), false, a);
+}
+
+extern "C" int nrt_stack_conv(const void* args, void* stream) {
+  RecurrenceArgs a;
+  memcpy(&a, args, sizeof(a));
+  if (a.rows < 1 || a.taps < 1 || a.hist_rows < 2 * (a.taps - 1) || a.hist_rows < 1 || a.width != a.blocks * a.block) return -3;
+  return launch_pdl(stack_conv_kernel, dim3(a.rows, (a.width + 255) / 256), dim3(256), 0, S(stream), false, a);
+}
+
+// The recurrence over the chunk's rows: pieces, then the scan with the state hand-over.
+extern "C" int nrt_stack_scan(const void* args, void* stream) {
+  RecurrenceArgs a;
+  memcpy(&a, args, sizeof(a));
+  if (a.rows < 1 || a.width != a.blocks * a.block) return -3;
+  const int pieces = (a.rows + kScanTokens - 1) / kScanTokens;
+  const dim3 grid(pieces, (a.width + 127) / 128);
+  int rc = 0;
+  if (pieces > 1 && (rc = launch_pdl(stack_scan_pieces_kernel, grid, dim3(128), 0, S(stream), false, a))) return rc;
+  return launch_pdl(stack_scan_kernel, grid, dim3(128), 0, S(stream), false, a);
+}
+
+extern "C" int nrt_stack_route(const void* args, int groups, int keep, void* stream) {
+  RouterArgs a;
+  memcpy(&a, args, sizeof(a));
+  if (a.rows < 1 || a.experts > 256 || a.top_k > 32 || groups < 1 || groups > 32 || a.experts % groups || !a.scores || a.probs) return -3;
+  return launch_pdl(stack_route_kernel, dim3((a.rows + kRouterRows - 1) / kRouterRows), dim3(256), 0, S(stream), false, a, groups, keep);
+}
+
+extern "C" int nrt_moe_gather(const void* args, void* stream) {
+  MoeGatherArgs a;
+  memcpy(&a, args, sizeof(a));
+  if (a.rows < 1 || a.row_bytes % 16 || a.h_ld % 16) return -3;
+  return launch_pdl(moe_gather_kernel, dim3(a.rows, a.top_k), dim3(128), 0, S(stream), false, a);
+}

@@ -1,0 +1,186 @@
+"""Models described as an ordered list of layers: each layer has a token mixer and, optionally, a feed-forward.
+
+The mechanisms are independent of one another and carry their own sizes and constants, so a design is a list of
+``LayerSpec`` plus the sizes of its stream.  ``StackSpec`` offers what the rest of the framework asks of a model
+(vocabulary, stop tokens, cache bytes); the runtime that executes it is ``runtime/stack.py``.
+
+A *run* is one execution of a layer: a layer inside the loop runs once per pass with the same weights, and every run
+has its own cache or state.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass, replace
+from typing import List, Optional, Tuple, Union
+
+from .spec import MoeRoutingSpec
+
+# widths of the kernels (csrc/stack*.cu, csrc/router.cuh)
+MAX_EXPERTS, MAX_TOP_K, MAX_GROUPS = 256, 32, 32
+MAX_HEAD_DIM = 512
+MAX_RANK = 4096
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Causal softmax attention without positions over one cached, normed latent per token, with an output gate."""
+
+    heads: int
+    dim: int                # query / key width of a head
+    vdim: int               # value width of a head
+    kv_rank: int            # cached latent
+    q_rank: int             # query latent
+    scale: float
+    kind: str = "latent_attention"
+
+
+@dataclass(frozen=True)
+class GatedRecurrenceSpec:
+    """Two branches of ``width``: a GELU gate and a short causal convolution feeding a gated linear recurrence whose
+    gates are block-diagonal products (``log a = -decay * r * softplus(lam)``)."""
+
+    width: int
+    blocks: int
+    taps: int
+    decay: float = 8.0
+    kind: str = "rglru"
+
+    @property
+    def block(self) -> int:
+        return self.width // self.blocks
+
+    @property
+    def hist_rows(self) -> int:
+        """Ring rows of the convolution history: a step writes its input while the previous ``taps - 1`` are read."""
+        return max(1, 2 * (self.taps - 1))
+
+
+@dataclass(frozen=True)
+class ClampedGluSpec:
+    """min(g, limit) * sigmoid(alpha * g) * (clamp(u, -limit, limit) + 1) between two products."""
+
+    ff: int
+    limit: float
+    alpha: float = 1.702
+    kind: str = "dense"
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    """Routed SiLU-GLU experts; ``routing`` carries scores, group limit and weights."""
+
+    routing: MoeRoutingSpec
+    kind: str = "moe"
+
+    @property
+    def ff(self) -> int:
+        return self.routing.intermediate
+
+
+Mixer = Union[LatentAttentionSpec, GatedRecurrenceSpec]
+FeedForward = Union[ClampedGluSpec, ExpertsSpec]
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: Mixer
+    mlp: Optional[FeedForward]
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row; a learned vector is added to the stream ahead of each pass."""
+
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    run: int                         # index among all runs: owns a cache or state
+    layer: int                       # whose weights
+    pass_start: Optional[int]        # pass whose vector is added to the stream first
+
+
+@dataclass(frozen=True)
+class StackSpec:
+    name: str
+    architecture: str
+    hidden: int
+    vocab: int
+    layers: Tuple[LayerSpec, ...]
+    norm_eps: float
+    embed_scale: float = 1.0
+    logit_scale: float = 1.0
+    loop: Optional[LoopSpec] = None
+    stop_token_ids: Tuple[int, ...] = ()
+    think_end_token_id: int = -1
+    draft: None = None               # no block draft: rounds commit one token
+
+    @property
+    def layer_count(self) -> int:
+        return len(self.layers)
+
+    def runs(self) -> List[LayerRun]:
+        out: List[Tuple[int, Optional[int]]] = []
+        n, lp = len(self.layers), self.loop
+        if lp is None:
+            out = [(i, None) for i in range(n)]
+        else:
+            out = [(i, None) for i in range(lp.start)]
+            for t in range(lp.times):
+                out += [(i, t if i == lp.start else None) for i in range(lp.start, lp.stop)]
+            out += [(i, None) for i in range(lp.stop, n)]
+        return [LayerRun(k, i, t) for k, (i, t) in enumerate(out)]
+
+    def vocab_shard(self, tp: int) -> int:
+        if tp != 1:
+            raise ValueError(f"{self.architecture} runs on one GPU (tp=1); tp={tp} was asked for")
+        return self.vocab
+
+    def with_layers(self, n: int) -> "StackSpec":
+        """The first ``n`` layers (a loop that would be cut is dropped)."""
+        if not 1 <= n <= len(self.layers):
+            raise ValueError(f"layer count {n} outside 1..{len(self.layers)}")
+        loop = self.loop if self.loop is not None and self.loop.stop <= n else None
+        return replace(self, name=f"{self.name}-L{n}", layers=self.layers[:n], loop=loop)
+
+    def kv_bytes_per_token(self, tp: int = 1, element_bytes: int = 2) -> int:
+        self.vocab_shard(tp)
+        return sum(_pad(self.layers[r.layer].mixer.kv_rank, 16) * element_bytes
+                   for r in self.runs() if self.layers[r.layer].mixer.kind == "latent_attention")
+
+    def validate(self) -> "StackSpec":
+        """Refuse what the kernels cannot run, by name, before anything is allocated."""
+        def need(ok: bool, what: str) -> None:
+            if not ok:
+                raise ValueError(f"{self.name}: {what}")
+        need(self.hidden >= 1 and self.vocab >= 1 and len(self.layers) >= 1, "empty model")
+        need(self.hidden <= 25600, "width above 25600")
+        for i, layer in enumerate(self.layers):
+            m, f = layer.mixer, layer.mlp
+            if m.kind == "latent_attention":
+                need(min(m.heads, m.dim, m.vdim, m.kv_rank, m.q_rank) >= 1, f"layer {i}: empty attention size")
+                need(m.dim <= MAX_HEAD_DIM and m.vdim <= MAX_HEAD_DIM, f"layer {i}: head width above {MAX_HEAD_DIM}")
+                need(m.kv_rank <= MAX_RANK, f"layer {i}: kv_rank above {MAX_RANK}")
+            elif m.kind == "rglru":
+                need(min(m.width, m.blocks, m.taps) >= 1 and m.width % m.blocks == 0, f"layer {i}: width does not split into blocks")
+            else:
+                need(False, f"layer {i}: unknown mixer {m.kind!r}")
+            if f is not None and f.kind == "moe":
+                r = f.routing
+                need(r.score_func == "sigmoid", f"layer {i}: router scores {r.score_func!r}")
+                need(1 <= r.top_k <= min(MAX_TOP_K, r.expert_count) and r.expert_count <= MAX_EXPERTS,
+                     f"layer {i}: router of {r.expert_count} experts, top {r.top_k}")
+                need(1 <= r.limited_group_count <= r.group_count <= MAX_GROUPS and r.expert_count % r.group_count == 0,
+                     f"layer {i}: expert groups")
+                need(r.top_k <= r.expert_count // r.group_count * r.limited_group_count, f"layer {i}: fewer eligible experts than top_k")
+            elif f is not None and f.kind != "dense":
+                need(False, f"layer {i}: unknown feed-forward {f.kind!r}")
+        if self.loop is not None:
+            need(0 <= self.loop.start < self.loop.stop <= len(self.layers) and self.loop.times >= 1, "loop bounds")
+        return self
+
+
+def _pad(n: int, to: int) -> int:
+    return -(-n // to) * to

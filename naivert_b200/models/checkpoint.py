@@ -461,6 +461,44 @@ def load_draft_rank_weights(spec: ModelSpec, root: str, rank: int, tp: int, devi
     return _to_device(shard_draft_weights(spec, prepare_draft_weights(spec, sd), rank, tp), device), ckpt.identity()
 
 
+# --------------------------------------------------------------------------- layer-stack designs
+def validate_stack_layout(spec, ckpt: LocalCheckpoint) -> None:
+    """Every tensor of the design present with the shape the configuration implies."""
+    from .registry import design_of
+    want = design_of(spec).tensor_shapes(spec)
+    missing = sorted(set(want) - set(ckpt.weight_map))
+    if missing:
+        raise CheckpointError(f"checkpoint lacks {len(missing)} tensors, e.g. {missing[:3]}")
+    for n, shape in want.items():
+        have = tuple(ckpt.headers[ckpt.weight_map[n]][n]["shape"])
+        if have != shape:
+            raise CheckpointError(f"tensor {n} has shape {have}, the configuration needs {shape}")
+
+
+def load_stack_weights(spec, root: str, device="cpu") -> dict:
+    """The weights of a layer-stack checkpoint (``config.json`` and one or more safetensors files), grouped by layer."""
+    from .registry import design_of
+    ckpt = LocalCheckpoint(root)
+    validate_stack_layout(spec, ckpt)
+    rd = SliceReader(ckpt)
+    try:
+        return design_of(spec).gather_weights(spec, lambda n: rd.full(n).to(device))
+    finally:
+        rd.close()
+
+
+def write_stack_checkpoint(root: str, spec, seed: int = 0, state_dict: Optional[StateDict] = None) -> CheckpointIdentity:
+    from safetensors.torch import save_file
+    from .registry import design_of
+    os.makedirs(root, exist_ok=True)
+    design = design_of(spec)
+    sd = state_dict if state_dict is not None else design.init_state_dict(spec, seed)
+    with open(os.path.join(root, "config.json"), "w") as f:
+        json.dump(design.config_from_spec(spec), f, indent=1)
+    save_file({k: v.contiguous() for k, v in sd.items()}, os.path.join(root, "model.safetensors"))
+    return LocalCheckpoint(root).identity()
+
+
 def _to_device(obj, device):
     if isinstance(obj, torch.Tensor):
         return obj.to(device)

@@ -116,3 +116,12 @@ def init_draft_rank_weights_device(spec: ModelSpec, rank: int, tp: int, seed: in
             "wv": _randn(kvg, nkv * hd, Hd, std=std), "wo": _randn(shd, Hd, nh * hd, std=std),
             "gate": _randn(shd, I, Hd, std=std), "up": _randn(shd, I, Hd, std=std), "down": _randn(shd, Hd, I, std=std)})
     return out
+
+
+def init_stack_weights_device(spec, seed: int = 0, device="cuda") -> dict:
+    """Random weights of a layer-stack model, drawn on the device and grouped by layer (experts drawn as one stack)."""
+    from .registry import design_of
+    design = design_of(spec)
+    g = torch.Generator(device=device).manual_seed(seed)
+    shapes = design.tensor_shapes(spec)
+    return design.gather_weights(spec, lambda n: design.random_tensor(n, shapes[n], g, device))

@@ -1,16 +1,32 @@
-"""Served-model registry (reference naivert/models/registry.py:25-44)."""
+"""Served-model registry (reference naivert/models/registry.py:25-44).
+
+A model is named (``resolve_model``) or described by a checkpoint's ``config.json`` (``resolve_checkpoint_model``):
+``architecture`` names a layer-stack design, ``model_type`` the speculative-decoding target.
+"""
 from __future__ import annotations
 
+import json
+import os
+from typing import Union
+
+from . import tumatar
+from .blocks import StackSpec
 from .naive_n0p5 import NAIVE_N0P5, small_w8a8_spec, tiny_spec
 from .spec import ModelSpec
 
 MODELS = {
     "naive-n0.5": NAIVE_N0P5,
     "naive-n0.5-preview": NAIVE_N0P5,
+    "tumatar-small": tumatar.small_spec(),
+    "tumatar-bench": tumatar.bench_spec(),
+    "tumatar-bench-dense": tumatar.bench_spec(experts=False),
 }
 
+# config.json "architecture" -> design module (spec_from_config, tensor_shapes, gather_weights, ...)
+DESIGNS = {tumatar.ARCHITECTURE: tumatar}
 
-def resolve_model(name: str) -> ModelSpec:
+
+def resolve_model(name: str) -> Union[ModelSpec, StackSpec]:
     if name in MODELS:
         return MODELS[name]
     if name.startswith("tiny"):
@@ -18,3 +34,28 @@ def resolve_model(name: str) -> ModelSpec:
     if name.startswith("small"):
         return small_w8a8_spec()
     raise KeyError(f"unknown model {name!r}; known: {sorted(MODELS)}")
+
+
+def design_of(spec: StackSpec):
+    return DESIGNS[spec.architecture]
+
+
+def spec_from_config(cfg: dict, name: str = "") -> Union[ModelSpec, StackSpec]:
+    """The model a ``config.json`` describes."""
+    arch = cfg.get("architecture")
+    if arch in DESIGNS:
+        return DESIGNS[arch].spec_from_config(cfg, name or arch.lower())
+    if cfg.get("model_type") == "naive_n0p5":
+        from .checkpoint import target_config
+        for spec in MODELS.values():
+            if isinstance(spec, ModelSpec) and target_config(spec)["hidden_size"] == cfg.get("hidden_size") \
+                    and spec.layer_count == cfg.get("num_hidden_layers"):
+                return spec
+    raise KeyError(f"no registered model for config.json (architecture {arch!r}, model_type {cfg.get('model_type')!r}); "
+                   f"designs: {sorted(DESIGNS)}")
+
+
+def resolve_checkpoint_model(root: str) -> Union[ModelSpec, StackSpec]:
+    """The model of a checkpoint directory, chosen by its ``config.json``."""
+    with open(os.path.join(root, "config.json")) as f:
+        return spec_from_config(json.load(f), os.path.basename(os.path.abspath(root)))

@@ -170,6 +170,21 @@ def generate(name: str, parsed: Optional[Dict[str, List[Field]]] = None, _cache:
     return cache[name]
 
 
+def generate_from(source: str, names: List[str]) -> Dict[str, type]:
+    """ctypes classes of the structs ``names`` declared in one CUDA source, for bindings that keep no mirror by hand."""
+    parsed: Dict[str, List[Field]] = {}
+    known: Dict[str, Tuple[int, int]] = {}
+    for name in names:
+        body = struct_body(os.path.join(CSRC, source), name)
+        if body is None:
+            raise ValueError(f"{name}: not found in {source}")
+        parsed[name] = parse_fields(body, known)
+        _, size, align = layout(parsed[name])
+        known[name] = (size, align)
+    cache: dict = {}
+    return {n: generate(n, parsed, cache) for n in names}
+
+
 def emit_module() -> str:
     """Python source of all generated classes (the starting point of a new binding)."""
     parsed = parse_all()

@@ -147,14 +147,14 @@ class TensorMap:
     """A 128-byte CUtensorMap kept alive with the tensor it describes."""
 
     def __init__(self, t: torch.Tensor, dims: Sequence[int], strides_bytes: Sequence[int], box: Sequence[int],
-                 dtype_code: int, swizzle: int = 3):
+                 dtype_code: int, swizzle: int = 3, library=None):
         self.tensor = t
         self.buf = (C.c_ubyte * 128)()
         rank = len(dims)
         d = (C.c_uint64 * 5)(*dims)
         s = (C.c_uint64 * 5)(*strides_bytes)
         b = (C.c_uint32 * 5)(*box)
-        check(lib().nrt_tmap_encode(C.byref(self.buf), dtype_code, rank, d, s, b, swizzle, VP(t.data_ptr())),
+        check((library or lib()).nrt_tmap_encode(C.byref(self.buf), dtype_code, rank, d, s, b, swizzle, VP(t.data_ptr())),
               "cuTensorMapEncodeTiled")
 
 

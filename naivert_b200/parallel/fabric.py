@@ -118,6 +118,7 @@ _SITE_CLASSES = {
     0x600: "a cluster partner did not arrive",
     0x700: "a small-message exchange did not complete",
     0x800: "an in-grid hand-over did not complete",
+    0x900: "a recurrent layer holds no state for the position the step starts at (a step was skipped or repeated out of order)",
 }
 
 

@@ -13,10 +13,11 @@ from __future__ import annotations
 
 import time
 from dataclasses import dataclass, field
-from typing import Iterator, List, Optional
+from typing import Iterator, List, Optional, Union
 
 import torch
 
+from ..models.blocks import StackSpec
 from ..models.spec import ModelSpec, SamplingParams
 from ..parallel.fabric import Fabric
 from .round import RING_SIZE, RoundRecord, RuntimeContractError, SpeculativeRound
@@ -54,13 +55,24 @@ class Engine:
 
     # ------------------------------------------------------------------ construction
     @classmethod
-    def build(cls, spec: ModelSpec, rank: int = 0, tp: int = 1, group=None, capacity: int = 16384, seed: int = 0,
+    def build(cls, spec: Union[ModelSpec, StackSpec], rank: int = 0, tp: int = 1, group=None, capacity: int = 16384, seed: int = 0,
               target_ckpt: Optional[str] = None, draft_ckpt: Optional[str] = None, device=None,
               weights: Optional[dict] = None, draft_weights: Optional[dict] = None, pdl: Optional[bool] = None,
               shape_tp: int = 0, device_chain: Optional[bool] = None, prefill_chunk: int = 0,
-              ep_weights: Optional[list] = None, ring_size: int = 0) -> "Engine":
+              ep_weights: Optional[list] = None, ring_size: int = 0, dtype: str = "bf16") -> "Engine":
         """``prefill_chunk`` > 0 adds the chunked native prefill (rows per chunk); ``ep_weights`` (whole experts of
-        this rank per layer, ``models.weights.shard_expert_weights``) selects its expert-parallel MoE path."""
+        this rank per layer, ``models.weights.shard_expert_weights``) selects its expert-parallel MoE path.
+        A layer-stack model (``models.blocks.StackSpec``) is built by ``runtime.stack_engine``; ``dtype`` is its numeric
+        form (``bf16`` or ``fp32``)."""
+        if isinstance(spec, StackSpec):
+            from .stack_engine import build_stack_engine
+            if draft_ckpt is not None or draft_weights is not None or ep_weights is not None or shape_tp:
+                raise RuntimeContractError(f"{spec.architecture} has no draft and no expert-parallel copies")
+            return build_stack_engine(spec, rank=rank, tp=tp, capacity=capacity, seed=seed, target_ckpt=target_ckpt, device=device,
+                                      weights=weights, pdl=pdl, device_chain=device_chain, prefill_chunk=prefill_chunk,
+                                      ring_size=ring_size, dtype=dtype)
+        if dtype != "bf16":
+            raise RuntimeContractError("the W8A8 target has no 32-bit form on the GPU")
         device = device or torch.device("cuda", torch.cuda.current_device())
         if pdl is None:
             # Programmatic dependent launch on every kernel (NAIVERT_PDL=0 turns it off): the next kernel's launch,
@@ -169,7 +181,7 @@ class Engine:
         return res
 
     def kv_bytes(self) -> int:
-        return self.target.kv_bytes() + self.round.draft.kv_bytes()
+        return self.target.kv_bytes() + (self.round.draft.kv_bytes() if self.round.draft is not None else 0)
 
     def close(self) -> None:
         if self.prefill is not None:

@@ -100,6 +100,8 @@ MODES: Dict[str, DecodeMode] = {m.mode_id: m for m in (
     DecodeMode("verify8", 8, False, _STEP + ("nrt_argmax_rows",), buffer_table(8, False, False)),
     DecodeMode("speculative_round", 8, True, _ROUND, buffer_table(8, True, True)),
     DecodeMode("prefill_replay", 8, True, _ROUND, buffer_table(8, True, False)),
+    # layer-stack models: their own step kernels (ops.stack_kernels checks that library), the shared sampler and tail
+    DecodeMode("stack_round", 1, False, ("nrt_sampler_persistent", "nrt_sampler_run", "nrt_tail_commit"), buffer_table(1, False, True)),
     DecodeMode("prefill_native", 0, True,
                ("nrt_wide_gemm_launch", "nrt_attn_post", "nrt_attn_group", "nrt_index_sweep", "nrt_topk_rows_grid", "nrt_router",
                 "nrt_ep_count", "nrt_ep_dispatch", "nrt_ep_combine", "nrt_ag_push"), buffer_table(0, True, False)),

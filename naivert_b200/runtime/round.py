@@ -2,6 +2,7 @@
 sharded sampler / verify -> tail commit, captured once as a CUDA graph per rank whose kernels
 are chained with programmatic dependent launch.  Ranks stay in lockstep purely through the
 tagged words of the fabric; the host only launches graphs ahead and polls a pinned ring.
+``DecodeRound`` is the same without a draft: one step, one token.
 
 Control block (int32, device): [0] position of the anchor row, [1] rows to ingest,
 [2] first ingest position, [4] stopped, [5] stop reason, [6] tokens produced, [7] token limit,
@@ -75,11 +76,14 @@ class HostRing:
             self.host = 0
 
 
-class SpeculativeRound:
-    def __init__(self, spec: ModelSpec, target: TargetRuntime, draft_weights: dict, capacity: int, pdl: bool = True,
-                 device_chain: bool = False, ring_size: int = RING_SIZE):
-        if target.rows != spec.draft.rows:
-            raise RuntimeContractError("the verify runtime must run block_size + 1 rows")
+class DecodeRound:
+    """Rounds of a model without a draft: one target step, the sampler on its last row, the tail commit - one token per
+    round.  ``target`` is any runtime with the step contract (``rows``, ``ctrl``, ``tokens``, ``logits``, ``step(head)``)
+    whose step may be repeated at the same position.  ``SpeculativeRound`` adds the draft."""
+
+    draft: Optional[DraftRuntime] = None
+
+    def __init__(self, spec, target, capacity: int, pdl: bool = True, device_chain: bool = False, ring_size: int = RING_SIZE):
         self.spec, self.t, self.fab, self.pdl = spec, target, target.fab, pdl
         dev = target.dev
         self.tp, self.rank = target.tp, target.rank
@@ -96,7 +100,7 @@ class SpeculativeRound:
         self.sampler_one_launch = target.fused and os.environ.get("NAIVERT_SAMPLER_PERSISTENT", "1") == "1"
         self.sampler_sync = torch.zeros(2, dtype=torch.int64, device=dev)
         self.ring = HostRing(ring_size)
-        self.draft = DraftRuntime(spec, draft_weights, target, capacity, self.seed, self.params, self.block_ids, pdl=pdl)
+        self._make_draft(capacity)
         self.capacity = capacity
         self.graph: Optional[torch.cuda.CUDAGraph] = None
         self.prefill_graph: Optional[torch.cuda.CUDAGraph] = None
@@ -114,15 +118,19 @@ class SpeculativeRound:
         self._build_args()
         self.stream = torch.cuda.Stream(device=dev)
 
+    def _make_draft(self, capacity: int) -> None:
+        pass
+
     def _build_args(self):
         s = K.SamplerArgs()
         s.zp, s.ldp = self.t.logits.data_ptr(), self.t.logits.shape[1]
-        s.zq, s.ldq = self.draft.zq.data_ptr(), self.draft.zq.shape[1]
+        if self.draft is not None:
+            s.zq, s.ldq = self.draft.zq.data_ptr(), self.draft.zq.shape[1]
         s.vlocal, s.vbase, s.e = self.vlocal, self.vbase, self.codes.data_ptr()
         s.counts = None
         s.params, s.seed = self.params.data_ptr(), self.seed.data_ptr()
         s.ctrl, s.block_ids = self.t.ctrl.data_ptr(), self.block_ids.data_ptr()
-        s.n_rows_p, s.n_rows_q = 8, 7
+        s.n_rows_p, s.n_rows_q = (8, 7) if self.draft is not None else (1, 0)
         s.st = self.state.data_ptr()
         s.x = self.fab.xchg_args()
         self.args_sampler = s
@@ -131,7 +139,7 @@ class SpeculativeRound:
         t.st, t.ring, t.ring_size = self.state.data_ptr(), self.ring.dev, self.ring.size
         t.cancel, t.stop_ids, t.n_stop = self.ring.cancel_dev, self.stop_ids.data_ptr(), len(self.spec.stop_token_ids)
         t.counts, t.vbase, t.vlocal = None, self.vbase, self.vlocal
-        t.status, t.n_rows_q = self.fab.status.data_ptr(), 7
+        t.status, t.n_rows_q = self.fab.status.data_ptr(), s.n_rows_q
         t.host_consumed = self.ring.consumed_dev if self.device_chain else None     # pause consensus of the chain
         t.x = self.fab.xchg_args()
         self.args_tail = t
@@ -154,9 +162,6 @@ class SpeculativeRound:
     # ------------------------------------------------------------------ phases
     def phases(self) -> None:
         """Enqueue one round on the current stream."""
-        self.draft.ingest()
-        self.draft.block()
-        self.draft.propose()
         self.t.step()
         self.sample()
         K.tail_commit(self.args_tail, pdl=self.pdl)
@@ -172,10 +177,9 @@ class SpeculativeRound:
         K.sampler_run(self.args_sampler, domain=domain, pdl=self.pdl)
 
     def prefill_phases(self) -> None:
-        """One 8-row prompt replay step: target rows (no head) + draft ingest of their features."""
+        """One prompt replay step: the next rows of the prompt through the target, without its head."""
         K.prefill_cursor(self.prompt_dev, -1, self.t.rows, self.t.ctrl, self.t.tokens, pdl=self.pdl)
         self.t.step(head=False)
-        self.draft.ingest()
         K.epoch_advance(self.fab.epoch, pdl=self.pdl)
 
     def _capture(self, fn) -> torch.cuda.CUDAGraph:
@@ -255,7 +259,8 @@ class SpeculativeRound:
         """Capture the round graph; the warm-up run inside capture mutates session state, so
         the control block, the block ids and the feature rows of the last replay chunk are restored
         (KV rows it wrote lie at or beyond the anchor and are rewritten by round 0)."""
-        saved_ctrl, saved_ids, saved_feats = self.t.ctrl.clone(), self.block_ids.clone(), self.t.feats.clone()
+        saved_ctrl, saved_ids = self.t.ctrl.clone(), self.block_ids.clone()
+        saved_feats = None if self.draft is None else self.t.feats.clone()
         self.ring.cancel.value = 1                       # the warm-up round commits nothing
         before = K.LAUNCHES["count"]
         if self.device_chain:
@@ -268,7 +273,8 @@ class SpeculativeRound:
         self.ring.clear()
         self.t.ctrl.copy_(saved_ctrl)
         self.block_ids.copy_(saved_ids)
-        self.t.feats.copy_(saved_feats)                  # round 0 re-ingests the last replay chunk's features
+        if saved_feats is not None:
+            self.t.feats.copy_(saved_feats)              # round 0 re-ingests the last replay chunk's features
         self.fab.status.zero_()
         torch.cuda.synchronize()
 
@@ -342,3 +348,32 @@ class SpeculativeRound:
 
     def close(self) -> None:
         self.ring.close()
+
+
+class SpeculativeRound(DecodeRound):
+    """Rounds with a block draft: ingest, block, proposals, verify, sampler, tail."""
+
+    def __init__(self, spec: ModelSpec, target: TargetRuntime, draft_weights: dict, capacity: int, pdl: bool = True,
+                 device_chain: bool = False, ring_size: int = RING_SIZE):
+        if target.rows != spec.draft.rows:
+            raise RuntimeContractError("the verify runtime must run block_size + 1 rows")
+        self._draft_weights = draft_weights
+        super().__init__(spec, target, capacity, pdl=pdl, device_chain=device_chain, ring_size=ring_size)
+
+    def _make_draft(self, capacity: int) -> None:
+        self.draft = DraftRuntime(self.spec, self._draft_weights, self.t, capacity, self.seed, self.params, self.block_ids, pdl=self.pdl)
+        del self._draft_weights
+
+    def phases(self) -> None:
+        """Enqueue one round on the current stream."""
+        self.draft.ingest()
+        self.draft.block()
+        self.draft.propose()
+        super().phases()
+
+    def prefill_phases(self) -> None:
+        """One 8-row prompt replay step: target rows (no head) + draft ingest of their features."""
+        K.prefill_cursor(self.prompt_dev, -1, self.t.rows, self.t.ctrl, self.t.tokens, pdl=self.pdl)
+        self.t.step(head=False)
+        self.draft.ingest()
+        K.epoch_advance(self.fab.epoch, pdl=self.pdl)

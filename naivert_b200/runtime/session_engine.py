@@ -19,7 +19,7 @@ from typing import Dict, List, Optional, Sequence
 
 import torch
 
-from ..models.spec import FULL_DSA, SamplingParams
+from ..models.spec import SamplingParams
 from .engine import Engine
 from .prefix_store import PrefixStore, best_prefix_match, common_prefix, park_name, select_resume
 from .round import RuntimeContractError
@@ -153,7 +153,7 @@ class Session:
                 self.accepted.append(rec.accepted)
                 if rec.stop_reason is not None:
                     self.done, self.stop_reason = True, rec.stop_reason
-        if self._launched:
+        if self._launched and r.draft is not None:
             r.launch(1, force=True)                       # one more pass completes the draft context of the last rows
         r.stream.synchronize()
         eng.fabric.check()
@@ -175,14 +175,10 @@ class SessionEngine:
         self.tokenizer = tokenizer                       # optional: enables incremental tokenisation in align_prompt
         spec = engine.spec
         self.config = EngineConfig(engine.round.capacity, max_output_tokens, tuple(spec.stop_token_ids), spec.think_end_token_id)
-        full, rings = [], []
-        for d in engine.target.layers:
-            if d["kind"] == FULL_DSA:
-                full += [d["k"], d["v"], d["ik"], d["iks"]]
-            else:
-                rings += [d["k"], d["v"]]
-        for L in engine.round.draft.layers:
-            full += [L["k"], L["v"]]
+        full, rings = engine.target.cache_tensors()
+        if engine.round.draft is not None:
+            for L in engine.round.draft.layers:
+                full += [L["k"], L["v"]]
         self.store = PrefixStore(full, rings, int(store_gb * (1 << 30)), host=host_store)
         self.active: Optional[Session] = None
         self._sampled: Dict[str, List[int]] = {}
@@ -260,7 +256,8 @@ class SessionEngine:
                 log.info("no parked prefix resumes this prompt; closest is %s: %d of its %d parked tokens match, the prompt "
                          "departs at token %d", near[0], near[1], self.store.entries[near[0]].position, near[1])
         t1 = time.perf_counter()
-        path = prefill_path(n - 1 - start, self.resume_policy, native_ready=self.engine.prefill is not None)
+        policy = self.resume_policy if self.engine.spec.draft is not None or self.resume_policy == "replay" else "native"
+        path = prefill_path(n - 1 - start, policy, native_ready=self.engine.prefill is not None)
         prompt = torch.tensor(tokens, dtype=torch.int32)
         replay_from = start
         if path == "native":

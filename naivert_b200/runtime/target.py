@@ -498,6 +498,16 @@ class TargetRuntime:
         self.tokens[: t.numel()].copy_(t.to(self.dev))
         self.ctrl[0] = pos0
 
+    def cache_tensors(self):
+        """(position-indexed caches, sliding-window rings) for prefix parking."""
+        full, rings = [], []
+        for d in self.layers:
+            if d["kind"] == FULL_DSA:
+                full += [d["k"], d["v"], d["ik"], d["iks"]]
+            else:
+                rings += [d["k"], d["v"]]
+        return full, rings
+
     def kv_bytes(self) -> int:
         n = 0
         for d in self.layers:

@@ -105,7 +105,7 @@ def test_index_checking_build_records_the_first_bad_index_and_stays_clean_on_a_r
     from naivert_b200.ops import build as B
     lib = os.path.join(B.LIB_DIR, B.BOUNDS_LIB_NAME)
     man = os.path.join(B.LIB_DIR, "manifest_bounds.json")
-    if not (os.path.isfile(lib) and os.path.isfile(man) and json.load(open(man)).get("digest") == B.source_digest()):
+    if not (os.path.isfile(lib) and os.path.isfile(man) and json.load(open(man)).get("digest") == B.source_digest("main")):
         pytest.skip("the checking flavour is not built (python -m naivert_b200.ops.build --bounds)")
     env = dict(os.environ, NAIVERT_BOUNDS_CHECK="1")
     root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))

@@ -328,11 +328,11 @@ def test_status_words_are_explained():
     assert "sampler phase 2" in explain_status(0x800 | 0x42) and "Markov step 3" in explain_status(0x800 | 0x23)
     assert "fused MoE arrival" in explain_status(0x801) and "mailbox" in explain_status(0x501)
     assert "return slot 3" in explain_status(0x583) and "all-gather flag of source rank 2" in explain_status(0x562)
-    assert "unknown" in explain_status(0x999)
+    assert "unknown" in explain_status(0xB99)
     # the classes are the enumerators of the device header
     src = open(os.path.join(ROOT, "naivert_b200", "csrc", "ptx.cuh")).read()
     for name, value in (("kSiteTmaFull", 0x100), ("kSiteStageEmpty", 0x200), ("kSiteAccFull", 0x300), ("kSiteAccEmpty", 0x400),
-                        ("kSiteMailbox", 0x500), ("kSiteCluster", 0x600), ("kSiteRendezvous", 0x700), ("kSiteGrid", 0x800)):
+                        ("kSiteMailbox", 0x500), ("kSiteCluster", 0x600), ("kSiteRendezvous", 0x700), ("kSiteGrid", 0x800), ("kSiteState", 0x900)):
         assert f"{name} = 0x{value:x}" in src
 
 
