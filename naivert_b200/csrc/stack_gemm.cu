@@ -162,7 +162,8 @@ stack_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant
       const Item it = item_of(p, item, row_tiles, NTOK, na);
       if (!it.live) continue;
       const int buf = t & 1;
-      if (!mbar_wait(&tail->acc_full[buf], (t >> 1) & 1, p.status, kSiteAccFull | buf)) { ok = false; break; }
+      ok = __all_sync(0xffffffffu, mbar_wait(&tail->acc_full[buf], (t >> 1) & 1, p.status, kSiteAccFull | buf));
+      if (!ok) break;
       tc_fence_after();
       const int n = tile * kFeat + feat;
       const bool live = n < p.n;

@@ -174,7 +174,10 @@ __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs
     }
   };
 
-  if (!ROUTE && (int)blockIdx.x < tiles) fetch(blockIdx.x, lig);
+  // each CTA owns a contiguous run of tiles, so a per-group input is loaded once per group it meets
+  const int per_cta = (tiles + (int)gridDim.x - 1) / (int)gridDim.x;
+  const int tile_lo = (int)blockIdx.x * per_cta, tile_hi = min(tiles, tile_lo + per_cta);
+  if (!ROUTE && tile_lo < tile_hi) fetch(tile_lo, lig);
   griddep_wait();
   griddep_launch();
   const int pos = a.pos0 ? *reinterpret_cast<const volatile int*>(a.pos0) : 0;
@@ -200,7 +203,7 @@ __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs
       store_act(a.lat_cache, (long long)pos * a.lat_ld + c, __ldcg(a.lat_in + c) * rs * bf(a.lat_w + c), a.f32);
   }
   int cur = -1;
-  for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x) {
+  for (int tile = tile_lo; tile < tile_hi; ++tile) {
     const int g = tile / tiles_g;
     if (PER_GROUP && g != cur) {
       if (cur >= 0) __syncthreads();
@@ -212,7 +215,7 @@ __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs
     for (int i = 0; i < RU; ++i) acc[i] = acc2[i] = 0.f;
 #pragma unroll 1
     for (int c0 = lig; c0 < k8 || c0 == lig; c0 += G * U) {
-      if (c0 != lig || ROUTE || tile != (int)blockIdx.x) fetch(tile, c0);
+      if (c0 != lig || ROUTE || tile != tile_lo) fetch(tile, c0);
 #pragma unroll
       for (int q = 0; q < U; ++q) {
         const int c = c0 + q * G;
@@ -319,7 +322,7 @@ int launch_step(const StepArgs& a, const RouterArgs& r, int groups, int keep, cu
   const long long tiles = (long long)a.groups * ((a.n + rows_tile - 1) / rows_tile);
   const size_t smem = (size_t)k8 * 32;
   if (smem > kMaxStepSmem || tiles < 1 || tiles > 0x7fffffffLL) return -7;
-  const int cap = 148 * 4;
+  const int cap = PRO == kProMerge ? 148 * 2 : 148 * 4;
   return launch_pdl(kern, dim3((unsigned)(tiles < cap ? tiles : cap)), dim3(kStepThreads), smem, stream, pdl, a, r, groups, keep, G);
 }
 

@@ -29,6 +29,7 @@ TEPI_STORE, TEPI_CONV, TEPI_GATE, TEPI_GLU, TEPI_RECUR = 0, 1, 2, 3, 4
 ENTRIES = {"nrt_stack_gemm": ("StackGemmArgs", "nrt_stack_gemm_args_size"), "nrt_stack_gemm_f32": ("StackGemmArgs", "nrt_stack_gemm_args_size"),
            "nrt_stack_rows": ("StackRowArgs", "nrt_stack_row_args_size"), "nrt_latent_prep": ("LatentPrepArgs", "nrt_latent_prep_args_size"),
            "nrt_latent_attn_rows": ("LatentAttnArgs", "nrt_latent_attn_args_size"),
+           "nrt_latent_attn_tc": ("LatentAttnArgs", "nrt_latent_attn_args_size"),
            "nrt_latent_decode": ("LatentDecodeArgs", "nrt_latent_decode_args_size"),
            "nrt_stack_conv": ("RecurrenceArgs", "nrt_recurrence_args_size"), "nrt_stack_scan": ("RecurrenceArgs", "nrt_recurrence_args_size"),
            "nrt_moe_gather": ("MoeGatherArgs", "nrt_moe_gather_args_size"), "nrt_stack_step": ("StepArgs", "nrt_step_args_size"),
@@ -69,6 +70,11 @@ def token_map(t: torch.Tensor, k: int, zcount: int, zstride: int, rows: int, ld:
     return K.TensorMap(view, (k, zcount, rows), ((zstride if zcount > 1 else ld) * 2, ld * 2), (64, 1, box_rows), 1, library=lib())
 
 
+def value_map(v: torch.Tensor, keys: int, features: int, box: int) -> K.TensorMap:
+    """Feature-major values [features, keys] -> boxes of ``box`` features x 64 keys."""
+    return K.TensorMap(v, (keys, features), (keys * 2,), (64, box), 1, library=lib())
+
+
 def gemm(epi: int, ntok: int, w: K.TensorMap, w2: Optional[K.TensorMap], x: K.TensorMap, args: StackGemmArgs, items_fastest: bool) -> None:
     K.check(lib().nrt_stack_gemm(epi, ntok, C.byref(w.buf), C.byref(w2.buf) if w2 is not None else None, C.byref(x.buf),
                                  C.byref(args), int(items_fastest), _stream()), "stack gemm")
@@ -88,6 +94,10 @@ def latent_prep(args: LatentPrepArgs) -> None:
 
 def latent_attn_rows(args: LatentAttnArgs) -> None:
     K.check(lib().nrt_latent_attn_rows(C.byref(args), _stream()), "latent attention (rows)")
+
+
+def latent_attn_tc(q: K.TensorMap, k: K.TensorMap, v: K.TensorMap, args: LatentAttnArgs) -> None:
+    K.check(lib().nrt_latent_attn_tc(C.byref(q.buf), C.byref(k.buf), C.byref(v.buf), C.byref(args), _stream()), "latent attention (chunk)")
 
 
 def latent_decode(args: LatentDecodeArgs, pdl: bool) -> None:

@@ -76,7 +76,8 @@ class StackPrefill:
             self.ey = z(self.cap * s.hidden)
         self.head_rows = 256
         self.hw = torch.zeros(self.head_rows, self.h_ld, dtype=self.act, device=dev)
-        self.maps: Dict[tuple, K.TensorMap] = {}
+        self.tensor_cores = not self.f32              # attention of chunk rows on tcgen05 (else the plain kernel)
+        self.maps: Dict[tuple, object] = {}
         self.phases: dict = {}
 
     @staticmethod
@@ -136,6 +137,13 @@ class StackPrefill:
         wbytes = w.nbytes * (2 if dual else 1)
         S.gemm(epi, ntok, self._wmap(w), self._wmap(w2) if dual else None, xm, a, items is None and wbytes > (96 << 20))
 
+    def _attn_maps(self, heads: int, dp: int, vp: int) -> Tuple[K.TensorMap, ...]:
+        key = ("attn", heads, dp, vp)
+        if key not in self.maps:
+            self.maps[key] = (S.token_map(self.q, dp, heads, dp, self.C, heads * dp, 128), S.token_map(self.kx, dp, heads, dp, self.kv_block, heads * dp, 64),
+                              S.value_map(self.vx, self.kv_block, heads * vp, pad(vp, 16)))
+        return self.maps[key]
+
     # ------------------------------------------------------------------ one chunk
     def _rows(self, R: int, *, embed: bool = False, y: Optional[torch.Tensor] = None, post=None, moe=None, add=None, pre=None) -> None:
         s, a = self.spec, S.StackRowArgs()
@@ -177,10 +185,15 @@ class StackPrefill:
             off = kv0 * cache.shape[1]
             kw = dict(x_off=off, x_rows=t.capacity - kv0)
             self._gemm(S.EPI_STORE, d["uk"], cache, cache.shape[1], n, self.kx, hq, **kw)
-            self._gemm(S.EPI_STORE, d["uv"], cache, cache.shape[1], n, self.vx, hv, **kw)
-            a.v_ld = hv
             a.kv0, a.kv_rows, a.first, a.last = kv0, n, int(kv0 == 0), int(kv0 + n == total)
-            S.latent_attn_rows(a)
+            if self.tensor_cores and max(dp, vp) <= 256:
+                a.v_ld = self.kv_block                 # values feature-major: the K-major operand of P V
+                self._gemm(S.EPI_TRANSPOSE, d["uv"], cache, cache.shape[1], n, self.vx, self.kv_block, **kw)
+                S.latent_attn_tc(*self._attn_maps(m.heads, dp, vp), a)
+            else:
+                a.v_ld = hv
+                self._gemm(S.EPI_STORE, d["uv"], cache, cache.shape[1], n, self.vx, hv, **kw)
+                S.latent_attn_rows(a)
         self._gemm(S.EPI_STORE, d["o"], self.o, hv, R, self.y, self.spec.hidden)
 
     def _recurrence(self, r: dict, R: int) -> None:
