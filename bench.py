@@ -120,6 +120,17 @@ class ClockSampler(threading.Thread):
                 "reasons": sorted(reasons), "samples": len(self.samples)}
 
 
+def stack_workload(a) -> int:
+    if a.gpus != 1:
+        raise SystemExit("layer-stack models run on one GPU")
+    import torch
+    from naivert_b200.runtime.stack_bench import run
+    torch.cuda.set_device(0)
+    model = a.model if a.model != "naive-n0.5" else "tumatar-bench"
+    print(json.dumps(run(model, a.prompt, a.steps, a.warmup, a.prefill_chunk or 2048, a.kernels, layers=a.layers, clocks=ClockSampler(0))))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -141,10 +152,15 @@ def main() -> int:
     ap.add_argument("--no-check", action="store_true", help="skip the small-geometry correctness self-check (outside the timed region)")
     ap.add_argument("--prefill-chunk", type=int, default=2048,
                     help="rows per chunk of the native prompt ingestion (0: eight-row replay only); outside the timed rounds")
+    ap.add_argument("--workload", choices=("speculative", "stack"), default="speculative",
+                    help="stack: prefill and decode of a layer-stack model (--model, default tumatar-bench) on one GPU")
+    ap.add_argument("--kernels", action="store_true", help="stack workload: add per-kernel tables")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_arm(a)
     a.warmup = max(3, a.warmup)
+    if a.workload == "stack":
+        return stack_workload(a)
 
     import torch
     import torch.distributed as dist

@@ -173,11 +173,11 @@ def small_spec() -> StackSpec:
                      norm_eps=1e-6, embed_scale=18.0, logit_scale=0.5, loop=LoopSpec(1, 3, 2)).validate()
 
 
-def bench_spec(layers: int = 8, experts: bool = True) -> StackSpec:
+def bench_spec(layers: int = 6, experts: bool = True) -> StackSpec:
     """Layers of a real model's size (random weights): alternating recurrence and latent attention at width 4096."""
     attn = LatentAttentionSpec(heads=64, dim=128, vdim=128, kv_rank=512, q_rank=1536, scale=128 ** -0.5)
     rec = GatedRecurrenceSpec(width=4096, blocks=16, taps=4)
-    moe = ExpertsSpec(MoeRoutingSpec(expert_count=128, top_k=8, intermediate=2048, normalize_top_k=False, group_count=8, limited_group_count=4))
+    moe = ExpertsSpec(MoeRoutingSpec(expert_count=256, top_k=8, intermediate=2048, normalize_top_k=False, group_count=8, limited_group_count=4))
     dense = ClampedGluSpec(ff=16384, limit=7.0)
     body: List[LayerSpec] = []
     for i in range(layers):

@@ -13,6 +13,7 @@ the step continues from.
 """
 from __future__ import annotations
 
+from contextlib import contextmanager
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
@@ -79,6 +80,26 @@ class StackPrefill:
         self.tensor_cores = not self.f32              # attention of chunk rows on tcgen05 (else the plain kernel)
         self.maps: Dict[tuple, object] = {}
         self.phases: dict = {}
+        self.profile = False                          # per-stage CUDA-event timing (adds an event pair per stage)
+        self._timed: Dict[str, list] = {}
+
+    @contextmanager
+    def _stage(self, name: str):
+        if not self.profile:
+            yield
+            return
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        yield
+        b.record()
+        self._timed.setdefault(name, []).append((a, b))
+
+    def stage_ms(self) -> Dict[str, Tuple[float, int]]:
+        """(device milliseconds, calls) per stage since the last call (``profile`` must be on); waits for the stream."""
+        torch.cuda.current_stream().synchronize()
+        out = {k: (sum(a.elapsed_time(b) for a, b in v), len(v)) for k, v in self._timed.items()}
+        self._timed = {}
+        return out
 
     @staticmethod
     def _item_rows(rows: int, routing, f32: bool = False) -> int:
@@ -157,22 +178,26 @@ class StackPrefill:
         a.x, a.width, a.rows, a.eps = self.x.data_ptr(), s.hidden, R, s.norm_eps
         a.pre_w = None if pre is None else pre.data_ptr()
         a.h, a.h_f32, a.h_ld = self.h.data_ptr(), int(self.f32), self.h_ld
-        S.rows(a)
+        with self._stage("rows"):
+            S.rows(a)
 
     def _attention(self, r: dict, R: int, pos0: int) -> None:
         d, t = r["layer"], self.t
         m, dp, vp = d["spec"].mixer, d["dp"], d["vp"]
         n_in, qp = d["in"].n, pad(m.q_rank, 8)
-        self._gemm(S.EPI_STORE, d["in"], self.h, self.h_ld, R, self.proj, n_in)
+        with self._stage("attn_in"):
+            self._gemm(S.EPI_STORE, d["in"], self.h, self.h_ld, R, self.proj, n_in)
         p = S.LatentPrepArgs()
         p.proj, p.ld, p.rows, p.q_rank, p.kv_rank = self.proj.data_ptr(), n_in, R, m.q_rank, m.kv_rank
         p.q_w, p.kv_w, p.eps = d["dq_norm"].data_ptr(), d["dkv_norm"].data_ptr(), self.spec.norm_eps
         cache = r["cache"]
         p.cq, p.cq_ld, p.cache, p.cache_ld = self.cq.data_ptr(), qp, cache.data_ptr(), cache.shape[1]
         p.f32, p.pos0, p.capacity = int(self.f32), self.pos.data_ptr(), t.capacity
-        S.latent_prep(p)
+        with self._stage("latent_prep"):
+            S.latent_prep(p)
         hq, hv = m.heads * dp, m.heads * vp
-        self._gemm(S.EPI_STORE, d["uq"], self.cq, qp, R, self.q, hq)
+        with self._stage("queries"):
+            self._gemm(S.EPI_STORE, d["uq"], self.cq, qp, R, self.q, hq)
         a = S.LatentAttnArgs()
         a.q, a.k, a.v, a.out, a.f32 = self.q.data_ptr(), self.kx.data_ptr(), self.vx.data_ptr(), self.o.data_ptr(), int(self.f32)
         a.gate, a.gate_ld = self.proj.data_ptr() + 4 * (m.q_rank + m.kv_rank), n_in
@@ -184,23 +209,29 @@ class StackPrefill:
             n = min(self.kv_block, total - kv0)
             off = kv0 * cache.shape[1]
             kw = dict(x_off=off, x_rows=t.capacity - kv0)
-            self._gemm(S.EPI_STORE, d["uk"], cache, cache.shape[1], n, self.kx, hq, **kw)
+            with self._stage("expand_k"):
+                self._gemm(S.EPI_STORE, d["uk"], cache, cache.shape[1], n, self.kx, hq, **kw)
             a.kv0, a.kv_rows, a.first, a.last = kv0, n, int(kv0 == 0), int(kv0 + n == total)
             if self.tensor_cores and max(dp, vp) <= 256:
                 a.v_ld = self.kv_block                 # values feature-major: the K-major operand of P V
-                self._gemm(S.EPI_TRANSPOSE, d["uv"], cache, cache.shape[1], n, self.vx, self.kv_block, **kw)
-                S.latent_attn_tc(*self._attn_maps(m.heads, dp, vp), a)
+                with self._stage("expand_v"):
+                    self._gemm(S.EPI_TRANSPOSE, d["uv"], cache, cache.shape[1], n, self.vx, self.kv_block, **kw)
+                with self._stage("attention"):
+                    S.latent_attn_tc(*self._attn_maps(m.heads, dp, vp), a)
             else:
                 a.v_ld = hv
                 self._gemm(S.EPI_STORE, d["uv"], cache, cache.shape[1], n, self.vx, hv, **kw)
-                S.latent_attn_rows(a)
-        self._gemm(S.EPI_STORE, d["o"], self.o, hv, R, self.y, self.spec.hidden)
+                with self._stage("attention_plain"):
+                    S.latent_attn_rows(a)
+        with self._stage("attn_out"):
+            self._gemm(S.EPI_STORE, d["o"], self.o, hv, R, self.y, self.spec.hidden)
 
     def _recurrence(self, r: dict, R: int) -> None:
         d = r["layer"]
         m = d["spec"].mixer
         bp, wp = pad(m.block, 8), pad(m.width, 8)
-        self._gemm(S.EPI_BIAS, d["in"], self.h, self.h_ld, R, self.xy, 2 * m.width, bias=d["in_b"], act_cols=m.width)
+        with self._stage("rec_in"):
+            self._gemm(S.EPI_BIAS, d["in"], self.h, self.h_ld, R, self.xy, 2 * m.width, bias=d["in_b"], act_cols=m.width)
         a = S.RecurrenceArgs()
         a.xy, a.xy_ld, a.conv, a.conv_b, a.taps = self.xy.data_ptr(), 2 * m.width, d["conv"].data_ptr(), d["conv_b"].data_ptr(), m.taps
         a.history, a.hist_rows, a.u = r["history"].data_ptr(), m.hist_rows, self.u.data_ptr()
@@ -209,27 +240,35 @@ class StackPrefill:
         a.out, a.out_ld, a.f32, a.rows = self.o.data_ptr(), wp, int(self.f32), R
         a.width, a.blocks, a.block, a.block_pad = m.width, m.blocks, m.block, bp
         a.pos0, a.status = self.pos.data_ptr(), self.t.fab.status.data_ptr()
-        S.conv(a)
-        self._gemm(S.EPI_BIAS, d["gates"], self.u, m.blocks * bp, R, self.gates, 2 * m.width, z=m.blocks, x_z=bp, out_z=2 * m.block,
-                   bias=d["gates_b"])
-        S.scan(a)
-        self._gemm(S.EPI_STORE, d["o"], self.o, wp, R, self.y, self.spec.hidden)
+        with self._stage("conv"):
+            S.conv(a)
+        with self._stage("rec_gates"):
+            self._gemm(S.EPI_BIAS, d["gates"], self.u, m.blocks * bp, R, self.gates, 2 * m.width, z=m.blocks, x_z=bp, out_z=2 * m.block,
+                       bias=d["gates_b"])
+        with self._stage("scan"):
+            S.scan(a)
+        with self._stage("rec_out"):
+            self._gemm(S.EPI_STORE, d["o"], self.o, wp, R, self.y, self.spec.hidden)
 
     def _feed_forward(self, d: dict, R: int) -> torch.Tensor:
         """Returns the buffer that holds the result rows (sorted by expert for routed layers)."""
         f, W = d["spec"].mlp, self.spec.hidden
         fp = pad(f.ff, 8)
         if f.kind == "dense":
-            self._gemm(S.EPI_CLAMPED_GLU, d["gate"], self.h, self.h_ld, R, self.ff, fp, w2=d["up"], limit=f.limit, alpha=f.alpha)
-            self._gemm(S.EPI_STORE, d["down"], self.ff, fp, R, self.y, W)
+            with self._stage("dense_gate_up"):
+                self._gemm(S.EPI_CLAMPED_GLU, d["gate"], self.h, self.h_ld, R, self.ff, fp, w2=d["up"], limit=f.limit, alpha=f.alpha)
+            with self._stage("dense_down"):
+                self._gemm(S.EPI_STORE, d["down"], self.ff, fp, R, self.y, W)
             return self.y
         rt = f.routing
-        self._gemm(S.EPI_STORE, d["router"], self.h, self.h_ld, R, self.scores, rt.expert_count)
+        with self._stage("router"):
+            self._gemm(S.EPI_STORE, d["router"], self.h, self.h_ld, R, self.scores, rt.expert_count)
         q = K.RouterArgs()
         q.bias, q.hidden, q.experts, q.rows, q.top_k = d["correction"].data_ptr(), W, rt.expert_count, R, rt.top_k
         q.sigmoid, q.normalize, q.route_scale = 1, int(rt.normalize_top_k), rt.route_scale
         q.scores, q.topk_ids, q.topk_p = self.scores.data_ptr(), self.ids.data_ptr(), self.probs.data_ptr()
-        S.route(q, rt.group_count, rt.limited_group_count)
+        with self._stage("choice"):
+            S.route(q, rt.group_count, rt.limited_group_count)
         ir = self._item_rows(R, rt, self.f32)
         items = self._items(R, rt, ir)
         e = K.EpArgs()
@@ -238,15 +277,19 @@ class StackPrefill:
         e.slot_of, e.n_items, e.item_expert, e.item_row = (self.slot_of.data_ptr(), self.n_items.data_ptr(), self.item_z.data_ptr(),
                                                            self.item_row.data_ptr())
         e.seg_rows, e.max_items, e.item_rows, e.x_args = self.seg_rows.data_ptr(), items, ir, self.t.fab.xchg_args()
-        S.moe_count(e)
+        with self._stage("expert_count"):
+            S.moe_count(e)
         g = S.MoeGatherArgs()
         eb = self.h.element_size()
         g.h, g.h_ld, g.sorted, g.slot_of = self.h.data_ptr(), self.h_ld * eb, self.sorted.data_ptr(), self.slot_of.data_ptr()
         g.rows, g.top_k, g.row_bytes, g.cap = R, rt.top_k, self.h_ld * eb, self.cap
-        S.moe_gather(g)
+        with self._stage("expert_gather"):
+            S.moe_gather(g)
         seg = dict(items=(ir, items))
-        self._gemm(S.EPI_SILU_GLU, d["gate"], self.sorted, self.h_ld, ir, self.ea, fp, w2=d["up"], x_rows=self.cap, **seg)
-        self._gemm(S.EPI_STORE, d["down"], self.ea, fp, ir, self.ey, W, x_rows=self.cap, **seg)
+        with self._stage("expert_gate_up"):
+            self._gemm(S.EPI_SILU_GLU, d["gate"], self.sorted, self.h_ld, ir, self.ea, fp, w2=d["up"], x_rows=self.cap, **seg)
+        with self._stage("expert_down"):
+            self._gemm(S.EPI_STORE, d["down"], self.ea, fp, ir, self.ey, W, x_rows=self.cap, **seg)
         return self.ey
 
     def _chunk(self, pos0: int, R: int, want: Sequence[int] = (), trace: Optional[list] = None) -> Optional[torch.Tensor]:

@@ -1,0 +1,219 @@
+"""Throughput of layer-stack models at the sizes of a real model's layers (random weights on the device).
+
+    python bench.py --workload stack [--model tumatar-bench|tumatar-bench-dense] [--prompt 8192] [--steps 64] [--kernels]
+
+Prefill: one prompt through the chunk path, CUDA events around the run.  Decode: rounds of the captured graph behind that
+prompt (step + sampler + tail), CUDA events around K replays.  ``--kernels`` adds tables with one row per kernel kind: time,
+the bytes it must move or the FLOPs it must do, and the fraction of the copy bandwidth / dense bf16 rate that is.  Weights of one
+token or chunk exceed the 126 MB L2, so no flush is needed between iterations.
+"""
+from __future__ import annotations
+
+import json
+import os
+from typing import Dict, List, Tuple
+
+import torch
+
+from ..models.registry import resolve_model
+from ..models.spec import SamplingParams
+from .engine import Engine
+
+FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
+
+
+def peaks() -> dict:
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
+    if os.path.isfile(path):
+        d = json.load(open(path))
+        return {"hbm_gbs": float(d["hbm_gbs"]), "bf16_tflops": float(d["bf16_tflops"]), "source": "measured"}
+    return FALLBACK_PEAKS
+
+
+# --------------------------------------------------------------------------- work per kernel kind
+def chunk_work(eng, pos0: int, R: int) -> Dict[str, Tuple[float, float]]:
+    """stage -> (FLOPs, bytes) over all runs of one chunk at ``pos0``; bytes are the operands once."""
+    spec, pf = eng.spec, eng.prefill
+    W, es = spec.hidden, 4 if eng.target.f32 else 2
+    out: Dict[str, List[float]] = {}
+
+    def add(name: str, flops: float, nbytes: float) -> None:
+        a = out.setdefault(name, [0.0, 0.0])
+        a[0] += flops
+        a[1] += nbytes
+
+    def gemm(name: str, n: int, k: int, rows: int, out_bytes: int, z: int = 1, mats: int = 1) -> None:
+        add(name, 2.0 * n * k * rows * z * mats, z * (mats * n * k * 2 + rows * k * es + rows * n * out_bytes))
+
+    ctx = pos0 + R
+    for r in eng.target.runs:
+        d = r["layer"]
+        m, f = d["spec"].mixer, d["spec"].mlp
+        add("rows", 0, R * W * (4 + 4 + 4 + es))
+        if m.kind == "latent_attention":
+            hq, hv = m.heads * d["dp"], m.heads * d["vp"]
+            gemm("attn_in", d["in"].n, W, R, 4)
+            add("latent_prep", 0, R * (m.q_rank + m.kv_rank) * (4 + es))
+            gemm("queries", hq, m.q_rank, R, es)
+            gemm("expand_k", hq, m.kv_rank, ctx, es)
+            gemm("expand_v", hv, m.kv_rank, ctx, es)
+            pairs = R * pos0 + R * (R + 1) / 2
+            add("attention", 2.0 * pairs * (hq + hv), R * (hq + 2 * hv) * es + ctx * (hq + hv) * es)
+            gemm("attn_out", W, hv, R, 4)
+        else:
+            gemm("rec_in", 2 * m.width, W, R, es)
+            add("conv", 0, R * m.width * 2 * es)
+            gemm("rec_gates", 2 * m.block, m.block, R, 4, z=m.blocks)
+            add("scan", 0, R * m.width * (2 * 8 + 2 * es + es + es))
+            gemm("rec_out", W, m.width, R, 4)
+        if f is None:
+            continue
+        add("rows", 0, R * W * (4 + 4 + 4 + es))
+        if f.kind == "dense":
+            gemm("dense_gate_up", f.ff, W, R, es, mats=2)
+            gemm("dense_down", W, f.ff, R, 4)
+        else:
+            rt = f.routing
+            P = R * rt.top_k
+            used = min(rt.expert_count, P)
+            gemm("router", rt.expert_count, W, R, 4)
+            add("choice", 0, R * rt.expert_count * 4)
+            add("expert_count", 0, P * 8)
+            add("expert_gather", 0, 2 * P * W * es)
+            add("expert_gate_up", 4.0 * P * W * f.ff, used * 2 * W * f.ff * 2 + P * (W + f.ff) * es)
+            add("expert_down", 2.0 * P * W * f.ff, used * W * f.ff * 2 + P * (f.ff * es + W * 4))
+    return {k: (v[0], v[1]) for k, v in out.items()}
+
+
+def step_work(eng, pos: int) -> List[Tuple[str, float]]:
+    """(kind, bytes that must be read) of every launch of the step, in launch order."""
+    out = []
+    t = eng.target
+    for r in t.runs:
+        d = r["layer"]
+        m, f = d["spec"].mixer, d["spec"].mlp
+        if m.kind == "latent_attention":
+            out += [("attn_in", d["in"].nbytes), ("queries", d["uq"].nbytes), ("latent_query", d["uk_t"].nbytes),
+                    ("attention", (pos + 1) * m.kv_rank * (4 if t.f32 else 2)), ("values", d["uv"].nbytes), ("attn_out", d["o"].nbytes)]
+        else:
+            out += [("rec_in", d["in"].nbytes), ("rec_gates", d["gates"].nbytes), ("rec_out", d["o"].nbytes)]
+        if f is None:
+            continue
+        if f.kind == "dense":
+            out += [("dense_gate_up", 2 * d["gate"].nbytes), ("dense_down", d["down"].nbytes)]
+        else:
+            per = d["gate"].n * d["gate"].ld * 2
+            k = f.routing.top_k
+            out += [("router", d["router"].nbytes), ("expert_gate_up", 2 * k * per), ("expert_down", k * d["down"].n * d["down"].ld * 2)]
+    return out + [("head", t.head.nbytes)]
+
+
+# --------------------------------------------------------------------------- measurements
+def chunk_table(eng, prompt: torch.Tensor, pos0: int, R: int) -> List[dict]:
+    pf, pk = eng.prefill, peaks()
+    pf.extend(prompt[pos0:pos0 + R], pos0)
+    pf.profile = True
+    reps = 3
+    for _ in range(reps):
+        pf.extend(prompt[pos0:pos0 + R], pos0)          # recurrent layers restart from the slot tagged pos0
+    ms = pf.stage_ms()
+    pf.profile = False
+    work = chunk_work(eng, pos0, R)
+    rows = []
+    for name, (total, calls) in sorted(ms.items(), key=lambda kv: -kv[1][0]):
+        t = total / reps * 1e-3
+        fl, by = work.get(name, (0.0, 0.0))
+        bound = max(fl / (pk["bf16_tflops"] * 1e12), by / (pk["hbm_gbs"] * 1e9))
+        rows.append({"kernel": name, "calls": calls // reps, "ms": round(t * 1e3, 3), "tflops": round(fl / t * 1e-12, 1),
+                     "gbs": round(by / t * 1e-9, 1), "roofline": round(bound / t, 3)})
+    return rows
+
+
+def step_table(eng, pos: int, steps: int = 4) -> List[dict]:
+    """Kernel times of the step without programmatic overlap (CUPTI records), matched to the launch list in order."""
+    from torch.profiler import ProfilerActivity, profile
+    t, pk = eng.target, peaks()
+    pdl, t.pdl = t.pdl, False
+    t.set_inputs([1], pos)
+    t.step()
+    torch.cuda.synchronize()
+    with profile(activities=[ProfilerActivity.CUDA]) as prof:
+        for _ in range(steps):
+            t.step()
+        torch.cuda.synchronize()
+    t.pdl = pdl
+    ev = sorted((e for e in prof.events() if "stack_" in e.name or "latent_" in e.name), key=lambda e: e.time_range.start)
+    work = step_work(eng, pos)
+    if len(ev) != steps * len(work):
+        raise RuntimeError(f"{len(ev)} kernel records for {steps} x {len(work)} launches")
+    agg: Dict[str, List[float]] = {}
+    for i, e in enumerate(ev):
+        name, nbytes = work[i % len(work)]
+        a = agg.setdefault(name, [0.0, 0.0, 0])
+        a[0] += e.device_time if hasattr(e, "device_time") else e.cuda_time
+        a[1] += nbytes
+        a[2] += 1
+    return [{"kernel": k, "calls": v[2] // steps, "us_each": round(v[0] / v[2], 2), "mb_each": round(v[1] / v[2] / 1e6, 2),
+             "gbs": round(v[1] / v[0] * 1e-3, 1), "roofline": round(v[1] / v[0] * 1e-3 / pk["hbm_gbs"], 3)}
+            for k, v in sorted(agg.items(), key=lambda kv: -kv[1][0])]
+
+
+def run(model: str, prompt_len: int, steps: int, warmup: int, chunk: int, kernels: bool, layers: int = 0, clocks=None) -> dict:
+    spec = resolve_model(model)
+    if layers:
+        spec = spec.with_layers(layers)
+    dev = torch.device("cuda", torch.cuda.current_device())
+    capacity = prompt_len + steps + warmup + 128
+    eng = Engine.build(spec, capacity=capacity, device=dev, prefill_chunk=chunk)
+    try:
+        g = torch.Generator().manual_seed(0)
+        prompt = torch.randint(0, spec.vocab, (prompt_len,), generator=g, dtype=torch.int32).pin_memory()
+        eng.prefill.warm_chunks([chunk])
+        eng.prefill.run(prompt, 0, prompt_len - 1)
+        torch.cuda.synchronize()
+        pre = []
+        for _ in range(3):
+            eng.prefill.run(prompt, 0, prompt_len - 1)
+            pre.append(eng.prefill.executor_ms())
+        pre_ms = sorted(pre)[1]
+        sp = SamplingParams(temperature=1.0, top_p=1e-6, seed=1)
+        eng.open(prompt, steps + warmup + 8, sp)
+        r = eng.round
+        r.stop_ids.fill_(-1)
+        r.launch(warmup)
+        torch.cuda.synchronize()
+        if clocks is not None:
+            clocks.start()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        with torch.cuda.stream(r.stream):
+            a.record()
+        r.launch(steps)
+        with torch.cuda.stream(r.stream):
+            b.record()
+        torch.cuda.synchronize()
+        if clocks is not None:
+            clocks.stop_flag.set()
+            clocks.join()
+        dec_ms = a.elapsed_time(b) / steps
+        eng.fabric.check()
+        read = sum(n for _, n in step_work(eng, prompt_len))
+        out = {"metric": "layer-stack decode tokens/s (one sequence)", "value": round(1e3 / dec_ms, 2), "unit": "tokens/s", "n_gpus": 1,
+               "steps": steps, "warmup": warmup, "ms_per_step": round(dec_ms, 4), "higher_is_better": True, "dtype": "bf16",
+               "data": "synthetic: random weights drawn on the device, uniform random prompt ids",
+               "decode_bytes_per_token": int(read), "decode_roofline": round(read / (dec_ms * 1e-3) * 1e-9 / peaks()["hbm_gbs"], 3),
+               "prefill": {"tokens_per_s": round((prompt_len - 1) / (pre_ms * 1e-3), 1), "ms": round(pre_ms, 3), "chunk": chunk},
+               "config": {"model": spec.name, "layers": spec.layer_count, "hidden": spec.hidden, "seq_len": prompt_len, "global_batch": 1,
+                          "kernels_per_round": r.kernels_per_round, "l2": "weights of a step exceed the 126 MB L2"},
+               "peaks": peaks(), "gpu_launches": int(r.kernels_per_round * steps)}
+        if clocks is not None:
+            out["clocks"] = clocks.summary()
+        if kernels:
+            n0 = min(prompt_len // 2, prompt_len - 1 - chunk) if prompt_len > chunk else 0
+            eng.prefill.run(prompt, 0, n0) if n0 else None
+            out["chunk_kernels"] = {"pos0": n0, "rows": chunk, "table": chunk_table(eng, prompt, n0, min(chunk, prompt_len - n0))}
+            eng.prefill.run(prompt, 0, prompt_len - 1)
+            out["step_kernels"] = {"pos": prompt_len - 1, "table": step_table(eng, prompt_len - 1)}
+        eng.fabric.check()
+        return out
+    finally:
+        eng.close()
