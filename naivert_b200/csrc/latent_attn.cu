@@ -335,7 +335,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
   const int h = blockIdx.x, sp_i = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = *a.pos0 + 1;
-  const int per = ((n + a.splits - 1) / a.splits + kDecTile - 1) / kDecTile * kDecTile;
+  const int per = latent_split_rows(n, a.splits);
   const int j_lo = min(n, sp_i * per), j_hi = min(n, j_lo + per);
   float* q = sh;
   float* o = sh + a.rank;
@@ -374,15 +374,15 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
     }
     __syncthreads();
   }
-  float* out = a.part + ((size_t)sp_i * a.heads + h) * (a.rank + 2);
+  float* out = a.part + ((size_t)sp_i * a.heads + h) * latent_part_row(a.rank);
   if (threadIdx.x == 0) { out[0] = m; out[1] = l; }
-  for (int c = threadIdx.x; c < a.rank; c += 256) out[2 + c] = o[c];
+  for (int c = threadIdx.x; c < a.rank; c += 256) out[4 + c] = o[c];
 }
 
 // ------------------------------------------------------------------------------------ one-token step, tensor-core form
-// grid (head tiles, splits).  Up to 64 heads of a CTA share every cached latent: the heads are the M side of bf16 m16n8k16
+// grid (head tiles, splits).  Up to 32 heads of a CTA share every cached latent: the heads are the M side of bf16 m16n8k16
 // MMAs, the latents (64 per tile, two cp.async stages) serve as keys and, through ldmatrix.trans, as values.  tcgen05 is not
-// used: the kernel streams the cache once, and with 64 live query rows at most half of its M = 128 would work.
+// used: the kernel streams the cache once, and with at most 64 or so live query rows half of its M = 128 would idle.
 __device__ __forceinline__ void cp16(void* dst, const void* src, bool valid) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
 }
@@ -421,11 +421,10 @@ __global__ void __launch_bounds__(256, 1) latent_decode_tc_kernel(const LatentDe
   float* scorr = sl + HT;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int h0 = blockIdx.x * HT;
-  // the position and the rows of earlier steps do not depend on the predecessor; the row it appends does
-  griddep_wait();
-  griddep_launch();
+  // The position and the cache rows (the newest was appended two launches back) do not depend on the predecessor: the first
+  // tile is requested before the wait for it.
   const int n = *reinterpret_cast<const volatile int*>(a.pos0) + 1;
-  const int per = ((n + a.splits - 1) / a.splits + kDecTile - 1) / kDecTile * kDecTile;
+  const int per = latent_split_rows(n, a.splits);
   const int j_lo = min(n, (int)blockIdx.y * per), j_hi = min(n, j_lo + per);
   const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(a.cache);
   const int pieces = rp / 8;
@@ -438,6 +437,18 @@ __global__ void __launch_bounds__(256, 1) latent_decode_tc_kernel(const LatentDe
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (j_lo < j_hi) request(j_lo, 0);
+  griddep_wait();
+  griddep_launch();
+  if (j_lo >= j_hi) return;                           // an unused split: nobody reads its partial
+  if (a.rank % 4 == 0) {
+#pragma unroll 4
+    for (int i = tid; i < HT * rp / 4; i += 256) {
+      const int t = i / (rp / 4), c = (i - t * (rp / 4)) * 4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (h0 + t < a.heads && c < a.rank) v = __ldcg(reinterpret_cast<const float4*>(a.q + (size_t)(h0 + t) * a.rank + c));
+      *reinterpret_cast<uint2*>(sq + t * pitch + c) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+    }
+  } else
   for (int i = tid; i < HT * rp; i += 256) {
     const int t = i / rp, c = i - t * rp;
     const float v = h0 + t < a.heads && c < a.rank ? __ldcg(a.q + (size_t)(h0 + t) * a.rank + c) : 0.f;
@@ -535,13 +546,13 @@ __global__ void __launch_bounds__(256, 1) latent_decode_tc_kernel(const LatentDe
     for (int half = 0; half < 2; ++half) {
       const int t = i * 16 + fr + 8 * half;
       if (h0 + t >= a.heads) continue;
-      float* out = a.part + ((size_t)blockIdx.y * a.heads + h0 + t) * (a.rank + 2);
+      float* out = a.part + ((size_t)blockIdx.y * a.heads + h0 + t) * latent_part_row(a.rank);
       if (warp == 0 && (lane & 3) == 0) { out[0] = sm[t]; out[1] = sl[t]; }
 #pragma unroll
       for (int q = 0; q < kNT; ++q) {
         const int c = (warp + 8 * q) * 8 + fc;
-        if (c < a.rank) out[2 + c] = o[i][q][2 * half];
-        if (c + 1 < a.rank) out[2 + c + 1] = o[i][q][2 * half + 1];
+        if (c < a.rank) out[4 + c] = o[i][q][2 * half];
+        if (c + 1 < a.rank) out[4 + c + 1] = o[i][q][2 * half + 1];
       }
     }
 }
@@ -593,13 +604,12 @@ extern "C" int nrt_latent_attn_tc(const void* tmQ, const void* tmK, const void* 
 extern "C" int nrt_latent_decode(const void* args, void* stream, int pdl) {
   LatentDecodeArgs a;
   memcpy(&a, args, sizeof(a));
-  if (!a.f32 && a.rank >= 1 && a.rank <= kMaxDecRank && a.splits >= 1 && a.cache_ld >= (a.rank + 15) / 16 * 16) {
+  if (!a.f32 && a.rank >= 1 && a.rank <= kMaxDecRank && a.splits >= 1 && a.splits <= kMaxSplits && a.cache_ld >= (a.rank + 15) / 16 * 16) {
     cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
     if (a.heads <= 16) return launch_decode_tc<1>(a, s, pdl != 0);
-    if (a.heads <= 32) return launch_decode_tc<2>(a, s, pdl != 0);
-    return launch_decode_tc<4>(a, s, pdl != 0);
+    return launch_decode_tc<2>(a, s, pdl != 0);
   }
   const size_t smem = (size_t)a.rank * 8;
-  if (a.rank < 1 || a.splits < 1 || smem > 48 * 1024) return -3;
+  if (a.rank < 1 || a.splits < 1 || a.splits > kMaxSplits || smem > 48 * 1024) return -3;
   return launch_pdl(latent_decode_kernel, dim3(a.heads, a.splits), dim3(256), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
 }

@@ -109,7 +109,7 @@ struct LatentDecodeArgs {
   int heads, rank;
   float scale;
   const int* pos0;
-  float* part;                  // [splits][heads][rank + 2]: max, sum, unnormalised latent output
+  float* part;                  // [splits][heads][latent_part_row(rank)]: max, sum, -, -, unnormalised latent output
   int splits;
 };
 
@@ -125,7 +125,8 @@ struct RecurrenceArgs {
   int hist_rows;
   void* u;                      // [rows][blocks][block_pad]
   // recurrence
-  const float* gates;           // [rows][blocks][2 * block]: pre-activation r | i of every block
+  const float* gates;           // [rows][blocks][2 * block]: pre-activation r | i of every block (scratch: the scan
+                                // replaces them by decay and drive)
   const float* softplus_lam;    // [width]
   float decay;                  // log a = -decay * r * softplus(lam)
   float* state;                 // [2][width] state after a position
@@ -229,6 +230,12 @@ struct StepDownArgs {            // routed experts, second product: out[n] = sum
   int top_k, k, n;
   float* out;
 };
+
+// Context splits of the one-token attention: rows per split (a multiple of the kernels' 64-row tile) and the layout of a
+// partial result.
+constexpr int kMaxSplits = 256;
+__host__ __device__ inline int latent_split_rows(int n, int splits) { return ((n + splits - 1) / splits + 63) / 64 * 64; }
+__host__ __device__ inline int latent_part_row(int rank) { return (rank + 3) / 4 * 4 + 4; }
 
 // ------------------------------------------------------------------------------------ math
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }

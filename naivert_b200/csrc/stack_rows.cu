@@ -12,12 +12,86 @@ namespace {
 
 // ------------------------------------------------------------------------------------ stream update + norms
 // One CTA per row.  x (+ embedding) -> x += rms(y) * post_w + add -> h = rms(x) * pre_w, all in float.
+__device__ __forceinline__ float4 bf4(const __nv_bfloat16* p) {
+  const uint2 v = __ldg(reinterpret_cast<const uint2*>(p));
+  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
+}
+__device__ __forceinline__ float dot4(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// widths that are multiples of four: 16-byte accesses, several in flight per thread
+__device__ __forceinline__ void rows_vec4(const StackRowArgs& a, int r, float4* buf, float* red) {
+  const int W4 = a.width / 4;
+  float4* sy = buf;
+  float4* sx = buf + W4;
+  float ry = 0.f;
+  float4* xrow = reinterpret_cast<float4*>(a.x + (size_t)r * a.width);
+  if (a.y) {
+    float ss = 0.f;
+    if (a.slot_of) {
+      for (int c = threadIdx.x; c < W4; c += 256) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int j = 0; j < a.top_k; ++j) {
+          const float p = a.probs[(size_t)r * a.top_k + j];
+          const float4 t = reinterpret_cast<const float4*>(a.y + (long long)a.slot_of[(size_t)r * a.top_k + j] * a.y_ld)[c];
+          v = make_float4(fmaf(p, t.x, v.x), fmaf(p, t.y, v.y), fmaf(p, t.z, v.z), fmaf(p, t.w, v.w));
+        }
+        sy[c] = v;
+        ss += dot4(v);
+      }
+    } else {
+      const float4* y = reinterpret_cast<const float4*>(a.y + (long long)r * a.y_ld);
+#pragma unroll 4
+      for (int c = threadIdx.x; c < W4; c += 256) {
+        const float4 v = y[c];
+        sy[c] = v;
+        ss += dot4(v);
+      }
+    }
+    ry = 1.0f / sqrtf(block_sum_f(ss, red) / (float)a.width + a.eps);
+  }
+  const __nv_bfloat16* emb = nullptr;
+  if (a.tokens) {
+    int t = a.tokens[r];
+    t = t < 0 ? 0 : t >= a.vocab ? a.vocab - 1 : t;
+    emb = a.table + (size_t)t * a.width;
+  }
+  float sq = 0.f;
+#pragma unroll 4
+  for (int c = threadIdx.x; c < W4; c += 256) {
+    float4 v;
+    if (emb) { v = bf4(emb + c * 4); v = make_float4(v.x * a.embed_scale, v.y * a.embed_scale, v.z * a.embed_scale, v.w * a.embed_scale); }
+    else v = xrow[c];
+    if (a.y) {
+      const float4 y = sy[c], w = bf4(a.post_w + c * 4);
+      v = make_float4(fmaf(y.x * ry, w.x, v.x), fmaf(y.y * ry, w.y, v.y), fmaf(y.z * ry, w.z, v.z), fmaf(y.w * ry, w.w, v.w));
+    }
+    if (a.add) { const float4 t = bf4(a.add + c * 4); v = make_float4(v.x + t.x, v.y + t.y, v.z + t.z, v.w + t.w); }
+    xrow[c] = v;
+    sx[c] = v;
+    sq += dot4(v);
+  }
+  if (!a.pre_w) return;
+  const float rx = 1.0f / sqrtf(block_sum_f(sq, red) / (float)a.width + a.eps);
+#pragma unroll 4
+  for (int c = threadIdx.x; c < W4; c += 256) {
+    const float4 v = sx[c], w = bf4(a.pre_w + c * 4);
+    const float4 o = make_float4(v.x * rx * w.x, v.y * rx * w.y, v.z * rx * w.z, v.w * rx * w.w);
+    if (a.h_f32) reinterpret_cast<float4*>(reinterpret_cast<float*>(a.h) + (long long)r * a.h_ld)[c] = o;
+    else reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.h) + (long long)r * a.h_ld)[c] =
+        make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
+  }
+}
 __global__ void __launch_bounds__(256) stack_rows_kernel(const StackRowArgs a) {
-  extern __shared__ float buf[];                 // [2][width]: sublayer row, stream row
+  extern __shared__ __align__(16) float buf[];   // [2][width]: sublayer row, stream row
   __shared__ float red[33];
   griddep_wait();
   griddep_launch();
   const int r = blockIdx.x, W = a.width;
+  if (((W | (int)a.y_ld | (int)a.h_ld) & 3) == 0) {
+    rows_vec4(a, r, reinterpret_cast<float4*>(buf), red);
+    return;
+  }
   float* sy = buf;
   float* sx = buf + W;
   float ss = 0.f;
@@ -82,41 +156,64 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepArgs a
 }
 
 // ------------------------------------------------------------------------------------ short convolution
-// grid (rows, channel blocks): u[r][c] = b[c] + sum_j k[c][j] x[position of tap j], zeros before the sequence.
-__global__ void __launch_bounds__(256) stack_conv_kernel(const RecurrenceArgs a) {
+// u[r][c] = b[c] + sum_j k[c][j] x[position of tap j], zeros before the sequence.  One thread owns a channel of a strip of
+// rows; up to kConvWin taps stay in a register window, longer kernels re-read their inputs.
+constexpr int kConvRows = 32, kConvWin = 4, kBatch = 8;
+
+__device__ __forceinline__ float conv_input(const RecurrenceArgs& a, int r, int c, int pos0) {     // x at row r (negative: history)
+  if (pos0 + r < 0) return 0.f;
+  return r >= 0 ? load_act(a.xy, (long long)r * a.xy_ld + a.width + c, a.f32)
+                : a.history[(long long)((pos0 + r) % a.hist_rows) * a.width + c];
+}
+
+__global__ void __launch_bounds__(128) stack_conv_kernel(const RecurrenceArgs a) {
   griddep_wait();
   griddep_launch();
-  const int r = blockIdx.x, c = blockIdx.y * 256 + threadIdx.x;
+  const int r0 = blockIdx.x * kConvRows, c = blockIdx.y * 128 + threadIdx.x;
   if (c >= a.width) return;
-  const int pos = *a.pos0 + r;
-  float v = bf(a.conv_b + c);
-  for (int j = 0; j < a.taps; ++j) {
-    const int back = a.taps - 1 - j;              // tokens before the current one
-    if (back > pos) continue;
-    const float x = back <= r ? load_act(a.xy, (long long)(r - back) * a.xy_ld + a.width + c, a.f32)
-                              : a.history[(long long)((pos - back) % a.hist_rows) * a.width + c];
-    v = fmaf(bf(a.conv + (size_t)c * a.taps + j), x, v);
-  }
+  const int pos0 = *a.pos0, rows = min(kConvRows, a.rows - r0);
   const int b = c / a.block;
-  store_act(a.u, ((long long)r * a.blocks + b) * a.block_pad + (c - b * a.block), v, a.f32);
+  const long long u0 = ((long long)r0 * a.blocks + b) * a.block_pad + (c - b * a.block), ustep = (long long)a.blocks * a.block_pad;
+  const float bias = bf(a.conv_b + c);
+  if (a.taps <= kConvWin) {
+    float k[kConvWin], x[kConvWin];                  // newest last; missing taps are zero
+#pragma unroll
+    for (int j = 0; j < kConvWin; ++j) {
+      const int t = j - (kConvWin - a.taps);
+      k[j] = t >= 0 ? bf(a.conv + (size_t)c * a.taps + t) : 0.f;
+    }
+#pragma unroll
+    for (int j = 1; j < kConvWin; ++j) x[j] = j > kConvWin - a.taps ? conv_input(a, r0 - (kConvWin - j), c, pos0) : 0.f;
+#pragma unroll 1
+    for (int i0 = 0; i0 < rows; i0 += kBatch) {
+      float in[kBatch];                              // requested together: the stores below could alias later loads
+#pragma unroll
+      for (int i = 0; i < kBatch; ++i) in[i] = i0 + i < rows ? load_act(a.xy, (long long)(r0 + i0 + i) * a.xy_ld + a.width + c, a.f32) : 0.f;
+#pragma unroll
+      for (int i = 0; i < kBatch; ++i) {
+#pragma unroll
+        for (int j = 0; j + 1 < kConvWin; ++j) x[j] = x[j + 1];
+        x[kConvWin - 1] = in[i];
+        float v = bias;
+#pragma unroll
+        for (int j = 0; j < kConvWin; ++j) v = fmaf(k[j], x[j], v);
+        if (i0 + i < rows) store_act(a.u, u0 + (i0 + i) * ustep, v, a.f32);
+      }
+    }
+  } else {
+    for (int i = 0; i < rows; ++i) {
+      float v = bias;
+      for (int j = 0; j < a.taps; ++j) v = fmaf(bf(a.conv + (size_t)c * a.taps + j), conv_input(a, r0 + i - (a.taps - 1 - j), c, pos0), v);
+      store_act(a.u, u0 + i * ustep, v, a.f32);
+    }
+  }
 }
 
 // ------------------------------------------------------------------------------------ gated linear recurrence
 constexpr int kScanTokens = 64;               // tokens per CTA of the scan
 
-struct Gate { float a, drive; };
-__device__ __forceinline__ Gate gate_of(const RecurrenceArgs& p, int r, int c, int b, int cb, float sp) {
-  const float* g = p.gates + ((long long)r * p.blocks + b) * 2 * p.block;
-  const float rg = sigmoid_f(g[cb]), ig = sigmoid_f(g[p.block + cb]);
-  const float la = -p.decay * rg * sp;
-  const float u = load_act(p.u, ((long long)r * p.blocks + b) * p.block_pad + cb, p.f32);
-  Gate o;
-  o.a = expf(la);
-  o.drive = sqrtf(-expm1f(2.0f * la)) * ig * u;
-  return o;
-}
-
-// pass 1: decay product and end state (from zero) of every 64-token piece
+// Pass 1: decay and drive of every token replace the gate pre-activations in place; decay product and end state (from zero)
+// of every 64-token piece.
 __global__ void __launch_bounds__(128) stack_scan_pieces_kernel(const RecurrenceArgs p) {
   griddep_wait();
   griddep_launch();
@@ -125,11 +222,29 @@ __global__ void __launch_bounds__(128) stack_scan_pieces_kernel(const Recurrence
   const int b = c / p.block, cb = c - b * p.block;
   const float sp = p.softplus_lam[c];
   const int r0 = blockIdx.x * kScanTokens, r1 = min(p.rows, r0 + kScanTokens);
+  float* g = const_cast<float*>(p.gates) + (long long)b * 2 * p.block + cb;
+  const long long gs = (long long)p.blocks * 2 * p.block, u0 = (long long)b * p.block_pad + cb, us = (long long)p.blocks * p.block_pad;
   float prod = 1.f, s = 0.f;
-  for (int r = r0; r < r1; ++r) {
-    const Gate g = gate_of(p, r, c, b, cb, sp);
-    prod *= g.a;
-    s = fmaf(g.a, s, g.drive);
+#pragma unroll 1
+  for (int q0 = r0; q0 < r1; q0 += kBatch) {
+    float zr[kBatch], zi[kBatch], u[kBatch];
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int r = min(q0 + i, r1 - 1);
+      zr[i] = g[r * gs];
+      zi[i] = g[r * gs + p.block];
+      u[i] = load_act(p.u, u0 + r * us, p.f32);
+    }
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      if (q0 + i >= r1) break;
+      const float la = -p.decay * sigmoid_f(zr[i]) * sp;
+      const float a = expf(la), drive = sqrtf(-expm1f(2.0f * la)) * sigmoid_f(zi[i]) * u[i];
+      g[(q0 + i) * gs] = a;
+      g[(q0 + i) * gs + p.block] = drive;
+      prod *= a;
+      s = fmaf(a, s, drive);
+    }
   }
   float* o = p.agg + (size_t)blockIdx.x * 2 * p.width;
   o[c] = prod;
@@ -148,17 +263,31 @@ __global__ void __launch_bounds__(128) stack_scan_kernel(const RecurrenceArgs p)
   if (slot < 0) return;
   if (c < p.width) {
     const int b = c / p.block, cb = c - b * p.block;
-    const float sp = p.softplus_lam[c];
     float s = pos0 == 0 ? 0.f : p.state[(size_t)slot * p.width + c];
+#pragma unroll 8
     for (int q = 0; q < (int)blockIdx.x; ++q) {
       const float* g = p.agg + (size_t)q * 2 * p.width;
       s = fmaf(g[c], s, g[p.width + c]);
     }
     const int r0 = blockIdx.x * kScanTokens, r1 = min(p.rows, r0 + kScanTokens);
-    for (int r = r0; r < r1; ++r) {
-      const Gate g = gate_of(p, r, c, b, cb, sp);
-      s = fmaf(g.a, s, g.drive);
-      store_act(p.out, (long long)r * p.out_ld + c, s * load_act(p.xy, (long long)r * p.xy_ld + c, p.f32), p.f32);
+    const float* g = p.gates + (long long)b * 2 * p.block + cb;
+    const long long gs = (long long)p.blocks * 2 * p.block;
+#pragma unroll 1
+    for (int q0 = r0; q0 < r1; q0 += kBatch) {
+      float ga[kBatch], gd[kBatch], y[kBatch];
+#pragma unroll
+      for (int i = 0; i < kBatch; ++i) {
+        const int r = min(q0 + i, r1 - 1);
+        ga[i] = g[r * gs];
+        gd[i] = g[r * gs + p.block];
+        y[i] = load_act(p.xy, (long long)r * p.xy_ld + c, p.f32);
+      }
+#pragma unroll
+      for (int i = 0; i < kBatch; ++i) {
+        if (q0 + i >= r1) break;
+        s = fmaf(ga[i], s, gd[i]);
+        store_act(p.out, (long long)(q0 + i) * p.out_ld + c, s * y[i], p.f32);
+      }
     }
     if (last) {
       p.state[(size_t)(1 - slot) * p.width + c] = s;
@@ -236,7 +365,7 @@ extern "C" int nrt_stack_conv(const void* args, void* stream) {
   RecurrenceArgs a;
   memcpy(&a, args, sizeof(a));
   if (a.rows < 1 || a.taps < 1 || a.hist_rows < 2 * (a.taps - 1) || a.hist_rows < 1 || a.width != a.blocks * a.block) return -3;
-  return launch_pdl(stack_conv_kernel, dim3(a.rows, (a.width + 255) / 256), dim3(256), 0, S(stream), false, a);
+  return launch_pdl(stack_conv_kernel, dim3((a.rows + kConvRows - 1) / kConvRows, (a.width + 127) / 128), dim3(128), 0, S(stream), false, a);
 }
 
 // The recurrence over the chunk's rows: pieces, then the scan with the state hand-over.
@@ -247,7 +376,7 @@ extern "C" int nrt_stack_scan(const void* args, void* stream) {
   const int pieces = (a.rows + kScanTokens - 1) / kScanTokens;
   const dim3 grid(pieces, (a.width + 127) / 128);
   int rc = 0;
-  if (pieces > 1 && (rc = launch_pdl(stack_scan_pieces_kernel, grid, dim3(128), 0, S(stream), false, a))) return rc;
+  if ((rc = launch_pdl(stack_scan_pieces_kernel, grid, dim3(128), 0, S(stream), false, a))) return rc;
   return launch_pdl(stack_scan_kernel, grid, dim3(128), 0, S(stream), false, a);
 }
 

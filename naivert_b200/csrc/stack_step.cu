@@ -41,62 +41,181 @@ __device__ __forceinline__ uint4 ld_stream(const uint4* p) {           // weight
   return v;
 }
 
+// Values of the first kPreSpan elements that do not depend on the predecessor kernel, requested before the wait for it: the
+// norm weights, and the stream itself (written at least two launches back).
+constexpr int kPreSpan = kStepThreads * 16;
+struct Pre {
+  float4 x[4];
+  uint2 post[4], in[4];
+};
+__device__ __forceinline__ float4 bf4(const uint2& v) { return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y)); }
+__device__ __forceinline__ float4 ldcg4(const float* p) { return __ldcg(reinterpret_cast<const float4*>(p)); }
+__device__ __forceinline__ uint2 ldw4(const __nv_bfloat16* p) { return __ldg(reinterpret_cast<const uint2*>(p)); }
+__device__ __forceinline__ float dot4(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+__device__ __forceinline__ float4 fma4(const float4& a, const float4& b, float s, const float4& c) {      // a * b * s + c
+  return make_float4(fmaf(a.x * s, b.x, c.x), fmaf(a.y * s, b.y, c.y), fmaf(a.z * s, b.z, c.z), fmaf(a.w * s, b.w, c.w));
+}
+
 template <int PRO>
-__device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, float* hs, float* red) {
-  const int K = a.k;
-  if (PRO == kProResidual) {
-    float ss = 0.f;
-    if (a.y) {
-      for (int c = threadIdx.x; c < K; c += kStepThreads) { const float v = __ldcg(a.y + c); ss = fmaf(v, v, ss); }
-      ss = block_sum_f(ss, red);
+__device__ __forceinline__ void preload(const StepArgs& a, Pre& p) {
+  if (a.k & 3) return;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
+    p.x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    p.post[i] = p.in[i] = make_uint2(0u, 0u);
+    if (e < a.k) {
+      p.in[i] = ldw4(a.in_w + e);
+      if (PRO == kProResidual) {
+        if (a.y) p.post[i] = ldw4(a.post_w + e);
+        if (!a.tokens) p.x[i] = ldcg4(a.x + e);
+      }
     }
-    const float ry = a.y ? 1.0f / sqrtf(ss / (float)K + a.eps) : 0.f;
+  }
+}
+
+template <int PRO>
+__device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, float* hs, float* red, const Pre& p, int pos) {
+  const int K = a.k;
+  float4* hs4 = reinterpret_cast<float4*>(hs);
+  // element e (a multiple of four) of the input -> its float4 in the two planes
+  auto at4 = [&](int e) -> float4& { return hs4[((e >> 2) & 1) * k8 + (e >> 3)]; };
+  if (PRO == kProResidual || PRO == kProNorm) {
     const __nv_bfloat16* emb = nullptr;
-    if (a.tokens) {
-      int t = *a.tokens;
+    if (PRO == kProResidual && a.tokens) {
+      int t = *reinterpret_cast<const volatile int*>(a.tokens);
       t = t < 0 ? 0 : t >= a.vocab ? a.vocab - 1 : t;
       emb = a.table + (size_t)t * K;
     }
-    float sq = 0.f;
-    for (int c = threadIdx.x; c < K; c += kStepThreads) {
-      float v = emb ? bf(emb + c) * a.embed_scale : __ldcg(a.x + c);
-      if (a.y) v += __ldcg(a.y + c) * ry * bf(a.post_w + c);
-      if (a.add) v += bf(a.add + c);
-      hs[plane_at(c, k8)] = v;
-      if (blockIdx.x == 0) a.x_out[c] = v;
-      sq = fmaf(v, v, sq);
+    if ((K & 3) == 0) {
+      float4 v[4];
+      float ss = 0.f, sq = 0.f;
+      if (PRO == kProResidual && a.y) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
+          v[i] = e < K ? ldcg4(a.y + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ss += dot4(v[i]);
+        for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) ss += dot4(ldcg4(a.y + e));
+        ss = block_sum_f(ss, red);
+      } else if (PRO == kProNorm) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
+          v[i] = e < K ? ldcg4(a.in_ + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+      }
+      const float ry = PRO == kProResidual && a.y ? 1.0f / sqrtf(ss / (float)K + a.eps) : 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
+        if (e >= K) continue;
+        if (PRO == kProResidual) {
+          float4 x = p.x[i];
+          if (emb) { const float4 t = bf4(ldw4(emb + e)); x = make_float4(t.x * a.embed_scale, t.y * a.embed_scale, t.z * a.embed_scale, t.w * a.embed_scale); }
+          if (a.y) x = fma4(v[i], bf4(p.post[i]), ry, x);
+          if (a.add) { const float4 t = bf4(ldw4(a.add + e)); x = make_float4(x.x + t.x, x.y + t.y, x.z + t.z, x.w + t.w); }
+          if (blockIdx.x == 0) *reinterpret_cast<float4*>(a.x_out + e) = x;
+          v[i] = x;
+        }
+        sq += dot4(v[i]);
+      }
+      for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) {
+        float4 x;
+        if (PRO == kProResidual) {
+          if (emb) { const float4 t = bf4(ldw4(emb + e)); x = make_float4(t.x * a.embed_scale, t.y * a.embed_scale, t.z * a.embed_scale, t.w * a.embed_scale); }
+          else x = ldcg4(a.x + e);
+          if (a.y) x = fma4(ldcg4(a.y + e), bf4(ldw4(a.post_w + e)), ry, x);
+          if (a.add) { const float4 t = bf4(ldw4(a.add + e)); x = make_float4(x.x + t.x, x.y + t.y, x.z + t.z, x.w + t.w); }
+          if (blockIdx.x == 0) *reinterpret_cast<float4*>(a.x_out + e) = x;
+        } else {
+          x = ldcg4(a.in_ + e);
+        }
+        at4(e) = x;
+        sq += dot4(x);
+      }
+      sq = block_sum_f(sq, red);
+      const float rx = 1.0f / sqrtf(sq / (float)K + a.eps);
+      const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
+        if (e < K) at4(e) = fma4(v[i], bf4(p.in[i]), rx, zero);
+      }
+      for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) at4(e) = fma4(at4(e), bf4(ldw4(a.in_w + e)), rx, zero);
+    } else {
+      float ss = 0.f, sq = 0.f;
+      if (PRO == kProResidual && a.y) {
+        for (int c = threadIdx.x; c < K; c += kStepThreads) { const float v = __ldcg(a.y + c); ss = fmaf(v, v, ss); }
+        ss = block_sum_f(ss, red);
+      }
+      const float ry = PRO == kProResidual && a.y ? 1.0f / sqrtf(ss / (float)K + a.eps) : 0.f;
+      for (int c = threadIdx.x; c < K; c += kStepThreads) {
+        float v = PRO == kProNorm ? __ldcg(a.in_ + c) : emb ? bf(emb + c) * a.embed_scale : __ldcg(a.x + c);
+        if (PRO == kProResidual) {
+          if (a.y) v += __ldcg(a.y + c) * ry * bf(a.post_w + c);
+          if (a.add) v += bf(a.add + c);
+          if (blockIdx.x == 0) a.x_out[c] = v;
+        }
+        hs[plane_at(c, k8)] = v;
+        sq = fmaf(v, v, sq);
+      }
+      sq = block_sum_f(sq, red);
+      const float rx = 1.0f / sqrtf(sq / (float)K + a.eps);
+      for (int c = threadIdx.x; c < K; c += kStepThreads) hs[plane_at(c, k8)] *= rx * bf(a.in_w + c);
     }
-    sq = block_sum_f(sq, red);
-    const float rx = 1.0f / sqrtf(sq / (float)K + a.eps);
-    for (int c = threadIdx.x; c < K; c += kStepThreads) hs[plane_at(c, k8)] *= rx * bf(a.in_w + c);
-  } else if (PRO == kProNorm) {
-    float sq = 0.f;
-    for (int c = threadIdx.x; c < K; c += kStepThreads) {
-      const float v = __ldcg(a.in_ + c);
-      hs[plane_at(c, k8)] = v;
-      sq = fmaf(v, v, sq);
-    }
-    sq = block_sum_f(sq, red);
-    const float rx = 1.0f / sqrtf(sq / (float)K + a.eps);
-    for (int c = threadIdx.x; c < K; c += kStepThreads) hs[plane_at(c, k8)] *= rx * bf(a.in_w + c);
   } else if (PRO == kProLoad) {
     const float* in = a.in_ + g * a.in_gstride;
-    for (int c = threadIdx.x; c < K; c += kStepThreads) hs[plane_at(c, k8)] = __ldcg(in + c);
-  } else {                                                             // kProMerge
-    const size_t row = K + 2, hstride = (size_t)a.groups * row;
-    const float* p0 = a.part + g * row;
-    float m = -FLT_MAX, l = 0.f;
-    for (int s = 0; s < a.splits; ++s) m = fmaxf(m, __ldcg(p0 + s * hstride));
-    for (int s = 0; s < a.splits; ++s) l += __ldcg(p0 + s * hstride + 1) * expf(__ldcg(p0 + s * hstride) - m);
-    const float inv = 1.0f / l;
-    for (int c = threadIdx.x; c < K; c += kStepThreads) {
-      float v = 0.f;
-      for (int s = 0; s < a.splits; ++s) {
-        const float ms = __ldcg(p0 + s * hstride);
-        if (ms > -FLT_MAX) v = fmaf(__ldcg(p0 + s * hstride + 2 + c), expf(ms - m), v);
-      }
-      hs[plane_at(c, k8)] = v * inv;
+    if (((K | (int)a.in_gstride) & 3) == 0) {
+#pragma unroll 4
+      for (int e = (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) at4(e) = ldcg4(in + e);
+    } else {
+      for (int c = threadIdx.x; c < K; c += kStepThreads) hs[plane_at(c, k8)] = __ldcg(in + c);
     }
+  } else {                                                             // kProMerge
+    // weights of the used splits, then a weighted sum of their outputs; threads beyond the row's float4 columns take other splits
+    __shared__ float ws[kMaxSplits];
+    const int n = pos + 1, per = latent_split_rows(n, a.splits), used = (n + per - 1) / per;
+    const int row = latent_part_row(K), k4 = (K + 3) / 4;
+    const size_t hstride = (size_t)a.groups * row;
+    const float* p0 = a.part + (size_t)g * row;
+    float ms = -FLT_MAX, ls = 0.f;
+    if ((int)threadIdx.x < used) { ms = __ldcg(p0 + threadIdx.x * hstride); ls = __ldcg(p0 + threadIdx.x * hstride + 1); }
+    float m = ms;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = m;
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kStepThreads / 32; ++i) m = fmaxf(m, red[i]);
+    const float w = (int)threadIdx.x < used ? expf(ms - m) : 0.f;
+    const float l = block_sum_f(ls * w, red);
+    if ((int)threadIdx.x < used) ws[threadIdx.x] = w / l;
+    int cols = 1;
+    while (cols < k4 && cols < kStepThreads) cols *= 2;
+    const int subs = kStepThreads / cols, sub = (int)threadIdx.x / cols, c0 = (int)threadIdx.x & (cols - 1);
+    __syncthreads();
+    for (int i = threadIdx.x; i < 2 * k8; i += kStepThreads) hs4[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    __syncthreads();
+    for (int cb = 0; cb < k4; cb += cols) {
+      const int c = cb + c0;
+      float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+      for (int s = sub; s < used && c < k4; s += subs) {
+        const float4 v = ldcg4(p0 + s * hstride + 4 + c * 4);
+        const float wv = ws[s];
+        acc = make_float4(fmaf(v.x, wv, acc.x), fmaf(v.y, wv, acc.y), fmaf(v.z, wv, acc.z), fmaf(v.w, wv, acc.w));
+      }
+      // sub-sums join in a fixed order
+      for (int q = 0; q < subs; ++q) {
+        if (sub == q && c < k4) { float4& d = at4(c * 4); d = make_float4(d.x + acc.x, d.y + acc.y, d.z + acc.z, d.w + acc.w); }
+        if (subs > 1) __syncthreads();
+      }
+    }
+    __syncthreads();
   }
   for (int c = K + threadIdx.x; c < k8 * 8; c += kStepThreads) hs[plane_at(c, k8)] = 0.f;
   __syncthreads();
@@ -140,6 +259,8 @@ __device__ __forceinline__ void finish_row(const StepArgs& a, int g, int row, fl
   }
 }
 
+constexpr int kMaxStepSmem = 200 * 1024;
+
 template <int PRO, int EPI, int RU, int U, bool ROUTE>
 __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs a, const RouterArgs ra, const int rgroups,
                                                                   const int rkeep, const int G) {
@@ -178,6 +299,8 @@ __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs
   const int per_cta = (tiles + (int)gridDim.x - 1) / (int)gridDim.x;
   const int tile_lo = (int)blockIdx.x * per_cta, tile_hi = min(tiles, tile_lo + per_cta);
   if (!ROUTE && tile_lo < tile_hi) fetch(tile_lo, lig);
+  Pre pre;
+  if constexpr (PRO == kProResidual) preload<PRO>(a, pre);       // (a normed input vector may come from the predecessor itself)
   griddep_wait();
   griddep_launch();
   const int pos = a.pos0 ? *reinterpret_cast<const volatile int*>(a.pos0) : 0;
@@ -193,7 +316,8 @@ __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs
     slot = state_slot(a.tags, pos, a.status);
     if (slot < 0) return;
   }
-  if (!PER_GROUP) load_input<PRO>(a, 0, k8, hs, red);
+  if constexpr (PRO == kProNorm) preload<PRO>(a, pre);
+  if (!PER_GROUP) load_input<PRO>(a, 0, k8, hs, red, pre, pos);
   if (PRO == kProNorm && a.lat_in && blockIdx.x == gridDim.x - 1 && pos >= 0 && pos < a.capacity) {
     // append the token's key/value latent to the cache
     float sq = 0.f;
@@ -207,7 +331,7 @@ __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs
     const int g = tile / tiles_g;
     if (PER_GROUP && g != cur) {
       if (cur >= 0) __syncthreads();
-      load_input<PRO>(a, g, k8, hs, red);
+      load_input<PRO>(a, g, k8, hs, red, pre, pos);
       cur = g;
     }
     float acc[RU], acc2[RU];
@@ -272,26 +396,25 @@ __global__ void __launch_bounds__(kStepThreads) stack_down_kernel(const StepDown
 #pragma unroll
     for (int i = 0; i < RU; ++i) acc[i] = 0.f;
 #pragma unroll 1
-    for (int c0 = lane; c0 < total; c0 += 32 * U) {
-      uint4 wv[RU][U];
+    for (int j = 0; j < a.top_k; ++j) {
+      const uint4* base = reinterpret_cast<const uint4*>(a.w + s_ids[j] * a.w_gstride + (long long)row0 * a.w_ld);
+      const int ld8 = (int)(a.w_ld / 8);
+#pragma unroll 1
+      for (int c0 = lane; c0 < k8; c0 += 32 * U) {
+        uint4 wv[RU][U];
 #pragma unroll
-      for (int q = 0; q < U; ++q) {
-        const int c = c0 + q * 32;
-        const int j = c / k8;
-        const bool in = c < total;
-        const __nv_bfloat16* base = a.w + (in ? s_ids[j] : 0) * a.w_gstride;
+        for (int q = 0; q < U; ++q)
 #pragma unroll
-        for (int i = 0; i < RU; ++i)
-          wv[i][q] = in && row0 + i < a.n ? ld_stream(reinterpret_cast<const uint4*>(base + (long long)(row0 + i) * a.w_ld) + (c - j * k8))
-                                          : make_uint4(0u, 0u, 0u, 0u);
-      }
+          for (int i = 0; i < RU; ++i)
+            wv[i][q] = c0 + q * 32 < k8 && row0 + i < a.n ? ld_stream(base + i * ld8 + c0 + q * 32) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
-      for (int q = 0; q < U; ++q) {
-        const int c = c0 + q * 32;
-        if (c < total) {
-          const float4 x0 = hs4[c], x1 = hs4[total + c];
+        for (int q = 0; q < U; ++q) {
+          const int c = c0 + q * 32;
+          if (c < k8) {
+            const float4 x0 = hs4[j * k8 + c], x1 = hs4[total + j * k8 + c];
 #pragma unroll
-          for (int i = 0; i < RU; ++i) acc[i] = dot8(wv[i][q], x0, x1, acc[i]);
+            for (int i = 0; i < RU; ++i) acc[i] = dot8(wv[i][q], x0, x1, acc[i]);
+          }
         }
       }
     }
@@ -304,43 +427,62 @@ __global__ void __launch_bounds__(kStepThreads) stack_down_kernel(const StepDown
   }
 }
 
-constexpr int kMaxStepSmem = 200 * 1024;
-
-template <int PRO, int EPI, int RU, int U, bool ROUTE>
-int launch_step(const StepArgs& a, const RouterArgs& r, int groups, int keep, cudaStream_t stream, bool pdl) {
-  auto* kern = stack_step_kernel<PRO, EPI, RU, U, ROUTE>;
-  static bool configured = false;
-  if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxStepSmem);
-    if (e != cudaSuccess) return (int)e;
-    configured = true;
-  }
-  const int k8 = (a.k + 7) / 8;
+int lanes_of(int k8) {
   int G = 4;
   while (G < 32 && G < k8) G *= 2;
-  const int rows_tile = kStepThreads / G * RU;
-  const long long tiles = (long long)a.groups * ((a.n + rows_tile - 1) / rows_tile);
-  const size_t smem = (size_t)k8 * 32;
-  if (smem > kMaxStepSmem || tiles < 1 || tiles > 0x7fffffffLL) return -7;
-  const int cap = PRO == kProMerge ? 148 * 2 : 148 * 4;
-  return launch_pdl(kern, dim3((unsigned)(tiles < cap ? tiles : cap)), dim3(kStepThreads), smem, stream, pdl, a, r, groups, keep, G);
+  return G;
 }
 
-// Rows per lane group: as many as still leave every SM two CTAs.
+template <int PRO, int EPI, int RU, int U, bool ROUTE>
+struct StepLaunch {
+  // CTAs of this kernel that are resident at once with `smem` bytes each
+  static int resident(size_t smem) {
+    static size_t seen[8];
+    static int value[8], count = 0;
+    for (int i = 0; i < count; ++i)
+      if (seen[i] == smem) return value[i];
+    auto* kern = stack_step_kernel<PRO, EPI, RU, U, ROUTE>;
+    if (count == 0 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxStepSmem) != cudaSuccess) return -1;
+    int per = 0, dev = 0, sms = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per, kern, kStepThreads, smem) != cudaSuccess || per < 1) per = 1;
+    if (count < 8) { seen[count] = smem; value[count] = per * sms; ++count; }
+    return per * sms;
+  }
+  static long long tiles(const StepArgs& a) {
+    const int rows_tile = kStepThreads / lanes_of((a.k + 7) / 8) * RU;
+    return (long long)a.groups * ((a.n + rows_tile - 1) / rows_tile);
+  }
+  static double balance(const StepArgs& a) {            // busy share of the resident CTAs
+    const long long t = tiles(a), res = resident((size_t)((a.k + 7) / 8) * 32);
+    if (res < 1) return 0.0;
+    const long long grid = t < res ? t : res, per = (t + grid - 1) / grid;
+    return (double)t / (double)(per * res);
+  }
+  static int run(const StepArgs& a, const RouterArgs& r, int groups, int keep, cudaStream_t stream, bool pdl) {
+    const int k8 = (a.k + 7) / 8;
+    const size_t smem = (size_t)k8 * 32;
+    const long long t = tiles(a);
+    if (smem > kMaxStepSmem || t < 1 || t > 0x7fffffffLL) return -7;
+    const int res = resident(smem);
+    if (res < 1) return -8;
+    return launch_pdl(stack_step_kernel<PRO, EPI, RU, U, ROUTE>, dim3((unsigned)(t < res ? t : res)), dim3(kStepThreads), smem, stream, pdl, a,
+                      r, groups, keep, lanes_of(k8));
+  }
+};
+
+// Rows per lane group: the largest count that still spreads the rows evenly over the resident CTAs.
 template <int PRO, int EPI, bool ROUTE>
 int pick_step(const StepArgs& a, const RouterArgs& r, int groups, int keep, cudaStream_t stream, bool pdl) {
-  const long long rows = (long long)a.groups * a.n;
-  const int k8 = (a.k + 7) / 8;
-  int G = 4;
-  while (G < 32 && G < k8) G *= 2;
-  const long long per = kStepThreads / G;
   if constexpr (EPI == kTEpiGlu || EPI == kTEpiRecur) {
-    if (rows >= 2 * per * 296) return launch_step<PRO, EPI, 2, 2, ROUTE>(a, r, groups, keep, stream, pdl);
-    return launch_step<PRO, EPI, 1, 4, ROUTE>(a, r, groups, keep, stream, pdl);
+    using A = StepLaunch<PRO, EPI, 2, 2, ROUTE>;
+    using B = StepLaunch<PRO, EPI, 1, 4, ROUTE>;
+    return A::balance(a) + 0.05 >= B::balance(a) ? A::run(a, r, groups, keep, stream, pdl) : B::run(a, r, groups, keep, stream, pdl);
   } else {
-    if (rows >= 4 * per * 296) return launch_step<PRO, EPI, 4, 2, ROUTE>(a, r, groups, keep, stream, pdl);
-    if (rows >= 2 * per * 296) return launch_step<PRO, EPI, 2, 4, ROUTE>(a, r, groups, keep, stream, pdl);
-    return launch_step<PRO, EPI, 1, 8, ROUTE>(a, r, groups, keep, stream, pdl);
+    using A = StepLaunch<PRO, EPI, 2, 4, ROUTE>;
+    using B = StepLaunch<PRO, EPI, 1, 8, ROUTE>;
+    return A::balance(a) + 0.05 >= B::balance(a) ? A::run(a, r, groups, keep, stream, pdl) : B::run(a, r, groups, keep, stream, pdl);
   }
 }
 
