@@ -235,32 +235,33 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
       tc_fence_before();
       mbar_arrive(&bar->s_empty);
       const int k0 = j * kKeys;
-      float mx = -INFINITY;
+      float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains: the row's 64 values are one thread's
       if (k0 + kKeys <= vis) {
 #pragma unroll
-        for (int i = 0; i < kKeys; ++i) mx = fmaxf(mx, __uint_as_float(s[i]));
+        for (int i = 0; i < kKeys; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(s[i]));
       } else {
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) {
           if (k0 + i >= vis) s[i] = 0xff800000u;
-          mx = fmaxf(mx, __uint_as_float(s[i]));
+          mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(s[i]));
         }
       }
+      float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       mx *= c2;                                                        // scale > 0 keeps the order
       float corr = 1.f;
       bool grow = false;
       if (m == -INFINITY) m = mx;
       else if (mx > m + 8.f) { corr = exp2_approx(m - mx); m = mx; grow = true; }
       const float base = m == -INFINITY ? 0.f : m;
-      float sum = 0.f;
+      float sum4[4] = {0.f, 0.f, 0.f, 0.f};
       uint32_t pk[kKeys / 2];
 #pragma unroll
       for (int i = 0; i < kKeys; i += 2) {
         const float p0 = exp2_approx(fmaf(__uint_as_float(s[i]), c2, -base)), p1 = exp2_approx(fmaf(__uint_as_float(s[i + 1]), c2, -base));
-        sum += p0 + p1;
+        sum4[(i >> 1) & 3] += p0 + p1;
         pk[i / 2] = pack_bf16x2(p0, p1);
       }
-      l = fmaf(l, corr, sum);
+      l = fmaf(l, corr, (sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
       if (j > 0) ok = __all_sync(0xffffffffu, mbar_wait(&bar->pv_done, (j - 1) & 1, a.status, kSiteAccFull | 1));
       if (!ok) break;
       if ((j > 0 || !a.first) && __any_sync(0xffffffffu, grow)) {
@@ -427,12 +428,15 @@ __global__ void __launch_bounds__(256, 1) latent_decode_tc_kernel(const LatentDe
   const int per = latent_split_rows(n, a.splits);
   const int j_lo = min(n, (int)blockIdx.y * per), j_hi = min(n, j_lo + per);
   const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(a.cache);
-  const int pieces = rp / 8;
+  const int pieces = rp / 8, t_first = tid / pieces, c_first = tid - t_first * pieces, t_step = 256 / pieces, c_step = 256 - t_step * pieces;
   auto request = [&](int j0, int stage) {
-    for (int i = tid; i < kDecTile * pieces; i += 256) {
-      const int t = i / pieces, c = i - t * pieces;
+    int t = t_first, c = c_first;                     // piece (t, c) of the tile; steps of 256 pieces without divisions
+    while (t < kDecTile) {
       const bool in = j0 + t < j_hi;
       cp16(sc + (stage * kDecTile + t) * pitch + c * 8, cache + (long long)(in ? j0 + t : j_lo) * a.cache_ld + c * 8, in);
+      c += c_step;
+      t += t_step;
+      if (c >= pieces) { c -= pieces; ++t; }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -463,6 +467,7 @@ __global__ void __launch_bounds__(256, 1) latent_decode_tc_kernel(const LatentDe
 #pragma unroll
       for (int q = 0; q < 4; ++q) o[i][t][q] = 0.f;
   const int ntiles = rp / 8;
+  const float c2 = a.scale * 1.4426950408889634f;     // scores in powers of two
   int stage = 0;
   for (int j0 = j_lo; j0 < j_hi; j0 += kDecTile, stage ^= 1) {
     if (j0 + kDecTile < j_hi) {
@@ -492,20 +497,22 @@ __global__ void __launch_bounds__(256, 1) latent_decode_tc_kernel(const LatentDe
 #pragma unroll
     for (int i = 0; i < MT; ++i) {
       float* d = ss + (i * 16 + fr) * kSP + warp * 8 + fc;
-      d[0] = acc[i][0] * a.scale;
-      d[1] = acc[i][1] * a.scale;
-      d[8 * kSP] = acc[i][2] * a.scale;
-      d[8 * kSP + 1] = acc[i][3] * a.scale;
+      d[0] = acc[i][0] * c2;
+      d[1] = acc[i][1] * c2;
+      d[8 * kSP] = acc[i][2] * c2;
+      d[8 * kSP + 1] = acc[i][3] * c2;
     }
     __syncthreads();
     const int live = j_hi - j0;
-    for (int t = warp; t < HT; t += 8) {
+#pragma unroll
+    for (int ti = 0; ti < HT / 8; ++ti) {
+      const int t = warp + 8 * ti;
       const float s0 = lane < live ? ss[t * kSP + lane] : -FLT_MAX, s1 = lane + 32 < live ? ss[t * kSP + lane + 32] : -FLT_MAX;
       float mt = fmaxf(s0, s1);
 #pragma unroll
       for (int off = 16; off > 0; off >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, off));
-      const float m_old = sm[t], mn = fmaxf(m_old, mt), corr = expf(m_old - mn);
-      const float p0 = lane < live ? expf(s0 - mn) : 0.f, p1 = lane + 32 < live ? expf(s1 - mn) : 0.f;
+      const float m_old = sm[t], mn = fmaxf(m_old, mt), corr = exp2_approx(m_old - mn);
+      const float p0 = lane < live ? exp2_approx(s0 - mn) : 0.f, p1 = lane + 32 < live ? exp2_approx(s1 - mn) : 0.f;
       const float l = lane_sum(p0 + p1);
       sp[t * kPP + lane] = __float2bfloat16_rn(p0);
       sp[t * kPP + lane + 32] = __float2bfloat16_rn(p1);
@@ -547,7 +554,7 @@ __global__ void __launch_bounds__(256, 1) latent_decode_tc_kernel(const LatentDe
       const int t = i * 16 + fr + 8 * half;
       if (h0 + t >= a.heads) continue;
       float* out = a.part + ((size_t)blockIdx.y * a.heads + h0 + t) * latent_part_row(a.rank);
-      if (warp == 0 && (lane & 3) == 0) { out[0] = sm[t]; out[1] = sl[t]; }
+      if (warp == 0 && (lane & 3) == 0) { out[0] = sm[t] * 0.6931471805599453f; out[1] = sl[t]; }     // maximum in natural units
 #pragma unroll
       for (int q = 0; q < kNT; ++q) {
         const int c = (warp + 8 * q) * 8 + fc;

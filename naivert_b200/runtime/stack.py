@@ -191,7 +191,9 @@ class StackRuntime:
         self.sq = z(max([m.heads * d["dp"] for m, d in attn], default=1))
         self.sqlat = z(max([m.heads * m.kv_rank for m, _ in attn], default=1))
         self.so = z(max([m.heads * d["vp"] for m, d in attn], default=1))
-        self.splits = max(8, min(64, self.capacity // 256))          # context splits of the step's attention
+        # context splits of the step's attention: one 64-row tile each while that fills the SMs once
+        heads = max([m.heads for m, _ in attn], default=1)
+        self.splits = max(1, min(-(-self.capacity // 64), 148 // -(-heads // 32), 148))
         self.spart = z(max([self.splits * m.heads * (pad(m.kv_rank, 4) + 4) for m, _ in attn], default=1))
         self.sgate, self.su, self.srec = (z(max([m.width for m in rec], default=1)) for _ in range(3))
         self.sact = z(max([f.ff * (f.routing.top_k if f.kind == "moe" else 1) for f in ffs], default=1))
