@@ -122,7 +122,8 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
   uint8_t* sP = sV + 2 * N * 128;
   TcBars* bar = reinterpret_cast<TcBars*>(sP + 16384);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int h = blockIdx.x, r0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * kQRows;      // long rows first
+  // query tiles of one head run side by side (they share its keys in L2), the longest first
+  const int h = blockIdx.y, r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kQRows;
   const uint32_t cols = tc_tmem_cols(a.vdim);
   if ((smem_u32(smem) & 1023u) != 0u) {                    // the swizzle pattern counts from a 1024-byte boundary
     if (threadIdx.x == 0) report(a.status, kSiteGrid | 0x10);
@@ -287,6 +288,7 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
     if (ok) {
       tc_fence_after();
       const float inv = 1.0f / l;
+      const bool gate_vec = ((reinterpret_cast<uintptr_t>(a.gate) & 15) | (a.gate_ld & 3)) == 0;
       if (!a.last && live) { st_row[0] = m; st_row[1] = l; }
       for (int c = 0; c < N; c += 16) {
         uint32_t v[16];
@@ -309,8 +311,16 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
               for (int i = 0; i < 8; ++i) st_row[2 + c + 8 * q + i] = __uint_as_float(v[8 * q + i]);
             } else {
               float x[8];
+              if (gate_vec) {
+                const float4 g0 = *reinterpret_cast<const float4*>(g + 8 * q), g1 = *reinterpret_cast<const float4*>(g + 8 * q + 4);
+                x[0] = g0.x; x[1] = g0.y; x[2] = g0.z; x[3] = g0.w;
+                x[4] = g1.x; x[5] = g1.y; x[6] = g1.z; x[7] = g1.w;
+              } else {
 #pragma unroll
-              for (int i = 0; i < 8; ++i) x[i] = __uint_as_float(v[8 * q + i]) * inv * sigmoid_f(g[8 * q + i]);
+                for (int i = 0; i < 8; ++i) x[i] = g[8 * q + i];
+              }
+#pragma unroll
+              for (int i = 0; i < 8; ++i) x[i] = __uint_as_float(v[8 * q + i]) * inv * sigmoid_f(x[i]);
               *reinterpret_cast<uint4*>(o + 8 * q) =
                   make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
             }
@@ -604,7 +614,7 @@ extern "C" int nrt_latent_attn_tc(const void* tmQ, const void* tmK, const void* 
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  return launch_pdl(latent_attn_tc_kernel, dim3(a.heads, (a.rows + kQRows - 1) / kQRows), dim3(kTcThreads), smem,
+  return launch_pdl(latent_attn_tc_kernel, dim3((a.rows + kQRows - 1) / kQRows, a.heads), dim3(kTcThreads), smem,
                     reinterpret_cast<cudaStream_t>(stream), false, q, k, v, a);
 }
 
