@@ -3,7 +3,8 @@
 set -euo pipefail
 cd "$(dirname "$0")/.."
 GPUS="${NAIVERT_GPUS:-8}"
-ARGS=(--host "${NAIVERT_HOST:-0.0.0.0}" --port "${NAIVERT_PORT:-8080}" --model "${NAIVERT_MODEL:-naive-n0.5}")
+ARGS=(--host "${NAIVERT_HOST:-0.0.0.0}" --port "${NAIVERT_PORT:-8080}")
+[[ -n "${NAIVERT_MODEL:-}" ]] && ARGS+=(--model "$NAIVERT_MODEL")
 [[ -n "${NAIVERT_TARGET_CHECKPOINT:-}" ]] && ARGS+=(--target "$NAIVERT_TARGET_CHECKPOINT")
 [[ -n "${NAIVERT_DRAFT_CHECKPOINT:-}" ]] && ARGS+=(--draft "$NAIVERT_DRAFT_CHECKPOINT")
 [[ "${NAIVERT_RANDOM_INIT:-0}" == "1" ]] && ARGS+=(--random-init)

@@ -43,10 +43,13 @@ def compile_all() -> dict:
     from naivert_b200.ops import build
     t0 = time.time()
     path = build.compile_library()
+    stack_path = build.compile_library(group="stack")
     from naivert_b200.ops import kernels
-    res = {"library": path, "seconds": round(time.time() - t0, 1), "units": [u for u in build.source_inventory() if u.endswith(".cu")]}
+    res = {"library": path, "stack_library": stack_path, "seconds": round(time.time() - t0, 1), "units": [u for u in build.source_inventory() if u.endswith(".cu")]}
     try:
         kernels.aux_lib()
+        from naivert_b200.ops import stack_kernels
+        stack_kernels.lib()                                # entry points and struct sizes of the layer-stack library
         res["bindings"] = "ok"
     except OSError as e:
         res["bindings"] = f"not loadable here ({e})"

@@ -2,6 +2,7 @@
 """Serve the Anthropic-Messages-compatible API from one node.
 
     python examples/serve_sessions.py --model naive-n0.5 --target /ckpt/target --draft /ckpt/draft
+    python examples/serve_sessions.py --target /ckpt/tumatar            # the model is chosen by the checkpoint's config.json
     python -m torch.distributed.run --nproc-per-node 8 --master-addr 127.0.0.1 examples/serve_sessions.py ...
 
 Rank 0 runs the HTTP server; with more than one process the other ranks follow its engine calls.
@@ -24,10 +25,12 @@ def parse_args(argv=None):
     ap.add_argument("--port", type=int, default=int(os.environ.get("NAIVERT_PORT", "8080")))
     ap.add_argument("--cors-origin", default=None)
     ap.add_argument("--cors-credentials", action="store_true")
-    ap.add_argument("--model", default="naive-n0.5", help="registry name of the architecture")
+    ap.add_argument("--model", default=None,
+                    help="registry name of the architecture (default: what the target checkpoint's config.json says, else naive-n0.5)")
+    ap.add_argument("--dtype", choices=("bf16", "fp32"), default="bf16", help="numeric form of a layer-stack model")
     ap.add_argument("--target", default=os.environ.get("NAIVERT_TARGET_CHECKPOINT"), help="target checkpoint directory or short name")
     ap.add_argument("--draft", "--checkpoint", dest="draft", default=os.environ.get("NAIVERT_DRAFT_CHECKPOINT"),
-                    help="draft checkpoint directory or short name")
+                    help="draft checkpoint directory or short name (models with a draft)")
     ap.add_argument("--list-weights", action="store_true",
                     help="print the checkpoints found under NAIVERT_MODEL_ROOTS / NAIVERT_DRAFT_ROOTS and exit")
     ap.add_argument("--random-init", action="store_true", help="draw weights on device instead of loading checkpoints")
@@ -63,6 +66,17 @@ def parse_args(argv=None):
     return ap.parse_args(argv)
 
 
+def choose_model(model, target):
+    """The named model, else the one the target checkpoint describes, else the default."""
+    from naivert_b200.models.registry import resolve_checkpoint_model, resolve_model
+    if model is None and target is not None:
+        try:
+            return resolve_checkpoint_model(target)
+        except (KeyError, OSError):
+            pass                                           # a checkpoint of the default model in another size
+    return resolve_model(model or "naive-n0.5")
+
+
 def main(argv=None) -> int:
     a = parse_args(argv)
     if a.list_weights:
@@ -78,7 +92,6 @@ def main(argv=None) -> int:
     import torch.distributed as dist
 
     from naivert_b200.models.checkpoint import resolve_checkpoint
-    from naivert_b200.models.registry import resolve_model
     from naivert_b200.runtime.engine import Engine
     from naivert_b200.runtime.session_engine import SessionEngine
     from naivert_b200.runtime.tp_frontend import Commands, LeaderEngine, follower_loop
@@ -87,6 +100,18 @@ def main(argv=None) -> int:
     from naivert_b200.serve.http import build_app, run_app
     from naivert_b200.serve.messages_api import ServerDefaults
 
+    target = draft = None
+    if not a.random_init:
+        if not a.target:
+            raise SystemExit("--target is required unless --random-init is given")
+        target = resolve_checkpoint(a.target)
+    spec = choose_model(a.model, target)
+    if spec.draft is not None and target is not None:
+        if not a.draft:
+            raise SystemExit(f"{spec.name} is served with a draft: --draft is required unless --random-init is given")
+        draft = resolve_checkpoint(a.draft, "NAIVERT_DRAFT_ROOTS")
+    if a.layers:
+        spec = spec.with_layers(a.layers)
     world, rank, local = (int(os.environ.get(k, d)) for k, d in (("WORLD_SIZE", "1"), ("RANK", "0"), ("LOCAL_RANK", "0")))
     torch.cuda.set_device(local)
     dev = torch.device("cuda", local)
@@ -96,15 +121,6 @@ def main(argv=None) -> int:
         dist.init_process_group("nccl", device_id=dev)
         group = dist.group.WORLD
         cpu_group = dist.new_group(backend="gloo")
-    spec = resolve_model(a.model)
-    if a.layers:
-        spec = spec.with_layers(a.layers)
-    target = draft = None
-    if not a.random_init:
-        if not a.target or not a.draft:
-            raise SystemExit("--target and --draft are required unless --random-init is given")
-        target, draft = resolve_checkpoint(a.target), resolve_checkpoint(a.draft, "NAIVERT_DRAFT_ROOTS")
-
     def build_engine() -> SessionEngine:
         ep_w = None
         if a.prefill == "native" and a.prefill_experts == "ep" and world > 1:
@@ -113,8 +129,8 @@ def main(argv=None) -> int:
             from naivert_b200.models.device_init import init_expert_rank_weights_device
             ep_w = init_expert_rank_weights_device(spec, rank, world, seed=a.seed, device=dev)
         eng = Engine.build(spec, rank=rank, tp=world, group=group, capacity=a.capacity, seed=a.seed, target_ckpt=target,
-                           draft_ckpt=draft, device=dev, prefill_chunk=a.prefill_chunk if a.prefill == "native" else 0,
-                           ep_weights=ep_w)
+                           draft_ckpt=draft, device=dev, dtype=a.dtype, ep_weights=ep_w,
+                           prefill_chunk=a.prefill_chunk if a.prefill == "native" or spec.draft is None else 0)
         if eng.prefill is not None and a.prefill_warm_chunks:
             with torch.cuda.stream(eng.round.stream):
                 eng.prefill.warm_chunks()
@@ -124,7 +140,7 @@ def main(argv=None) -> int:
         follower_loop(build_engine(), Commands(cpu_group))
         return 0
 
-    defaults = ServerDefaults(served_model=a.served_model_name or a.model, temperature=a.temperature, top_p=a.top_p, seed=a.seed,
+    defaults = ServerDefaults(served_model=a.served_model_name or a.model or spec.name, temperature=a.temperature, top_p=a.top_p, seed=a.seed,
                               repetition_penalty=a.repetition_penalty, frequency_penalty=a.frequency_penalty,
                               presence_penalty=a.presence_penalty, max_output_tokens=a.max_decode_tokens)
 

@@ -158,6 +158,59 @@ def step_table(eng, pos: int, steps: int = 4) -> List[dict]:
             for k, v in sorted(agg.items(), key=lambda kv: -kv[1][0])]
 
 
+def closest(prompt_len: int, chunk: int, layers: int, steps: int) -> dict:
+    """The speculative target (W8A8, same width, heads and experts) at equal depth: chunked prefill, its eight-row step, and the
+    kernels of both with the weight bytes they must read or the FLOPs they must do."""
+    from torch.profiler import ProfilerActivity, profile
+    spec, pk = resolve_model("naive-n0.5").with_layers(layers), peaks()
+    dev = torch.device("cuda", torch.cuda.current_device())
+    eng = Engine.build(spec, capacity=-(-(prompt_len + 256) // 128) * 128, device=dev, prefill_chunk=chunk)
+    try:
+        g = torch.Generator().manual_seed(0)
+        prompt = torch.randint(0, spec.vocab - 16, (prompt_len + 1,), generator=g, dtype=torch.int32).pin_memory()
+        pf, t = eng.prefill, eng.target
+        pf.warm_chunks([pf.quantum, chunk])
+        pf.run(prompt, 0, prompt_len)
+        pre_ms = sorted((pf.run(prompt, 0, prompt_len), pf.executor_ms())[1] for _ in range(3))[1]
+        pf.profile = True
+        pf.run(prompt, prompt_len - chunk, prompt_len)
+        stages = pf.stage_ms()
+        pf.profile = False
+        flops = {"qkv_gemm": sum(d["wqkv"].numel() for d in t.layers), "o_gemm": sum(d["wo"].w.numel() for d in t.layers)}
+        table = [{"stage": k, "ms": v, **({"tflops": round(2.0 * flops[k] * chunk / v * 1e-9, 1),
+                                          "roofline": round(2.0 * flops[k] * chunk / v * 1e-9 / pk["bf16_tflops"], 3)} if k in flops else {})}
+                 for k, v in sorted(stages.items(), key=lambda kv: -kv[1])]
+        pdl, t.pdl = t.pdl, False
+        t.set_inputs(torch.arange(8), prompt_len)
+        for _ in range(3):
+            t.step()
+        torch.cuda.synchronize()
+        with profile(activities=[ProfilerActivity.CUDA]) as prof:
+            for _ in range(steps):
+                t.step()
+            torch.cuda.synchronize()
+        t.pdl = pdl
+        by_name: Dict[str, List[float]] = {}
+        for e in prof.events():
+            n = e.name.split("(")[0]
+            by_name.setdefault(n, []).append(e.device_time if hasattr(e, "device_time") else e.cuda_time)
+        rt = spec.routing
+        active = rt.expert_count * (1 - (1 - rt.top_k / rt.expert_count) ** 8)
+        moe_bytes = active * 3 * rt.intermediate * spec.hidden
+        mean = {"moe_layer_kernel": moe_bytes, "6": sum(d["wqkv"].numel() for d in t.layers) / layers * 2}
+        rows = []
+        for n, v in sorted(by_name.items(), key=lambda kv: -sum(kv[1])):
+            r = {"kernel": n[-90:], "calls": len(v) // steps, "us_each": round(sum(v) / len(v), 2)}
+            by = moe_bytes if "moe_layer" in n else mean["6"] if "false, false, 6" in n else None
+            if by:
+                r.update(mb_each=round(by / 1e6, 1), roofline=round(by / (sum(v) / len(v)) * 1e-3 / pk["hbm_gbs"], 3))
+            rows.append(r)
+        return {"model": spec.name, "dtype": "fp8 weights and activations", "prefill_tokens_per_s": round(prompt_len / (pre_ms * 1e-3), 1),
+                "prefill_stages_last_chunk": table, "step8_kernels": rows, "step8_us_no_overlap": round(sum(sum(v) for v in by_name.values()) / steps, 1)}
+    finally:
+        eng.close()
+
+
 def run(model: str, prompt_len: int, steps: int, warmup: int, chunk: int, kernels: bool, layers: int = 0, clocks=None) -> dict:
     spec = resolve_model(model)
     if layers:

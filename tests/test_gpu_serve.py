@@ -21,9 +21,9 @@ def _free_port():
     return p
 
 
-def _serve(nproc):
+def _serve(nproc, model="small"):
     port = _free_port()
-    args = [os.path.join(ROOT, "examples", "serve_sessions.py"), "--model", "small", "--random-init", "--capacity", "4096",
+    args = [os.path.join(ROOT, "examples", "serve_sessions.py"), "--model", model, "--random-init", "--capacity", "4096",
             "--port", str(port), "--max-decode-tokens", "2048", "--log-level", "warning"]
     if nproc == 1:
         cmd = [sys.executable] + args
@@ -47,8 +47,8 @@ def _serve(nproc):
     raise RuntimeError("server did not become ready")
 
 
-def _check(base):
-    body = {"model": "small", "max_tokens": 48, "temperature": 0.8, "seed": 7,
+def _check(base, model="small"):
+    body = {"model": model, "max_tokens": 48, "temperature": 0.8, "seed": 7,
             "messages": [{"role": "user", "content": "Tell me about caches. " * 4}]}
     a = httpx.post(base + "/v1/messages", json=body, headers={"x-session-id": "s"}, timeout=120)
     assert a.status_code == 200, a.text
@@ -70,13 +70,13 @@ def _check(base):
     assert httpx.get(base + "/health").json()["slot"] == "IDLE"
 
 
-@pytest.mark.parametrize("nproc", [1, 2])
-def test_server_process(nproc):
+@pytest.mark.parametrize("nproc,model", [(1, "small"), (2, "small"), (1, "tumatar-small")])
+def test_server_process(nproc, model):
     if torch.cuda.device_count() < nproc:
         pytest.skip(f"needs {nproc} GPUs")
-    proc, base = _serve(nproc)
+    proc, base = _serve(nproc, model)
     try:
-        _check(base)
+        _check(base, model)
     finally:
         proc.terminate()
         try:

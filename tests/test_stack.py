@@ -121,6 +121,20 @@ def test_segment_bound_covers_every_distribution():
             assert worst <= bound
 
 
+def test_server_chooses_the_model_by_the_checkpoint(tmp_path):
+    import sys
+    sys.path.insert(0, os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "examples"))
+    import serve_sessions
+    spec, cfg = small()
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    assert serve_sessions.choose_model(None, str(tmp_path)).layers == spec.layers
+    assert serve_sessions.choose_model("tumatar-small", None) is resolve_model("tumatar-small")
+    assert serve_sessions.choose_model(None, None).name == "naive-n0.5"
+    assert serve_sessions.parse_args(["--dtype", "fp32"]).dtype == "fp32"
+    with pytest.raises(SystemExit):
+        serve_sessions.main(["--model", "tumatar-small", "--log-level", "error"])          # neither a checkpoint nor --random-init
+
+
 # --------------------------------------------------------------------------- the plain implementation
 def test_plain_convolution_and_recurrence_by_hand():
     x = torch.tensor([[1.0], [2.0], [3.0]], dtype=torch.float64)
