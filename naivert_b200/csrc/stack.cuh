@@ -155,6 +155,7 @@ enum StepPro : int {
   kProNorm = 1,        // input = rms(in) * in_w
   kProLoad = 2,        // input = in + group * in_gstride
   kProMerge = 3,       // input = softmax-merged latent output of head `group` from the attention partials
+  kProExperts = 4,     // inputs of the chosen experts side by side, each times its weight: out = sum_j W[ids[j]] (p[j] in[j])
 };
 enum StepEpi : int {
   kTEpiStore = 0,      // acc * scale; rows from `sig_from` on through a sigmoid
@@ -188,7 +189,9 @@ struct StepArgs {
   const __nv_bfloat16* w2;
   long long w_ld, w_gstride, w2_gstride;
   int groups, n;                // groups x n output rows
-  const int* group_ids;         // weight group of each output group (routed experts), null: identity
+  int segs;                     // chosen experts whose products are summed (kProExperts), else 1
+  const int* ids;               // [segs] their weight groups
+  const float* probs;           // [segs] their weights
   // output
   float* out;                   // [groups][n]
   float scale;
@@ -219,16 +222,6 @@ struct StepArgs {
   const int* pos0;
   int capacity;
   uint32_t* status;
-};
-
-struct StepDownArgs {            // routed experts, second product: out[n] = sum_j p[j] * (W[id_j] act_j)[n]
-  const float* act;             // [top_k][k]
-  const __nv_bfloat16* w;       // [experts][n][w_ld]
-  long long w_ld, w_gstride;
-  const int* ids;
-  const float* probs;
-  int top_k, k, n;
-  float* out;
 };
 
 // Context splits of the one-token attention: rows per split (a multiple of the kernels' 64-row tile) and the layout of a

@@ -6,8 +6,11 @@
 //              segment, plain load per group, merge of the attention partials
 //   epilogues  store / sigmoid, biased branches with the short convolution, output gate, two-product activations, the
 //              recurrence step
-// The first weights of a CTA are requested before griddepcontrol.wait: with programmatic dependent launch they travel under
-// the predecessor's tail.
+// Weights stream through shared memory: each of the sixteen warps owns a run of output rows and a ring of its own (three 4 KiB
+// slots) that one lane fills with bulk copies, so no two warps wait for one another inside the product.  The ring is filled
+// before griddepcontrol.wait, where the choice of weights does not depend on the predecessor.  Measured on B200: smaller rings
+// that let two kernels share an SM are slower (the successor's copies compete with the running product), and eight warps do not
+// keep up with the copies.
 #include "stack.cuh"
 #include "launch.hpp"
 #include "router.cuh"
@@ -18,35 +21,37 @@ using namespace nrt;
 
 namespace {
 
-constexpr int kStepThreads = 256;
+constexpr int kStepThreads = 512;
+constexpr int kPreN = 4096 / (kStepThreads * 4);       // float4 values per thread that cover the first 4096 elements
 
 // The input vector lives in shared memory as two planes of float4: chunk c of eight elements is plane0[c], plane1[c], so that
 // neighbouring lanes read neighbouring 16-byte words.
 __device__ __forceinline__ int plane_at(int c, int k8) { return ((c >> 2) & 1) * k8 * 4 + (c >> 3) * 4 + (c & 3); }
 
 __device__ __forceinline__ float dot8(const uint4& w, const float4& a, const float4& b, float acc) {
+  float t = bf16_lo(w.z) * b.x;                  // two chains
   acc = fmaf(bf16_lo(w.x), a.x, acc);
+  t = fmaf(bf16_hi(w.z), b.y, t);
   acc = fmaf(bf16_hi(w.x), a.y, acc);
+  t = fmaf(bf16_lo(w.w), b.z, t);
   acc = fmaf(bf16_lo(w.y), a.z, acc);
+  t = fmaf(bf16_hi(w.w), b.w, t);
   acc = fmaf(bf16_hi(w.y), a.w, acc);
-  acc = fmaf(bf16_lo(w.z), b.x, acc);
-  acc = fmaf(bf16_hi(w.z), b.y, acc);
-  acc = fmaf(bf16_lo(w.w), b.z, acc);
-  acc = fmaf(bf16_hi(w.w), b.w, acc);
-  return acc;
+  return acc + t;
 }
-__device__ __forceinline__ uint4 ld_stream(const uint4* p) {           // weights: read once per step
-  uint4 v;
-  asm volatile("ld.global.nc.L1::no_allocate.v4.b32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
-  return v;
+// untiled bulk copy of weights that are read once per step (16-byte addresses and size)
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar, uint64_t policy) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes.L2::cache_hint [%0], [%1], %2, [%3], %4;"
+               ::"r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)), "l"(policy)
+               : "memory");
 }
 
 // Values of the first kPreSpan elements that do not depend on the predecessor kernel, requested before the wait for it: the
 // norm weights, and the stream itself (written at least two launches back).
-constexpr int kPreSpan = kStepThreads * 16;
+constexpr int kPreSpan = kStepThreads * 4 * kPreN;
 struct Pre {
-  float4 x[4];
-  uint2 post[4], in[4];
+  float4 x[kPreN];
+  uint2 post[kPreN], in[kPreN];
 };
 __device__ __forceinline__ float4 bf4(const uint2& v) { return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y)); }
 __device__ __forceinline__ float4 ldcg4(const float* p) { return __ldcg(reinterpret_cast<const float4*>(p)); }
@@ -60,7 +65,7 @@ template <int PRO>
 __device__ __forceinline__ void preload(const StepArgs& a, Pre& p) {
   if (a.k & 3) return;
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
+  for (int i = 0; i < kPreN; ++i) {
     const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
     p.x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     p.post[i] = p.in[i] = make_uint2(0u, 0u);
@@ -88,28 +93,28 @@ __device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, flo
       emb = a.table + (size_t)t * K;
     }
     if ((K & 3) == 0) {
-      float4 v[4];
+      float4 v[kPreN];
       float ss = 0.f, sq = 0.f;
       if (PRO == kProResidual && a.y) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
+        for (int i = 0; i < kPreN; ++i) {
           const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
           v[i] = e < K ? ldcg4(a.y + e) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) ss += dot4(v[i]);
+        for (int i = 0; i < kPreN; ++i) ss += dot4(v[i]);
         for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) ss += dot4(ldcg4(a.y + e));
         ss = block_sum_f(ss, red);
       } else if (PRO == kProNorm) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
+        for (int i = 0; i < kPreN; ++i) {
           const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
           v[i] = e < K ? ldcg4(a.in_ + e) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
       }
       const float ry = PRO == kProResidual && a.y ? 1.0f / sqrtf(ss / (float)K + a.eps) : 0.f;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
+      for (int i = 0; i < kPreN; ++i) {
         const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
         if (e >= K) continue;
         if (PRO == kProResidual) {
@@ -140,7 +145,7 @@ __device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, flo
       const float rx = 1.0f / sqrtf(sq / (float)K + a.eps);
       const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
+      for (int i = 0; i < kPreN; ++i) {
         const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
         if (e < K) at4(e) = fma4(v[i], bf4(p.in[i]), rx, zero);
       }
@@ -174,6 +179,15 @@ __device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, flo
     } else {
       for (int c = threadIdx.x; c < K; c += kStepThreads) hs[plane_at(c, k8)] = __ldcg(in + c);
     }
+  } else if (PRO == kProExperts) {
+    const int total = a.segs * k8;
+    for (int j = 0; j < a.segs; ++j) {
+      const float pj = __ldcg(a.probs + j);
+      for (int c = threadIdx.x; c < k8 * 8; c += kStepThreads)
+        hs[plane_at(j * k8 * 8 + c, total)] = c < K ? __ldcg(a.in_ + (size_t)j * K + c) * pj : 0.f;
+    }
+    __syncthreads();
+    return;
   } else {                                                             // kProMerge
     // weights of the used splits, then a weighted sum of their outputs; threads beyond the row's float4 columns take other splits
     __shared__ float ws[kMaxSplits];
@@ -193,9 +207,9 @@ __device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, flo
     for (int i = 0; i < kStepThreads / 32; ++i) m = fmaxf(m, red[i]);
     const float w = (int)threadIdx.x < used ? expf(ms - m) : 0.f;
     const float l = block_sum_f(ls * w, red);
-    if ((int)threadIdx.x < used) ws[threadIdx.x] = w / l;
+    if ((int)threadIdx.x < used) ws[threadIdx.x] = w / l;           // used <= kMaxSplits <= threads
     int cols = 1;
-    while (cols < k4 && cols < kStepThreads) cols *= 2;
+    while (cols < k4 && cols < kStepThreads) cols *= 2;         // (both powers of two)
     const int subs = kStepThreads / cols, sub = (int)threadIdx.x / cols, c0 = (int)threadIdx.x & (cols - 1);
     __syncthreads();
     for (int i = threadIdx.x; i < 2 * k8; i += kStepThreads) hs4[i] = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -259,48 +273,101 @@ __device__ __forceinline__ void finish_row(const StepArgs& a, int g, int row, fl
   }
 }
 
-constexpr int kMaxStepSmem = 200 * 1024;
+constexpr int kWarps = kStepThreads / 32;
+constexpr int kSlot = 4096;                   // bytes of one ring slot of a warp
+constexpr int kMaxStepSmem = 225 * 1024;
 
-template <int PRO, int EPI, int RU, int U, bool ROUTE>
-__global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs a, const RouterArgs ra, const int rgroups,
-                                                                  const int rkeep, const int G) {
+// How a launch cuts its rows: host-computed, the same for every CTA.
+struct StepShape {
+  int k8;            // 16-byte pieces of a row (per expert)
+  int per_seg;       // slots of one row of one expert
+  int rows_slot;     // > 0: short rows, this many per slot (row-block form)
+  int G;             // lanes per row of the row-block form
+  int q, units, parts;   // rows per unit, units, units per group (per-group inputs)
+  int slots;         // ring slots per warp
+};
+
+template <int PRO, int EPI, bool ROUTE>
+__global__ void __launch_bounds__(kStepThreads, 2) stack_step_kernel(const StepArgs a, const RouterArgs ra, const int rgroups,
+                                                                     const int rkeep, const StepShape sh) {
   constexpr bool DUAL = EPI == kTEpiGlu || EPI == kTEpiRecur;
   constexpr bool PER_GROUP = PRO == kProLoad || PRO == kProMerge;
-  extern __shared__ float4 hs4[];
+  constexpr int CUT = DUAL ? kSlot / 32 : kSlot / 16;                  // pieces per slot and matrix
+  extern __shared__ __align__(128) uint8_t dyn[];
   __shared__ float red[33];
   __shared__ int s_ids[32];
-  float* hs = reinterpret_cast<float*>(hs4);
-  const int k8 = (a.k + 7) / 8;
-  const int lig = threadIdx.x & (G - 1), grp = threadIdx.x / G, gpc = kStepThreads / G;
-  const int rows_tile = gpc * RU;
-  const int tiles_g = (a.n + rows_tile - 1) / rows_tile;
-  const int tiles = a.groups * tiles_g;
-  uint4 wv[RU][U], wv2[DUAL ? RU : 1][DUAL ? U : 1];
+  __shared__ uint64_t bars[kWarps * 3];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  uint8_t* ring = dyn + warp * sh.slots * kSlot;
+  float* hs = reinterpret_cast<float*>(dyn + kWarps * sh.slots * kSlot);
+  const float4* hs4 = reinterpret_cast<const float4*>(hs);
+  uint64_t* bar = bars + warp * 3;
+  const int k8 = sh.k8, ld8 = (int)(a.w_ld / 8), total = a.segs * k8;
+  const int R = a.groups * a.n;
+  if (lane == 0) {
+    for (int i = 0; i < sh.slots; ++i) mbar_init(&bar[i], 1);
+    mbar_fence_init();
+  }
+  __syncwarp();
+  const uint64_t policy = l2_policy_evict_first();
 
-  auto fetch = [&](int tile, int c0) {
-    const int g = tile / tiles_g;
-    const int wg = ROUTE ? s_ids[g] : g;
-    const int row0 = (tile - g * tiles_g) * rows_tile + grp * RU;
-#pragma unroll
-    for (int i = 0; i < RU; ++i) {
-      const bool in = row0 + i < a.n;
-      const uint4* p = reinterpret_cast<const uint4*>(a.w + wg * a.w_gstride + (long long)(row0 + i) * a.w_ld);
-      const uint4* p2 = DUAL ? reinterpret_cast<const uint4*>(a.w2 + wg * a.w2_gstride + (long long)(row0 + i) * a.w_ld) : nullptr;
-#pragma unroll
-      for (int q = 0; q < U; ++q) {
-        const int c = c0 + q * G;
-        wv[i][q] = in && c < k8 ? ld_stream(p + c) : make_uint4(0u, 0u, 0u, 0u);
-        if (DUAL) wv2[DUAL ? i : 0][DUAL ? q : 0] = in && c < k8 ? ld_stream(p2 + c) : make_uint4(0u, 0u, 0u, 0u);
-      }
+  // this warp's rows of a unit; the request cursor runs ahead of the consuming one by up to `slots`
+  int w_end = 0, i_row = 0, i_seg = 0, i_sub = 0, i_slot = 0, issued = 0, used = 0;
+  auto group_of = [&](int row) { return a.groups == 1 ? 0 : row / a.n; };
+  auto rows_at = [&](int row) { return min(min(sh.rows_slot, w_end - row), a.n * (group_of(row) + 1) - row); };
+  auto open_unit = [&](int u) {
+    int lo, hi;
+    if (PER_GROUP) {
+      const int g = u / sh.parts, part = u - g * sh.parts;
+      lo = g * a.n + min(a.n, part * sh.q);
+      hi = g * a.n + min(a.n, (part + 1) * sh.q);
+    } else {
+      lo = min(R, u * sh.q);
+      hi = min(R, lo + sh.q);
+    }
+    const int per = (hi - lo + kWarps - 1) / kWarps;
+    i_row = min(hi, lo + warp * per);
+    w_end = min(hi, i_row + per);
+    i_seg = i_sub = 0;
+    return i_row;
+  };
+  auto request = [&]() {
+    const int slot = i_slot, g = group_of(i_row), r = i_row - g * a.n;
+    uint8_t* dst = ring + slot * kSlot;
+    long long off;
+    int count, rows = 1, wg = ROUTE ? s_ids[g] : PRO == kProExperts ? s_ids[0] : g;
+    if (sh.rows_slot > 0) {
+      rows = rows_at(i_row);
+      count = rows * ld8;
+      off = (long long)r * a.w_ld;
+    } else {
+      if (PRO == kProExperts) wg = s_ids[i_seg];
+      count = min(CUT, k8 - i_sub * CUT);
+      off = (long long)r * a.w_ld + i_sub * CUT * 8;
+    }
+    if (lane == 0) {
+      mbar_expect_tx(&bar[slot], (DUAL ? 2u : 1u) * count * 16u);
+      bulk_load(dst, a.w + wg * a.w_gstride + off, count * 16u, &bar[slot], policy);
+      if (DUAL) bulk_load(dst + CUT * 16, a.w2 + wg * a.w2_gstride + off, count * 16u, &bar[slot], policy);
+    }
+    ++issued;
+    if (++i_slot == sh.slots) i_slot = 0;
+    if (sh.rows_slot > 0) i_row += rows;
+    else if (++i_sub == sh.per_seg) {
+      i_sub = 0;
+      if (++i_seg == a.segs) { i_seg = 0; ++i_row; }
     }
   };
+  auto fill = [&]() {
+    while (i_row < w_end && issued - used < sh.slots) request();
+  };
 
-  // each CTA owns a contiguous run of tiles, so a per-group input is loaded once per group it meets
-  const int per_cta = (tiles + (int)gridDim.x - 1) / (int)gridDim.x;
-  const int tile_lo = (int)blockIdx.x * per_cta, tile_hi = min(tiles, tile_lo + per_cta);
-  if (!ROUTE && tile_lo < tile_hi) fetch(tile_lo, lig);
+  int unit = blockIdx.x;
+  int row = open_unit(unit);
+  constexpr bool EARLY = !ROUTE && PRO != kProExperts;                 // which weights is known before the predecessor ends
+  if (EARLY) fill();
   Pre pre;
-  if constexpr (PRO == kProResidual) preload<PRO>(a, pre);       // (a normed input vector may come from the predecessor itself)
+  if constexpr (PRO == kProResidual) preload<PRO>(a, pre);             // (a normed input may come from the predecessor itself)
   griddep_wait();
   griddep_launch();
   const int pos = a.pos0 ? *reinterpret_cast<const volatile int*>(a.pos0) : 0;
@@ -311,11 +378,13 @@ __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs
     if ((int)threadIdx.x < ra.top_k) s_ids[threadIdx.x] = sm.tk_id[0][threadIdx.x];
     __syncthreads();
   }
-  int slot = 1;
-  if (EPI == kTEpiRecur) {
-    slot = state_slot(a.tags, pos, a.status);
-    if (slot < 0) return;
+  if (PRO == kProExperts) {
+    if ((int)threadIdx.x < a.segs) s_ids[threadIdx.x] = __ldcg(a.ids + threadIdx.x);
+    __syncthreads();
   }
+  if (!EARLY) fill();
+  int slot = 1;
+  if (EPI == kTEpiRecur) slot = state_slot(a.tags, pos, a.status);
   if constexpr (PRO == kProNorm) preload<PRO>(a, pre);
   if (!PER_GROUP) load_input<PRO>(a, 0, k8, hs, red, pre, pos);
   if (PRO == kProNorm && a.lat_in && blockIdx.x == gridDim.x - 1 && pos >= 0 && pos < a.capacity) {
@@ -326,170 +395,153 @@ __global__ void __launch_bounds__(kStepThreads) stack_step_kernel(const StepArgs
     for (int c = threadIdx.x; c < a.lat_rank; c += kStepThreads)
       store_act(a.lat_cache, (long long)pos * a.lat_ld + c, __ldcg(a.lat_in + c) * rs * bf(a.lat_w + c), a.f32);
   }
-  int cur = -1;
-  for (int tile = tile_lo; tile < tile_hi; ++tile) {
-    const int g = tile / tiles_g;
-    if (PER_GROUP && g != cur) {
-      if (cur >= 0) __syncthreads();
-      load_input<PRO>(a, g, k8, hs, red, pre, pos);
-      cur = g;
-    }
-    float acc[RU], acc2[RU];
+
+  bool ok = true;
+  int u_slot = 0;
+  uint32_t u_phase = 0;
+  while (true) {
+    if (PER_GROUP) load_input<PRO>(a, unit / sh.parts, k8, hs, red, pre, pos);
+    // results of up to 32 finished rows wait in the lanes, then all lanes run the epilogue at once
+    float acc = 0.f, acc2 = 0.f, res = 0.f, res2 = 0.f;
+    int ready = 0, first = row, seg = 0, sub = 0;
+    auto flush = [&]() {
+      if (lane < ready && slot >= 0) {
+        const int at = first + lane, g = group_of(at);
+        finish_row<EPI>(a, g, at - g * a.n, res, res2, pos, slot);
+      }
+      first += ready;
+      ready = 0;
+      __syncwarp();
+    };
+    while (row < w_end && ok) {
+      const int s = u_slot;
+      ok = __all_sync(0xffffffffu, mbar_wait(&bar[s], u_phase, a.status, kSiteTmaFull | (warp & 7)));
+      if (!ok) break;
+      const uint4* w0 = reinterpret_cast<const uint4*>(ring + s * kSlot);
+      const uint4* w1 = w0 + CUT;
+      if (sh.rows_slot > 0) {
+        const int rows = rows_at(row), lig = lane & (sh.G - 1), mine = lane / sh.G, per = 32 / sh.G;
+        if (ready + rows > 32) flush();
+        for (int r0 = 0; r0 < rows; r0 += per) {
+          const int rr = r0 + mine;
+          float v = 0.f, v2 = 0.f;
+          if (rr < rows)
+            for (int c = lig; c < k8; c += sh.G) {
+              const float4 x0 = hs4[c], x1 = hs4[total + c];
+              v = dot8(w0[rr * ld8 + c], x0, x1, v);
+              if (DUAL) v2 = dot8(w1[rr * ld8 + c], x0, x1, v2);
+            }
+          for (int o = sh.G >> 1; o > 0; o >>= 1) {
+            v += __shfl_xor_sync(0xffffffffu, v, o);
+            if (DUAL) v2 += __shfl_xor_sync(0xffffffffu, v2, o);
+          }
+          const int want = lane - (ready + r0);                        // row of this pass that belongs to this lane
+          const int src = (want * sh.G) & 31;
+          const float t = __shfl_sync(0xffffffffu, v, src), t2 = DUAL ? __shfl_sync(0xffffffffu, v2, src) : 0.f;
+          if (want >= 0 && want < per && r0 + want < rows) { res = t; res2 = t2; }
+        }
+        ready += rows;
+        row += rows;
+      } else {
+        const int count = min(CUT, k8 - sub * CUT);
+        const float4* h0 = hs4 + seg * k8 + sub * CUT;
+        const float4* h1 = h0 + total;
 #pragma unroll
-    for (int i = 0; i < RU; ++i) acc[i] = acc2[i] = 0.f;
-#pragma unroll 1
-    for (int c0 = lig; c0 < k8 || c0 == lig; c0 += G * U) {
-      if (c0 != lig || ROUTE || tile != tile_lo) fetch(tile, c0);
-#pragma unroll
-      for (int q = 0; q < U; ++q) {
-        const int c = c0 + q * G;
-        if (c < k8) {
-          const float4 x0 = hs4[c], x1 = hs4[k8 + c];
-#pragma unroll
-          for (int i = 0; i < RU; ++i) {
-            acc[i] = dot8(wv[i][q], x0, x1, acc[i]);
-            if (DUAL) acc2[i] = dot8(wv2[DUAL ? i : 0][DUAL ? q : 0], x0, x1, acc2[i]);
+        for (int i = 0; i < CUT / 32; ++i) {
+          const int c = lane + 32 * i;
+          if (c < count) {
+            const float4 x0 = h0[c], x1 = h1[c];
+            acc = dot8(w0[c], x0, x1, acc);
+            if (DUAL) acc2 = dot8(w1[c], x0, x1, acc2);
           }
         }
+        if (++sub == sh.per_seg) { sub = 0; ++seg; }
+        if (seg == a.segs) {
+          seg = 0;
+          const float v = lane_sum(acc), v2 = DUAL ? lane_sum(acc2) : 0.f;
+          acc = acc2 = 0.f;
+          if (lane == ready) { res = v; res2 = v2; }
+          ++row;
+          if (++ready == 32) flush();
+        }
       }
+      ++used;
+      if (++u_slot == sh.slots) { u_slot = 0; u_phase ^= 1; }
+      __syncwarp();                                                    // every lane has read the slot before it is requested anew
+      fill();
     }
-#pragma unroll
-    for (int i = 0; i < RU; ++i)
-      for (int o = G >> 1; o > 0; o >>= 1) {
-        acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], o);
-        if (DUAL) acc2[i] += __shfl_xor_sync(0xffffffffu, acc2[i], o);
-      }
-    if (lig == 0) {
-      const int row0 = (tile - g * tiles_g) * rows_tile + grp * RU;
-#pragma unroll
-      for (int i = 0; i < RU; ++i)
-        if (row0 + i < a.n) finish_row<EPI>(a, g, row0 + i, acc[i], acc2[i], pos, slot);
-    }
-    __syncwarp();
+    flush();
+    unit += gridDim.x;
+    if (unit >= sh.units) break;
+    row = open_unit(unit);
+    if (ok) fill();
+    __syncthreads();                                                   // the input vector is replaced
   }
   // A CTA that starts after this store still finds `pos` in its own slot: only the other slot's tag changes.
-  if (EPI == kTEpiRecur && blockIdx.x == 0 && threadIdx.x == 0) {
+  if (EPI == kTEpiRecur && slot >= 0 && blockIdx.x == 0 && threadIdx.x == 0) {
     a.tags[1 - slot] = pos + 1;
     if (pos == 0) a.tags[1] = -1;
   }
+  if (!ok) drain_on_error(a.status);
 }
 
-// Second product of the routed experts: out[n] = sum_j p_j (W[id_j] act_j)[n], warp per RU rows.
-template <int RU, int U>
-__global__ void __launch_bounds__(kStepThreads) stack_down_kernel(const StepDownArgs a) {
-  extern __shared__ float4 hs4[];
-  __shared__ int s_ids[32];
-  float* hs = reinterpret_cast<float*>(hs4);
-  const int k8 = (a.k + 7) / 8, total = a.top_k * k8;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  griddep_wait();
-  griddep_launch();
-  if ((int)threadIdx.x < a.top_k) s_ids[threadIdx.x] = __ldcg(a.ids + threadIdx.x);
-  for (int j = 0; j < a.top_k; ++j) {
-    const float p = __ldcg(a.probs + j);
-    for (int c = threadIdx.x; c < k8 * 8; c += kStepThreads)
-      hs[plane_at(j * k8 * 8 + c, total)] = c < a.k ? __ldcg(a.act + (size_t)j * a.k + c) * p : 0.f;
-  }
-  __syncthreads();
-  for (int row0 = (blockIdx.x * 8 + warp) * RU; row0 < a.n; row0 += gridDim.x * 8 * RU) {
-    float acc[RU];
-#pragma unroll
-    for (int i = 0; i < RU; ++i) acc[i] = 0.f;
-#pragma unroll 1
-    for (int j = 0; j < a.top_k; ++j) {
-      const uint4* base = reinterpret_cast<const uint4*>(a.w + s_ids[j] * a.w_gstride + (long long)row0 * a.w_ld);
-      const int ld8 = (int)(a.w_ld / 8);
-#pragma unroll 1
-      for (int c0 = lane; c0 < k8; c0 += 32 * U) {
-        uint4 wv[RU][U];
-#pragma unroll
-        for (int q = 0; q < U; ++q)
-#pragma unroll
-          for (int i = 0; i < RU; ++i)
-            wv[i][q] = c0 + q * 32 < k8 && row0 + i < a.n ? ld_stream(base + i * ld8 + c0 + q * 32) : make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll
-        for (int q = 0; q < U; ++q) {
-          const int c = c0 + q * 32;
-          if (c < k8) {
-            const float4 x0 = hs4[j * k8 + c], x1 = hs4[total + j * k8 + c];
-#pragma unroll
-            for (int i = 0; i < RU; ++i) acc[i] = dot8(wv[i][q], x0, x1, acc[i]);
-          }
-        }
-      }
-    }
-    __syncwarp();
-#pragma unroll
-    for (int i = 0; i < RU; ++i) {
-      const float v = lane_sum(acc[i]);
-      if (lane == 0 && row0 + i < a.n) a.out[row0 + i] = v;
-    }
-  }
-}
-
-int lanes_of(int k8) {
-  int G = 4;
-  while (G < 32 && G < k8) G *= 2;
-  return G;
-}
-
-template <int PRO, int EPI, int RU, int U, bool ROUTE>
-struct StepLaunch {
-  // CTAs of this kernel that are resident at once with `smem` bytes each
-  static int resident(size_t smem) {
-    static size_t seen[8];
-    static int value[8], count = 0;
-    for (int i = 0; i < count; ++i)
-      if (seen[i] == smem) return value[i];
-    auto* kern = stack_step_kernel<PRO, EPI, RU, U, ROUTE>;
-    if (count == 0 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxStepSmem) != cudaSuccess) return -1;
-    int per = 0, dev = 0, sms = 148;
+int step_sms() {
+  static int sms = 0;
+  if (!sms) {
+    int dev = 0;
     cudaGetDevice(&dev);
-    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per, kern, kStepThreads, smem) != cudaSuccess || per < 1) per = 1;
-    if (count < 8) { seen[count] = smem; value[count] = per * sms; ++count; }
-    return per * sms;
+    if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms < 1) sms = 148;
   }
-  static long long tiles(const StepArgs& a) {
-    const int rows_tile = kStepThreads / lanes_of((a.k + 7) / 8) * RU;
-    return (long long)a.groups * ((a.n + rows_tile - 1) / rows_tile);
-  }
-  static double balance(const StepArgs& a) {            // busy share of the resident CTAs
-    const long long t = tiles(a), res = resident((size_t)((a.k + 7) / 8) * 32);
-    if (res < 1) return 0.0;
-    const long long grid = t < res ? t : res, per = (t + grid - 1) / grid;
-    return (double)t / (double)(per * res);
-  }
-  static int run(const StepArgs& a, const RouterArgs& r, int groups, int keep, cudaStream_t stream, bool pdl) {
-    const int k8 = (a.k + 7) / 8;
-    const size_t smem = (size_t)k8 * 32;
-    const long long t = tiles(a);
-    if (smem > kMaxStepSmem || t < 1 || t > 0x7fffffffLL) return -7;
-    const int res = resident(smem);
-    if (res < 1) return -8;
-    return launch_pdl(stack_step_kernel<PRO, EPI, RU, U, ROUTE>, dim3((unsigned)(t < res ? t : res)), dim3(kStepThreads), smem, stream, pdl, a,
-                      r, groups, keep, lanes_of(k8));
-  }
-};
+  return sms;
+}
 
-// Rows per lane group: the largest count that still spreads the rows evenly over the resident CTAs.
 template <int PRO, int EPI, bool ROUTE>
-int pick_step(const StepArgs& a, const RouterArgs& r, int groups, int keep, cudaStream_t stream, bool pdl) {
-  if constexpr (EPI == kTEpiGlu || EPI == kTEpiRecur) {
-    using A = StepLaunch<PRO, EPI, 2, 2, ROUTE>;
-    using B = StepLaunch<PRO, EPI, 1, 4, ROUTE>;
-    return A::balance(a) + 0.05 >= B::balance(a) ? A::run(a, r, groups, keep, stream, pdl) : B::run(a, r, groups, keep, stream, pdl);
-  } else {
-    using A = StepLaunch<PRO, EPI, 2, 4, ROUTE>;
-    using B = StepLaunch<PRO, EPI, 1, 8, ROUTE>;
-    return A::balance(a) + 0.05 >= B::balance(a) ? A::run(a, r, groups, keep, stream, pdl) : B::run(a, r, groups, keep, stream, pdl);
+int launch_step(const StepArgs& a, const RouterArgs& r, int groups, int keep, cudaStream_t stream, bool pdl) {
+  constexpr bool DUAL = EPI == kTEpiGlu || EPI == kTEpiRecur;
+  constexpr bool PER_GROUP = PRO == kProLoad || PRO == kProMerge;
+  constexpr int CUT = DUAL ? kSlot / 32 : kSlot / 16;
+  auto* kern = stack_step_kernel<PRO, EPI, ROUTE>;
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxStepSmem - (ROUTE ? 8192 : 0));
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
   }
+  const long long R = (long long)a.groups * a.n;
+  if (R > 0x7fffffffLL) return -3;
+  StepShape s = {};
+  s.k8 = (a.k + 7) / 8;
+  const int ld8 = (int)(a.w_ld / 8);
+  if (a.segs == 1 && ld8 * 2 <= CUT) {                   // short rows travel in blocks
+    s.rows_slot = CUT / ld8 < 32 ? CUT / ld8 : 32;
+    s.G = 1;
+    while (s.G < 32 && s.G < s.k8) s.G *= 2;
+  } else {
+    s.per_seg = (s.k8 + CUT - 1) / CUT;
+  }
+  const int sms = step_sms();
+  if (PER_GROUP) {
+    s.parts = sms / a.groups > 1 ? sms / a.groups : 1;
+    s.q = (a.n + s.parts - 1) / s.parts;
+    s.parts = (a.n + s.q - 1) / s.q;
+    s.units = a.groups * s.parts;
+  } else {
+    const long long want = (R + kWarps - 1) / kWarps;
+    const int grid = (int)(want < sms ? want : sms);
+    s.q = (int)((R + grid - 1) / grid);
+    s.units = (int)((R + s.q - 1) / s.q);
+    s.parts = 1;
+  }
+  const int hs_bytes = a.segs * s.k8 * 32, limit = kMaxStepSmem - (ROUTE ? 8192 : 0);
+  for (s.slots = 3; s.slots > 1 && kWarps * s.slots * kSlot + hs_bytes > limit; --s.slots) {}
+  const int smem = kWarps * s.slots * kSlot + hs_bytes;
+  if (smem > limit) return -7;
+  return launch_pdl(kern, dim3(s.units < sms ? s.units : sms), dim3(kStepThreads), smem, stream, pdl, a, r, groups, keep, s);
 }
 
 }  // namespace
 
 extern "C" int nrt_step_args_size() { return (int)sizeof(StepArgs); }
-extern "C" int nrt_step_down_args_size() { return (int)sizeof(StepDownArgs); }
 
 // `router` (expert form of the two-product epilogue): RouterArgs with the token's filled score row; the selection runs in every
 // CTA and CTA 0 publishes it.
@@ -499,37 +551,22 @@ extern "C" int nrt_stack_step(int pro, int epi, const void* args, const void* ro
   RouterArgs r;
   memset(&r, 0, sizeof(r));
   if (router) memcpy(&r, router, sizeof(r));
-  if (a.n < 1 || a.k < 1 || a.groups < 1 || a.w_ld % 8 || a.w_gstride % 8 || a.w2_gstride % 8) return -3;
+  if (a.n < 1 || a.k < 1 || a.groups < 1 || a.segs < 1 || a.segs > 32 || (a.segs > 1 && pro != kProExperts) || a.w_ld % 8 || a.w_gstride % 8 || a.w2_gstride % 8) return -3;
   if (router && (r.experts > 256 || r.top_k > 32 || r.rows != 1 || groups < 1 || groups > 32 || r.experts % groups)) return -3;
   if (epi == kTEpiConv && (a.hist_rows < 1 || a.hist_rows < 2 * (a.taps - 1) || a.groups != 1)) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const bool p = pdl != 0;
 #define NRT_CASE(P, E) \
-  if (pro == P && epi == E && !router) return pick_step<P, E, false>(a, r, groups, keep, s, p);
+  if (pro == P && epi == E && !router) return launch_step<P, E, false>(a, r, groups, keep, s, p);
   NRT_CASE(kProResidual, kTEpiStore)
   NRT_CASE(kProResidual, kTEpiConv)
   NRT_CASE(kProResidual, kTEpiGlu)
   NRT_CASE(kProNorm, kTEpiStore)
   NRT_CASE(kProLoad, kTEpiStore)
+  NRT_CASE(kProExperts, kTEpiStore)
   NRT_CASE(kProMerge, kTEpiGate)
   NRT_CASE(kProLoad, kTEpiRecur)
 #undef NRT_CASE
-  if (pro == kProNorm && epi == kTEpiGlu && router) return pick_step<kProNorm, kTEpiGlu, true>(a, r, groups, keep, s, p);
+  if (pro == kProNorm && epi == kTEpiGlu && router) return launch_step<kProNorm, kTEpiGlu, true>(a, r, groups, keep, s, p);
   return -2;
-}
-
-extern "C" int nrt_stack_down(const void* args, void* stream, int pdl) {
-  StepDownArgs a;
-  memcpy(&a, args, sizeof(a));
-  if (a.n < 1 || a.k < 1 || a.top_k < 1 || a.top_k > 32 || a.w_ld % 8 || a.w_gstride % 8) return -3;
-  const size_t smem = (size_t)a.top_k * ((a.k + 7) / 8) * 32;
-  if (smem > kMaxStepSmem) return -7;
-  auto run = [&](auto* kern, int ru) {
-    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxStepSmem);
-    if (e != cudaSuccess) return (int)e;
-    const int tiles = (a.n + 8 * ru - 1) / (8 * ru);
-    return launch_pdl(kern, dim3(tiles < 592 ? tiles : 592), dim3(kStepThreads), smem, reinterpret_cast<cudaStream_t>(stream), pdl != 0, a);
-  };
-  if (a.n >= 8 * 2 * 296) return run(stack_down_kernel<2, 4>, 2);
-  return run(stack_down_kernel<1, 8>, 1);
 }

@@ -18,6 +18,7 @@ from .spec import MoeRoutingSpec
 MAX_EXPERTS, MAX_TOP_K, MAX_GROUPS = 256, 32, 32
 MAX_HEAD_DIM = 512
 MAX_RANK = 4096
+MAX_STEP_INPUT = 40000           # values a product of the one-token step can take in
 
 
 @dataclass(frozen=True)
@@ -157,6 +158,12 @@ class StackSpec:
                 raise ValueError(f"{self.name}: {what}")
         need(self.hidden >= 1 and self.vocab >= 1 and len(self.layers) >= 1, "empty model")
         need(self.hidden <= 25600, "width above 25600")
+        for i, layer in enumerate(self.layers):
+            m, f = layer.mixer, layer.mlp
+            widest = m.heads * _pad(m.vdim, 8) if m.kind == "latent_attention" else getattr(m, "width", 0)
+            if f is not None:
+                widest = max(widest, _pad(f.ff, 8) * (f.routing.top_k if f.kind == "moe" else 1))
+            need(widest <= MAX_STEP_INPUT, f"layer {i}: a product of the step would take in {widest} values, at most {MAX_STEP_INPUT}")
         for i, layer in enumerate(self.layers):
             m, f = layer.mixer, layer.mlp
             if m.kind == "latent_attention":

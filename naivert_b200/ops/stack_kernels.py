@@ -16,13 +16,13 @@ from .build import load_library
 
 VP = C.c_void_p
 _G = generate_from("stack.cuh", ["StackGemmArgs", "StackRowArgs", "LatentPrepArgs", "LatentAttnArgs", "LatentDecodeArgs",
-                                 "RecurrenceArgs", "MoeGatherArgs", "StepArgs", "StepDownArgs"])
+                                 "RecurrenceArgs", "MoeGatherArgs", "StepArgs"])
 StackGemmArgs, StackRowArgs, LatentPrepArgs = _G["StackGemmArgs"], _G["StackRowArgs"], _G["LatentPrepArgs"]
 LatentAttnArgs, LatentDecodeArgs, RecurrenceArgs = _G["LatentAttnArgs"], _G["LatentDecodeArgs"], _G["RecurrenceArgs"]
-MoeGatherArgs, StepArgs, StepDownArgs = _G["MoeGatherArgs"], _G["StepArgs"], _G["StepDownArgs"]
+MoeGatherArgs, StepArgs = _G["MoeGatherArgs"], _G["StepArgs"]
 
 EPI_STORE, EPI_BIAS, EPI_TRANSPOSE, EPI_CLAMPED_GLU, EPI_SILU_GLU = 0, 1, 2, 3, 4
-PRO_RESIDUAL, PRO_NORM, PRO_LOAD, PRO_MERGE = 0, 1, 2, 3
+PRO_RESIDUAL, PRO_NORM, PRO_LOAD, PRO_MERGE, PRO_EXPERTS = 0, 1, 2, 3, 4
 TEPI_STORE, TEPI_CONV, TEPI_GATE, TEPI_GLU, TEPI_RECUR = 0, 1, 2, 3, 4
 
 # library entry points of the family and the argument struct each reads
@@ -32,8 +32,7 @@ ENTRIES = {"nrt_stack_gemm": ("StackGemmArgs", "nrt_stack_gemm_args_size"), "nrt
            "nrt_latent_attn_tc": ("LatentAttnArgs", "nrt_latent_attn_args_size"),
            "nrt_latent_decode": ("LatentDecodeArgs", "nrt_latent_decode_args_size"),
            "nrt_stack_conv": ("RecurrenceArgs", "nrt_recurrence_args_size"), "nrt_stack_scan": ("RecurrenceArgs", "nrt_recurrence_args_size"),
-           "nrt_moe_gather": ("MoeGatherArgs", "nrt_moe_gather_args_size"), "nrt_stack_step": ("StepArgs", "nrt_step_args_size"),
-           "nrt_stack_down": ("StepDownArgs", "nrt_step_down_args_size")}
+           "nrt_moe_gather": ("MoeGatherArgs", "nrt_moe_gather_args_size"), "nrt_stack_step": ("StepArgs", "nrt_step_args_size")}
 
 _lib = None
 
@@ -132,6 +131,3 @@ def step(pro: int, epi: int, args: StepArgs, router: Optional[K.RouterArgs], gro
     K.check(lib().nrt_stack_step(pro, epi, C.byref(args), C.byref(router) if router is not None else None, groups, keep, _stream(),
                                  int(pdl)), "stack step")
 
-
-def down(args: StepDownArgs, pdl: bool) -> None:
-    K.check(lib().nrt_stack_down(C.byref(args), _stream(), int(pdl)), "expert down")

@@ -203,14 +203,14 @@ class StackRuntime:
     def _args(self, w: Packed, out: torch.Tensor, groups: int = 1, n: Optional[int] = None) -> "S.StepArgs":
         a = S.StepArgs()
         a.w, a.w_ld, a.k = w.w.data_ptr(), w.ld, w.k
-        a.groups, a.n = groups, w.n if n is None else n
+        a.groups, a.n, a.segs = groups, w.n if n is None else n, 1
         a.w_gstride = w.n * w.ld if w.z > 1 else a.n * w.ld
         a.out, a.scale, a.sig_from, a.eps = out.data_ptr(), 1.0, 0x7FFFFFFF, self.spec.norm_eps
         a.pos0, a.capacity, a.status, a.f32 = self.ctrl.data_ptr(), self.capacity, self.fab.status.data_ptr(), int(self.f32)
         return a
 
     def _build_step(self) -> None:
-        """Launch list: ("step", prologue, epilogue, args, router, groups, keep) | ("attn", args) | ("down", args)."""
+        """Launch list: ("step", prologue, epilogue, args, router, groups, keep) | ("attn", args)."""
         s = self.spec
         ops: List[tuple] = []
         cur = 0                                                       # buffer that holds the stream
@@ -300,11 +300,9 @@ class StackRuntime:
                 q.sigmoid, q.normalize, q.route_scale = 1, int(rt.normalize_top_k), rt.route_scale
                 q.scores, q.topk_ids, q.topk_p = self.sscores.data_ptr(), self.sids.data_ptr(), self.sprobs.data_ptr()
                 step(S.PRO_NORM, S.TEPI_GLU, a, q, rt.group_count, rt.limited_group_count)
-                b = S.StepDownArgs()
-                b.act, b.w, b.w_ld, b.w_gstride = self.sact.data_ptr(), d["down"].w.data_ptr(), d["down"].ld, d["down"].n * d["down"].ld
-                b.ids, b.probs, b.top_k, b.k, b.n, b.out = (self.sids.data_ptr(), self.sprobs.data_ptr(), rt.top_k, f.ff, s.hidden,
-                                                            self.sy.data_ptr())
-                ops.append(("down", b))
+                a = self._args(d["down"], self.sy)
+                a.in_, a.segs, a.ids, a.probs = self.sact.data_ptr(), rt.top_k, self.sids.data_ptr(), self.sprobs.data_ptr()
+                step(S.PRO_EXPERTS, S.TEPI_STORE, a)
             y_from = d["norm2b"]
         self._body = ops
         a = residual(self._args(self.head, self.logits), self.g_final)
@@ -316,10 +314,8 @@ class StackRuntime:
         for op in self._body + ([self._head_op] if head else []):
             if op[0] == "step":
                 S.step(op[1], op[2], op[3], op[4], op[5], op[6], pdl)
-            elif op[0] == "attn":
-                S.latent_decode(op[1], pdl)
             else:
-                S.down(op[1], pdl)
+                S.latent_decode(op[1], pdl)
 
     # ------------------------------------------------------------------ host helpers (not on the hot path)
     def set_inputs(self, tokens, pos0: int) -> None:

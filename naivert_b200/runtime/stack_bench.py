@@ -192,7 +192,7 @@ def closest(prompt_len: int, chunk: int, layers: int, steps: int) -> dict:
         t.pdl = pdl
         by_name: Dict[str, List[float]] = {}
         for e in prof.events():
-            n = e.name.split("(")[0]
+            n = e.name.replace("(anonymous namespace)::", "").split("(")[0]
             by_name.setdefault(n, []).append(e.device_time if hasattr(e, "device_time") else e.cuda_time)
         rt = spec.routing
         active = rt.expert_count * (1 - (1 - rt.top_k / rt.expert_count) ** 8)
