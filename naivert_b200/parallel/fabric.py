@@ -100,6 +100,8 @@ class Fabric:
             raise RuntimeError(f"device wait gave up at site 0x{code:x} (rank {self.rank}): {explain_status(code)}")
 
     def close(self) -> None:
+        if not self._opened and not self._local:          # a single rank has no peer memory to give back
+            return
         L = K.lib()
         for q in self._opened:
             L.nrt_ipc_close(C.c_void_p(q))

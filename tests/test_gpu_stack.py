@@ -441,6 +441,15 @@ def test_replayed_prompt_equals_chunks():
         eng.close()
 
 
+def test_stepwise_use_loads_only_the_stack_library():
+    """A process that feeds tokens step by step never builds or loads the speculative target's library."""
+    code = ("import torch; from naivert_b200.models import tumatar; from naivert_b200.ops import build; from naivert_b200.runtime.engine import Engine\n"
+            "e = Engine.build(tumatar.small_spec(), capacity=64, device=torch.device('cuda', 0))\n"
+            "e.extend([1, 2, 3], [2]); e.extend([4], [0]); e.close(); print(sorted(build._LIBS))")
+    r = subprocess.run([sys.executable, "-c", code], cwd=ROOT, capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0 and r.stdout.split("\n")[-2] == "['stack']", r.stdout + r.stderr[-2000:]
+
+
 def test_checkpoint_and_trace_program(tmp_path):
     """A written checkpoint, replayed by the command line program in both numeric forms."""
     from naivert_b200.models import tumatar
