@@ -14,7 +14,6 @@ is captured into the round's CUDA graph.  Prompt chunks go through ``prefill/sta
 """
 from __future__ import annotations
 
-import ctypes as C
 from dataclasses import dataclass
 from typing import Dict, List, Optional, Tuple
 
