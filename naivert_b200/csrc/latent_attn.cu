@@ -1,6 +1,8 @@
 // Latent attention: causal softmax attention whose keys and values are linear images of one cached latent per token.
 //   chunk path   keys and values of a block of cached positions are expanded by products (stack_gemm.cu), then
 //                attended by the rows of the chunk; the output gate is applied as the result is stored
+//                (the same kernels serve grouped-query attention from a key / value cache: `group` heads share a key head,
+//                `window` limits a query to the keys of its own chunk)
 //   one-token    the query is taken into the latent space instead, and the cached latents serve as keys and values
 //                of all heads at once (kernels below: split over the context, merged by the next product)
 #include "stack.cuh"
@@ -23,9 +25,11 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(const LatentAttnA
   if (unit >= a.rows * a.heads) return;
   const int r = unit / a.heads, h = unit % a.heads;
   const int pos = *a.pos0 + r;
-  const int n = min(a.kv_rows, pos + 1 - a.kv0);            // visible keys of this block
-  const long long kld = (long long)a.heads * a.dim, vld = (long long)a.heads * a.vdim;
-  for (int d = lane; d < a.dim; d += 32) sq[warp][d] = load_act(a.q, (long long)r * kld + h * a.dim + d, a.f32);
+  const int n = min(a.kv_rows, pos + 1 - a.kv0);            // visible keys of this block: [first_key, n)
+  const int first_key = max(0, (a.window > 0 ? pos / a.window * a.window : 0) - a.kv0);
+  const int hk = h / a.group, kv_heads = a.heads / a.group;
+  const long long kld = (long long)kv_heads * a.dim, vld = (long long)kv_heads * a.vdim;
+  for (int d = lane; d < a.dim; d += 32) sq[warp][d] = load_act(a.q, ((long long)r * a.heads + h) * a.dim + d, a.f32);
   __syncwarp();
   float o[16];
 #pragma unroll
@@ -39,12 +43,12 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(const LatentAttnA
     for (int i = 0; i < 16; ++i)
       if (lane + 32 * i < a.vdim) o[i] = st[2 + lane + 32 * i];
   }
-  for (int j0 = 0; j0 < n; j0 += 32) {
+  for (int j0 = first_key; j0 < n; j0 += 32) {
     const int j = j0 + lane;
     float s = -FLT_MAX;
     if (j < n) {
       s = 0.f;
-      const long long base = (long long)j * kld + h * a.dim;
+      const long long base = (long long)j * kld + hk * a.dim;
       for (int d = 0; d < a.dim; ++d) s = fmaf(sq[warp][d], load_act(a.k, base + d, a.f32), s);
       s *= a.scale;
     }
@@ -60,7 +64,7 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(const LatentAttnA
     const int live = min(32, n - j0);
     for (int t = 0; t < live; ++t) {
       const float pt = __shfl_sync(0xffffffffu, p, t);
-      const long long base = (long long)(j0 + t) * vld + h * a.vdim;
+      const long long base = (long long)(j0 + t) * vld + hk * a.vdim;
 #pragma unroll
       for (int i = 0; i < 16; ++i)
         if (lane + 32 * i < a.vdim) o[i] = fmaf(pt, load_act(a.v, base + lane + 32 * i, a.f32), o[i]);
@@ -78,8 +82,8 @@ __global__ void __launch_bounds__(128) latent_attn_rows_kernel(const LatentAttnA
   for (int i = 0; i < 16; ++i) {
     const int c = lane + 32 * i;
     if (c < a.vdim) {
-      const float g = sigmoid_f(a.gate[(long long)r * a.gate_ld + h * a.vdim + c]);
-      store_act(a.out, (long long)r * vld + h * a.vdim + c, o[i] * inv * g, a.f32);
+      const float g = a.gate ? sigmoid_f(a.gate[(long long)r * a.gate_ld + h * a.vdim + c]) : 1.f;
+      store_act(a.out, ((long long)r * a.heads + h) * a.vdim + c, o[i] * inv * g, a.f32);
     }
   }
 }
@@ -151,7 +155,10 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
   const int pos0 = *a.pos0;
   const int last_row = min(r0 + kQRows, a.rows) - 1;
   const int seen = min(a.kv_rows, pos0 + last_row + 1 - a.kv0);
-  const int tiles = seen > 0 ? (seen + kKeys - 1) / kKeys : 0;
+  // tiles of keys that no row of this CTA sees (earlier chunks of the mask) are left out
+  const int tile0 = max(0, (a.window > 0 ? (pos0 + r0) / a.window * a.window : 0) - a.kv0) / kKeys;
+  const int tiles = seen > tile0 * kKeys ? (seen + kKeys - 1) / kKeys - tile0 : 0;
+  const int hk = h / a.group;
 
   if (warp == 0) {
     if (elect_one() && tiles > 0) {
@@ -162,10 +169,10 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
         const uint32_t ph = ((j >> 1) & 1) ^ 1;
         if (j >= 2 && !mbar_wait(&bar->k_empty[st], ph, a.status, kSiteStageEmpty | st)) break;
         mbar_expect_tx(&bar->k_full[st], chunks * 8192);
-        for (int c = 0; c < chunks; ++c) tma_load_3d(sK + (st * chunks + c) * 8192, &tmK, &bar->k_full[st], c * 64, h, j * kKeys);
+        for (int c = 0; c < chunks; ++c) tma_load_3d(sK + (st * chunks + c) * 8192, &tmK, &bar->k_full[st], c * 64, hk, a.k_row0 + (tile0 + j) * kKeys);
         if (j >= 2 && !mbar_wait(&bar->v_empty[st], ph, a.status, kSiteStageEmpty | 8 | st)) break;
         mbar_expect_tx(&bar->v_full[st], N * 128);
-        tma_load_2d(sV + st * N * 128, &tmV, &bar->v_full[st], j * kKeys, h * a.vdim);
+        tma_load_2d(sV + st * N * 128, &tmV, &bar->v_full[st], (tile0 + j) * kKeys, hk * a.vdim);
       }
     }
   } else if (warp == 1) {
@@ -206,7 +213,8 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
     const int quad = warp & 3, row = quad * 32 + lane, r = r0 + row;
     const uint32_t lane_off = uint32_t(quad * 32) << 16;
     const bool live = r < a.rows;
-    const int vis = min(a.kv_rows, pos0 + r + 1 - a.kv0);              // visible keys of this row in the block
+    const int vis = min(a.kv_rows, pos0 + r + 1 - a.kv0);              // visible keys of this row in the block: [low, vis)
+    const int low = a.window > 0 ? (pos0 + r) / a.window * a.window - a.kv0 : 0;
     const float c2 = a.scale * 1.4426950408889634f;                    // scores in powers of two
     float* st_row = a.state ? a.state + ((size_t)min(r, a.rows - 1) * a.heads + h) * (a.vdim + 2) : nullptr;
     float m = -INFINITY, l = 0.f;                                      // m in scaled (base 2) units
@@ -235,15 +243,15 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
       tmem_ld_wait();
       tc_fence_before();
       mbar_arrive(&bar->s_empty);
-      const int k0 = j * kKeys;
+      const int k0 = (tile0 + j) * kKeys;
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains: the row's 64 values are one thread's
-      if (k0 + kKeys <= vis) {
+      if (k0 + kKeys <= vis && k0 >= low) {
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(s[i]));
       } else {
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) {
-          if (k0 + i >= vis) s[i] = 0xff800000u;
+          if (k0 + i >= vis || k0 + i < low) s[i] = 0xff800000u;
           mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(s[i]));
         }
       }
@@ -301,7 +309,7 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
           for (int i = 0; i < 16; ++i) v[i] = c + i < a.vdim ? __float_as_uint(st_row[2 + c + i]) : 0u;
         }
         if (live) {
-          const float* g = a.gate + (long long)r * a.gate_ld + (long long)h * a.vdim + c;
+          const float* g = a.gate ? a.gate + (long long)r * a.gate_ld + (long long)h * a.vdim + c : nullptr;
           __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(a.out) + ((long long)r * a.heads + h) * a.vdim + c;
 #pragma unroll
           for (int q = 0; q < 2; ++q) {
@@ -311,7 +319,8 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
               for (int i = 0; i < 8; ++i) st_row[2 + c + 8 * q + i] = __uint_as_float(v[8 * q + i]);
             } else {
               float x[8];
-              if (gate_vec) {
+              if (!a.gate) {
+              } else if (gate_vec) {
                 const float4 g0 = *reinterpret_cast<const float4*>(g + 8 * q), g1 = *reinterpret_cast<const float4*>(g + 8 * q + 4);
                 x[0] = g0.x; x[1] = g0.y; x[2] = g0.z; x[3] = g0.w;
                 x[4] = g1.x; x[5] = g1.y; x[6] = g1.z; x[7] = g1.w;
@@ -320,7 +329,7 @@ __global__ void __launch_bounds__(kTcThreads) latent_attn_tc_kernel(const __grid
                 for (int i = 0; i < 8; ++i) x[i] = g[8 * q + i];
               }
 #pragma unroll
-              for (int i = 0; i < 8; ++i) x[i] = __uint_as_float(v[8 * q + i]) * inv * sigmoid_f(x[i]);
+              for (int i = 0; i < 8; ++i) x[i] = __uint_as_float(v[8 * q + i]) * inv * (a.gate ? sigmoid_f(x[i]) : 1.f);
               *reinterpret_cast<uint4*>(o + 8 * q) =
                   make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
             }
@@ -593,7 +602,7 @@ extern "C" int nrt_latent_decode_args_size() { return (int)sizeof(LatentDecodeAr
 extern "C" int nrt_latent_attn_rows(const void* args, void* stream) {
   LatentAttnArgs a;
   memcpy(&a, args, sizeof(a));
-  if (a.rows < 1 || a.dim > 512 || a.vdim > 512 || ((!a.first || !a.last) && !a.state)) return -3;
+  if (a.rows < 1 || a.group < 1 || a.heads % a.group || a.window < 0 || a.dim > 512 || a.vdim > 512 || ((!a.first || !a.last) && !a.state)) return -3;
   return launch_pdl(latent_attn_rows_kernel, dim3((a.rows * a.heads + 3) / 4), dim3(128), 0, reinterpret_cast<cudaStream_t>(stream), false, a);
 }
 
@@ -606,7 +615,7 @@ extern "C" int nrt_latent_attn_tc(const void* tmQ, const void* tmK, const void* 
   memcpy(&v, tmV, sizeof(v));
   LatentAttnArgs a;
   memcpy(&a, args, sizeof(a));
-  if (a.rows < 1 || a.f32 || a.dim > 256 || a.vdim > 256 || a.dim % 8 || a.vdim % 8 || !(a.scale > 0.f) || ((!a.first || !a.last) && !a.state)) return -3;
+  if (a.rows < 1 || a.group < 1 || a.heads % a.group || a.window < 0 || a.f32 || a.dim > 256 || a.vdim > 256 || a.dim % 8 || a.vdim % 8 || !(a.scale > 0.f) || ((!a.first || !a.last) && !a.state)) return -3;
   const int smem = tc_smem(a.dim, a.vdim);
   static bool configured = false;
   if (!configured) {

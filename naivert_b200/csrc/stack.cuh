@@ -1,6 +1,6 @@
 // Argument structs and small device helpers of the layer-stack kernels: the mechanisms from which models of
-// freely ordered layers (latent attention, gated linear recurrence, dense and expert feed-forwards, sandwich norms,
-// looped layers) are put together.  Every size and constant is a field; nothing here belongs to one model.
+// freely ordered layers (latent and chunked grouped-query attention, gated linear recurrence, matrix-state recurrences,
+// dense and expert feed-forwards, norms before and after a sublayer, looped layers) are put together.  Every size and constant is a field; nothing here belongs to one model.
 //
 // Activation buffers come in two forms: bf16 (`f32` = 0: tensor-core products) and float (`f32` = 1: everything in
 // true 32-bit on the CUDA cores).  Weights are bf16 in both.  The residual stream, norms, routers, attention scores,
@@ -19,6 +19,10 @@ enum StackEpi : int {
   kSEpiTranspose = 2,  // acc stored feature-major: out[feature][token] (bf16)
   kSEpiClampedGlu = 3, // two products g, u: g = min(g, limit), u = clamp(u), g * sigmoid(alpha g) * (u + 1)
   kSEpiSiluGlu = 4,    // two products g, u: silu(g) * u
+  kSEpiRelu2 = 5,      // relu(acc)^2
+  kSEpiTanh = 6,       // tanh(acc)
+  kSEpiDecaySoft = 7,  // exp(-rate * softplus(acc + bias)), rate per feature
+  kSEpiDecayExp = 8,   // exp(-exp(acc + bias))
 };
 
 struct StackGemmArgs {
@@ -37,12 +41,18 @@ struct StackGemmArgs {
   int out_f32;                  // element type of `out`
   long long out_ld, out_zstride;
   const __nv_bfloat16* bias;    // [zcount][n]
+  const float* rate;            // [n] (kSEpiDecaySoft)
   int act_cols;
   float scale, limit, alpha;
   uint32_t* status;
 };
 
 // ------------------------------------------------------------------------------------ rows
+enum NormKind : int {
+  kNormRms = 0,        // x / sqrt(mean(x^2) + eps) * w
+  kNormLayer = 1,      // (x - mean) / sqrt(mean((x - mean)^2) + eps) * w
+};
+
 struct StackRowArgs {
   // where the stream comes from: an embedding gather (tokens != null), else x as it stands
   const int* tokens;
@@ -56,9 +66,15 @@ struct StackRowArgs {
   const float* probs;           // [rows][top_k]
   int top_k;
   const __nv_bfloat16* post_w;
+  // second half of a sublayer of two mixers side by side (null: none): y becomes half the sum of both, each RMS-normed first
+  const float* y2;
+  const __nv_bfloat16* join_w;
+  const __nv_bfloat16* join_w2;
   const __nv_bfloat16* add;     // vector added to the stream afterwards (null: none)
   float* x;                     // [rows][width] in / out
   const __nv_bfloat16* pre_w;   // norm of the next sublayer (null: none)
+  int norm;                     // NormKind of post_w and pre_w
+  int copy_h;                   // without pre_w: the stream itself is the next sublayer's input
   void* h;
   int h_f32;
   long long h_ld;
@@ -83,12 +99,17 @@ struct LatentPrepArgs {
   int capacity;
 };
 
+// Attention of chunk rows over a block of keys.  Query head h uses key / value head h / group.  With `window` > 0 positions are
+// cut into chunks of that many, counted from position 0, and a query sees only keys of its own chunk.
 struct LatentAttnArgs {
   const void* q;                // [rows][heads * dim]
-  const void* k;                // keys of the block [kv_rows][heads * dim]
-  const void* v;                // simple form: [kv_rows][heads * vdim]; tensor-core form: feature-major [heads * vdim][v_ld]
+  const void* k;                // keys of the block [kv_rows][heads / group * dim]
+  const void* v;                // simple form: [kv_rows][heads / group * vdim]; tensor-core form: feature-major [heads / group * vdim][v_ld]
   long long v_ld;
-  const float* gate;            // raw output gate, element (row, head * vdim + j) at row * gate_ld + ...
+  int group;                    // query heads per key / value head
+  int window;                   // chunk length of the mask, 0: causal only
+  int k_row0;                   // tensor-core form: row of the key map that holds position kv0
+  const float* gate;            // raw output gate (null: none), element (row, head * vdim + j) at row * gate_ld + ...
   long long gate_ld;
   void* out;                    // [rows][heads * vdim]
   int f32;
@@ -140,6 +161,163 @@ struct RecurrenceArgs {
   uint32_t* status;
 };
 
+// ------------------------------------------------------------------------------------ chunked grouped-query attention
+// Queries, keys and values of a token as one product left them (biases added); norms per head, rotation of the first
+// rot_dims columns (halves paired, angle = position * freq[i]), queries times `scale`.
+struct GroupPrepArgs {
+  const float* proj;            // [rows][ld]: queries from q_off, keys from k_off, values from v_off
+  long long ld;
+  int q_off, k_off, v_off;
+  int rows, heads, kv_heads, dim, vdim, dp, vp;      // dp, vp: storage widths of a head
+  const __nv_bfloat16* q_norm;  // [dim] (null: none)
+  const __nv_bfloat16* k_norm;
+  const float* freq;            // [rot_dims / 2]
+  int rot_dims;
+  float eps, scale;
+  void* q;                      // [rows][heads * dp]
+  void* k_cache;                // [capacity][kv_heads * dp], row = position
+  void* v_cache;                // [capacity][kv_heads * vp]
+  int f32;
+  const int* pos0;
+  int capacity;
+};
+
+struct TransposeArgs {
+  const __nv_bfloat16* src;     // [rows][cols]
+  __nv_bfloat16* dst;           // [cols][dst_ld]
+  long long dst_ld;
+  int rows, cols;
+};
+
+// One token: preparation as above, then attention over the visible keys, split over a cluster that merges its parts.
+struct GroupDecodeArgs {
+  GroupPrepArgs p;              // rows = 1; q unused
+  int window;                   // chunk length of the mask, 0: causal only
+  int splits;                   // cluster size
+  float* out;                   // [heads * vdim]
+};
+
+// ------------------------------------------------------------------------------------ matrix-state recurrences
+// Every head carries a matrix S [dim x vdim] (stored per value column: [vdim][dim4], dim4 = dim rounded up to four).
+enum StateKind : int {
+  kStateDelta = 0,     // S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q
+  kStateBonus = 1,     // o = (S + diag(u) k v^T)^T q; S <- g S + k v^T
+  kStateNormalized = 2,// S <- a S + b k v^T, n likewise with k alone, stabilised by a running maximum; o = S^T q, with n . q beside it
+};
+enum GateKind : int { kGateSigmoid = 0, kGateSilu = 1 };
+
+struct StateChunkArgs {
+  const float* q;               // element (row, key head, d) at row * q_ld + key head * dim + d
+  const float* k;
+  const float* v;               // element (row, head, j) at row * v_ld + head * vdim + j
+  const float* g;               // decay per head and key channel (delta, bonus)
+  long long q_ld, k_ld, v_ld, g_ld;
+  int rows, heads, kv_heads, dim, vdim;
+  float q_scale;
+  const float* beta;            // delta: raw step size, element (row, head) at row * beta_ld + head
+  long long beta_ld;
+  const __nv_bfloat16* u;       // bonus: [heads][dim]
+  const float* gi;              // normalized: raw input and forget gates, element (row, head) at row * gate_ld + head
+  const float* gf;
+  long long gate_ld;
+  float cap;
+  float* o;                     // [rows][heads * vdim]
+  float* den;                   // normalized: [rows][heads][2] = n . q, exp(-m)
+  float* state;                 // [2][state_stride]: heads x columns x dim4, then (normalized) the running maxima
+  long long state_stride;
+  int* tags;                    // [2]: number of tokens each state slot has seen
+  // inputs of a short convolution whose last rows are kept for the next chunk (null: none)
+  const float* hist_src;        // [rows][hist_ld], first hist_cols columns
+  long long hist_ld;
+  int hist_cols, taps, hist_rows;
+  float* history;               // [hist_rows][hist_cols], slot = position % hist_rows
+  const int* pos0;
+  uint32_t* status;
+};
+
+// Short causal convolution + SiLU of the q | k | v columns of a projection; q and k heads become unit vectors (q times q_scale).
+// The remaining columns named by `low` are copied to an operand buffer.
+struct ShortConvArgs {
+  const float* proj;            // [rows][ld]: q [kv_heads * dim] | k [kv_heads * dim] | v [heads * vdim] | ...
+  long long ld;
+  int rows, heads, kv_heads, dim, vdim, taps;
+  const __nv_bfloat16* conv;    // [columns][taps]
+  const float* history;         // [hist_rows][columns]
+  int hist_rows;
+  float q_scale;
+  float* q;                     // [rows][kv_heads * dim]
+  float* k;
+  float* v;                     // [rows][heads * vdim]
+  int low_off, low_cols;        // columns copied to `low` [rows][low_ld]
+  int low2_off, low2_cols, low2_at;   // and from low2_at on
+  void* low;
+  long long low_ld;
+  int f32;
+  const int* pos0;
+};
+
+// Mixes of a token with its predecessor: out[row][s] = x + (x_before - x) * mu[s]
+struct TokenMixArgs {
+  const float* x;               // [rows][width]
+  int rows, width, mixes;
+  const __nv_bfloat16* mu;      // [mixes][width]
+  void* out;                    // [rows][mixes][out_ld]
+  long long out_ld;
+  int f32;
+  float* shift;                 // state slot s keeps the last row at shift + s * state_stride
+  long long state_stride;
+  const int* tags;
+  const int* pos0;
+  uint32_t* status;
+};
+
+// Read-out of a matrix state: each head divided by its root mean square, times a weight, times a gate.
+struct HeadGateArgs {
+  const float* o;               // [rows][heads * vdim]
+  const float* den;             // [rows][heads][2] (null: none): o is first divided by max(|n . q|, exp(-m)) + 1e-6
+  const __nv_bfloat16* norm;    // [vdim] shared (norm_per_head = 0) or [heads * vdim]
+  int norm_per_head;
+  const float* gate;            // raw, element (row, head * vdim + j) at row * gate_ld + ...
+  long long gate_ld;
+  int gate_kind;
+  void* out;                    // [rows][out_ld]
+  long long out_ld;
+  int f32, rows, heads, vdim;
+  float eps;
+};
+
+// One token of a matrix-state mixer: unit vectors, low-rank decay and gate, state update, read-out, head norm and gate.
+struct StateStepArgs {
+  int kind, heads, kv_heads, dim, vdim;
+  const float* proj;            // the token's projections; offsets of its parts
+  int q_off, k_off, v_off;
+  int unit;                     // q and k become unit vectors
+  float q_scale;
+  int beta_off;                 // delta
+  const __nv_bfloat16* u;       // bonus
+  int gi_off, gf_off;           // normalized
+  float cap;
+  // decay = exp(-rate softplus(z + bias)) (rate != null) or exp(-exp(z + bias)), z = decay_w act(in)
+  int low_off, low_rank, low_tanh;
+  const __nv_bfloat16* decay_w; // [heads * dim][decay_ld]
+  long long decay_ld;
+  const __nv_bfloat16* decay_b; // [heads * dim]
+  const float* rate;            // [heads * dim]
+  // gate: raw columns of the projection, or low-rank (gate_w != null)
+  int gate_off, gate_rank, gate_kind;
+  const __nv_bfloat16* gate_w;  // [heads * vdim][gate_ld]
+  long long gate_ld;
+  const __nv_bfloat16* norm;
+  int norm_per_head;
+  float eps;
+  float* state;
+  long long state_stride;
+  int* tags;
+  float* out;                   // [heads * vdim]
+  const int* pos0;
+  uint32_t* status;
+};
+
 struct MoeGatherArgs {
   const void* h;                // [rows][h_ld]
   long long h_ld;
@@ -155,14 +333,17 @@ enum StepPro : int {
   kProNorm = 1,        // input = rms(in) * in_w
   kProLoad = 2,        // input = in + group * in_gstride
   kProMerge = 3,       // input = softmax-merged latent output of head `group` from the attention partials
+  kProMix = 5,         // stream update, then input of group g = x_out + (x_before - x_out) * mu[g] (x_before: the previous token's)
   kProExperts = 4,     // inputs of the chosen experts side by side, each times its weight: out = sum_j W[ids[j]] (p[j] in[j])
 };
 enum StepEpi : int {
-  kTEpiStore = 0,      // acc * scale; rows from `sig_from` on through a sigmoid
+  kTEpiStore = 0,      // acc * scale (+ bias); rows from `sig_from` on through a sigmoid
   kTEpiConv = 1,       // + bias; rows < width: GELU (tanh form); others: convolution input -> u, history
   kTEpiGate = 2,       // acc * gate[row]
   kTEpiGlu = 3,        // two products: clamped GLU (glu_kind 0) or SiLU GLU (1)
   kTEpiRecur = 4,      // two products (r, i) + biases: recurrence step, times the gate branch
+  kTEpiConvSilu = 5,   // rows < conv_rows: short convolution without a bias, SiLU; others: stored
+  kTEpiRelu2 = 6,      // relu(acc)^2
 };
 
 struct StepArgs {
@@ -174,6 +355,14 @@ struct StepArgs {
   const float* x;
   const float* y;
   const __nv_bfloat16* post_w;
+  const float* y2;              // second half of a sublayer of two mixers (StackRowArgs)
+  const __nv_bfloat16* join_w;
+  const __nv_bfloat16* join_w2;
+  int norm;                     // NormKind of post_w and in_w (stream prologues)
+  int raw_in;                   // the stream itself is the input (no in_w)
+  const __nv_bfloat16* mu;      // kProMix: [groups][k]
+  float* shift;                 // kProMix: the previous token's stream, state slot s at shift + s * state_stride
+  long long state_stride;
   const __nv_bfloat16* add;
   float* x_out;
   const float* in_;
@@ -189,6 +378,8 @@ struct StepArgs {
   const __nv_bfloat16* w2;
   long long w_ld, w_gstride, w2_gstride;
   int groups, n;                // groups x n output rows
+  int n_last;                   // rows of the last group (0: n)
+  int conv_rows;                // kTEpiConvSilu
   int segs;                     // chosen experts whose products are summed (kProExperts), else 1
   const int* ids;               // [segs] their weight groups
   const float* probs;           // [segs] their weights
@@ -241,6 +432,12 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit, floa
   return g * sigmoid_f(alpha * g) * (u + 1.0f);
 }
 __device__ __forceinline__ float silu_glu(float g, float u) { return g * sigmoid_f(g) * u; }
+__device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
+__device__ __forceinline__ float relu2_f(float z) { z = fmaxf(z, 0.f); return z * z; }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
+__device__ __forceinline__ float decay_soft(float z, float rate) { return expf(-rate * softplus_f(z)); }
+__device__ __forceinline__ float decay_exp(float z) { return expf(-expf(z)); }
 
 __device__ __forceinline__ float lane_sum(float v) {
 #pragma unroll

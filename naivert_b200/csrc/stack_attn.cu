@@ -1,0 +1,309 @@
+// Grouped-query attention of layer stacks around the chunk kernels of latent_attn.cu: preparation of queries, keys and values
+// (norm per head, rotary positions, cache rows), the feature-major copy of the values, and the one-token step.
+#include "stack.cuh"
+#include "launch.hpp"
+
+#include <string.h>
+
+using namespace nrt;
+
+namespace {
+
+constexpr int kMaxHead = 512;                 // head width the kernels hold in shared memory
+
+// One head of a token, by one warp: x[0, n) -> normed (w != null) and rotated by the angles in (cs, sn), times `scale`, in `out`
+// (shared, n values).  All reads of `src` happen before the first write of `out`.
+__device__ __forceinline__ void head_vector(const float* src, int n, const __nv_bfloat16* w, float eps, int half, const float* cs, const float* sn,
+                                            float scale, float* out, int lane) {
+  float ss = 0.f;
+  for (int c = lane; c < n; c += 32) {
+    const float v = __ldcg(src + c);
+    out[c] = v;
+    ss = fmaf(v, v, ss);
+  }
+  if (w) {
+    const float r = 1.0f / sqrtf(lane_sum(ss) / (float)n + eps);
+    for (int c = lane; c < n; c += 32) out[c] = out[c] * r * bf(w + c);
+  }
+  __syncwarp();
+  for (int i = lane; i < half; i += 32) {
+    const float u = out[i], v = out[i + half], c = cs[i], s = sn[i];
+    out[i] = u * c - v * s;
+    out[i + half] = v * c + u * s;
+  }
+  __syncwarp();
+  if (scale != 1.f)
+    for (int c = lane; c < n; c += 32) out[c] *= scale;
+  __syncwarp();
+}
+__device__ __forceinline__ void angles(const GroupPrepArgs& p, int pos, float* cs, float* sn) {
+  for (int i = threadIdx.x; i < p.rot_dims / 2; i += blockDim.x) sincosf((float)pos * p.freq[i], sn + i, cs + i);
+}
+
+// ------------------------------------------------------------------------------------ chunk path: preparation
+// One CTA per row; a warp takes one head at a time: queries, then keys, then values.
+__global__ void __launch_bounds__(256) group_prep_kernel(const GroupPrepArgs p) {
+  __shared__ float buf[8][kMaxHead], cs[kMaxHead / 2], sn[kMaxHead / 2];
+  griddep_wait();
+  griddep_launch();
+  const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dims / 2;
+  const int pos = *p.pos0 + r;
+  if (pos < 0 || pos >= p.capacity) return;
+  angles(p, pos, cs, sn);
+  __syncthreads();
+  const float* row = p.proj + r * p.ld;
+  for (int u = warp; u < p.heads + 2 * p.kv_heads; u += 8) {
+    if (u < p.heads + p.kv_heads) {
+      const bool is_q = u < p.heads;
+      const int h = is_q ? u : u - p.heads;
+      head_vector(row + (is_q ? p.q_off : p.k_off) + h * p.dim, p.dim, is_q ? p.q_norm : p.k_norm, p.eps, half, cs, sn, is_q ? p.scale : 1.f, buf[warp], lane);
+      void* dst = is_q ? p.q : p.k_cache;
+      const long long at = is_q ? ((long long)r * p.heads + h) * p.dp : ((long long)pos * p.kv_heads + h) * p.dp;
+      for (int c = lane; c < p.dp; c += 32) store_act(dst, at + c, c < p.dim ? buf[warp][c] : 0.f, p.f32);
+      __syncwarp();
+    } else {
+      const int h = u - p.heads - p.kv_heads;
+      for (int c = lane; c < p.vdim; c += 32) store_act(p.v_cache, ((long long)pos * p.kv_heads + h) * p.vp + c, __ldg(row + p.v_off + h * p.vdim + c), p.f32);
+    }
+  }
+}
+
+// dst[c][r] = src[r][c], 64 x 64 tiles
+__global__ void __launch_bounds__(256) transpose_kernel(const TransposeArgs a) {
+  __shared__ __nv_bfloat16 tile[64][66];
+  griddep_wait();
+  griddep_launch();
+  const int r0 = blockIdx.x * 64, c0 = blockIdx.y * 64, tx = threadIdx.x & 63, ty = threadIdx.x >> 6;
+  for (int i = ty; i < 64; i += 4)
+    if (r0 + i < a.rows && c0 + tx < a.cols) tile[i][tx] = a.src[(long long)(r0 + i) * a.cols + c0 + tx];
+  __syncthreads();
+  for (int i = ty; i < 64; i += 4)
+    if (c0 + i < a.cols && r0 + tx < a.rows) a.dst[(long long)(c0 + i) * a.dst_ld + r0 + tx] = tile[tx][i];
+}
+
+// ------------------------------------------------------------------------------------ one token
+// grid (splits, key heads, groups of eight query heads); the splits of one key head are a cluster.  Eight lanes share a key, the
+// query heads of the CTA are scored together; then threads own value columns.  The partial results meet through distributed shared
+// memory.  Every CTA whose keys end at the token itself prepares and stores the token's key and value first (equal values).
+constexpr int kHB = 8, kTile = 64, kDecThreads = 256;
+
+__device__ __forceinline__ float ld_cluster_f32(const float* p, uint32_t rank) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(mapa_shared(smem_u32(p), rank)) : "memory");
+  return v;
+}
+__host__ __device__ inline int group_smem_floats(int dp, int vp) { return kHB * dp + kMaxHead + kTile * kHB + 3 * kHB + kHB * vp; }
+
+template <bool F32, int VC>                    // VC value columns per thread
+__global__ void __launch_bounds__(kDecThreads) group_decode_kernel(const GroupDecodeArgs a) {
+  extern __shared__ __align__(16) float sh[];
+  const GroupPrepArgs& p = a.p;
+  float* sq = sh;                              // [8][dp]
+  float* cs = sq + kHB * p.dp;
+  float* sn = cs + kMaxHead / 2;
+  float* sp = sn + kMaxHead / 2;               // [64][8]
+  float* sm = sp + kTile * kHB;
+  float* sl = sm + kHB;
+  float* scorr = sl + kHB;
+  float* so = scorr + kHB;                     // [8][vp]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & 7;
+  const int split = blockIdx.x, hk = blockIdx.y, group = p.heads / p.kv_heads, h0 = blockIdx.z * kHB, nh = min(kHB, group - h0);
+  const int half = p.rot_dims / 2;
+  griddep_wait();
+  griddep_launch();
+  const int pos = *reinterpret_cast<const volatile int*>(p.pos0);
+  const int start = a.window > 0 ? pos / a.window * a.window : 0, n = pos + 1 - start;
+  const int per = ((n + a.splits - 1) / a.splits + kTile - 1) / kTile * kTile;
+  const int j_lo = min(n, split * per), j_hi = min(n, j_lo + per);
+  const bool inside = pos >= 0 && pos < p.capacity;
+  angles(p, pos, cs, sn);
+  for (int i = tid; i < kHB * p.dp; i += kDecThreads) sq[i] = 0.f;
+  for (int i = tid; i < kHB * p.vp; i += kDecThreads) so[i] = 0.f;
+  if (tid < kHB) { sm[tid] = -FLT_MAX; sl[tid] = 0.f; }
+  __syncthreads();
+  if (inside && j_lo < j_hi) {
+    if (j_hi == n) {
+      // the token's own key and value (sp is free until the first tile)
+      if (warp == 0) {
+        head_vector(p.proj + p.k_off + hk * p.dim, p.dim, p.k_norm, p.eps, half, cs, sn, 1.f, sp, lane);
+        for (int c = lane; c < p.dim; c += 32) store_act(p.k_cache, ((long long)pos * p.kv_heads + hk) * p.dp + c, sp[c], F32);
+      } else if (warp == 1) {
+        for (int c = lane; c < p.vdim; c += 32)
+          store_act(p.v_cache, ((long long)pos * p.kv_heads + hk) * p.vp + c, __ldcg(p.proj + p.v_off + hk * p.vdim + c), F32);
+      }
+    }
+    for (int h = warp; h < nh; h += kDecThreads / 32)
+      head_vector(p.proj + p.q_off + (hk * group + h0 + h) * p.dim, p.dim, p.q_norm, p.eps, half, cs, sn, p.scale, sq + h * p.dp, lane);
+    __syncthreads();
+    const int pieces = p.dp / 8;
+    int vc = 32;
+    while (vc < p.vdim && vc < kDecThreads) vc *= 2;
+    const int subs = kDecThreads / vc, sub = tid / vc, c0 = tid & (vc - 1);
+    float acc[kHB][VC];
+#pragma unroll
+    for (int h = 0; h < kHB; ++h)
+#pragma unroll
+      for (int i = 0; i < VC; ++i) acc[h][i] = 0.f;
+    float m = -FLT_MAX, sum = 0.f;                                       // of head `warp`
+    for (int j0 = j_lo; j0 < j_hi; j0 += kTile) {
+      const int live = min(kTile, j_hi - j0);
+#pragma unroll
+      for (int t0 = 0; t0 < kTile; t0 += kDecThreads / 8) {
+        const int t = t0 + tid / 8;
+        float d[kHB];
+#pragma unroll
+        for (int h = 0; h < kHB; ++h) d[h] = 0.f;
+        if (t < live) {
+          const long long at = ((long long)(start + j0 + t) * p.kv_heads + hk) * p.dp;
+#pragma unroll 2
+          for (int i = l; i < pieces; i += 8) {
+            float4 x, y;
+            if (F32) {
+              const float4* k = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.k_cache) + at + i * 8);
+              x = __ldcg(k);
+              y = __ldcg(k + 1);
+            } else {
+              const uint4 k = __ldcg(reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.k_cache) + at + i * 8));
+              x = make_float4(bf16_lo(k.x), bf16_hi(k.x), bf16_lo(k.y), bf16_hi(k.y));
+              y = make_float4(bf16_lo(k.z), bf16_hi(k.z), bf16_lo(k.w), bf16_hi(k.w));
+            }
+#pragma unroll
+            for (int h = 0; h < kHB; ++h) {
+              const float4 q0 = *reinterpret_cast<const float4*>(sq + h * p.dp + i * 8), q1 = *reinterpret_cast<const float4*>(sq + h * p.dp + i * 8 + 4);
+              d[h] = fmaf(x.x, q0.x, fmaf(x.y, q0.y, fmaf(x.z, q0.z, fmaf(x.w, q0.w, d[h]))));
+              d[h] = fmaf(y.x, q1.x, fmaf(y.y, q1.y, fmaf(y.z, q1.z, fmaf(y.w, q1.w, d[h]))));
+            }
+          }
+        }
+        float mine = 0.f;
+#pragma unroll
+        for (int h = 0; h < kHB; ++h) {
+          float v = d[h];
+          v += __shfl_xor_sync(0xffffffffu, v, 1);
+          v += __shfl_xor_sync(0xffffffffu, v, 2);
+          v += __shfl_xor_sync(0xffffffffu, v, 4);
+          if (h == l) mine = v;
+        }
+        sp[t * kHB + l] = mine;
+      }
+      __syncthreads();
+      {                                                                  // softmax of head `warp`
+        const float s0 = lane < live ? sp[lane * kHB + warp] : -FLT_MAX, s1 = lane + 32 < live ? sp[(lane + 32) * kHB + warp] : -FLT_MAX;
+        float mt = fmaxf(s0, s1);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, o));
+        const float mn = fmaxf(m, mt), corr = expf(m - mn);
+        const float p0 = lane < live ? expf(s0 - mn) : 0.f, p1 = lane + 32 < live ? expf(s1 - mn) : 0.f;
+        sum = fmaf(sum, corr, lane_sum(p0 + p1));
+        m = mn;
+        sp[lane * kHB + warp] = p0;
+        sp[(lane + 32) * kHB + warp] = p1;
+        if (lane == 0) scorr[warp] = corr;
+      }
+      __syncthreads();
+#pragma unroll
+      for (int h = 0; h < kHB; ++h)
+#pragma unroll
+        for (int i = 0; i < VC; ++i) acc[h][i] *= scorr[h];
+#pragma unroll 4
+      for (int t = sub; t < live; t += subs) {
+        const float4 pa = *reinterpret_cast<const float4*>(sp + t * kHB), pb = *reinterpret_cast<const float4*>(sp + t * kHB + 4);
+        const long long at = ((long long)(start + j0 + t) * p.kv_heads + hk) * p.vp;
+#pragma unroll
+        for (int i = 0; i < VC; ++i) {
+          const int c = c0 + i * kDecThreads;
+          if (c < p.vdim) {
+            const float v = F32 ? __ldcg(reinterpret_cast<const float*>(p.v_cache) + at + c)
+                                : __bfloat162float(__ldcg(reinterpret_cast<const __nv_bfloat16*>(p.v_cache) + at + c));
+            acc[0][i] = fmaf(pa.x, v, acc[0][i]);
+            acc[1][i] = fmaf(pa.y, v, acc[1][i]);
+            acc[2][i] = fmaf(pa.z, v, acc[2][i]);
+            acc[3][i] = fmaf(pa.w, v, acc[3][i]);
+            acc[4][i] = fmaf(pb.x, v, acc[4][i]);
+            acc[5][i] = fmaf(pb.y, v, acc[5][i]);
+            acc[6][i] = fmaf(pb.z, v, acc[6][i]);
+            acc[7][i] = fmaf(pb.w, v, acc[7][i]);
+          }
+        }
+      }
+      __syncthreads();                                                   // sp is rewritten
+    }
+    if (lane == 0) { sm[warp] = m; sl[warp] = sum; }
+    // key subsets join in a fixed order
+    for (int s = 0; s < subs; ++s) {
+      if (sub == s) {
+#pragma unroll
+        for (int h = 0; h < kHB; ++h)
+#pragma unroll
+          for (int i = 0; i < VC; ++i)
+            if (c0 + i * kDecThreads < p.vdim) so[h * p.vp + c0 + i * kDecThreads] += acc[h][i];
+      }
+      __syncthreads();
+    }
+  }
+  cluster_sync_all();
+  // every CTA of the cluster finishes a share of the heads' columns
+  for (int i = split * kDecThreads + tid; i < nh * p.vdim; i += a.splits * kDecThreads) {
+    const int h = i / p.vdim, c = i - h * p.vdim;
+    float m = -FLT_MAX, o = 0.f, sum = 0.f;
+    for (int s = 0; s < a.splits; ++s) m = fmaxf(m, ld_cluster_f32(sm + h, s));
+    for (int s = 0; s < a.splits; ++s) {
+      const float w = expf(ld_cluster_f32(sm + h, s) - m);
+      sum = fmaf(w, ld_cluster_f32(sl + h, s), sum);
+      o = fmaf(w, ld_cluster_f32(so + h * p.vp + c, s), o);
+    }
+    a.out[(long long)(hk * group + h0 + h) * p.vp + c] = o / sum;
+  }
+  cluster_sync_all();                                                    // nobody leaves while its shared memory is read
+}
+
+template <bool F32, int VC>
+int launch_decode(const GroupDecodeArgs& a, cudaStream_t stream, bool pdl) {
+  const int smem = 4 * group_smem_floats(a.p.dp, a.p.vp);
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(group_decode_kernel<F32, VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  const int group = a.p.heads / a.p.kv_heads;
+  return launch_cluster(group_decode_kernel<F32, VC>, dim3(a.splits, a.p.kv_heads, (group + kHB - 1) / kHB), dim3(kDecThreads), dim3(a.splits, 1, 1), smem, stream,
+                        pdl, a);
+}
+
+bool prep_ok(const GroupPrepArgs& p) {
+  return p.heads >= 1 && p.kv_heads >= 1 && p.heads % p.kv_heads == 0 && p.dim >= 1 && p.dim <= p.dp && p.dp <= kMaxHead && p.vdim >= 1 &&
+         p.vdim <= p.vp && p.vp <= kMaxHead && p.dp % 8 == 0 && p.vp % 8 == 0 && p.rot_dims >= 0 && p.rot_dims % 2 == 0 && p.rot_dims <= p.dim &&
+         (p.rot_dims == 0 || p.freq) && p.rows >= 1;
+}
+
+}  // namespace
+
+#define S(stream) reinterpret_cast<cudaStream_t>(stream)
+
+extern "C" int nrt_group_prep_args_size() { return (int)sizeof(GroupPrepArgs); }
+extern "C" int nrt_transpose_args_size() { return (int)sizeof(TransposeArgs); }
+extern "C" int nrt_group_decode_args_size() { return (int)sizeof(GroupDecodeArgs); }
+
+extern "C" int nrt_group_prep(const void* args, void* stream) {
+  GroupPrepArgs p;
+  memcpy(&p, args, sizeof(p));
+  if (!prep_ok(p) || !p.q) return -3;
+  return launch_pdl(group_prep_kernel, dim3(p.rows), dim3(256), 0, S(stream), false, p);
+}
+
+extern "C" int nrt_transpose(const void* args, void* stream) {
+  TransposeArgs a;
+  memcpy(&a, args, sizeof(a));
+  if (a.rows < 1 || a.cols < 1 || a.dst_ld < a.rows) return -3;
+  return launch_pdl(transpose_kernel, dim3((a.rows + 63) / 64, (a.cols + 63) / 64), dim3(256), 0, S(stream), false, a);
+}
+
+extern "C" int nrt_group_decode(const void* args, void* stream, int pdl) {
+  GroupDecodeArgs a;
+  memcpy(&a, args, sizeof(a));
+  if (!prep_ok(a.p) || a.p.rows != 1 || a.splits < 1 || a.splits > 8 || a.window < 0) return -3;
+  const bool wide = a.p.vdim > kDecThreads, p = pdl != 0;
+  if (a.p.f32) return wide ? launch_decode<true, 2>(a, S(stream), p) : launch_decode<true, 1>(a, S(stream), p);
+  return wide ? launch_decode<false, 2>(a, S(stream), p) : launch_decode<false, 1>(a, S(stream), p);
+}

@@ -56,13 +56,20 @@ __device__ __forceinline__ Item item_of(const StackGemmArgs& p, int item, int ro
 }
 
 template <int EPI>
-__device__ __forceinline__ float epi_value(const StackGemmArgs& p, float a0, float a1, int n, float bias) {
+constexpr bool epi_has_bias() { return EPI == kSEpiBias || EPI == kSEpiDecaySoft || EPI == kSEpiDecayExp; }
+
+template <int EPI>
+__device__ __forceinline__ float epi_value(const StackGemmArgs& p, float a0, float a1, int n, float bias, float rate) {
   if (EPI == kSEpiBias) {
     const float v = a0 + bias;
     return n < p.act_cols ? gelu_tanh_f(v) : v;
   }
   if (EPI == kSEpiClampedGlu) return clamped_glu(a0, a1, p.limit, p.alpha);
   if (EPI == kSEpiSiluGlu) return silu_glu(a0, a1);
+  if (EPI == kSEpiRelu2) return relu2_f(a0);
+  if (EPI == kSEpiTanh) return tanhf(a0);
+  if (EPI == kSEpiDecaySoft) return decay_soft(a0 + bias, rate);
+  if (EPI == kSEpiDecayExp) return decay_exp(a0 + bias);
   return a0 * p.scale;
 }
 
@@ -167,7 +174,8 @@ stack_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant
       tc_fence_after();
       const int n = tile * kFeat + feat;
       const bool live = n < p.n;
-      const float bias = (EPI == kSEpiBias && live) ? bf(p.bias + (size_t)it.z * p.n + n) : 0.f;
+      const float bias = (epi_has_bias<EPI>() && live) ? bf(p.bias + (size_t)it.z * p.n + n) : 0.f;
+      const float rate = (EPI == kSEpiDecaySoft && live) ? p.rate[n] : 0.f;
       const long long zoff = p.n_items ? 0 : it.z * p.out_zstride;
       const uint32_t acc = tmem + (uint32_t(quad * 32) << 16) + buf * C::kAccCols + half * kHalf;
       const int row_end = p.n_items ? 0x7fffffff : p.rows;
@@ -209,14 +217,14 @@ stack_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant
 #pragma unroll
             for (int r = 0; r < 32; ++r)
               if (row + r < row_end)
-                o[(long long)r * p.out_ld] = epi_value<EPI>(p, __uint_as_float(v0[r]), DUAL ? __uint_as_float(v1[DUAL ? r : 0]) : 0.f, n, bias);
+                o[(long long)r * p.out_ld] = epi_value<EPI>(p, __uint_as_float(v0[r]), DUAL ? __uint_as_float(v1[DUAL ? r : 0]) : 0.f, n, bias, rate);
           } else {
             __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + at;
 #pragma unroll
             for (int r = 0; r < 32; ++r)
               if (row + r < row_end)
                 o[(long long)r * p.out_ld] = __float2bfloat16_rn(
-                    epi_value<EPI>(p, __uint_as_float(v0[r]), DUAL ? __uint_as_float(v1[DUAL ? r : 0]) : 0.f, n, bias));
+                    epi_value<EPI>(p, __uint_as_float(v0[r]), DUAL ? __uint_as_float(v1[DUAL ? r : 0]) : 0.f, n, bias, rate));
           }
         }
       }
@@ -327,8 +335,9 @@ __global__ void __launch_bounds__(256) stack_gemm_f32_kernel(const StackGemmArgs
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       if (n >= p.n) continue;
-      const float bias = EPI == kSEpiBias ? bf(p.bias + (size_t)it.z * p.n + n) : 0.f;
-      const float v = epi_value<EPI>(p, acc[i][j], acc2[i][j], n, bias);
+      const float bias = epi_has_bias<EPI>() ? bf(p.bias + (size_t)it.z * p.n + n) : 0.f;
+      const float rate = EPI == kSEpiDecaySoft ? p.rate[n] : 0.f;
+      const float v = epi_value<EPI>(p, acc[i][j], acc2[i][j], n, bias, rate);
       store_act(p.out, (long long)row * p.out_ld + (p.n_items ? 0 : it.z * p.out_zstride) + n, v, p.out_f32);
     }
   }
@@ -356,6 +365,7 @@ extern "C" int nrt_stack_gemm(int epi, int ntok, const void* tmW, const void* tm
   StackGemmArgs a;
   memcpy(&a, args, sizeof(a));
   if (a.n < 1 || a.k < 1 || a.rows < 1 || (a.n_items && a.item_rows != ntok)) return -3;
+  if (((epi == kSEpiBias || epi == kSEpiDecaySoft || epi == kSEpiDecayExp) && !a.bias) || (epi == kSEpiDecaySoft && (!a.rate || a.zcount != 1))) return -3;
   if (epi == kSEpiTranspose && (a.out_f32 || a.out_ld % 8 || a.out_zstride % 8)) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define NRT_CASE(N, E) \
@@ -365,6 +375,10 @@ extern "C" int nrt_stack_gemm(int epi, int ntok, const void* tmW, const void* tm
   NRT_CASE(64, kSEpiTranspose) NRT_CASE(256, kSEpiTranspose)
   NRT_CASE(64, kSEpiClampedGlu) NRT_CASE(128, kSEpiClampedGlu)
   NRT_CASE(64, kSEpiSiluGlu) NRT_CASE(128, kSEpiSiluGlu)
+  NRT_CASE(64, kSEpiRelu2) NRT_CASE(128, kSEpiRelu2) NRT_CASE(256, kSEpiRelu2)
+  NRT_CASE(64, kSEpiTanh) NRT_CASE(256, kSEpiTanh)
+  NRT_CASE(64, kSEpiDecaySoft) NRT_CASE(256, kSEpiDecaySoft)
+  NRT_CASE(64, kSEpiDecayExp) NRT_CASE(256, kSEpiDecayExp)
 #undef NRT_CASE
   return -2;
 }
@@ -379,6 +393,10 @@ extern "C" int nrt_stack_gemm_f32(int epi, const void* args, void* stream) {
     case kSEpiBias: return launch_f32<kSEpiBias>(a, s);
     case kSEpiClampedGlu: return launch_f32<kSEpiClampedGlu>(a, s);
     case kSEpiSiluGlu: return launch_f32<kSEpiSiluGlu>(a, s);
+    case kSEpiRelu2: return launch_f32<kSEpiRelu2>(a, s);
+    case kSEpiTanh: return launch_f32<kSEpiTanh>(a, s);
+    case kSEpiDecaySoft: return launch_f32<kSEpiDecaySoft>(a, s);
+    case kSEpiDecayExp: return launch_f32<kSEpiDecayExp>(a, s);
   }
   return -2;
 }

@@ -11,19 +11,38 @@ using namespace nrt;
 namespace {
 
 // ------------------------------------------------------------------------------------ stream update + norms
-// One CTA per row.  x (+ embedding) -> x += rms(y) * post_w + add -> h = rms(x) * pre_w, all in float.
+// One CTA per row.  x (+ embedding) -> x += norm(y) * post_w + add -> h = norm(x) * pre_w (or x itself), all in float.
 __device__ __forceinline__ float4 bf4(const __nv_bfloat16* p) {
   const uint2 v = __ldg(reinterpret_cast<const uint2*>(p));
   return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
 }
 __device__ __forceinline__ float dot4(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+__device__ __forceinline__ float sum4(const float4& v) { return (v.x + v.y) + (v.z + v.w); }
+__device__ __forceinline__ float4 minus4(const float4& v, float m) { return make_float4(v.x - m, v.y - m, v.z - m, v.w - m); }
+
+// What a row is shifted and scaled by: `part` is the thread's sum of squares (RMS) or of values (layer norm: the squared
+// deviations are summed in a second pass over the thread's own values, `again(mean)`).
+struct RowNorm { float mean, r; };
+template <class Again>
+__device__ __forceinline__ RowNorm row_norm(int kind, float part, int width, float eps, float* red, Again again) {
+  RowNorm n;
+  n.mean = 0.f;
+  float sq = block_sum_f(part, red);
+  if (kind == kNormLayer) {
+    n.mean = sq / (float)width;
+    sq = block_sum_f(again(n.mean), red);
+  }
+  n.r = 1.0f / sqrtf(sq / (float)width + eps);
+  return n;
+}
 
 // widths that are multiples of four: 16-byte accesses, several in flight per thread
 __device__ __forceinline__ void rows_vec4(const StackRowArgs& a, int r, float4* buf, float* red) {
   const int W4 = a.width / 4;
+  const bool layer = a.norm == kNormLayer;
   float4* sy = buf;
   float4* sx = buf + W4;
-  float ry = 0.f;
+  RowNorm ny = {0.f, 0.f};
   float4* xrow = reinterpret_cast<float4*>(a.x + (size_t)r * a.width);
   if (a.y) {
     float ss = 0.f;
@@ -37,7 +56,28 @@ __device__ __forceinline__ void rows_vec4(const StackRowArgs& a, int r, float4* 
           v = make_float4(fmaf(p, t.x, v.x), fmaf(p, t.y, v.y), fmaf(p, t.z, v.z), fmaf(p, t.w, v.w));
         }
         sy[c] = v;
-        ss += dot4(v);
+        ss += layer ? sum4(v) : dot4(v);
+      }
+    } else if (a.y2) {
+      const float4* y = reinterpret_cast<const float4*>(a.y + (long long)r * a.y_ld);
+      const float4* y2 = reinterpret_cast<const float4*>(a.y2 + (long long)r * a.y_ld);
+      float s1 = 0.f, s2 = 0.f;
+#pragma unroll 4
+      for (int c = threadIdx.x; c < W4; c += 256) {
+        const float4 v = y[c], w = y2[c];
+        sy[c] = v;
+        sx[c] = w;
+        s1 += dot4(v);
+        s2 += dot4(w);
+      }
+      const float r1 = 0.5f / sqrtf(block_sum_f(s1, red) / (float)a.width + a.eps), r2 = 0.5f / sqrtf(block_sum_f(s2, red) / (float)a.width + a.eps);
+#pragma unroll 4
+      for (int c = threadIdx.x; c < W4; c += 256) {
+        const float4 v = sy[c], w = sx[c], wv = bf4(a.join_w + c * 4), ww = bf4(a.join_w2 + c * 4);
+        const float4 t = make_float4(fmaf(v.x * r1, wv.x, w.x * r2 * ww.x), fmaf(v.y * r1, wv.y, w.y * r2 * ww.y),
+                                     fmaf(v.z * r1, wv.z, w.z * r2 * ww.z), fmaf(v.w * r1, wv.w, w.w * r2 * ww.w));
+        sy[c] = t;
+        ss += layer ? sum4(t) : dot4(t);
       }
     } else {
       const float4* y = reinterpret_cast<const float4*>(a.y + (long long)r * a.y_ld);
@@ -45,10 +85,14 @@ __device__ __forceinline__ void rows_vec4(const StackRowArgs& a, int r, float4* 
       for (int c = threadIdx.x; c < W4; c += 256) {
         const float4 v = y[c];
         sy[c] = v;
-        ss += dot4(v);
+        ss += layer ? sum4(v) : dot4(v);
       }
     }
-    ry = 1.0f / sqrtf(block_sum_f(ss, red) / (float)a.width + a.eps);
+    ny = row_norm(a.norm, ss, a.width, a.eps, red, [&](float mean) {
+      float sq = 0.f;
+      for (int c = threadIdx.x; c < W4; c += 256) sq += dot4(minus4(sy[c], mean));
+      return sq;
+    });
   }
   const __nv_bfloat16* emb = nullptr;
   if (a.tokens) {
@@ -56,27 +100,36 @@ __device__ __forceinline__ void rows_vec4(const StackRowArgs& a, int r, float4* 
     t = t < 0 ? 0 : t >= a.vocab ? a.vocab - 1 : t;
     emb = a.table + (size_t)t * a.width;
   }
-  float sq = 0.f;
+  float part = 0.f;
 #pragma unroll 4
   for (int c = threadIdx.x; c < W4; c += 256) {
     float4 v;
     if (emb) { v = bf4(emb + c * 4); v = make_float4(v.x * a.embed_scale, v.y * a.embed_scale, v.z * a.embed_scale, v.w * a.embed_scale); }
     else v = xrow[c];
     if (a.y) {
-      const float4 y = sy[c], w = bf4(a.post_w + c * 4);
-      v = make_float4(fmaf(y.x * ry, w.x, v.x), fmaf(y.y * ry, w.y, v.y), fmaf(y.z * ry, w.z, v.z), fmaf(y.w * ry, w.w, v.w));
+      const float4 y = minus4(sy[c], ny.mean), w = bf4(a.post_w + c * 4);
+      v = make_float4(fmaf(y.x * ny.r, w.x, v.x), fmaf(y.y * ny.r, w.y, v.y), fmaf(y.z * ny.r, w.z, v.z), fmaf(y.w * ny.r, w.w, v.w));
     }
     if (a.add) { const float4 t = bf4(a.add + c * 4); v = make_float4(v.x + t.x, v.y + t.y, v.z + t.z, v.w + t.w); }
     xrow[c] = v;
     sx[c] = v;
-    sq += dot4(v);
+    part += layer ? sum4(v) : dot4(v);
   }
-  if (!a.pre_w) return;
-  const float rx = 1.0f / sqrtf(block_sum_f(sq, red) / (float)a.width + a.eps);
+  if (!a.pre_w && !a.copy_h) return;
+  RowNorm nx = {0.f, 1.f};
+  if (a.pre_w)
+    nx = row_norm(a.norm, part, a.width, a.eps, red, [&](float mean) {
+      float sq = 0.f;
+      for (int c = threadIdx.x; c < W4; c += 256) sq += dot4(minus4(sx[c], mean));
+      return sq;
+    });
 #pragma unroll 4
   for (int c = threadIdx.x; c < W4; c += 256) {
-    const float4 v = sx[c], w = bf4(a.pre_w + c * 4);
-    const float4 o = make_float4(v.x * rx * w.x, v.y * rx * w.y, v.z * rx * w.z, v.w * rx * w.w);
+    float4 o = sx[c];
+    if (a.pre_w) {
+      const float4 v = minus4(o, nx.mean), w = bf4(a.pre_w + c * 4);
+      o = make_float4(v.x * nx.r * w.x, v.y * nx.r * w.y, v.z * nx.r * w.z, v.w * nx.r * w.w);
+    }
     if (a.h_f32) reinterpret_cast<float4*>(reinterpret_cast<float*>(a.h) + (long long)r * a.h_ld)[c] = o;
     else reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.h) + (long long)r * a.h_ld)[c] =
         make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
@@ -92,47 +145,65 @@ __global__ void __launch_bounds__(256) stack_rows_kernel(const StackRowArgs a) {
     rows_vec4(a, r, reinterpret_cast<float4*>(buf), red);
     return;
   }
+  const bool layer = a.norm == kNormLayer;
   float* sy = buf;
   float* sx = buf + W;
-  float ss = 0.f;
+  RowNorm ny = {0.f, 0.f};
   if (a.y) {
-    if (a.slot_of) {
+    float ss = 0.f;
+    if (a.y2) {
+      float s1 = 0.f, s2 = 0.f;
+      for (int c = threadIdx.x; c < W; c += 256) {
+        const float v = a.y[(long long)r * a.y_ld + c], w = a.y2[(long long)r * a.y_ld + c];
+        sy[c] = v;
+        sx[c] = w;
+        s1 = fmaf(v, v, s1);
+        s2 = fmaf(w, w, s2);
+      }
+      const float r1 = 0.5f / sqrtf(block_sum_f(s1, red) / (float)W + a.eps), r2 = 0.5f / sqrtf(block_sum_f(s2, red) / (float)W + a.eps);
+      for (int c = threadIdx.x; c < W; c += 256) sy[c] = sy[c] * r1 * bf(a.join_w + c) + sx[c] * r2 * bf(a.join_w2 + c);
+    } else if (a.slot_of) {
       for (int c = threadIdx.x; c < W; c += 256) {
         float v = 0.f;
         for (int j = 0; j < a.top_k; ++j)
           v = fmaf(a.probs[(size_t)r * a.top_k + j], a.y[(long long)a.slot_of[(size_t)r * a.top_k + j] * a.y_ld + c], v);
         sy[c] = v;
-        ss = fmaf(v, v, ss);
       }
     } else {
-      for (int c = threadIdx.x; c < W; c += 256) {
-        const float v = a.y[(long long)r * a.y_ld + c];
-        sy[c] = v;
-        ss = fmaf(v, v, ss);
-      }
+      for (int c = threadIdx.x; c < W; c += 256) sy[c] = a.y[(long long)r * a.y_ld + c];
     }
-    ss = block_sum_f(ss, red);
+    for (int c = threadIdx.x; c < W; c += 256) ss += layer ? sy[c] : sy[c] * sy[c];
+    ny = row_norm(a.norm, ss, W, a.eps, red, [&](float mean) {
+      float sq = 0.f;
+      for (int c = threadIdx.x; c < W; c += 256) sq = fmaf(sy[c] - mean, sy[c] - mean, sq);
+      return sq;
+    });
   }
-  const float ry = a.y ? 1.0f / sqrtf(ss / (float)W + a.eps) : 0.f;
   const __nv_bfloat16* emb = nullptr;
   if (a.tokens) {
     int t = a.tokens[r];
     t = t < 0 ? 0 : t >= a.vocab ? a.vocab - 1 : t;
     emb = a.table + (size_t)t * W;
   }
-  float sq = 0.f;
+  float part = 0.f;
   for (int c = threadIdx.x; c < W; c += 256) {
     float v = emb ? bf(emb + c) * a.embed_scale : a.x[(size_t)r * W + c];
-    if (a.y) v += sy[c] * ry * bf(a.post_w + c);
+    if (a.y) v += (sy[c] - ny.mean) * ny.r * bf(a.post_w + c);
     if (a.add) v += bf(a.add + c);
     a.x[(size_t)r * W + c] = v;
     sx[c] = v;
-    sq = fmaf(v, v, sq);
+    part += layer ? v : v * v;
   }
-  if (!a.pre_w) return;
-  sq = block_sum_f(sq, red);
-  const float rx = 1.0f / sqrtf(sq / (float)W + a.eps);
-  for (int c = threadIdx.x; c < W; c += 256) store_act(a.h, (long long)r * a.h_ld + c, sx[c] * rx * bf(a.pre_w + c), a.h_f32);
+  if (!a.pre_w && !a.copy_h) return;
+  RowNorm nx = {0.f, 1.f};
+  if (a.pre_w)
+    nx = row_norm(a.norm, part, W, a.eps, red, [&](float mean) {
+      float sq = 0.f;
+      for (int c = threadIdx.x; c < W; c += 256) sq = fmaf(sx[c] - mean, sx[c] - mean, sq);
+      return sq;
+    });
+  for (int c = threadIdx.x; c < W; c += 256)
+    store_act(a.h, (long long)r * a.h_ld + c, a.pre_w ? (sx[c] - nx.mean) * nx.r * bf(a.pre_w + c) : sx[c], a.h_f32);
 }
 
 // ------------------------------------------------------------------------------------ latent preparation
@@ -342,7 +413,7 @@ extern "C" int nrt_stack_scan_tokens() { return kScanTokens; }
 extern "C" int nrt_stack_rows(const void* args, void* stream) {
   StackRowArgs a;
   memcpy(&a, args, sizeof(a));
-  if (a.rows < 1 || a.width < 1 || (a.y && !a.post_w)) return -3;
+  if (a.rows < 1 || a.width < 1 || (a.y && !a.post_w) || (a.y2 && (!a.y || a.slot_of || !a.join_w || !a.join_w2))) return -3;
   const size_t smem = (size_t)a.width * 8;
   if (smem > 200 * 1024) return -7;
   static bool configured = false;

@@ -2,10 +2,10 @@
 //
 // A single token reads every weight once, so the step is bound by HBM and the CUDA cores keep up with it; activations stay
 // fp32 throughout.  Each launch is (prologue) -> W h -> (epilogue):
-//   prologues  stream update + norm (every CTA repeats it: two row-sized L2 reads instead of a launch of its own), norm of a
-//              segment, plain load per group, merge of the attention partials
-//   epilogues  store / sigmoid, biased branches with the short convolution, output gate, two-product activations, the
-//              recurrence step
+//   prologues  stream update + norms (every CTA repeats it: two row-sized L2 reads instead of a launch of its own), the same
+//              with a mix of the previous token per group, norm of a segment, plain load per group, merge of the attention partials
+//   epilogues  store / sigmoid / bias / squared relu, branches with the short convolution, output gate, two-product activations,
+//              the recurrence step
 // Weights stream through shared memory: each of the sixteen warps owns a run of output rows and a ring of its own (three 4 KiB
 // slots) that one lane fills with bulk copies, so no two warps wait for one another inside the product.  The ring is filled
 // before griddepcontrol.wait, where the choice of weights does not depend on the predecessor.  Measured on B200: smaller rings
@@ -70,8 +70,8 @@ __device__ __forceinline__ void preload(const StepArgs& a, Pre& p) {
     p.x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     p.post[i] = p.in[i] = make_uint2(0u, 0u);
     if (e < a.k) {
-      p.in[i] = ldw4(a.in_w + e);
-      if (PRO == kProResidual) {
+      if (a.in_w) p.in[i] = ldw4(a.in_w + e);
+      if (PRO == kProResidual || PRO == kProMix) {
         if (a.y) p.post[i] = ldw4(a.post_w + e);
         if (!a.tokens) p.x[i] = ldcg4(a.x + e);
       }
@@ -79,97 +79,157 @@ __device__ __forceinline__ void preload(const StepArgs& a, Pre& p) {
   }
 }
 
+__device__ __forceinline__ float sum4(const float4& v) { return (v.x + v.y) + (v.z + v.w); }
+__device__ __forceinline__ float4 minus4(const float4& v, float m) { return make_float4(v.x - m, v.y - m, v.z - m, v.w - m); }
+__device__ __forceinline__ float4 scale4(const float4& v, float s) { return make_float4(v.x * s, v.y * s, v.z * s, v.w * s); }
+__device__ __forceinline__ float4 add4(const float4& a, const float4& b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+
+// The input of one group in shared memory.  `slot`: state slot of the previous token (kProMix).
 template <int PRO>
-__device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, float* hs, float* red, const Pre& p, int pos) {
+__device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, float* hs, float* red, const Pre& p, int pos, int slot) {
   const int K = a.k;
   float4* hs4 = reinterpret_cast<float4*>(hs);
   // element e (a multiple of four) of the input -> its float4 in the two planes
   auto at4 = [&](int e) -> float4& { return hs4[((e >> 2) & 1) * k8 + (e >> 3)]; };
-  if (PRO == kProResidual || PRO == kProNorm) {
+  if (PRO == kProResidual || PRO == kProNorm || PRO == kProMix) {
+    constexpr bool STREAM = PRO != kProNorm;
+    const bool layer = STREAM && a.norm == kNormLayer;
     const __nv_bfloat16* emb = nullptr;
-    if (PRO == kProResidual && a.tokens) {
+    if (STREAM && a.tokens) {
       int t = *reinterpret_cast<const volatile int*>(a.tokens);
       t = t < 0 ? 0 : t >= a.vocab ? a.vocab - 1 : t;
       emb = a.table + (size_t)t * K;
     }
+    // kProMix: the previous token's stream (none at position 0), this group's mixing weights
+    const float* before = PRO == kProMix && pos > 0 && slot >= 0 ? a.shift + (long long)slot * a.state_stride : nullptr;
+    float* after = PRO == kProMix && blockIdx.x == 0 && slot >= 0 ? a.shift + (long long)(1 - slot) * a.state_stride : nullptr;
+    const __nv_bfloat16* mu = PRO == kProMix ? a.mu + (long long)g * K : nullptr;
     if ((K & 3) == 0) {
+      // the first kPreSpan elements stay in registers, the others in the input's own place
       float4 v[kPreN];
-      float ss = 0.f, sq = 0.f;
-      if (PRO == kProResidual && a.y) {
+      auto each = [&](auto&& f) {
 #pragma unroll
         for (int i = 0; i < kPreN; ++i) {
           const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
-          v[i] = e < K ? ldcg4(a.y + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+          if (e < K) f(e, v[i]);
         }
-#pragma unroll
-        for (int i = 0; i < kPreN; ++i) ss += dot4(v[i]);
-        for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) ss += dot4(ldcg4(a.y + e));
-        ss = block_sum_f(ss, red);
-      } else if (PRO == kProNorm) {
+        for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) f(e, at4(e));
+      };
+      float mean = 0.f, r = 0.f;
+      auto norm_of = [&](float part) {                   // sums of squares, or (layer norm) of values
+        float sq = block_sum_f(part, red);
+        mean = 0.f;
+        if (layer) {
+          mean = sq / (float)K;
+          float d = 0.f;
+          each([&](int, float4& t) { d += dot4(minus4(t, mean)); });
+          sq = block_sum_f(d, red);
+        }
+        r = 1.0f / sqrtf(sq / (float)K + a.eps);
+      };
+      float part = 0.f;
+      if (PRO == kProNorm) {
+        each([&](int e, float4& t) { t = ldcg4(a.in_ + e); part += dot4(t); });
+      } else {
+        if (a.y) {
+          if (a.y2) {
+            // two sublayers side by side: half the sum of both, each divided by its root mean square
+            float s1 = 0.f, s2 = 0.f;
+            each([&](int e, float4& t) { t = ldcg4(a.y + e); s1 += dot4(t); s2 += dot4(ldcg4(a.y2 + e)); });
+            const float r1 = 0.5f / sqrtf(block_sum_f(s1, red) / (float)K + a.eps), r2 = 0.5f / sqrtf(block_sum_f(s2, red) / (float)K + a.eps);
+            each([&](int e, float4& t) {
+              t = fma4(t, bf4(ldw4(a.join_w + e)), r1, fma4(ldcg4(a.y2 + e), bf4(ldw4(a.join_w2 + e)), r2, make_float4(0.f, 0.f, 0.f, 0.f)));
+              part += layer ? sum4(t) : dot4(t);
+            });
+          } else {
+            each([&](int e, float4& t) { t = ldcg4(a.y + e); part += layer ? sum4(t) : dot4(t); });
+          }
+          norm_of(part);
+        }
+        part = 0.f;
+        auto stream = [&](int e, float4& t, float4 x, const float4& w) {
+          if (emb) x = scale4(bf4(ldw4(emb + e)), a.embed_scale);
+          if (a.y) x = fma4(minus4(t, mean), w, r, x);
+          if (a.add) x = add4(x, bf4(ldw4(a.add + e)));
+          if (blockIdx.x == 0) *reinterpret_cast<float4*>(a.x_out + e) = x;
+          t = x;
+          part += layer ? sum4(x) : dot4(x);
+        };
 #pragma unroll
         for (int i = 0; i < kPreN; ++i) {
           const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
-          v[i] = e < K ? ldcg4(a.in_ + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+          if (e < K) stream(e, v[i], p.x[i], bf4(p.post[i]));
         }
+        for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4)
+          stream(e, at4(e), emb ? make_float4(0.f, 0.f, 0.f, 0.f) : ldcg4(a.x + e), a.y ? bf4(ldw4(a.post_w + e)) : make_float4(0.f, 0.f, 0.f, 0.f));
       }
-      const float ry = PRO == kProResidual && a.y ? 1.0f / sqrtf(ss / (float)K + a.eps) : 0.f;
+      if (PRO == kProMix) {
+        each([&](int e, float4& t) {
+          if (after) *reinterpret_cast<float4*>(after + e) = t;
+          const float4 b = before ? ldcg4(before + e) : make_float4(0.f, 0.f, 0.f, 0.f), m = bf4(ldw4(mu + e));
+          at4(e) = make_float4(fmaf(b.x - t.x, m.x, t.x), fmaf(b.y - t.y, m.y, t.y), fmaf(b.z - t.z, m.z, t.z), fmaf(b.w - t.w, m.w, t.w));
+        });
+      } else if (STREAM && a.raw_in) {
+        each([&](int e, float4& t) { at4(e) = t; });
+      } else {
+        norm_of(part);
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int i = 0; i < kPreN; ++i) {
-        const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
-        if (e >= K) continue;
-        if (PRO == kProResidual) {
-          float4 x = p.x[i];
-          if (emb) { const float4 t = bf4(ldw4(emb + e)); x = make_float4(t.x * a.embed_scale, t.y * a.embed_scale, t.z * a.embed_scale, t.w * a.embed_scale); }
-          if (a.y) x = fma4(v[i], bf4(p.post[i]), ry, x);
-          if (a.add) { const float4 t = bf4(ldw4(a.add + e)); x = make_float4(x.x + t.x, x.y + t.y, x.z + t.z, x.w + t.w); }
-          if (blockIdx.x == 0) *reinterpret_cast<float4*>(a.x_out + e) = x;
-          v[i] = x;
+        for (int i = 0; i < kPreN; ++i) {
+          const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
+          if (e < K) at4(e) = fma4(minus4(v[i], mean), bf4(p.in[i]), r, zero);
         }
-        sq += dot4(v[i]);
+        for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) at4(e) = fma4(minus4(at4(e), mean), bf4(ldw4(a.in_w + e)), r, zero);
       }
-      for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) {
-        float4 x;
-        if (PRO == kProResidual) {
-          if (emb) { const float4 t = bf4(ldw4(emb + e)); x = make_float4(t.x * a.embed_scale, t.y * a.embed_scale, t.z * a.embed_scale, t.w * a.embed_scale); }
-          else x = ldcg4(a.x + e);
-          if (a.y) x = fma4(ldcg4(a.y + e), bf4(ldw4(a.post_w + e)), ry, x);
-          if (a.add) { const float4 t = bf4(ldw4(a.add + e)); x = make_float4(x.x + t.x, x.y + t.y, x.z + t.z, x.w + t.w); }
-          if (blockIdx.x == 0) *reinterpret_cast<float4*>(a.x_out + e) = x;
-        } else {
-          x = ldcg4(a.in_ + e);
-        }
-        at4(e) = x;
-        sq += dot4(x);
-      }
-      sq = block_sum_f(sq, red);
-      const float rx = 1.0f / sqrtf(sq / (float)K + a.eps);
-      const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-      for (int i = 0; i < kPreN; ++i) {
-        const int e = (i * kStepThreads + (int)threadIdx.x) * 4;
-        if (e < K) at4(e) = fma4(v[i], bf4(p.in[i]), rx, zero);
-      }
-      for (int e = kPreSpan + (int)threadIdx.x * 4; e < K; e += kStepThreads * 4) at4(e) = fma4(at4(e), bf4(ldw4(a.in_w + e)), rx, zero);
     } else {
-      float ss = 0.f, sq = 0.f;
-      if (PRO == kProResidual && a.y) {
-        for (int c = threadIdx.x; c < K; c += kStepThreads) { const float v = __ldcg(a.y + c); ss = fmaf(v, v, ss); }
-        ss = block_sum_f(ss, red);
-      }
-      const float ry = PRO == kProResidual && a.y ? 1.0f / sqrtf(ss / (float)K + a.eps) : 0.f;
-      for (int c = threadIdx.x; c < K; c += kStepThreads) {
-        float v = PRO == kProNorm ? __ldcg(a.in_ + c) : emb ? bf(emb + c) * a.embed_scale : __ldcg(a.x + c);
-        if (PRO == kProResidual) {
-          if (a.y) v += __ldcg(a.y + c) * ry * bf(a.post_w + c);
-          if (a.add) v += bf(a.add + c);
-          if (blockIdx.x == 0) a.x_out[c] = v;
+      auto at = [&](int c) -> float& { return hs[plane_at(c, k8)]; };
+      float mean = 0.f, r = 0.f;
+      auto norm_of = [&]() {
+        float part = 0.f;
+        for (int c = threadIdx.x; c < K; c += kStepThreads) part += layer ? at(c) : at(c) * at(c);
+        float sq = block_sum_f(part, red);
+        mean = 0.f;
+        if (layer) {
+          mean = sq / (float)K;
+          float d = 0.f;
+          for (int c = threadIdx.x; c < K; c += kStepThreads) d = fmaf(at(c) - mean, at(c) - mean, d);
+          sq = block_sum_f(d, red);
         }
-        hs[plane_at(c, k8)] = v;
-        sq = fmaf(v, v, sq);
+        r = 1.0f / sqrtf(sq / (float)K + a.eps);
+      };
+      if (STREAM && a.y) {
+        float r1 = 1.f, r2 = 0.f;
+        if (a.y2) {
+          float s1 = 0.f, s2 = 0.f;
+          for (int c = threadIdx.x; c < K; c += kStepThreads) {
+            const float t = __ldcg(a.y + c), u = __ldcg(a.y2 + c);
+            s1 = fmaf(t, t, s1);
+            s2 = fmaf(u, u, s2);
+          }
+          r1 = 0.5f / sqrtf(block_sum_f(s1, red) / (float)K + a.eps);
+          r2 = 0.5f / sqrtf(block_sum_f(s2, red) / (float)K + a.eps);
+        }
+        for (int c = threadIdx.x; c < K; c += kStepThreads)
+          at(c) = a.y2 ? __ldcg(a.y + c) * r1 * bf(a.join_w + c) + __ldcg(a.y2 + c) * r2 * bf(a.join_w2 + c) : __ldcg(a.y + c);
+        norm_of();
       }
-      sq = block_sum_f(sq, red);
-      const float rx = 1.0f / sqrtf(sq / (float)K + a.eps);
-      for (int c = threadIdx.x; c < K; c += kStepThreads) hs[plane_at(c, k8)] *= rx * bf(a.in_w + c);
+      for (int c = threadIdx.x; c < K; c += kStepThreads) {
+        float x = PRO == kProNorm ? __ldcg(a.in_ + c) : emb ? bf(emb + c) * a.embed_scale : __ldcg(a.x + c);
+        if (STREAM) {
+          if (a.y) x += (at(c) - mean) * r * bf(a.post_w + c);
+          if (a.add) x += bf(a.add + c);
+          if (blockIdx.x == 0) a.x_out[c] = x;
+        }
+        if (PRO == kProMix) {
+          if (after) after[c] = x;
+          x = fmaf((before ? __ldcg(before + c) : 0.f) - x, bf(mu + c), x);
+        }
+        at(c) = x;
+      }
+      if (PRO == kProNorm || (PRO == kProResidual && !a.raw_in)) {
+        norm_of();
+        for (int c = threadIdx.x; c < K; c += kStepThreads) at(c) = (at(c) - mean) * r * bf(a.in_w + c);
+      }
     }
   } else if (PRO == kProLoad) {
     const float* in = a.in_ + g * a.in_gstride;
@@ -239,7 +299,22 @@ template <int EPI>
 __device__ __forceinline__ void finish_row(const StepArgs& a, int g, int row, float v, float v2, int pos, int slot) {
   const size_t at = (size_t)g * a.n + row;
   if (EPI == kTEpiStore) {
-    a.out[at] = row >= a.sig_from ? sigmoid_f(v) : v * a.scale;
+    v = row >= a.sig_from ? sigmoid_f(v) : v * a.scale;
+    a.out[at] = a.bias ? v + bf(a.bias + at) : v;
+  } else if (EPI == kTEpiRelu2) {
+    a.out[at] = relu2_f(v);
+  } else if (EPI == kTEpiConvSilu) {
+    if (row < a.conv_rows) {
+      float u = 0.f;
+      for (int j = 0; j < a.taps - 1; ++j) {
+        const int back = a.taps - 1 - j;
+        if (back <= pos) u = fmaf(bf(a.conv + (size_t)row * a.taps + j), a.history[(long long)((pos - back) % a.hist_rows) * a.conv_rows + row], u);
+      }
+      u = fmaf(bf(a.conv + (size_t)row * a.taps + a.taps - 1), v, u);
+      a.history[(long long)(pos % a.hist_rows) * a.conv_rows + row] = v;
+      v = silu_f(u);
+    }
+    a.out[at] = v;
   } else if (EPI == kTEpiGate) {
     a.out[at] = v * __ldcg(a.gate + at);
   } else if (EPI == kTEpiGlu) {
@@ -291,7 +366,7 @@ template <int PRO, int EPI, bool ROUTE>
 __global__ void __launch_bounds__(kStepThreads, 2) stack_step_kernel(const StepArgs a, const RouterArgs ra, const int rgroups,
                                                                      const int rkeep, const StepShape sh) {
   constexpr bool DUAL = EPI == kTEpiGlu || EPI == kTEpiRecur;
-  constexpr bool PER_GROUP = PRO == kProLoad || PRO == kProMerge;
+  constexpr bool PER_GROUP = PRO == kProLoad || PRO == kProMerge || PRO == kProMix;
   constexpr int CUT = DUAL ? kSlot / 32 : kSlot / 16;                  // pieces per slot and matrix
   extern __shared__ __align__(128) uint8_t dyn[];
   __shared__ float red[33];
@@ -303,7 +378,7 @@ __global__ void __launch_bounds__(kStepThreads, 2) stack_step_kernel(const StepA
   const float4* hs4 = reinterpret_cast<const float4*>(hs);
   uint64_t* bar = bars + warp * 3;
   const int k8 = sh.k8, ld8 = (int)(a.w_ld / 8), total = a.segs * k8;
-  const int R = a.groups * a.n;
+  const int n_last = a.n_last ? a.n_last : a.n, R = (a.groups - 1) * a.n + n_last;
   if (lane == 0) {
     for (int i = 0; i < sh.slots; ++i) mbar_init(&bar[i], 1);
     mbar_fence_init();
@@ -318,9 +393,9 @@ __global__ void __launch_bounds__(kStepThreads, 2) stack_step_kernel(const StepA
   auto open_unit = [&](int u) {
     int lo, hi;
     if (PER_GROUP) {
-      const int g = u / sh.parts, part = u - g * sh.parts;
-      lo = g * a.n + min(a.n, part * sh.q);
-      hi = g * a.n + min(a.n, (part + 1) * sh.q);
+      const int g = min(u / sh.parts, a.groups - 1), part = u - g * sh.parts, ng = g == a.groups - 1 ? n_last : a.n;
+      lo = g * a.n + min(ng, part * sh.q);
+      hi = g * a.n + min(ng, (part + 1) * sh.q);
     } else {
       lo = min(R, u * sh.q);
       hi = min(R, lo + sh.q);
@@ -367,7 +442,7 @@ __global__ void __launch_bounds__(kStepThreads, 2) stack_step_kernel(const StepA
   constexpr bool EARLY = !ROUTE && PRO != kProExperts;                 // which weights is known before the predecessor ends
   if (EARLY) fill();
   Pre pre;
-  if constexpr (PRO == kProResidual) preload<PRO>(a, pre);             // (a normed input may come from the predecessor itself)
+  if constexpr (PRO == kProResidual || PRO == kProMix) preload<PRO>(a, pre);   // (a normed input may come from the predecessor itself)
   griddep_wait();
   griddep_launch();
   const int pos = a.pos0 ? *reinterpret_cast<const volatile int*>(a.pos0) : 0;
@@ -384,9 +459,9 @@ __global__ void __launch_bounds__(kStepThreads, 2) stack_step_kernel(const StepA
   }
   if (!EARLY) fill();
   int slot = 1;
-  if (EPI == kTEpiRecur) slot = state_slot(a.tags, pos, a.status);
+  if (EPI == kTEpiRecur || PRO == kProMix) slot = state_slot(a.tags, pos, a.status);
   if constexpr (PRO == kProNorm) preload<PRO>(a, pre);
-  if (!PER_GROUP) load_input<PRO>(a, 0, k8, hs, red, pre, pos);
+  if (!PER_GROUP) load_input<PRO>(a, 0, k8, hs, red, pre, pos, slot);
   if (PRO == kProNorm && a.lat_in && blockIdx.x == gridDim.x - 1 && pos >= 0 && pos < a.capacity) {
     // append the token's key/value latent to the cache
     float sq = 0.f;
@@ -400,7 +475,7 @@ __global__ void __launch_bounds__(kStepThreads, 2) stack_step_kernel(const StepA
   int u_slot = 0;
   uint32_t u_phase = 0;
   while (true) {
-    if (PER_GROUP) load_input<PRO>(a, unit / sh.parts, k8, hs, red, pre, pos);
+    if (PER_GROUP) load_input<PRO>(a, min(unit / sh.parts, a.groups - 1), k8, hs, red, pre, pos, slot);
     // results of up to 32 finished rows wait in the lanes, then all lanes run the epilogue at once
     float acc = 0.f, acc2 = 0.f, res = 0.f, res2 = 0.f;
     int ready = 0, first = row, seg = 0, sub = 0;
@@ -498,7 +573,7 @@ int step_sms() {
 template <int PRO, int EPI, bool ROUTE>
 int launch_step(const StepArgs& a, const RouterArgs& r, int groups, int keep, cudaStream_t stream, bool pdl) {
   constexpr bool DUAL = EPI == kTEpiGlu || EPI == kTEpiRecur;
-  constexpr bool PER_GROUP = PRO == kProLoad || PRO == kProMerge;
+  constexpr bool PER_GROUP = PRO == kProLoad || PRO == kProMerge || PRO == kProMix;
   constexpr int CUT = DUAL ? kSlot / 32 : kSlot / 16;
   auto* kern = stack_step_kernel<PRO, EPI, ROUTE>;
   static bool configured = false;
@@ -507,7 +582,8 @@ int launch_step(const StepArgs& a, const RouterArgs& r, int groups, int keep, cu
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  const long long R = (long long)a.groups * a.n;
+  const int n_last = a.n_last ? a.n_last : a.n;
+  const long long R = (long long)(a.groups - 1) * a.n + n_last;
   if (R > 0x7fffffffLL) return -3;
   StepShape s = {};
   s.k8 = (a.k + 7) / 8;
@@ -521,10 +597,15 @@ int launch_step(const StepArgs& a, const RouterArgs& r, int groups, int keep, cu
   }
   const int sms = step_sms();
   if (PER_GROUP) {
-    s.parts = sms / a.groups > 1 ? sms / a.groups : 1;
-    s.q = (a.n + s.parts - 1) / s.parts;
+    // the most parts per group (a shorter last group gets fewer) that fill the SMs once
+    auto last = [&]() { return (n_last + s.q - 1) / s.q; };
+    s.parts = n_last < a.n && a.groups > 1 ? sms / (a.groups - 1) : sms / a.groups;
+    for (s.parts = s.parts > 1 ? s.parts : 1;; --s.parts) {
+      s.q = (a.n + s.parts - 1) / s.parts;
+      if (s.parts == 1 || (a.groups - 1) * ((a.n + s.q - 1) / s.q) + last() <= sms) break;
+    }
     s.parts = (a.n + s.q - 1) / s.q;
-    s.units = a.groups * s.parts;
+    s.units = (a.groups - 1) * s.parts + last();
   } else {
     const long long want = (R + kWarps - 1) / kWarps;
     const int grid = (int)(want < sms ? want : sms);
@@ -553,6 +634,11 @@ extern "C" int nrt_stack_step(int pro, int epi, const void* args, const void* ro
   if (router) memcpy(&r, router, sizeof(r));
   if (a.n < 1 || a.k < 1 || a.groups < 1 || a.segs < 1 || a.segs > 32 || (a.segs > 1 && pro != kProExperts) || a.w_ld % 8 || a.w_gstride % 8 || a.w2_gstride % 8) return -3;
   if (router && (r.experts > 256 || r.top_k > 32 || r.rows != 1 || groups < 1 || groups > 32 || r.experts % groups)) return -3;
+  if (a.n_last < 0 || a.n_last > a.n || (a.y2 && (!a.y || !a.join_w || !a.join_w2))) return -3;
+  if ((pro == kProResidual || pro == kProMix) && a.y && !a.post_w) return -3;
+  if (pro == kProResidual && !a.raw_in && !a.in_w) return -3;
+  if (pro == kProMix && (!a.mu || !a.shift || !a.tags)) return -3;
+  if (epi == kTEpiConvSilu && (a.hist_rows < 1 || a.hist_rows < 2 * (a.taps - 1) || a.groups != 1 || a.conv_rows > a.n)) return -3;
   if (epi == kTEpiConv && (a.hist_rows < 1 || a.hist_rows < 2 * (a.taps - 1) || a.groups != 1)) return -3;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const bool p = pdl != 0;
@@ -561,6 +647,9 @@ extern "C" int nrt_stack_step(int pro, int epi, const void* args, const void* ro
   NRT_CASE(kProResidual, kTEpiStore)
   NRT_CASE(kProResidual, kTEpiConv)
   NRT_CASE(kProResidual, kTEpiGlu)
+  NRT_CASE(kProResidual, kTEpiConvSilu)
+  NRT_CASE(kProResidual, kTEpiRelu2)
+  NRT_CASE(kProMix, kTEpiStore)
   NRT_CASE(kProNorm, kTEpiStore)
   NRT_CASE(kProLoad, kTEpiStore)
   NRT_CASE(kProExperts, kTEpiStore)

@@ -10,7 +10,7 @@ has its own cache or state.
 from __future__ import annotations
 
 from dataclasses import dataclass, replace
-from typing import List, Optional, Tuple, Union
+from typing import Dict, List, Optional, Tuple, Union
 
 from .spec import MoeRoutingSpec
 
@@ -19,6 +19,7 @@ MAX_EXPERTS, MAX_TOP_K, MAX_GROUPS = 256, 32, 32
 MAX_HEAD_DIM = 512
 MAX_RANK = 4096
 MAX_STEP_INPUT = 40000           # values a product of the one-token step can take in
+MAX_STATE_DIM = 512              # key width of a matrix state
 
 
 @dataclass(frozen=True)
@@ -56,6 +57,107 @@ class GatedRecurrenceSpec:
 
 
 @dataclass(frozen=True)
+class RotarySpec:
+    """Rotation of the first ``dims`` columns of a head (column i paired with i + dims / 2) by position * freq[i]."""
+
+    dims: int
+    base: float
+    factor: float = 1.0              # linear scaling: every frequency is divided by it
+
+    def frequencies(self) -> List[float]:
+        return [self.base ** (-2.0 * i / self.dims) / self.factor for i in range(self.dims // 2)]
+
+
+@dataclass(frozen=True)
+class GroupedAttentionSpec:
+    """Softmax attention with shared key / value heads, norms per head, rotary positions and biases; with ``window`` > 0
+    positions fall into chunks of that many (counted from 0) and a query sees its own chunk only."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rotary: Optional[RotarySpec] = None
+    window: int = 0
+    kind: str = "grouped_attention"
+
+
+@dataclass(frozen=True)
+class DeltaStateSpec:
+    """Gated delta rule with a decay per head and key channel; short convolutions ahead of q, k and v; the decay and the
+    output gate come through low-rank products (``decay_rank``, ``gate_rank``)."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+    decay_rank: int
+    gate_rank: int
+    kind: str = "channel_delta"
+
+    @property
+    def conv_columns(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    @property
+    def hist_rows(self) -> int:
+        """Ring rows of the convolution history (see ``GatedRecurrenceSpec.hist_rows``)."""
+        return max(1, 2 * (self.taps - 1))
+
+    def state_floats(self, hidden: int) -> int:
+        return _pad(self.heads * self.vdim * _pad(self.dim, 4), 4)
+
+
+@dataclass(frozen=True)
+class BonusStateSpec:
+    """Time mixing with the previous token ahead of every product, a data-dependent decay per channel (low-rank) and a bonus
+    for the current token."""
+
+    heads: int
+    dim: int
+    decay_rank: int
+    kind: str = "wkv"
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    def state_floats(self, hidden: int) -> int:
+        """The matrices, then the previous token's input."""
+        return self.shift_at + _pad(hidden, 4)
+
+    @property
+    def shift_at(self) -> int:
+        return self.heads * self.dim * _pad(self.dim, 4)
+
+
+@dataclass(frozen=True)
+class NormalizedStateSpec:
+    """Matrix memory with exponential gates (log gates capped at ``cap``), a normaliser and a running maximum."""
+
+    heads: int
+    dim: int
+    vdim: int
+    cap: float
+    kind: str = "mlstm"
+
+    def state_floats(self, hidden: int) -> int:
+        """The matrices with the normaliser as one more column, then the maxima."""
+        return _pad(self.heads * (self.vdim + 1) * _pad(self.dim, 4) + self.heads, 4)
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers that read the same input; the sublayer is half the sum of their outputs, each RMS-normed."""
+
+    left: GroupedAttentionSpec
+    right: NormalizedStateSpec
+    kind: str = "parallel"
+
+
+@dataclass(frozen=True)
 class ClampedGluSpec:
     """min(g, limit) * sigmoid(alpha * g) * (clamp(u, -limit, limit) + 1) between two products."""
 
@@ -63,6 +165,14 @@ class ClampedGluSpec:
     limit: float
     alpha: float = 1.702
     kind: str = "dense"
+
+
+@dataclass(frozen=True)
+class SquaredReluSpec:
+    """relu(.)^2 between two products."""
+
+    ff: int
+    kind: str = "relu2"
 
 
 @dataclass(frozen=True)
@@ -77,14 +187,15 @@ class ExpertsSpec:
         return self.routing.intermediate
 
 
-Mixer = Union[LatentAttentionSpec, GatedRecurrenceSpec]
-FeedForward = Union[ClampedGluSpec, ExpertsSpec]
+Mixer = Union[LatentAttentionSpec, GatedRecurrenceSpec, DeltaStateSpec, BonusStateSpec, ParallelSpec]
+FeedForward = Union[ClampedGluSpec, SquaredReluSpec, ExpertsSpec]
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: Mixer
     mlp: Optional[FeedForward]
+    weights_of: Optional[int] = None     # layer whose tensors this one uses (cache and state stay its own)
 
 
 @dataclass(frozen=True)
@@ -114,6 +225,9 @@ class StackSpec:
     embed_scale: float = 1.0
     logit_scale: float = 1.0
     loop: Optional[LoopSpec] = None
+    norm: str = "rms"                # kind of the norms around a sublayer and of the last one: "rms" or "layer"
+    pre_norm: bool = True            # a sublayer reads the normed stream (else the stream itself); its output is always normed
+    tied_head: bool = True           # the output product uses the embedding table
     stop_token_ids: Tuple[int, ...] = ()
     think_end_token_id: int = -1
     draft: None = None               # no block draft: rounds commit one token
@@ -121,6 +235,16 @@ class StackSpec:
     @property
     def layer_count(self) -> int:
         return len(self.layers)
+
+    def owner(self, i: int) -> int:
+        """The layer whose tensors layer ``i`` uses."""
+        seen = set()
+        while self.layers[i].weights_of is not None:
+            if i in seen:
+                raise ValueError(f"{self.name}: layer {i} borrows its weights in a circle")
+            seen.add(i)
+            i = self.layers[i].weights_of
+        return i
 
     def runs(self) -> List[LayerRun]:
         out: List[Tuple[int, Optional[int]]] = []
@@ -144,12 +268,24 @@ class StackSpec:
         if not 1 <= n <= len(self.layers):
             raise ValueError(f"layer count {n} outside 1..{len(self.layers)}")
         loop = self.loop if self.loop is not None and self.loop.stop <= n else None
-        return replace(self, name=f"{self.name}-L{n}", layers=self.layers[:n], loop=loop)
+        first: Dict[int, int] = {}                     # borrowers of a layer that is cut share among themselves
+        layers = []
+        for i, layer in enumerate(self.layers[:n]):
+            j = self.owner(i)
+            j = first.setdefault(j, i) if j >= n else j
+            layers.append(replace(layer, weights_of=None if j == i else j))
+        return replace(self, name=f"{self.name}-L{n}", layers=tuple(layers), loop=loop)
 
     def kv_bytes_per_token(self, tp: int = 1, element_bytes: int = 2) -> int:
         self.vocab_shard(tp)
-        return sum(_pad(self.layers[r.layer].mixer.kv_rank, 16) * element_bytes
-                   for r in self.runs() if self.layers[r.layer].mixer.kind == "latent_attention")
+        total = 0
+        for r in self.runs():
+            m = self.layers[r.layer].mixer
+            if m.kind == "latent_attention":
+                total += _pad(m.kv_rank, 16) * element_bytes
+            elif m.kind == "parallel":
+                total += m.left.kv_heads * (_pad(m.left.dim, 8) + _pad(m.left.vdim, 8)) * element_bytes
+        return total
 
     def validate(self) -> "StackSpec":
         """Refuse what the kernels cannot run, by name, before anything is allocated."""
@@ -160,10 +296,20 @@ class StackSpec:
         need(self.hidden <= 25600, "width above 25600")
         for i, layer in enumerate(self.layers):
             m, f = layer.mixer, layer.mlp
-            widest = m.heads * _pad(m.vdim, 8) if m.kind == "latent_attention" else getattr(m, "width", 0)
+            if m.kind == "parallel":
+                widest = max(m.left.heads * _pad(m.left.vdim, 8), m.right.heads * m.right.vdim)
+            else:
+                widest = m.width if m.kind == "rglru" else m.heads * _pad(m.vdim, 8)
             if f is not None:
                 widest = max(widest, _pad(f.ff, 8) * (f.routing.top_k if f.kind == "moe" else 1))
             need(widest <= MAX_STEP_INPUT, f"layer {i}: a product of the step would take in {widest} values, at most {MAX_STEP_INPUT}")
+        need(self.norm in ("rms", "layer"), f"unknown norm {self.norm!r}")
+        for i, layer in enumerate(self.layers):
+            j = layer.weights_of
+            if j is not None:
+                need(0 <= j < len(self.layers), f"layer {i}: no layer {j} to take weights from")
+                own = self.layers[self.owner(i)]
+                need((own.mixer, own.mlp) == (layer.mixer, layer.mlp), f"layer {i}: differs from layer {j}, whose weights it uses")
         for i, layer in enumerate(self.layers):
             m, f = layer.mixer, layer.mlp
             if m.kind == "latent_attention":
@@ -172,6 +318,23 @@ class StackSpec:
                 need(m.kv_rank <= MAX_RANK, f"layer {i}: kv_rank above {MAX_RANK}")
             elif m.kind == "rglru":
                 need(min(m.width, m.blocks, m.taps) >= 1 and m.width % m.blocks == 0, f"layer {i}: width does not split into blocks")
+            elif m.kind in ("channel_delta", "wkv"):
+                need(min(m.heads, m.dim, m.vdim, m.decay_rank) >= 1, f"layer {i}: empty mixer size")
+                need(m.dim <= MAX_STATE_DIM and m.vdim <= MAX_STATE_DIM, f"layer {i}: head width above {MAX_STATE_DIM}")
+                need(m.decay_rank <= MAX_RANK, f"layer {i}: decay rank above {MAX_RANK}")
+                if m.kind == "channel_delta":
+                    need(min(m.kv_heads, m.taps, m.gate_rank) >= 1, f"layer {i}: empty mixer size")
+                    need(m.gate_rank <= MAX_RANK, f"layer {i}: gate rank above {MAX_RANK}")
+                    need(m.heads % m.kv_heads == 0, f"layer {i}: {m.heads} heads over {m.kv_heads} key heads")
+            elif m.kind == "parallel":
+                a, b = m.left, m.right
+                need(min(a.heads, a.kv_heads, a.dim, a.vdim, b.heads, b.dim, b.vdim) >= 1, f"layer {i}: empty mixer size")
+                need(max(a.dim, a.vdim) <= MAX_HEAD_DIM and b.dim <= MAX_STATE_DIM, f"layer {i}: head width above {MAX_HEAD_DIM}")
+                need(b.vdim <= 4096, f"layer {i}: value width above 4096")
+                need(a.heads % a.kv_heads == 0, f"layer {i}: {a.heads} heads over {a.kv_heads} key heads")
+                need(a.window >= 0, f"layer {i}: negative chunk length")
+                need(a.rotary is None or (a.rotary.dims % 2 == 0 and 0 <= a.rotary.dims <= a.dim), f"layer {i}: rotated columns")
+                need(b.cap > 0, f"layer {i}: gate cap")
             else:
                 need(False, f"layer {i}: unknown mixer {m.kind!r}")
             if f is not None and f.kind == "moe":
@@ -182,7 +345,7 @@ class StackSpec:
                 need(1 <= r.limited_group_count <= r.group_count <= MAX_GROUPS and r.expert_count % r.group_count == 0,
                      f"layer {i}: expert groups")
                 need(r.top_k <= r.expert_count // r.group_count * r.limited_group_count, f"layer {i}: fewer eligible experts than top_k")
-            elif f is not None and f.kind != "dense":
+            elif f is not None and f.kind not in ("dense", "relu2"):
                 need(False, f"layer {i}: unknown feed-forward {f.kind!r}")
         if self.loop is not None:
             need(0 <= self.loop.start < self.loop.stop <= len(self.layers) and self.loop.times >= 1, "loop bounds")

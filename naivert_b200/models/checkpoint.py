@@ -116,6 +116,9 @@ class LocalCheckpoint:
             if name not in self.headers[f]:
                 raise CheckpointError(f"index maps {name} to {f}, which does not contain it")
 
+    def shapes(self) -> Dict[str, tuple]:
+        return {n: tuple(self.headers[f][n]["shape"]) for n, f in self.weight_map.items()}
+
     def identity(self) -> CheckpointIdentity:
         meta = {n: (self.headers[f][n]["dtype"], self.headers[f][n]["shape"], f, self.headers[f][n]["data_offsets"])
                 for n, f in self.weight_map.items()}

@@ -7,9 +7,9 @@ from __future__ import annotations
 
 import json
 import os
-from typing import Union
+from typing import Mapping, Optional, Tuple, Union
 
-from . import tumatar
+from . import tumatar, zuzupel
 from .blocks import StackSpec
 from .naive_n0p5 import NAIVE_N0P5, small_w8a8_spec, tiny_spec
 from .spec import ModelSpec
@@ -20,10 +20,12 @@ MODELS = {
     "tumatar-small": tumatar.small_spec(),
     "tumatar-bench": tumatar.bench_spec(),
     "tumatar-bench-dense": tumatar.bench_spec(experts=False),
+    "zuzupel-small": zuzupel.small_spec(),
+    "zuzupel-bench": zuzupel.bench_spec(),
 }
 
 # config.json "architecture" -> design module (spec_from_config, tensor_shapes, gather_weights, ...)
-DESIGNS = {tumatar.ARCHITECTURE: tumatar}
+DESIGNS = {tumatar.ARCHITECTURE: tumatar, zuzupel.ARCHITECTURE: zuzupel}
 
 
 def resolve_model(name: str) -> Union[ModelSpec, StackSpec]:
@@ -40,11 +42,14 @@ def design_of(spec: StackSpec):
     return DESIGNS[spec.architecture]
 
 
-def spec_from_config(cfg: dict, name: str = "") -> Union[ModelSpec, StackSpec]:
-    """The model a ``config.json`` describes."""
+def spec_from_config(cfg: dict, name: str = "", shapes: Optional[Mapping[str, Tuple[int, ...]]] = None) -> Union[ModelSpec, StackSpec]:
+    """The model a ``config.json`` describes; ``shapes`` (tensor name -> shape) for designs that leave sizes to their tensors."""
     arch = cfg.get("architecture")
     if arch in DESIGNS:
-        return DESIGNS[arch].spec_from_config(cfg, name or arch.lower())
+        design = DESIGNS[arch]
+        if getattr(design, "NEEDS_SHAPES", False):
+            return design.spec_from_config(cfg, name or arch.lower(), shapes)
+        return design.spec_from_config(cfg, name or arch.lower())
     if cfg.get("model_type") == "naive_n0p5":
         from .checkpoint import target_config
         for spec in MODELS.values():
@@ -58,4 +63,9 @@ def spec_from_config(cfg: dict, name: str = "") -> Union[ModelSpec, StackSpec]:
 def resolve_checkpoint_model(root: str) -> Union[ModelSpec, StackSpec]:
     """The model of a checkpoint directory, chosen by its ``config.json``."""
     with open(os.path.join(root, "config.json")) as f:
-        return spec_from_config(json.load(f), os.path.basename(os.path.abspath(root)))
+        cfg = json.load(f)
+    shapes = None
+    if getattr(DESIGNS.get(cfg.get("architecture")), "NEEDS_SHAPES", False):
+        from .checkpoint import LocalCheckpoint
+        shapes = LocalCheckpoint(root).shapes()
+    return spec_from_config(cfg, os.path.basename(os.path.abspath(root)), shapes)

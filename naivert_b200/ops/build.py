@@ -33,7 +33,7 @@ CSRC = os.path.join(_ROOT, "csrc")
 LIB_DIR = os.path.join(_ROOT, "_lib")
 LIB_NAME = "libnaivert_b200.so"
 STACK_LIB_NAME = "libnaivert_b200_stack.so"
-STACK_ONLY = ("latent_attn.cu", "stack_gemm.cu", "stack_rows.cu", "stack_step.cu")
+STACK_ONLY = ("latent_attn.cu", "stack_attn.cu", "stack_gemm.cu", "stack_rows.cu", "stack_state.cu", "stack_step.cu")
 GROUPS = ("main", "stack")
 _SHARED_WITH_STACK = ("ep.cu", "tmap.cu")           # compiled into both
 # The checking flavour: the same sources with -DNRT_BOUNDS_CHECK (every data-derived index is tested before use and the

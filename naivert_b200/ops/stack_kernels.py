@@ -16,14 +16,23 @@ from .build import load_library
 
 VP = C.c_void_p
 _G = generate_from("stack.cuh", ["StackGemmArgs", "StackRowArgs", "LatentPrepArgs", "LatentAttnArgs", "LatentDecodeArgs",
-                                 "RecurrenceArgs", "MoeGatherArgs", "StepArgs"])
+                                 "RecurrenceArgs", "MoeGatherArgs", "StepArgs", "GroupPrepArgs", "TransposeArgs", "GroupDecodeArgs",
+                                 "StateChunkArgs", "ShortConvArgs", "TokenMixArgs", "HeadGateArgs", "StateStepArgs"])
 StackGemmArgs, StackRowArgs, LatentPrepArgs = _G["StackGemmArgs"], _G["StackRowArgs"], _G["LatentPrepArgs"]
 LatentAttnArgs, LatentDecodeArgs, RecurrenceArgs = _G["LatentAttnArgs"], _G["LatentDecodeArgs"], _G["RecurrenceArgs"]
 MoeGatherArgs, StepArgs = _G["MoeGatherArgs"], _G["StepArgs"]
+GroupPrepArgs, TransposeArgs, GroupDecodeArgs = _G["GroupPrepArgs"], _G["TransposeArgs"], _G["GroupDecodeArgs"]
+StateChunkArgs, ShortConvArgs, TokenMixArgs = _G["StateChunkArgs"], _G["ShortConvArgs"], _G["TokenMixArgs"]
+HeadGateArgs, StateStepArgs = _G["HeadGateArgs"], _G["StateStepArgs"]
 
 EPI_STORE, EPI_BIAS, EPI_TRANSPOSE, EPI_CLAMPED_GLU, EPI_SILU_GLU = 0, 1, 2, 3, 4
-PRO_RESIDUAL, PRO_NORM, PRO_LOAD, PRO_MERGE, PRO_EXPERTS = 0, 1, 2, 3, 4
-TEPI_STORE, TEPI_CONV, TEPI_GATE, TEPI_GLU, TEPI_RECUR = 0, 1, 2, 3, 4
+EPI_RELU2, EPI_TANH, EPI_DECAY_SOFT, EPI_DECAY_EXP = 5, 6, 7, 8
+PRO_RESIDUAL, PRO_NORM, PRO_LOAD, PRO_MERGE, PRO_EXPERTS, PRO_MIX = 0, 1, 2, 3, 4, 5
+TEPI_STORE, TEPI_CONV, TEPI_GATE, TEPI_GLU, TEPI_RECUR, TEPI_CONV_SILU, TEPI_RELU2 = 0, 1, 2, 3, 4, 5, 6
+NORM = {"rms": 0, "layer": 1}
+STATE_DELTA, STATE_BONUS, STATE_NORMALIZED = 0, 1, 2
+GATE_SIGMOID, GATE_SILU = 0, 1
+MAX_SPLITS = 8                                        # context splits of the grouped one-token attention (a cluster)
 
 # library entry points of the family and the argument struct each reads
 ENTRIES = {"nrt_stack_gemm": ("StackGemmArgs", "nrt_stack_gemm_args_size"), "nrt_stack_gemm_f32": ("StackGemmArgs", "nrt_stack_gemm_args_size"),
@@ -32,7 +41,12 @@ ENTRIES = {"nrt_stack_gemm": ("StackGemmArgs", "nrt_stack_gemm_args_size"), "nrt
            "nrt_latent_attn_tc": ("LatentAttnArgs", "nrt_latent_attn_args_size"),
            "nrt_latent_decode": ("LatentDecodeArgs", "nrt_latent_decode_args_size"),
            "nrt_stack_conv": ("RecurrenceArgs", "nrt_recurrence_args_size"), "nrt_stack_scan": ("RecurrenceArgs", "nrt_recurrence_args_size"),
-           "nrt_moe_gather": ("MoeGatherArgs", "nrt_moe_gather_args_size"), "nrt_stack_step": ("StepArgs", "nrt_step_args_size")}
+           "nrt_moe_gather": ("MoeGatherArgs", "nrt_moe_gather_args_size"), "nrt_stack_step": ("StepArgs", "nrt_step_args_size"),
+           "nrt_group_prep": ("GroupPrepArgs", "nrt_group_prep_args_size"), "nrt_transpose": ("TransposeArgs", "nrt_transpose_args_size"),
+           "nrt_group_decode": ("GroupDecodeArgs", "nrt_group_decode_args_size"),
+           "nrt_state_chunk": ("StateChunkArgs", "nrt_state_chunk_args_size"), "nrt_state_step": ("StateStepArgs", "nrt_state_step_args_size"),
+           "nrt_short_conv": ("ShortConvArgs", "nrt_short_conv_args_size"), "nrt_token_mix": ("TokenMixArgs", "nrt_token_mix_args_size"),
+           "nrt_head_gate": ("HeadGateArgs", "nrt_head_gate_args_size")}
 
 _lib = None
 
@@ -115,6 +129,38 @@ def scan_tokens() -> int:
     return lib().nrt_stack_scan_tokens()
 
 
+def group_prep(args: GroupPrepArgs) -> None:
+    K.check(lib().nrt_group_prep(C.byref(args), _stream()), "grouped attention prep")
+
+
+def transpose(args: TransposeArgs) -> None:
+    K.check(lib().nrt_transpose(C.byref(args), _stream()), "transpose")
+
+
+def group_decode(args: GroupDecodeArgs, pdl: bool) -> None:
+    K.check(lib().nrt_group_decode(C.byref(args), _stream(), int(pdl)), "grouped attention (step)")
+
+
+def short_conv(args: ShortConvArgs) -> None:
+    K.check(lib().nrt_short_conv(C.byref(args), _stream()), "short convolution with SiLU")
+
+
+def token_mix(args: TokenMixArgs) -> None:
+    K.check(lib().nrt_token_mix(C.byref(args), _stream()), "token mixes")
+
+
+def state_chunk(kind: int, args: StateChunkArgs) -> None:
+    K.check(lib().nrt_state_chunk(kind, C.byref(args), _stream()), "matrix-state recurrence (chunk)")
+
+
+def state_step(args: StateStepArgs, pdl: bool) -> None:
+    K.check(lib().nrt_state_step(C.byref(args), _stream(), int(pdl)), "matrix-state recurrence (step)")
+
+
+def head_gate(args: HeadGateArgs) -> None:
+    K.check(lib().nrt_head_gate(C.byref(args), _stream()), "read-out norm and gate")
+
+
 def route(args: K.RouterArgs, groups: int, keep: int) -> None:
     K.check(lib().nrt_stack_route(C.byref(args), groups, keep, _stream()), "expert choice")
 
@@ -130,4 +176,3 @@ def moe_gather(args: MoeGatherArgs) -> None:
 def step(pro: int, epi: int, args: StepArgs, router: Optional[K.RouterArgs], groups: int, keep: int, pdl: bool) -> None:
     K.check(lib().nrt_stack_step(pro, epi, C.byref(args), C.byref(router) if router is not None else None, groups, keep, _stream(),
                                  int(pdl)), "stack step")
-

@@ -1,12 +1,9 @@
 """Chunk path of layer-stack models: R prompt rows go through every layer in one pass over the step's own caches.
 
     rows (stream update + norms)
-    latent attention   [dq | dkv | g] product -> norms, latent rows into the cache -> queries; keys and values of the
-                       cached positions expanded block by block -> causal attention, gated -> output product
-    recurrence         [y | x] product with biases and GELU -> short convolution -> block-diagonal gate products ->
-                       chunked scan from the carried state -> output product
-    feed-forward       two-product GLU -> down; routed experts: scores -> choice -> rows sorted by expert -> grouped
-                       products -> weighted sum inside the next row kernel
+    token mixer        one class per mechanism in ``prefill/stack_mixers.py``
+    feed-forward       two-product GLU -> down, or squared ReLU -> down; routed experts: scores -> choice -> rows sorted by
+                       expert -> grouped products -> weighted sum inside the next row kernel
 
 A chunk may start and end anywhere and has any length up to ``chunk`` rows; the caches and states it leaves are those
 the step continues from.
@@ -20,7 +17,9 @@ import torch
 
 from ..ops import kernels as K
 from ..ops import stack_kernels as S
-from ..runtime.stack import Packed, StackRuntime, pad
+from ..runtime.packing import Packed, pad
+from ..runtime.stack import StackRuntime
+from .stack_mixers import MIXERS
 
 SMS = 148
 
@@ -35,8 +34,6 @@ class StackPrefill:
         s, dev, C = self.spec, self.dev, chunk
         f32, i32 = torch.float32, torch.int32
         L = runtime.layers
-        attn = [(d["spec"].mixer, d) for d in L if d["kind"] == "latent_attention"]
-        rec = [(d["spec"].mixer, d) for d in L if d["kind"] == "rglru"]
         ffs = [d["spec"].mlp for d in L if d["spec"].mlp is not None]
         moe = [f for f in ffs if f.kind == "moe"]
         self.h_ld = pad(s.hidden, 8)
@@ -52,19 +49,14 @@ class StackPrefill:
         self.x = torch.zeros(C, s.hidden, dtype=f32, device=dev)
         self.h = torch.zeros(C, self.h_ld, dtype=self.act, device=dev)
         self.y = torch.zeros(C, s.hidden, dtype=f32, device=dev)
-        # one arena per role, shared by the layers (sizes differ from layer to layer)
-        self.proj = z(C * most(d["in"].n for _, d in attn))
-        self.cq = z(C * most(pad(m.q_rank, 8) for m, _ in attn), self.act)
-        self.q = z(C * most(m.heads * d["dp"] for m, d in attn), self.act)
-        self.kx = z(self.kv_block * most(m.heads * d["dp"] for m, d in attn), self.act)
-        self.vx = z(self.kv_block * most(m.heads * d["vp"] for m, d in attn), self.act)
-        self.o = z(C * max(most(m.heads * d["vp"] for m, d in attn), most(pad(m.width, 8) for m, _ in rec)), self.act)
-        self.carry = z(C * most(m.heads * (d["vp"] + 2) for m, d in attn)) if runtime.capacity > self.kv_block else None
-        self.xy = z(C * most(2 * m.width for m, _ in rec), self.act)
-        self.u = z(C * most(m.blocks * pad(m.block, 8) for m, _ in rec), self.act)
-        self.gates = z(C * most(2 * m.width for m, _ in rec))
-        self.agg = z(-(-C // S.scan_tokens()) * 2 * most(m.width for m, _ in rec))
-        self.ff = z(C * most(pad(f.ff, 8) for f in ffs if f.kind == "dense"), self.act)
+        self.y2 = torch.zeros(C, s.hidden, dtype=f32, device=dev) if any(d["kind"] == "parallel" for d in L) else None
+        # buffers of the mixers, one per role, shared by the layers (sizes differ from layer to layer)
+        sizes: Dict[tuple, int] = {}
+        for d in L:
+            for name, (n, t) in MIXERS[d["kind"]].scratch(self, d["spec"].mixer, d).items():
+                sizes[name, t] = max(n, sizes.get((name, t), 0))
+        self.buf = {name: z(n, t) for (name, t), n in sizes.items()}
+        self.ff = z(C * most(pad(f.ff, 8) for f in ffs if f.kind != "moe"), self.act)
         if moe:
             E, T = most(f.routing.expert_count for f in moe), most(f.routing.top_k for f in moe)
             self.scores, self.ids, self.probs = z(C * E), z(C * T, i32), z(C * T)
@@ -84,7 +76,7 @@ class StackPrefill:
         self._timed: Dict[str, list] = {}
 
     @contextmanager
-    def _stage(self, name: str):
+    def stage(self, name: str):
         if not self.profile:
             yield
             return
@@ -117,7 +109,7 @@ class StackPrefill:
 
     # ------------------------------------------------------------------ products
     def _wmap(self, p: Packed) -> K.TensorMap:
-        key = ("w", p.w.data_ptr())
+        key = ("w", p.w.data_ptr(), p.z, p.n)
         if key not in self.maps:
             self.maps[key] = S.weight_map(p.w, p.k)
         return self.maps[key]
@@ -128,14 +120,15 @@ class StackPrefill:
             self.maps[key] = S.token_map(t, k, zcount, zstride, rows, ld, box, offset)
         return self.maps[key]
 
-    def _gemm(self, epi: int, w: Packed, x: torch.Tensor, x_ld: int, rows: int, out: torch.Tensor, out_ld: int, *, w2: Optional[Packed] = None,
+    def gemm(self, epi: int, w: Packed, x: torch.Tensor, x_ld: int, rows: int, out: torch.Tensor, out_ld: int, *, w2: Optional[Packed] = None,
               z: int = 1, x_z: int = 0, out_z: int = 0, x_off: int = 0, x_rows: Optional[int] = None, items: Optional[tuple] = None,
-              bias: Optional[torch.Tensor] = None, act_cols: int = 0, scale: float = 1.0, limit: float = 0.0, alpha: float = 0.0) -> None:
+              bias: Optional[torch.Tensor] = None, rate: Optional[torch.Tensor] = None, act_cols: int = 0, scale: float = 1.0, limit: float = 0.0, alpha: float = 0.0) -> None:
         """out[row, z, :] = epilogue(W_z x[row, z, :]) for every token row; ``items`` = (segment rows, most segments)."""
         a = S.StackGemmArgs()
         a.n, a.k, a.rows, a.zcount = w.n, w.k, rows, z
         a.out, a.out_ld, a.out_zstride, a.out_f32 = out.data_ptr(), out_ld, out_z, int(out.dtype == torch.float32)
         a.bias = None if bias is None else bias.data_ptr()
+        a.rate = None if rate is None else rate.data_ptr()
         a.act_cols, a.scale, a.limit, a.alpha, a.status = act_cols, scale, limit, alpha, self.t.fab.status.data_ptr()
         if items is not None:
             a.n_items, a.item_z, a.item_row = self.n_items.data_ptr(), self.item_z.data_ptr(), self.item_row.data_ptr()
@@ -151,123 +144,58 @@ class StackPrefill:
             ntok = items[0]
         else:
             tiles = -(-w.n // 128) * z
-            sizes = (128, 64) if dual else (256, 128, 64) if epi == S.EPI_STORE else (256, 64)
+            sizes = (128, 64) if dual else (256, 128, 64) if epi in (S.EPI_STORE, S.EPI_RELU2) else (256, 64)
             ntok = next((t for t in sizes if tiles * -(-rows // t) >= SMS - 20), 64)
         live = x_rows if x_rows is not None else x.numel() // x_ld
         xm = self._xmap(x, w.k, z, x_z, live, x_ld, ntok, x_off)
         wbytes = w.nbytes * (2 if dual else 1)
         S.gemm(epi, ntok, self._wmap(w), self._wmap(w2) if dual else None, xm, a, items is None and wbytes > (96 << 20))
 
-    def _attn_maps(self, heads: int, dp: int, vp: int) -> Tuple[K.TensorMap, ...]:
-        key = ("attn", heads, dp, vp)
-        if key not in self.maps:
-            self.maps[key] = (S.token_map(self.q, dp, heads, dp, self.C, heads * dp, 128), S.token_map(self.kx, dp, heads, dp, self.kv_block, heads * dp, 64),
-                              S.value_map(self.vx, self.kv_block, heads * vp, pad(vp, 16)))
-        return self.maps[key]
-
     # ------------------------------------------------------------------ one chunk
-    def _rows(self, R: int, *, embed: bool = False, y: Optional[torch.Tensor] = None, post=None, moe=None, add=None, pre=None) -> None:
+    def _rows(self, R: int, *, embed: bool = False, y: Optional[torch.Tensor] = None, post=None, y2: Optional[torch.Tensor] = None, join=None,
+              moe=None, add=None, pre=None, copy: bool = False) -> None:
+        """Stream update; then the input rows ``h`` of the next sublayer: normed by ``pre``, or the stream itself (``copy``)."""
         s, a = self.spec, S.StackRowArgs()
         if embed:
             a.tokens, a.table, a.vocab, a.embed_scale = self.tokens.data_ptr(), self.t.embed.data_ptr(), s.vocab, s.embed_scale
         if y is not None:
             a.y, a.y_ld, a.post_w = y.data_ptr(), s.hidden, post.data_ptr()
+            if join is not None:
+                a.y2, a.join_w, a.join_w2 = y2.data_ptr(), join[0].data_ptr(), join[1].data_ptr()
             if moe is not None:
                 a.slot_of, a.probs, a.top_k = self.slot_of.data_ptr(), self.probs.data_ptr(), moe.top_k
         a.add = None if add is None else add.data_ptr()
         a.x, a.width, a.rows, a.eps = self.x.data_ptr(), s.hidden, R, s.norm_eps
         a.pre_w = None if pre is None else pre.data_ptr()
+        a.norm, a.copy_h = S.NORM[s.norm], int(copy)
         a.h, a.h_f32, a.h_ld = self.h.data_ptr(), int(self.f32), self.h_ld
-        with self._stage("rows"):
+        with self.stage("rows"):
             S.rows(a)
-
-    def _attention(self, r: dict, R: int, pos0: int) -> None:
-        d, t = r["layer"], self.t
-        m, dp, vp = d["spec"].mixer, d["dp"], d["vp"]
-        n_in, qp = d["in"].n, pad(m.q_rank, 8)
-        with self._stage("attn_in"):
-            self._gemm(S.EPI_STORE, d["in"], self.h, self.h_ld, R, self.proj, n_in)
-        p = S.LatentPrepArgs()
-        p.proj, p.ld, p.rows, p.q_rank, p.kv_rank = self.proj.data_ptr(), n_in, R, m.q_rank, m.kv_rank
-        p.q_w, p.kv_w, p.eps = d["dq_norm"].data_ptr(), d["dkv_norm"].data_ptr(), self.spec.norm_eps
-        cache = r["cache"]
-        p.cq, p.cq_ld, p.cache, p.cache_ld = self.cq.data_ptr(), qp, cache.data_ptr(), cache.shape[1]
-        p.f32, p.pos0, p.capacity = int(self.f32), self.pos.data_ptr(), t.capacity
-        with self._stage("latent_prep"):
-            S.latent_prep(p)
-        hq, hv = m.heads * dp, m.heads * vp
-        with self._stage("queries"):
-            self._gemm(S.EPI_STORE, d["uq"], self.cq, qp, R, self.q, hq)
-        a = S.LatentAttnArgs()
-        a.q, a.k, a.v, a.out, a.f32 = self.q.data_ptr(), self.kx.data_ptr(), self.vx.data_ptr(), self.o.data_ptr(), int(self.f32)
-        a.gate, a.gate_ld = self.proj.data_ptr() + 4 * (m.q_rank + m.kv_rank), n_in
-        a.rows, a.heads, a.dim, a.vdim, a.scale, a.pos0 = R, m.heads, dp, vp, m.scale, self.pos.data_ptr()
-        a.state = None if self.carry is None else self.carry.data_ptr()
-        a.status = t.fab.status.data_ptr()
-        total = pos0 + R
-        for kv0 in range(0, total, self.kv_block):
-            n = min(self.kv_block, total - kv0)
-            off = kv0 * cache.shape[1]
-            kw = dict(x_off=off, x_rows=t.capacity - kv0)
-            with self._stage("expand_k"):
-                self._gemm(S.EPI_STORE, d["uk"], cache, cache.shape[1], n, self.kx, hq, **kw)
-            a.kv0, a.kv_rows, a.first, a.last = kv0, n, int(kv0 == 0), int(kv0 + n == total)
-            if self.tensor_cores and max(dp, vp) <= 256:
-                a.v_ld = self.kv_block                 # values feature-major: the K-major operand of P V
-                with self._stage("expand_v"):
-                    self._gemm(S.EPI_TRANSPOSE, d["uv"], cache, cache.shape[1], n, self.vx, self.kv_block, **kw)
-                with self._stage("attention"):
-                    S.latent_attn_tc(*self._attn_maps(m.heads, dp, vp), a)
-            else:
-                a.v_ld = hv
-                self._gemm(S.EPI_STORE, d["uv"], cache, cache.shape[1], n, self.vx, hv, **kw)
-                with self._stage("attention_plain"):
-                    S.latent_attn_rows(a)
-        with self._stage("attn_out"):
-            self._gemm(S.EPI_STORE, d["o"], self.o, hv, R, self.y, self.spec.hidden)
-
-    def _recurrence(self, r: dict, R: int) -> None:
-        d = r["layer"]
-        m = d["spec"].mixer
-        bp, wp = pad(m.block, 8), pad(m.width, 8)
-        with self._stage("rec_in"):
-            self._gemm(S.EPI_BIAS, d["in"], self.h, self.h_ld, R, self.xy, 2 * m.width, bias=d["in_b"], act_cols=m.width)
-        a = S.RecurrenceArgs()
-        a.xy, a.xy_ld, a.conv, a.conv_b, a.taps = self.xy.data_ptr(), 2 * m.width, d["conv"].data_ptr(), d["conv_b"].data_ptr(), m.taps
-        a.history, a.hist_rows, a.u = r["history"].data_ptr(), m.hist_rows, self.u.data_ptr()
-        a.gates, a.softplus_lam, a.decay = self.gates.data_ptr(), d["sp"].data_ptr(), m.decay
-        a.state, a.tags, a.agg = r["state"].data_ptr(), r["tags"].data_ptr(), self.agg.data_ptr()
-        a.out, a.out_ld, a.f32, a.rows = self.o.data_ptr(), wp, int(self.f32), R
-        a.width, a.blocks, a.block, a.block_pad = m.width, m.blocks, m.block, bp
-        a.pos0, a.status = self.pos.data_ptr(), self.t.fab.status.data_ptr()
-        with self._stage("conv"):
-            S.conv(a)
-        with self._stage("rec_gates"):
-            self._gemm(S.EPI_BIAS, d["gates"], self.u, m.blocks * bp, R, self.gates, 2 * m.width, z=m.blocks, x_z=bp, out_z=2 * m.block,
-                       bias=d["gates_b"])
-        with self._stage("scan"):
-            S.scan(a)
-        with self._stage("rec_out"):
-            self._gemm(S.EPI_STORE, d["o"], self.o, wp, R, self.y, self.spec.hidden)
 
     def _feed_forward(self, d: dict, R: int) -> torch.Tensor:
         """Returns the buffer that holds the result rows (sorted by expert for routed layers)."""
         f, W = d["spec"].mlp, self.spec.hidden
         fp = pad(f.ff, 8)
+        if f.kind == "relu2":
+            with self.stage("ff_up"):
+                self.gemm(S.EPI_RELU2, d["up"], self.h, self.h_ld, R, self.ff, fp)
+            with self.stage("ff_down"):
+                self.gemm(S.EPI_STORE, d["down"], self.ff, fp, R, self.y, W)
+            return self.y
         if f.kind == "dense":
-            with self._stage("dense_gate_up"):
-                self._gemm(S.EPI_CLAMPED_GLU, d["gate"], self.h, self.h_ld, R, self.ff, fp, w2=d["up"], limit=f.limit, alpha=f.alpha)
-            with self._stage("dense_down"):
-                self._gemm(S.EPI_STORE, d["down"], self.ff, fp, R, self.y, W)
+            with self.stage("dense_gate_up"):
+                self.gemm(S.EPI_CLAMPED_GLU, d["gate"], self.h, self.h_ld, R, self.ff, fp, w2=d["up"], limit=f.limit, alpha=f.alpha)
+            with self.stage("dense_down"):
+                self.gemm(S.EPI_STORE, d["down"], self.ff, fp, R, self.y, W)
             return self.y
         rt = f.routing
-        with self._stage("router"):
-            self._gemm(S.EPI_STORE, d["router"], self.h, self.h_ld, R, self.scores, rt.expert_count)
+        with self.stage("router"):
+            self.gemm(S.EPI_STORE, d["router"], self.h, self.h_ld, R, self.scores, rt.expert_count)
         q = K.RouterArgs()
         q.bias, q.hidden, q.experts, q.rows, q.top_k = d["correction"].data_ptr(), W, rt.expert_count, R, rt.top_k
         q.sigmoid, q.normalize, q.route_scale = 1, int(rt.normalize_top_k), rt.route_scale
         q.scores, q.topk_ids, q.topk_p = self.scores.data_ptr(), self.ids.data_ptr(), self.probs.data_ptr()
-        with self._stage("choice"):
+        with self.stage("choice"):
             S.route(q, rt.group_count, rt.limited_group_count)
         ir = self._item_rows(R, rt, self.f32)
         items = self._items(R, rt, ir)
@@ -277,19 +205,19 @@ class StackPrefill:
         e.slot_of, e.n_items, e.item_expert, e.item_row = (self.slot_of.data_ptr(), self.n_items.data_ptr(), self.item_z.data_ptr(),
                                                            self.item_row.data_ptr())
         e.seg_rows, e.max_items, e.item_rows, e.x_args = self.seg_rows.data_ptr(), items, ir, self.t.fab.xchg_args()
-        with self._stage("expert_count"):
+        with self.stage("expert_count"):
             S.moe_count(e)
         g = S.MoeGatherArgs()
         eb = self.h.element_size()
         g.h, g.h_ld, g.sorted, g.slot_of = self.h.data_ptr(), self.h_ld * eb, self.sorted.data_ptr(), self.slot_of.data_ptr()
         g.rows, g.top_k, g.row_bytes, g.cap = R, rt.top_k, self.h_ld * eb, self.cap
-        with self._stage("expert_gather"):
+        with self.stage("expert_gather"):
             S.moe_gather(g)
         seg = dict(items=(ir, items))
-        with self._stage("expert_gate_up"):
-            self._gemm(S.EPI_SILU_GLU, d["gate"], self.sorted, self.h_ld, ir, self.ea, fp, w2=d["up"], x_rows=self.cap, **seg)
-        with self._stage("expert_down"):
-            self._gemm(S.EPI_STORE, d["down"], self.ea, fp, ir, self.ey, W, x_rows=self.cap, **seg)
+        with self.stage("expert_gate_up"):
+            self.gemm(S.EPI_SILU_GLU, d["gate"], self.sorted, self.h_ld, ir, self.ea, fp, w2=d["up"], x_rows=self.cap, **seg)
+        with self.stage("expert_down"):
+            self.gemm(S.EPI_STORE, d["down"], self.ea, fp, ir, self.ey, W, x_rows=self.cap, **seg)
         return self.ey
 
     def _chunk(self, pos0: int, R: int, want: Sequence[int] = (), trace: Optional[list] = None) -> Optional[torch.Tensor]:
@@ -301,15 +229,14 @@ class StackPrefill:
         for r in t.runs:
             d, run = r["layer"], r["run"]
             add = None if run.pass_start is None else t.loop_step[run.pass_start]
-            self._rows(R, add=add, pre=d["norm1"], **wait)
-            if d["kind"] == "latent_attention":
-                self._attention(r, R, pos0)
-            else:
-                self._recurrence(r, R)
+            self._rows(R, add=add, pre=d["norm1"], copy=d["norm1"] is None and d["kind"] != "wkv", **wait)
+            MIXERS[d["kind"]].run(self, r, R, pos0)
             wait = dict(y=self.y, post=d["norm1b"])
+            if d["kind"] == "parallel":
+                wait.update(y2=self.y2, join=(d["out"], d["out2"]))
             f = d["spec"].mlp
             if f is not None:
-                self._rows(R, pre=d["norm2"], **wait)
+                self._rows(R, pre=d["norm2"], copy=d["norm2"] is None, **wait)
                 wait = dict(y=self._feed_forward(d, R), post=d["norm2b"], moe=f.routing if f.kind == "moe" else None)
             if trace is not None:
                 self._rows(R, **wait)
@@ -323,7 +250,7 @@ class StackPrefill:
         for i in range(0, len(idx), self.head_rows):
             n = min(self.head_rows, len(idx) - i)
             self.hw[:n].copy_(self.h.index_select(0, idx[i:i + n]))
-            self._gemm(S.EPI_STORE, t.head, self.hw, self.h_ld, n, out[i:i + n], s.vocab, scale=s.logit_scale)
+            self.gemm(S.EPI_STORE, t.head, self.hw, self.h_ld, n, out[i:i + n], s.vocab, scale=s.logit_scale)
         return out
 
     # ------------------------------------------------------------------ public API (that of ``NativePrefill``)

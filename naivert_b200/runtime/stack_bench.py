@@ -1,10 +1,11 @@
 """Throughput of layer-stack models at the sizes of a real model's layers (random weights on the device).
 
-    python bench.py --workload stack [--model tumatar-bench|tumatar-bench-dense] [--prompt 8192] [--steps 64] [--kernels]
+    python bench.py --workload stack [--model tumatar-bench|tumatar-bench-dense|zuzupel-bench] [--prompt 8192] [--steps 64] [--kernels]
 
 Prefill: one prompt through the chunk path, CUDA events around the run.  Decode: rounds of the captured graph behind that
 prompt (step + sampler + tail), CUDA events around K replays.  ``--kernels`` adds tables with one row per kernel kind: time,
-the bytes it must move or the FLOPs it must do, and the fraction of the copy bandwidth / dense bf16 rate that is.  Weights of one
+the bytes it must move or the FLOPs it must do, and the fraction of the copy bandwidth / dense bf16 rate (recurrences on the
+CUDA cores: nominal fp32 rate) that is.  Weights of one
 token or chunk exceed the 126 MB L2, so no flush is needed between iterations.
 """
 from __future__ import annotations
@@ -17,8 +18,11 @@ import torch
 
 from ..models.registry import resolve_model
 from ..models.spec import SamplingParams
+from ..prefill.stack_mixers import MIXERS as CHUNK_MIXERS
+from .stack_mixers import MIXERS
 from .engine import Engine
 
+FP32_TFLOPS = 148 * 128 * 2 * 1.965e-3          # CUDA cores, nominal: SMs x lanes x FMA x boost clock
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
 
 
@@ -31,75 +35,69 @@ def peaks() -> dict:
 
 
 # --------------------------------------------------------------------------- work per kernel kind
-def chunk_work(eng, pos0: int, R: int) -> Dict[str, Tuple[float, float]]:
-    """stage -> (FLOPs, bytes) over all runs of one chunk at ``pos0``; bytes are the operands once."""
-    spec, pf = eng.spec, eng.prefill
+class Work:
+    """(tensor-core FLOPs, bytes, CUDA-core fp32 FLOPs) by stage; bytes are the operands once."""
+
+    def __init__(self, hidden: int, es: int):
+        self.W, self.es, self.stages = hidden, es, {}
+
+    def add(self, name: str, flops: float, nbytes: float, flops32: float = 0.0) -> None:
+        a = self.stages.setdefault(name, [0.0, 0.0, 0.0])
+        for i, v in enumerate((flops, nbytes, flops32)):
+            a[i] += v
+
+    def add32(self, name: str, flops32: float, nbytes: float) -> None:
+        self.add(name, 0.0, nbytes, flops32)
+
+    def gemm(self, name: str, n: int, k: int, rows: int, out_bytes: int, z: int = 1, mats: int = 1) -> None:
+        self.add(name, 2.0 * n * k * rows * z * mats, z * (mats * n * k * 2 + rows * k * self.es + rows * n * out_bytes))
+
+
+def chunk_work(eng, pos0: int, R: int) -> Dict[str, List[float]]:
+    """Work per stage over all runs of one chunk at ``pos0``."""
+    spec = eng.spec
     W, es = spec.hidden, 4 if eng.target.f32 else 2
-    out: Dict[str, List[float]] = {}
-
-    def add(name: str, flops: float, nbytes: float) -> None:
-        a = out.setdefault(name, [0.0, 0.0])
-        a[0] += flops
-        a[1] += nbytes
-
-    def gemm(name: str, n: int, k: int, rows: int, out_bytes: int, z: int = 1, mats: int = 1) -> None:
-        add(name, 2.0 * n * k * rows * z * mats, z * (mats * n * k * 2 + rows * k * es + rows * n * out_bytes))
-
-    ctx = pos0 + R
+    w = Work(W, es)
     for r in eng.target.runs:
         d = r["layer"]
         m, f = d["spec"].mixer, d["spec"].mlp
-        add("rows", 0, R * W * (4 + 4 + 4 + es))
-        if m.kind == "latent_attention":
-            hq, hv = m.heads * d["dp"], m.heads * d["vp"]
-            gemm("attn_in", d["in"].n, W, R, 4)
-            add("latent_prep", 0, R * (m.q_rank + m.kv_rank) * (4 + es))
-            gemm("queries", hq, m.q_rank, R, es)
-            gemm("expand_k", hq, m.kv_rank, ctx, es)
-            gemm("expand_v", hv, m.kv_rank, ctx, es)
-            pairs = R * pos0 + R * (R + 1) / 2
-            add("attention", 2.0 * pairs * (hq + hv), R * (hq + 2 * hv) * es + ctx * (hq + hv) * es)
-            gemm("attn_out", W, hv, R, 4)
-        else:
-            gemm("rec_in", 2 * m.width, W, R, es)
-            add("conv", 0, R * m.width * 2 * es)
-            gemm("rec_gates", 2 * m.block, m.block, R, 4, z=m.blocks)
-            add("scan", 0, R * m.width * (2 * 8 + 2 * es + es + es))
-            gemm("rec_out", W, m.width, R, 4)
+        w.add("rows", 0, R * W * (4 + 4 + 4 + es))
+        CHUNK_MIXERS[d["kind"]].work(w, m, d, pos0, R)
         if f is None:
             continue
-        add("rows", 0, R * W * (4 + 4 + 4 + es))
-        if f.kind == "dense":
-            gemm("dense_gate_up", f.ff, W, R, es, mats=2)
-            gemm("dense_down", W, f.ff, R, 4)
+        w.add("rows", 0, R * W * (4 + 4 + 4 + es))
+        if f.kind == "relu2":
+            w.gemm("ff_up", f.ff, W, R, es)
+            w.gemm("ff_down", W, f.ff, R, 4)
+        elif f.kind == "dense":
+            w.gemm("dense_gate_up", f.ff, W, R, es, mats=2)
+            w.gemm("dense_down", W, f.ff, R, 4)
         else:
             rt = f.routing
             P = R * rt.top_k
             used = min(rt.expert_count, P)
-            gemm("router", rt.expert_count, W, R, 4)
-            add("choice", 0, R * rt.expert_count * 4)
-            add("expert_count", 0, P * 8)
-            add("expert_gather", 0, 2 * P * W * es)
-            add("expert_gate_up", 4.0 * P * W * f.ff, used * 2 * W * f.ff * 2 + P * (W + f.ff) * es)
-            add("expert_down", 2.0 * P * W * f.ff, used * W * f.ff * 2 + P * (f.ff * es + W * 4))
-    return {k: (v[0], v[1]) for k, v in out.items()}
+            w.gemm("router", rt.expert_count, W, R, 4)
+            w.add("choice", 0, R * rt.expert_count * 4)
+            w.add("expert_count", 0, P * 8)
+            w.add("expert_gather", 0, 2 * P * W * es)
+            w.add("expert_gate_up", 4.0 * P * W * f.ff, used * 2 * W * f.ff * 2 + P * (W + f.ff) * es)
+            w.add("expert_down", 2.0 * P * W * f.ff, used * W * f.ff * 2 + P * (f.ff * es + W * 4))
+    return w.stages
 
 
 def step_work(eng, pos: int) -> List[Tuple[str, float]]:
-    """(kind, bytes that must be read) of every launch of the step, in launch order."""
-    out = []
+    """(kind, bytes that must move) of every launch of the step, in launch order."""
+    out: List[Tuple[str, float]] = []
     t = eng.target
     for r in t.runs:
         d = r["layer"]
-        m, f = d["spec"].mixer, d["spec"].mlp
-        if m.kind == "latent_attention":
-            out += [("attn_in", d["in"].nbytes), ("queries", d["uq"].nbytes), ("latent_query", d["uk_t"].nbytes),
-                    ("attention", (pos + 1) * m.kv_rank * (4 if t.f32 else 2)), ("values", d["uv"].nbytes), ("attn_out", d["o"].nbytes)]
-        else:
-            out += [("rec_in", d["in"].nbytes), ("rec_gates", d["gates"].nbytes), ("rec_out", d["o"].nbytes)]
+        f = d["spec"].mlp
+        out += MIXERS[d["kind"]].step_work(t, d["spec"].mixer, d, pos)
         if f is None:
             continue
-        if f.kind == "dense":
+        if f.kind == "relu2":
+            out += [("ff_up", d["up"].nbytes), ("ff_down", d["down"].nbytes)]
+        elif f.kind == "dense":
             out += [("dense_gate_up", 2 * d["gate"].nbytes), ("dense_down", d["down"].nbytes)]
         else:
             per = d["gate"].n * d["gate"].ld * 2
@@ -122,9 +120,9 @@ def chunk_table(eng, prompt: torch.Tensor, pos0: int, R: int) -> List[dict]:
     rows = []
     for name, (total, calls) in sorted(ms.items(), key=lambda kv: -kv[1][0]):
         t = total / reps * 1e-3
-        fl, by = work.get(name, (0.0, 0.0))
-        bound = max(fl / (pk["bf16_tflops"] * 1e12), by / (pk["hbm_gbs"] * 1e9))
-        rows.append({"kernel": name, "calls": calls // reps, "ms": round(t * 1e3, 3), "tflops": round(fl / t * 1e-12, 1),
+        fl, by, f32 = work.get(name, (0.0, 0.0, 0.0))
+        bound = max(fl / (pk["bf16_tflops"] * 1e12), by / (pk["hbm_gbs"] * 1e9), f32 / (FP32_TFLOPS * 1e12))
+        rows.append({"kernel": name, "calls": calls // reps, "ms": round(t * 1e3, 3), "tflops": round((fl + f32) / t * 1e-12, 1),
                      "gbs": round(by / t * 1e-9, 1), "roofline": round(bound / t, 3)})
     return rows
 
@@ -142,7 +140,7 @@ def step_table(eng, pos: int, steps: int = 4) -> List[dict]:
             t.step()
         torch.cuda.synchronize()
     t.pdl = pdl
-    ev = sorted((e for e in prof.events() if "stack_" in e.name or "latent_" in e.name), key=lambda e: e.time_range.start)
+    ev = sorted((e for e in prof.events() if any(x in e.name for x in ("stack_", "latent_", "state_step", "group_decode"))), key=lambda e: e.time_range.start)
     work = step_work(eng, pos)
     if len(ev) != steps * len(work):
         raise RuntimeError(f"{len(ev)} kernel records for {steps} x {len(work)} launches")

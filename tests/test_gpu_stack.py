@@ -305,7 +305,7 @@ def test_slow_decay_keeps_the_first_token():
 def test_products_against_torch(rows):
     """Every epilogue and tile width of the chunk product, sizes off every multiple."""
     from naivert_b200.ops import stack_kernels as S
-    from naivert_b200.runtime.stack import pack, pad
+    from naivert_b200.runtime.packing import pack, pad
     cfg = CASES["mixed"]
     eng = engine(cfg, weights(cfg), "bf16", capacity=1024, chunk=1024)
     pf = eng.prefill
@@ -324,7 +324,7 @@ def test_products_against_torch(rows):
 
             def run(epi, dtype=torch.float32, **more):
                 out = torch.full((rows, z, n), float("nan"), dtype=dtype, device="cuda")
-                pf._gemm(epi, p, x, z * kp, rows, out, z * n, **kw, **more)
+                pf.gemm(epi, p, x, z * kp, rows, out, z * n, **kw, **more)
                 torch.cuda.synchronize()
                 return out.double()
 
@@ -342,7 +342,7 @@ def test_products_against_torch(rows):
             if z == 1:
                 ld = pad(rows, 64)
                 out = torch.zeros(n, ld, dtype=torch.bfloat16, device="cuda")
-                pf._gemm(S.EPI_TRANSPOSE, p, x, kp, rows, out, ld, x_rows=rows)
+                pf.gemm(S.EPI_TRANSPOSE, p, x, kp, rows, out, ld, x_rows=rows)
                 close(out[:, :rows].t().double(), a[:, 0], 1e-2)
         eng.fabric.check()
     finally:

@@ -96,9 +96,9 @@ def test_engine_refuses_what_the_family_has_not():
 
 
 def test_head_padding_keeps_the_products():
-    from naivert_b200.runtime.stack import _head_rows, pack
+    from naivert_b200.runtime.packing import head_rows, pack
     w = torch.randn(3 * 5, 7)
-    p = _head_rows(w, 3, 5, 8)
+    p = head_rows(w, 3, 5, 8)
     assert p.shape == (24, 7) and torch.equal(p.view(3, 8, 7)[:, :5], w.view(3, 5, 7)) and not p.view(3, 8, 7)[:, 5:].any()
     k = pack(w, "cpu")
     assert (k.z, k.n, k.ld, k.k) == (1, 15, 8, 7) and not k.w[:, :, 7].any()
