@@ -403,24 +403,6 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeAr
 // grid (head tiles, splits).  Up to 32 heads of a CTA share every cached latent: the heads are the M side of bf16 m16n8k16
 // MMAs, the latents (64 per tile, two cp.async stages) serve as keys and, through ldmatrix.trans, as values.  tcgen05 is not
 // used: the kernel streams the cache once, and with at most 64 or so live query rows half of its M = 128 would idle.
-__device__ __forceinline__ void cp16(void* dst, const void* src, bool valid) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldsm2(uint32_t& r0, uint32_t& r1, const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldsm2t(uint32_t& r0, uint32_t& r1, const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(smem_u32(p)));
-}
-
 constexpr int kMaxDecRank = 512;
 __host__ __device__ inline int dec_pitch(int rank) { return (rank + 15) / 16 * 16 + 8; }        // bf16 elements; rows fall into distinct banks
 __host__ __device__ inline int dec_smem(int rank, int mt) {

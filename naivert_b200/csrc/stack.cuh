@@ -206,6 +206,18 @@ enum StateKind : int {
 };
 enum GateKind : int { kGateSigmoid = 0, kGateSilu = 1 };
 
+// Chunk rows are worked off in blocks of kStateBlock tokens.  With c_t the product of the block's decays up to token t (per key
+// channel), everything the block needs from the state S at its start are products with c_t k_t and c_t q_t, and what is left of the
+// tokens' influence on one another are a few numbers per pair.  `blocks` holds a record per (block, head), written by a kernel of its
+// own: [c_t k_t (delta only)] [c_t q_t] [k_t times the decays behind it], kStateBlock rows each, then the block's whole decay; rows are
+// padded with zeros to state_row(dim).  Then 64 pair coefficients, element [t][s]: s <= t: weight of token s's update in the
+// read-out of token t; s > t: what token t's update adds to S^T k at token s (delta).  Then the step sizes (delta).
+constexpr int kStateBlock = 8;
+__host__ __device__ inline int state_row(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : dim <= 256 ? 256 : 512; }
+__host__ __device__ inline int state_record(int kind, int dim) {
+  return ((kind == kStateDelta ? 3 : 2) * kStateBlock + 1) * state_row(dim) + kStateBlock * kStateBlock + kStateBlock;
+}
+
 struct StateChunkArgs {
   const float* q;               // element (row, key head, d) at row * q_ld + key head * dim + d
   const float* k;
@@ -221,6 +233,8 @@ struct StateChunkArgs {
   const float* gf;
   long long gate_ld;
   float cap;
+  float* keep;                  // normalized, scratch: [rows][heads][2] = factor on the state, factor on the new term
+  float* blocks;                // scratch: [blocks][heads][state_record]
   float* o;                     // [rows][heads * vdim]
   float* den;                   // normalized: [rows][heads][2] = n . q, exp(-m)
   float* state;                 // [2][state_stride]: heads x columns x dim4, then (normalized) the running maxima

@@ -82,16 +82,13 @@ __global__ void __launch_bounds__(256) transpose_kernel(const TransposeArgs a) {
 }
 
 // ------------------------------------------------------------------------------------ one token
-// grid (splits, key heads, groups of eight query heads); the splits of one key head are a cluster.  Eight lanes share a key, the
-// query heads of the CTA are scored together; then threads own value columns.  The partial results meet through distributed shared
-// memory.  Every CTA whose keys end at the token itself prepares and stores the token's key and value first (equal values).
+// The splits of the context of one key head are a cluster; their partial results meet through distributed shared memory.  Every CTA
+// whose keys end at the token itself prepares and stores the token's key and value (equal values where there are several).
+//
+// Plain form (32-bit caches, wide heads): grid (splits, key heads, groups of eight query heads); eight lanes share a key, the query
+// heads of the CTA are scored together; then threads own value columns.
 constexpr int kHB = 8, kTile = 64, kDecThreads = 256;
 
-__device__ __forceinline__ float ld_cluster_f32(const float* p, uint32_t rank) {
-  float v;
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(mapa_shared(smem_u32(p), rank)) : "memory");
-  return v;
-}
 __host__ __device__ inline int group_smem_floats(int dp, int vp) { return kHB * dp + kMaxHead + kTile * kHB + 3 * kHB + kHB * vp; }
 
 template <bool F32, int VC>                    // VC value columns per thread
@@ -257,6 +254,224 @@ __global__ void __launch_bounds__(kDecThreads) group_decode_kernel(const GroupDe
   cluster_sync_all();                                                    // nobody leaves while its shared memory is read
 }
 
+// Tensor-core form: grid (splits, key heads, tiles of 16 or 32 query heads).  The query heads of a key head are the M side of bf16
+// m16n8k16 MMAs; keys and values come 64 at a time through two cp.async stages, the first requested before the wait for the
+// predecessor (older rows do not depend on it; the token's own row is put into its tile by hand).  tcgen05 is not used: the kernel
+// streams the cache once, and most of its M = 128 rows would idle.
+constexpr int kTcHead = 256;
+__host__ __device__ inline int tc_pitch(int n) { return (n + 15) / 16 * 16 + 8; }              // bf16 elements; rows fall into distinct banks
+__host__ __device__ inline int group_tc_smem(int dp, int vp, int ht) {
+  return 2 * (ht + 2 * kTile) * tc_pitch(dp) + 2 * 2 * kTile * tc_pitch(vp) + 4 * ht * (kTile + 4) + 2 * ht * (kTile + 8) + 4 * 3 * ht + 4 * ht * vp +
+         4 * (8 * kTcHead + kTcHead) + 2 * (dp + vp);
+}
+
+template <int MT>
+__global__ void __launch_bounds__(kDecThreads, 1) group_decode_tc_kernel(const GroupDecodeArgs a) {
+  extern __shared__ __align__(16) uint8_t raw[];
+  constexpr int HT = MT * 16, kSP = kTile + 4, kPP = kTile + 8, kNT = kTcHead / 64;
+  const GroupPrepArgs& p = a.p;
+  const int kp = tc_pitch(p.dp), vpitch = tc_pitch(p.vp), rp = (p.dp + 15) / 16 * 16;
+  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(raw);             // [HT][kp]
+  __nv_bfloat16* sk = sq + HT * kp;                                      // [2][64][kp]
+  __nv_bfloat16* sv = sk + 2 * kTile * kp;                               // [2][64][vpitch]
+  __nv_bfloat16* sp = sv + 2 * kTile * vpitch;                           // [HT][kPP]
+  float* ss = reinterpret_cast<float*>(sp + HT * kPP);                   // [HT][kSP]
+  float* sm = ss + HT * kSP;
+  float* sl = sm + HT;
+  float* scorr = sl + HT;
+  float* so = scorr + HT;                                                // [HT][vp]
+  float* cs = so + HT * p.vp;
+  float* sn = cs + kTcHead / 2;
+  float* buf = sn + kTcHead / 2;                                         // [8][256]
+  __nv_bfloat16* new_k = reinterpret_cast<__nv_bfloat16*>(buf + 8 * kTcHead);
+  __nv_bfloat16* new_v = new_k + p.dp;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int split = blockIdx.x, hk = blockIdx.y, group = p.heads / p.kv_heads, h0 = blockIdx.z * HT, nh = min(HT, group - h0);
+  const int half = p.rot_dims / 2;
+  const int pos = *reinterpret_cast<const volatile int*>(p.pos0);
+  const bool inside = pos >= 0 && pos < p.capacity;
+  const int start = a.window > 0 ? pos / a.window * a.window : 0, n = inside ? pos + 1 - start : 0;
+  const int per = ((n + a.splits - 1) / a.splits + kTile - 1) / kTile * kTile;
+  const int j_lo = min(n, split * per), j_hi = min(n, j_lo + per);
+  const bool owner = j_hi == n && j_lo < j_hi;
+  {
+    uint4* z = reinterpret_cast<uint4*>(raw);                            // columns beyond a head stay zero
+    const int words = ((HT + 2 * kTile) * kp + 2 * kTile * vpitch) / 8;
+    for (int i = tid; i < words; i += kDecThreads) z[i] = make_uint4(0u, 0u, 0u, 0u);
+  }
+  for (int i = tid; i < HT * p.vp; i += kDecThreads) so[i] = 0.f;
+  for (int i = tid; i < HT; i += kDecThreads) { sm[i] = -FLT_MAX; sl[i] = 0.f; }
+  __syncthreads();
+  const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(p.k_cache) + (long long)hk * p.dp;
+  const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(p.v_cache) + (long long)hk * p.vp;
+  auto request = [&](int j0, int st) {
+    const int kpieces = p.dp / 8, pieces = kpieces + p.vp / 8;
+    for (int i = tid; i < kTile * pieces; i += kDecThreads) {
+      const int t = i / pieces, c = i - t * pieces;
+      const bool in = j0 + t < j_hi && j0 + t != n - 1;                  // the token's own row is not in the cache yet
+      const long long row = start + (in ? j0 + t : j_lo);
+      if (c < kpieces) cp16(sk + (st * kTile + t) * kp + c * 8, kc + row * p.kv_heads * p.dp + c * 8, in);
+      else cp16(sv + (st * kTile + t) * vpitch + (c - kpieces) * 8, vc + row * p.kv_heads * p.vp + (c - kpieces) * 8, in);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (j_lo < j_hi) request(j_lo, 0);
+  griddep_wait();
+  griddep_launch();
+  if (j_lo < j_hi) {
+    angles(p, pos, cs, sn);
+    __syncthreads();
+    for (int u = warp; u < nh + (owner ? 2 : 0); u += kDecThreads / 32) {
+      float* b = buf + warp * kTcHead;
+      if (u < nh) {
+        head_vector(p.proj + p.q_off + (hk * group + h0 + u) * p.dim, p.dim, p.q_norm, p.eps, half, cs, sn, p.scale, b, lane);
+        for (int c = lane; c < p.dim; c += 32) sq[u * kp + c] = __float2bfloat16_rn(b[c]);
+      } else if (u == nh) {
+        head_vector(p.proj + p.k_off + hk * p.dim, p.dim, p.k_norm, p.eps, half, cs, sn, 1.f, b, lane);
+        for (int c = lane; c < p.dp; c += 32) {
+          const __nv_bfloat16 x = __float2bfloat16_rn(c < p.dim ? b[c] : 0.f);
+          new_k[c] = x;
+          reinterpret_cast<__nv_bfloat16*>(p.k_cache)[((long long)pos * p.kv_heads + hk) * p.dp + c] = x;
+        }
+      } else {
+        for (int c = lane; c < p.vp; c += 32) {
+          const __nv_bfloat16 x = __float2bfloat16_rn(c < p.vdim ? __ldcg(p.proj + p.v_off + hk * p.vdim + c) : 0.f);
+          new_v[c] = x;
+          reinterpret_cast<__nv_bfloat16*>(p.v_cache)[((long long)pos * p.kv_heads + hk) * p.vp + c] = x;
+        }
+      }
+      __syncwarp();
+    }
+    float o[MT][kNT][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int t = 0; t < kNT; ++t)
+#pragma unroll
+        for (int q = 0; q < 4; ++q) o[i][t][q] = 0.f;
+    const int ntiles = p.vp / 8, fr = lane >> 2, fc = (lane & 3) * 2;
+    const float c2 = 1.4426950408889634f;                                // scores in powers of two
+    int st = 0;
+    for (int j0 = j_lo; j0 < j_hi; j0 += kTile, st ^= 1) {
+      if (j0 + kTile < j_hi) {
+        request(j0 + kTile, st ^ 1);
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+      } else {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+      }
+      __syncthreads();
+      if (owner && n - 1 < j0 + kTile) {                                 // the last tile: the token's own row
+        for (int c = tid; c < p.dp; c += kDecThreads) sk[(st * kTile + n - 1 - j0) * kp + c] = new_k[c];
+        for (int c = tid; c < p.vp; c += kDecThreads) sv[(st * kTile + n - 1 - j0) * vpitch + c] = new_v[c];
+        __syncthreads();
+      }
+      const __nv_bfloat16* kt = sk + st * kTile * kp;
+      const __nv_bfloat16* vt = sv + st * kTile * vpitch;
+      // scores: warp = 8 keys, all heads
+      float acc[MT][4];
+#pragma unroll
+      for (int i = 0; i < MT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll 4
+      for (int k = 0; k < rp; k += 16) {
+        uint32_t b0, b1;
+        ldsm2(b0, b1, kt + (warp * 8 + (lane & 7)) * kp + k + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+          uint32_t af[4];
+          ldsm4(af, sq + (i * 16 + (lane & 15)) * kp + k + (lane >> 4) * 8);
+          mma16816(acc[i], af, b0, b1);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        float* d = ss + (i * 16 + fr) * kSP + warp * 8 + fc;
+        d[0] = acc[i][0] * c2;
+        d[1] = acc[i][1] * c2;
+        d[8 * kSP] = acc[i][2] * c2;
+        d[8 * kSP + 1] = acc[i][3] * c2;
+      }
+      __syncthreads();
+      const int live = j_hi - j0;
+#pragma unroll
+      for (int ti = 0; ti < HT / 8; ++ti) {
+        const int t = warp + 8 * ti;
+        const float s0 = lane < live ? ss[t * kSP + lane] : -FLT_MAX, s1 = lane + 32 < live ? ss[t * kSP + lane + 32] : -FLT_MAX;
+        float mt = fmaxf(s0, s1);
+#pragma unroll
+        for (int off = 16; off > 0; off >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, off));
+        const float m_old = sm[t], mn = fmaxf(m_old, mt), corr = exp2_approx(m_old - mn);
+        const float p0 = lane < live ? exp2_approx(s0 - mn) : 0.f, p1 = lane + 32 < live ? exp2_approx(s1 - mn) : 0.f;
+        const float l = lane_sum(p0 + p1);
+        sp[t * kPP + lane] = __float2bfloat16_rn(p0);
+        sp[t * kPP + lane + 32] = __float2bfloat16_rn(p1);
+        __syncwarp();
+        if (lane == 0) { sm[t] = mn; sl[t] = sl[t] * corr + l; scorr[t] = corr; }
+      }
+      __syncthreads();
+      // outputs: warp = every eighth group of 8 value columns
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        const float ca = scorr[i * 16 + fr], cb = scorr[i * 16 + fr + 8];
+        uint32_t pf[4][4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) ldsm4(pf[k], sp + (i * 16 + (lane & 15)) * kPP + k * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int t = 0; t < kNT; ++t) {
+          const int nt = warp + 8 * t;
+          if (nt >= ntiles) continue;
+          o[i][t][0] *= ca;
+          o[i][t][1] *= ca;
+          o[i][t][2] *= cb;
+          o[i][t][3] *= cb;
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            uint32_t b0, b1;
+            ldsm2t(b0, b1, vt + (k * 16 + (lane & 15)) * vpitch + nt * 8);
+            mma16816(o[i][t], pf[k], b0, b1);
+          }
+        }
+      }
+      __syncthreads();                                                   // the stage and the P tile are free again
+    }
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int t = 0; t < kNT; ++t) {
+        const int c = (warp + 8 * t) * 8 + fc;
+        if (c >= p.vp) continue;
+        *reinterpret_cast<float2*>(so + (i * 16 + fr) * p.vp + c) = make_float2(o[i][t][0], o[i][t][1]);
+        *reinterpret_cast<float2*>(so + (i * 16 + fr + 8) * p.vp + c) = make_float2(o[i][t][2], o[i][t][3]);
+      }
+  }
+  cluster_sync_all();
+  // every CTA of the cluster finishes a share of the heads' columns
+  for (int i = split * kDecThreads + tid; i < nh * p.vdim && inside; i += a.splits * kDecThreads) {
+    const int h = i / p.vdim, c = i - h * p.vdim;
+    float m = -FLT_MAX, v = 0.f, sum = 0.f;
+    for (int s = 0; s < a.splits; ++s) m = fmaxf(m, ld_cluster_f32(sm + h, s));
+    for (int s = 0; s < a.splits; ++s) {
+      const float w = exp2_approx(ld_cluster_f32(sm + h, s) - m);
+      sum = fmaf(w, ld_cluster_f32(sl + h, s), sum);
+      v = fmaf(w, ld_cluster_f32(so + h * p.vp + c, s), v);
+    }
+    a.out[(long long)(hk * group + h0 + h) * p.vp + c] = v / sum;
+  }
+  cluster_sync_all();                                                    // nobody leaves while its shared memory is read
+}
+
+template <int MT>
+int launch_decode_tc(const GroupDecodeArgs& a, cudaStream_t stream, bool pdl) {
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(group_decode_tc_kernel<MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  const int group = a.p.heads / a.p.kv_heads;
+  return launch_cluster(group_decode_tc_kernel<MT>, dim3(a.splits, a.p.kv_heads, (group + MT * 16 - 1) / (MT * 16)), dim3(kDecThreads), dim3(a.splits, 1, 1),
+                        group_tc_smem(a.p.dp, a.p.vp, MT * 16), stream, pdl, a);
+}
+
 template <bool F32, int VC>
 int launch_decode(const GroupDecodeArgs& a, cudaStream_t stream, bool pdl) {
   const int smem = 4 * group_smem_floats(a.p.dp, a.p.vp);
@@ -304,6 +519,7 @@ extern "C" int nrt_group_decode(const void* args, void* stream, int pdl) {
   memcpy(&a, args, sizeof(a));
   if (!prep_ok(a.p) || a.p.rows != 1 || a.splits < 1 || a.splits > 8 || a.window < 0) return -3;
   const bool wide = a.p.vdim > kDecThreads, p = pdl != 0;
+  if (!a.p.f32 && a.p.dp <= kTcHead && a.p.vp <= kTcHead) return a.p.heads / a.p.kv_heads <= 16 ? launch_decode_tc<1>(a, S(stream), p) : launch_decode_tc<2>(a, S(stream), p);
   if (a.p.f32) return wide ? launch_decode<true, 2>(a, S(stream), p) : launch_decode<true, 1>(a, S(stream), p);
   return wide ? launch_decode<false, 2>(a, S(stream), p) : launch_decode<false, 1>(a, S(stream), p);
 }

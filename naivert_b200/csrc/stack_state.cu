@@ -3,9 +3,11 @@
 //                read-out norm and gate
 //   one token    one kernel: unit vectors, low-rank decay and gate, state update, read-out, norm and gate
 //
-// A value column of S evolves on its own given q, k and the decay, so columns are spread over the GPU and the tokens of a chunk run
-// one after the other, all in fp32 (packed pairs): eight lanes share a column, lane l holds the 16-byte pieces l, l + 8, ... of
-// its dim entries in registers for the whole chunk.  Rows arrive in shared memory tile by tile through cp.async, two tiles deep.
+// A value column of S evolves on its own given q, k and the decay, so columns are spread over the GPU; everything is fp32 (packed
+// pairs).  Chunks go in blocks of eight tokens (stack.cuh): L lanes share four columns, lane l holds the 16-byte pieces l, l + L, ...
+// of their dim entries in registers for the whole chunk; a block is two (delta: three) sets of independent products with the state and
+// one update, with a single reduction over the lanes.  One token after the other, each with a reduction of its own, left a scheduler
+// with one warp waiting for its own results two thirds of the time.
 #include "stack.cuh"
 #include "launch.hpp"
 
@@ -45,22 +47,6 @@ __device__ __forceinline__ float column_sum(float v) {                 // over t
   v += __shfl_xor_sync(0xffffffffu, v, 4);
   return v;
 }
-__device__ __forceinline__ void cp_async(float* dst, const float* src, bool vec) {
-  if (vec) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ bool quads(const float* p, long long ld, int n) {      // rows of n floats reachable in 16-byte pieces
-  return ((reinterpret_cast<uintptr_t>(p) & 15) | (uintptr_t)((ld | n) & 3)) == 0;
-}
-// Rows [0, n) of `cols` floats into shared rows of `pitch`.
-__device__ __forceinline__ void stage_rows(float* dst, int pitch, const float* src, long long ld, int n, int cols, bool vec) {
-  const int step = vec ? 4 : 1, per = cols / step;
-  for (int i = threadIdx.x; i < n * per; i += blockDim.x) {
-    const int t = i / per, c = (i - t * per) * step;
-    cp_async(dst + t * pitch + c, src + t * ld + c, vec);
-  }
-}
-
 __host__ __device__ inline int pad4(int n) { return (n + 3) / 4 * 4; }
 template <int KIND>
 __host__ __device__ constexpr int extra_columns() { return KIND == kStateNormalized ? 1 : 0; }      // the normaliser is a column with v = 1
@@ -123,148 +109,325 @@ __device__ __forceinline__ float column_step(u64 (&s)[2 * NV], const ulonglong2*
 __device__ __forceinline__ float log_input(float z, float cap) { return soft_cap(z, cap); }
 __device__ __forceinline__ float log_forget(float z, float cap) { return -softplus_f(-soft_cap(z, cap)); }
 
-// ------------------------------------------------------------------------------------ chunk path: the recurrence
-// grid (column tiles, heads); a warp holds four columns.
-__host__ __device__ inline int chunk_stage_floats(int kind, int dp, int cols, int tokens) {
-  return tokens * ((kind == kStateNormalized ? 2 : 3) * dp + cols + 4);
-}
+// ------------------------------------------------------------------------------------ chunk path: block records
+// Running maximum of the normalised form over the whole chunk, one CTA per head: m -> max(f + m, i) composes as (sum of f, max).
+constexpr int kScanT = 1024;
 
-template <int KIND, int NV>
-__global__ void __launch_bounds__(256) state_chunk_kernel(const StateChunkArgs a, const int tokens) {
-  constexpr int DP = NV * 4 * kLanes;
-  extern __shared__ __align__(16) float sh[];
+__global__ void __launch_bounds__(kScanT) gate_scan_kernel(const StateChunkArgs a) {
+  __shared__ float wf[32], wb[32];
   griddep_wait();
   griddep_launch();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane & (kLanes - 1);
-  const int cols = (blockDim.x >> 5) * 4, C = a.vdim + extra_columns<KIND>(), d4 = pad4(a.dim);
-  const int h = blockIdx.y, hk = h / (a.heads / a.kv_heads), c0 = blockIdx.x * cols, c = c0 + warp * 4 + lane / kLanes;
+  const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos0 = *a.pos0;
+  const int slot = state_slot(a.tags, pos0, a.status);
+  if (slot < 0) return;
+  const long long m_at = (long long)a.heads * (a.vdim + 1) * pad4(a.dim) + h;
+  float m = pos0 > 0 ? a.state[slot * a.state_stride + m_at] : 0.f;
+  for (int r0 = 0; r0 < a.rows; r0 += kScanT) {
+    const int r = r0 + threadIdx.x;
+    const bool in = r < a.rows;
+    const float zi = in ? log_input(a.gi[r * a.gate_ld + h], a.cap) : -FLT_MAX, zf = in ? log_forget(a.gf[r * a.gate_ld + h], a.cap) : 0.f;
+    float f = zf, b = zi;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float fp = __shfl_up_sync(0xffffffffu, f, o), bp = __shfl_up_sync(0xffffffffu, b, o);
+      if (lane >= o) {
+        b = fmaxf(f + bp, b);
+        f += fp;
+      }
+    }
+    if (lane == 31) { wf[warp] = f; wb[warp] = b; }
+    __syncthreads();
+    float before = m;                          // running maximum ahead of this warp, then ahead of this token
+    for (int w = 0; w < warp; ++w) before = fmaxf(wf[w] + before, wb[w]);
+    const float mt = fmaxf(f + before, b);
+    float mp = __shfl_up_sync(0xffffffffu, mt, 1);
+    if (lane == 0) mp = before;
+    if (in) {
+      *reinterpret_cast<float2*>(a.keep + ((long long)r * a.heads + h) * 2) = make_float2(expf(zf + mp - mt), expf(zi - mt));
+      a.den[((long long)r * a.heads + h) * 2 + 1] = expf(-mt);
+    }
+    for (int w = 0; w < kScanT / 32; ++w) m = fmaxf(wf[w] + m, wb[w]);
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) a.state[(1 - slot) * a.state_stride + m_at] = m;
+}
+
+// N values over the lanes -> N / L per lane: lane l keeps values N / L * l, ...
+template <int N, int L>
+__device__ __forceinline__ void scatter_sum(float (&v)[N], int l) {
+#pragma unroll
+  for (int o = L / 2, half = N / 2; o >= 1; o /= 2, half /= 2) {
+    const bool up = l & o;
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i)
+      if (i < half) {
+        const float keep = up ? v[i + half] : v[i], send = up ? v[i] : v[i + half];
+        v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+      }
+  }
+}
+
+// One warp per (block, head); lane = key channels lane, lane + 32, ... of a slice.
+template <int KIND, int NC>
+__global__ void __launch_bounds__(128) state_blocks_kernel(const StateChunkArgs a) {
+  griddep_wait();
+  griddep_launch();
+  constexpr int B = kStateBlock;
+  const int lane = threadIdx.x & 31, h = blockIdx.y * 4 + (threadIdx.x >> 5), r0 = blockIdx.x * B, n = min(B, a.rows - r0);
+  if (h >= a.heads) return;
+  const int hk = h / (a.heads / a.kv_heads), dp = state_row(a.dim);
+  float* rec = a.blocks + ((long long)blockIdx.x * a.heads + h) * state_record(KIND, a.dim);
+  float* k1 = rec;                             // (delta)
+  float* q1 = rec + (KIND == kStateDelta ? B * dp : 0);
+  float* k2 = q1 + B * dp;
+  float* whole = k2 + B * dp;
+  float* pairs = whole + dp;
+  float keep[B], add[B];
+#pragma unroll
+  for (int t = 0; t < B; ++t) {
+    keep[t] = add[t] = 1.f;
+    if (KIND == kStateNormalized && t < n) {
+      const float2 c = *reinterpret_cast<const float2*>(a.keep + ((long long)(r0 + t) * a.heads + h) * 2);
+      keep[t] = c.x;
+      add[t] = c.y;
+    }
+  }
+  float w[B * B];                              // pair coefficients, partial sums
+#pragma unroll
+  for (int i = 0; i < B * B; ++i) w[i] = 0.f;
+  for (int d0 = 0; d0 < dp; d0 += 32 * NC) {
+    float q[B][NC], k[B][NC], g[B][NC];
+#pragma unroll
+    for (int t = 0; t < B; ++t)
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+        const int d = d0 + lane + 32 * i;
+        const bool in = t < n && d < a.dim;
+        q[t][i] = in ? __ldg(a.q + (r0 + t) * a.q_ld + hk * a.dim + d) * a.q_scale : 0.f;
+        k[t][i] = in ? __ldg(a.k + (r0 + t) * a.k_ld + hk * a.dim + d) : 0.f;
+        g[t][i] = KIND == kStateNormalized ? keep[t] : in ? __ldg(a.g + (r0 + t) * a.g_ld + h * a.dim + d) : 1.f;
+      }
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int d = d0 + lane + 32 * i;
+      float c = 1.f;
+#pragma unroll
+      for (int t = 0; t < B; ++t) {
+        if (KIND == kStateBonus) q1[t * dp + d] = c * q[t][i];            // the read-out sees the state ahead of the token
+        c *= g[t][i];
+        if (KIND != kStateBonus) q1[t * dp + d] = c * q[t][i];
+        if (KIND == kStateDelta) k1[t * dp + d] = c * k[t][i];
+      }
+      whole[d] = c;
+      c = 1.f;
+#pragma unroll
+      for (int t = B - 1; t >= 0; --t) {
+        k2[t * dp + d] = c * add[t] * k[t][i];
+        c *= g[t][i];
+      }
+      const float bonus = KIND == kStateBonus && d < a.dim ? bf(a.u + (long long)h * a.dim + d) : 1.f;
+#pragma unroll
+      for (int s = 0; s < B; ++s) {
+        c = k[s][i] * add[s];
+        w[s * B + s] = fmaf(q[s][i], c * bonus, w[s * B + s]);
+#pragma unroll
+        for (int t = s + 1; t < B; ++t) {
+          if (KIND == kStateBonus) w[t * B + s] = fmaf(q[t][i], c, w[t * B + s]);
+          c *= g[t][i];
+          if (KIND != kStateBonus) w[t * B + s] = fmaf(q[t][i], c, w[t * B + s]);
+          if (KIND == kStateDelta) w[s * B + t] = fmaf(k[t][i], c, w[s * B + t]);
+        }
+      }
+    }
+  }
+  scatter_sum<B * B, 32>(w, lane);
+  *reinterpret_cast<float2*>(pairs + 2 * lane) = make_float2(w[0], w[1]);
+  if (lane < B) pairs[B * B + lane] = KIND == kStateDelta && lane < n ? sigmoid_f(a.beta[(r0 + lane) * a.beta_ld + h]) : 0.f;
+}
+
+// ------------------------------------------------------------------------------------ chunk path: the recurrence
+// grid (column tiles, heads); a warp holds 4 * 32 / L columns; records and values arrive three stages deep, the records as one bulk copy.
+constexpr int kQuad = 4, kStages = 3;
+
+template <int L, int NV>
+__device__ __forceinline__ void state_products(const u64 (&s)[kQuad][2 * NV], const ulonglong2* vec, float (&out)[32]) {
+  // out[value]: value = 32 / L * lane + i belongs to column lane & 3 and token (lane >> 2) + L / 4 * i
+  constexpr int VPL = 32 / L;
+  u64 acc[kStateBlock][kQuad];
+#pragma unroll
+  for (int t = 0; t < kStateBlock; ++t)
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const ulonglong2 x = vec[t * (NV * L) + i * L];
+#pragma unroll
+      for (int j = 0; j < kQuad; ++j) acc[t][j] = i == 0 ? mul2(s[j][0], x.x) : fma2(s[j][2 * i], x.x, acc[t][j]);
+#pragma unroll
+      for (int j = 0; j < kQuad; ++j) acc[t][j] = fma2(s[j][2 * i + 1], x.y, acc[t][j]);
+    }
+#pragma unroll
+  for (int v = 0; v < 32; ++v) out[v] = both(acc[(v / VPL >> 2) + L / 4 * (v % VPL)][v / VPL & 3]);
+}
+
+template <int KIND, int L, int NV>
+__global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArgs a) {
+  constexpr int B = kStateBlock, DP = NV * 4 * L, PER_WARP = 32 / L * kQuad, VPL = 32 / L;
+  constexpr int ROWS = (KIND == kStateDelta ? 3 : 2) * B, REC = (ROWS + 1) * DP + B * B + B;
+  extern __shared__ __align__(16) float sh[];
+  __shared__ uint64_t full[kStages];
+  griddep_wait();
+  griddep_launch();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane & (L - 1);
+  const int cols = (blockDim.x >> 5) * PER_WARP, C = a.vdim + extra_columns<KIND>(), d4 = pad4(a.dim);
+  const int h = blockIdx.y, c0 = blockIdx.x * cols, c = c0 + warp * PER_WARP + lane / L * kQuad;
   const int pos0 = *a.pos0;
   const int slot = state_slot(a.tags, pos0, a.status);
   if (slot < 0) return;
   const float* old = a.state + slot * a.state_stride;
   float* now = a.state + (1 - slot) * a.state_stride;
   const long long at = ((long long)h * C + c) * d4;
-  const bool live = c < C;
 
-  u64 s[2 * NV];
+  u64 s[kQuad][2 * NV];
 #pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    ulonglong2 v = make_ulonglong2(0ull, 0ull);
-    const int e = (l + kLanes * i) * 4;
-    if (live && pos0 > 0 && e < d4) v = *reinterpret_cast<const ulonglong2*>(old + at + e);
-    s[2 * i] = v.x;
-    s[2 * i + 1] = v.y;
-  }
-  float m = KIND == kStateNormalized && pos0 > 0 ? old[(long long)a.heads * C * d4 + h] : 0.f;
-
-  const int stage = chunk_stage_floats(KIND, DP, cols, tokens);
-  for (int i = threadIdx.x; i < 2 * stage; i += blockDim.x) sh[i] = 0.f;      // columns beyond dim stay zero
-  __syncthreads();
-  const float* q0 = a.q + (long long)hk * a.dim;
-  const float* k0 = a.k + (long long)hk * a.dim;
-  const float* g0 = KIND == kStateNormalized ? nullptr : a.g + (long long)h * a.dim;
-  const float* v0 = a.v + (long long)h * a.vdim + c0;
-  const int vcols = min(cols, a.vdim - c0);                              // (none in a tile that holds only the normaliser)
-  const bool qv = quads(q0, a.q_ld, a.dim), kv = quads(k0, a.k_ld, a.dim), gv = KIND != kStateNormalized && quads(g0, a.g_ld, a.dim),
-             vv = vcols > 0 && quads(v0, a.v_ld, vcols);
-  auto parts = [&](int st, float*& sk, float*& sq, float*& sg, float*& sv, float*& sc) {
-    sk = sh + st * stage;
-    sq = sk + tokens * DP;
-    sg = sq + tokens * DP;
-    sv = KIND == kStateNormalized ? sg : sg + tokens * DP;
-    sc = sv + tokens * cols;                                             // four scalars per token: two raw, two derived
-  };
-  auto request = [&](int r0, int st) {
-    const int n = min(tokens, a.rows - r0);
-    float *sk, *sq, *sg, *sv, *sc;
-    parts(st, sk, sq, sg, sv, sc);
-    stage_rows(sk, DP, k0 + r0 * a.k_ld, a.k_ld, n, a.dim, kv);
-    stage_rows(sq, DP, q0 + r0 * a.q_ld, a.q_ld, n, a.dim, qv);
-    if (KIND != kStateNormalized) stage_rows(sg, DP, g0 + r0 * a.g_ld, a.g_ld, n, a.dim, gv);
-    if (vcols > 0) stage_rows(sv, cols, v0 + r0 * a.v_ld, a.v_ld, n, vcols, vv);
-    if (KIND == kStateDelta) stage_rows(sc, 4, a.beta + r0 * a.beta_ld + h, a.beta_ld, n, 1, false);
-    if (KIND == kStateNormalized) {
-      stage_rows(sc, 4, a.gi + r0 * a.gate_ld + h, a.gate_ld, n, 1, false);
-      stage_rows(sc + 1, 4, a.gf + r0 * a.gate_ld + h, a.gate_ld, n, 1, false);
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-
-  request(0, 0);
-  int st = 0;
-  for (int r0 = 0; r0 < a.rows; r0 += tokens, st ^= 1) {
-    const int n = min(tokens, a.rows - r0);
-    if (r0 + tokens < a.rows) {
-      request(r0 + tokens, st ^ 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();
-    float *sk, *sq, *sg, *sv, *sc;
-    parts(st, sk, sq, sg, sv, sc);
-    // scalars of the tile's tokens
-    if (KIND == kStateDelta) {
-      if ((int)threadIdx.x < n) sc[threadIdx.x * 4 + 2] = sigmoid_f(sc[threadIdx.x * 4]);
-    } else if (KIND == kStateBonus) {
-      for (int t = warp; t < n; t += blockDim.x >> 5) {
-        float b = 0.f;
-        for (int d = lane; d < a.dim; d += 32) b = fmaf(sq[t * DP + d] * bf(a.u + (long long)h * a.dim + d), sk[t * DP + d], b);
-        b = lane_sum(b);
-        if (lane == 0) sc[t * 4 + 2] = b;
-      }
-    } else if (warp == 0) {
-      // running maximum over the tile: m -> max(f + m, i) composes as (sum of f, max), scanned over the lanes
-      const float zi = lane < n ? log_input(sc[lane * 4], a.cap) : 0.f, zf = lane < n ? log_forget(sc[lane * 4 + 1], a.cap) : 0.f;
-      float f = zf, b = lane < n ? zi : -FLT_MAX;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float fp = __shfl_up_sync(0xffffffffu, f, o), bp = __shfl_up_sync(0xffffffffu, b, o);
-        if (lane >= o) {
-          b = fmaxf(f + bp, b);
-          f += fp;
-        }
-      }
-      const float mt = fmaxf(f + m, b);
-      float before = __shfl_up_sync(0xffffffffu, mt, 1);
-      if (lane == 0) before = m;
-      if (lane < n) {
-        sc[lane * 4] = expf(-mt);
-        sc[lane * 4 + 2] = expf(zf + before - mt);
-        sc[lane * 4 + 3] = expf(zi - mt);
-      }
-      m = __shfl_sync(0xffffffffu, mt, n - 1);
-    }
-    __syncthreads();
-    const ulonglong2* q = reinterpret_cast<const ulonglong2*>(sq) + l;
-    const ulonglong2* k = reinterpret_cast<const ulonglong2*>(sk) + l;
-    const ulonglong2* g = reinterpret_cast<const ulonglong2*>(sg) + l;
-    const bool normaliser = KIND == kStateNormalized && c == a.vdim;
-    const float* vc = sv + (c - c0);
-    const bool vin = c < a.vdim;
-    float* o = a.o + ((long long)r0 * a.heads + h) * a.vdim + c;
-#pragma unroll 2
-    for (int t = 0; t < n; ++t) {
-      const float v = KIND == kStateNormalized && normaliser ? 1.f : vc[t * cols];
-      float r = column_step<KIND, NV>(s, q + t * (DP / 4), k + t * (DP / 4), g + t * (DP / 4), v, sc[t * 4 + 2], sc[t * 4 + 3]);
-      r = column_sum(r);
-      if (KIND == kStateBonus) r = fmaf(sc[t * 4 + 2], v, r);
-      if (l == 0) {
-        if (vin) o[(long long)t * a.heads * a.vdim] = r * a.q_scale;
-        else if (normaliser) *reinterpret_cast<float2*>(a.den + ((long long)(r0 + t) * a.heads + h) * 2) = make_float2(r * a.q_scale, sc[t * 4]);
-      }
-    }
-    __syncthreads();                                                     // the stage is free again
-  }
-
-  if (live) {
+  for (int j = 0; j < kQuad; ++j)
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int e = (l + kLanes * i) * 4;
-      if (e < d4) *reinterpret_cast<ulonglong2*>(now + at + e) = make_ulonglong2(s[2 * i], s[2 * i + 1]);
+      ulonglong2 v = make_ulonglong2(0ull, 0ull);
+      const int e = (l + L * i) * 4;
+      if (c + j < C && pos0 > 0 && e < d4) v = *reinterpret_cast<const ulonglong2*>(old + at + (long long)j * d4 + e);
+      s[j][2 * i] = v.x;
+      s[j][2 * i + 1] = v.y;
     }
+
+  float* sv = sh + kStages * REC;                                        // [stages][B][cols]
+  float* work = sv + kStages * B * cols + (warp * (32 / L) + lane / L) * 2 * B * kQuad;     // this lane group's: S^T k, updates [B][4]
+  for (int i = threadIdx.x; i < kStages * B * cols; i += blockDim.x) {
+    const int cc = c0 + i % cols;
+    sv[i] = KIND == kStateNormalized && cc == a.vdim ? 1.f : 0.f;         // the normaliser's column
   }
-  if (KIND == kStateNormalized && blockIdx.x == 0 && threadIdx.x == 0) now[(long long)a.heads * C * d4 + h] = m;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kStages; ++i) mbar_init(&full[i], 1);
+    mbar_fence_init();
+  }
+  __syncthreads();
+  const int blocks = (a.rows + B - 1) / B;
+  const float* v0 = a.v + (long long)h * a.vdim + c0;
+  const int vcols = min(cols, a.vdim - c0);                              // (none in a tile that holds only the normaliser)
+  const bool quads = vcols > 0 && ((reinterpret_cast<uintptr_t>(v0) & 15) | (uintptr_t)((a.v_ld | vcols) & 3)) == 0;
+  const int step = quads ? 4 : 1, per = max(vcols, 0) / step;
+  auto request = [&](int b, int st) {
+    if (threadIdx.x == 0) {
+      mbar_expect_tx(&full[st], REC * 4);
+      asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                   ::"r"(smem_u32(sh + st * REC)), "l"(a.blocks + ((long long)b * a.heads + h) * REC), "r"(REC * 4), "r"(smem_u32(&full[st]))
+                   : "memory");
+    }
+    const int n = min(B, a.rows - b * B);
+    for (int i = threadIdx.x; i < n * per; i += blockDim.x) {
+      const int t = i / per, e = (i - t * per) * step;
+      const uint32_t dst = smem_u32(sv + (st * B + t) * cols + e);
+      const float* src = v0 + (b * B + t) * a.v_ld + e;
+      if (quads) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+      else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory");
+    }
+  };
+  request(0, 0);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  if (blocks > 1) request(1, 1);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  const int col = l & 3, tq = l >> 2;                                    // this lane's column and first token among the reduced values
+  bool ok = true;
+  for (int b = 0, st = 0; b < blocks; ++b, st = st + 1 == kStages ? 0 : st + 1) {
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    ok = __syncthreads_and(mbar_wait(&full[st], (b / kStages) & 1, a.status, kSiteTmaFull | st));
+    if (!ok) break;
+    if (b + 2 < blocks) request(b + 2, st + 2 >= kStages ? st + 2 - kStages : st + 2);       // (its last reader has passed the barrier)
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    const float* rec = sh + st * REC;
+    const ulonglong2* vec = reinterpret_cast<const ulonglong2*>(rec) + l;
+    const float* pairs = rec + (ROWS + 1) * DP;
+    const float* vc = sv + st * B * cols + (c - c0);
+    float p[32], q[32];
+    if (KIND == kStateDelta) {
+      state_products<L, NV>(s, vec, p);
+      scatter_sum<32, L>(p, l);
+#pragma unroll
+      for (int i = 0; i < VPL; ++i) work[(tq + L / 4 * i) * kQuad + col] = p[i];
+    }
+    state_products<L, NV>(s, vec + (KIND == kStateDelta ? B * DP / 4 : 0), q);
+    scatter_sum<32, L>(q, l);
+    const float* upd = vc;                     // the tokens' updates of the group's columns, rows of `upd_ld`
+    int upd_ld = cols;
+    if (KIND == kStateDelta) {
+      __syncwarp();
+      float* us = work + B * kQuad;
+      if (l < kQuad) {
+        float r[B];
+#pragma unroll
+        for (int t = 0; t < B; ++t) r[t] = vc[t * cols + col] - work[t * kQuad + col];
+#pragma unroll
+        for (int t = 0; t < B; ++t) {
+          const float u = pairs[B * B + t] * r[t];
+          us[t * kQuad + col] = u;
+#pragma unroll
+          for (int x = t + 1; x < B; ++x) r[x] = fmaf(-pairs[t * B + x], u, r[x]);
+        }
+      }
+      __syncwarp();
+      upd = us;
+      upd_ld = kQuad;
+    }
+    // the state moves on by the whole block
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const ulonglong2 g = vec[ROWS * DP / 4 + i * L];
+#pragma unroll
+      for (int j = 0; j < kQuad; ++j) {
+        s[j][2 * i] = mul2(s[j][2 * i], g.x);
+        s[j][2 * i + 1] = mul2(s[j][2 * i + 1], g.y);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < B; ++t) {
+      const float4 u = *reinterpret_cast<const float4*>(upd + t * upd_ld);
+      const u64 uu[kQuad] = {pack2(u.x, u.x), pack2(u.y, u.y), pack2(u.z, u.z), pack2(u.w, u.w)};
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const ulonglong2 k = vec[(ROWS - B + t) * DP / 4 + i * L];
+#pragma unroll
+        for (int j = 0; j < kQuad; ++j) {
+          s[j][2 * i] = fma2(k.x, uu[j], s[j][2 * i]);
+          s[j][2 * i + 1] = fma2(k.y, uu[j], s[j][2 * i + 1]);
+        }
+      }
+    }
+    // read-outs: this lane's column at its tokens
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) {
+      const int t = tq + L / 4 * i;
+      float x = q[i];
+#pragma unroll
+      for (int e = 0; e < B; ++e) x = fmaf(e <= t ? pairs[t * B + e] : 0.f, upd[e * upd_ld + col], x);
+      const int r = b * B + t;
+      if (r < a.rows) {
+        if (c + col < a.vdim) a.o[((long long)r * a.heads + h) * a.vdim + c + col] = x;
+        else if (KIND == kStateNormalized && c + col == a.vdim) a.den[((long long)r * a.heads + h) * 2] = x;
+      }
+    }
+    if (KIND == kStateDelta) __syncwarp();                               // the work area is rewritten
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  if (!ok) {
+    drain_on_error(a.status);
+    return;
+  }
+#pragma unroll
+  for (int j = 0; j < kQuad; ++j)
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = (l + L * i) * 4;
+      if (c + j < C && e < d4) *reinterpret_cast<ulonglong2*>(now + at + (long long)j * d4 + e) = make_ulonglong2(s[j][2 * i], s[j][2 * i + 1]);
+    }
   if (a.history) {
     const int keep = min(a.taps - 1, a.rows), ctas = gridDim.x * gridDim.y, cta = blockIdx.y * gridDim.x + blockIdx.x;
     for (int i = cta * blockDim.x + threadIdx.x; i < keep * a.hist_cols; i += ctas * blockDim.x) {
@@ -281,7 +444,7 @@ __global__ void __launch_bounds__(256) state_chunk_kernel(const StateChunkArgs a
 
 // ------------------------------------------------------------------------------------ chunk path: around the recurrence
 // One warp per (head or operand copy, strip of rows).
-constexpr int kConvStrip = 8;
+constexpr int kConvStrip = 16, kConvWin = 4;  // rows per warp; taps that stay in a register window (longer kernels re-read their inputs)
 
 template <int NC>
 __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvArgs a) {
@@ -304,30 +467,78 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvArgs a) 
   float* out = is_v ? a.v + (seg - 2 * G) * a.vdim : (seg < G ? a.q : a.k) + (seg % G) * a.dim;
   const long long out_ld = (long long)(is_v ? a.heads * a.vdim : G * a.dim);
   const __nv_bfloat16* kern = a.conv + (long long)col * a.taps;
-  for (int r = r0; r < r1; ++r) {
-    float y[NC], ss = 0.f;
+  auto input = [&](int rr, int c) {            // row rr of the projection, or what earlier chunks left
+    if (rr >= 0) return __ldg(a.proj + rr * a.ld + col + c);
+    return pos0 + rr >= 0 ? a.history[(long long)((pos0 + rr) % a.hist_rows) * columns + col + c] : 0.f;
+  };
+  auto finish = [&](int r, float (&y)[NC]) {
+    float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
-      const int c = lane + 32 * i;
-      y[i] = 0.f;
-      if (c < w) {
-#pragma unroll 4
-        for (int j = 0; j < a.taps; ++j) {
-          const int rr = r - (a.taps - 1 - j);
-          float x = 0.f;
-          if (rr >= 0) x = __ldg(a.proj + rr * a.ld + col + c);
-          else if (pos0 + rr >= 0) x = a.history[(long long)((pos0 + rr) % a.hist_rows) * columns + col + c];
-          y[i] = fmaf(bf(kern + c * a.taps + j), x, y[i]);
-        }
-        y[i] = silu_f(y[i]);
-      }
+      y[i] = lane + 32 * i < w ? silu_f(y[i]) : 0.f;
       ss = fmaf(y[i], y[i], ss);
     }
     const float scale = is_v ? 1.f : (seg < G ? a.q_scale : 1.f) / sqrtf(lane_sum(ss) + kUnitEps);
 #pragma unroll
     for (int i = 0; i < NC; ++i)
       if (lane + 32 * i < w) out[r * out_ld + lane + 32 * i] = y[i] * scale;
+  };
+  if (a.taps <= kConvWin) {
+    constexpr int BATCH = NC <= 4 ? 4 : 1;     // rows requested together
+    float kw[NC][kConvWin], x[NC][kConvWin];   // newest last; missing taps are zero
+#pragma unroll
+    for (int i = 0; i < NC; ++i)
+#pragma unroll
+      for (int j = 0; j < kConvWin; ++j) {
+        const int c = lane + 32 * i, t = j - (kConvWin - a.taps);
+        kw[i][j] = c < w && t >= 0 ? bf(kern + c * a.taps + t) : 0.f;
+        x[i][j] = c < w && j > kConvWin - a.taps ? input(r0 - (kConvWin - j), c) : 0.f;
+      }
+#pragma unroll 1
+    for (int rb = r0; rb < r1; rb += BATCH) {
+      float in[BATCH][NC];
+#pragma unroll
+      for (int q = 0; q < BATCH; ++q)
+#pragma unroll
+        for (int i = 0; i < NC; ++i) in[q][i] = rb + q < r1 && lane + 32 * i < w ? __ldg(a.proj + (rb + q) * a.ld + col + lane + 32 * i) : 0.f;
+#pragma unroll
+      for (int q = 0; q < BATCH; ++q) {
+        if (rb + q >= r1) break;
+        float y[NC];
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+          y[i] = 0.f;
+#pragma unroll
+          for (int j = 0; j < kConvWin; ++j) {
+            x[i][j] = j + 1 < kConvWin ? x[i][j + 1] : in[q][i];
+            y[i] = fmaf(kw[i][j], x[i][j], y[i]);
+          }
+        }
+        finish(rb + q, y);
+      }
+    }
+    return;
   }
+  for (int r = r0; r < r1; ++r) {
+    float y[NC];
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = lane + 32 * i;
+      y[i] = 0.f;
+      if (c < w)
+        for (int j = 0; j < a.taps; ++j) y[i] = fmaf(bf(kern + c * a.taps + j), input(r - (a.taps - 1 - j), c), y[i]);
+    }
+    finish(r, y);
+  }
+}
+
+__device__ __forceinline__ float4 bf4(const __nv_bfloat16* p) {
+  const uint2 v = __ldg(reinterpret_cast<const uint2*>(p));
+  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
+}
+__device__ __forceinline__ void store_act4(void* base, long long i, const float4& v, int f32) {
+  if (f32) *reinterpret_cast<float4*>(reinterpret_cast<float*>(base) + i) = v;
+  else *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(base) + i) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
 }
 
 __global__ void __launch_bounds__(256) token_mix_kernel(const TokenMixArgs a) {
@@ -340,6 +551,20 @@ __global__ void __launch_bounds__(256) token_mix_kernel(const TokenMixArgs a) {
   const float* before = r > 0 ? x - a.width : pos0 > 0 ? a.shift + slot * a.state_stride : nullptr;
   float* keep = r == a.rows - 1 ? a.shift + (1 - slot) * a.state_stride : nullptr;
   const long long o0 = (long long)r * a.mixes * a.out_ld;
+  if (((a.width | (int)a.out_ld | (int)a.state_stride) & 3) == 0 && (reinterpret_cast<uintptr_t>(a.shift) & 15) == 0) {
+    for (int c = threadIdx.x * 4; c < a.width; c += 1024) {
+      const float4 v = __ldg(reinterpret_cast<const float4*>(x + c));
+      const float4 b = before ? *reinterpret_cast<const float4*>(before + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 d = make_float4(b.x - v.x, b.y - v.y, b.z - v.z, b.w - v.w);
+#pragma unroll 5
+      for (int s = 0; s < a.mixes; ++s) {
+        const float4 m = bf4(a.mu + (long long)s * a.width + c);
+        store_act4(a.out, o0 + s * a.out_ld + c, make_float4(fmaf(d.x, m.x, v.x), fmaf(d.y, m.y, v.y), fmaf(d.z, m.z, v.z), fmaf(d.w, m.w, v.w)), a.f32);
+      }
+      if (keep) *reinterpret_cast<float4*>(keep + c) = v;
+    }
+    return;
+  }
   for (int c = threadIdx.x; c < a.width; c += 256) {
     const float v = __ldg(x + c), d = (before ? before[c] : 0.f) - v;
     for (int s = 0; s < a.mixes; ++s) store_act(a.out, o0 + s * a.out_ld + c, fmaf(d, bf(a.mu + (long long)s * a.width + c), v), a.f32);
@@ -359,32 +584,60 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const HeadGateArgs a) {
     const float* d = a.den + ((long long)r * a.heads + h) * 2;
     inv = 1.0f / (fmaxf(fabsf(d[0]), d[1]) + 1e-6f);
   }
+  const float* g = a.gate + (long long)r * a.gate_ld + (long long)h * a.vdim;
+  const __nv_bfloat16* w = a.norm + (a.norm_per_head ? (long long)h * a.vdim : 0);
+  const long long at = (long long)r * a.out_ld + (long long)h * a.vdim;
+  auto gated = [&](float z) { return a.gate_kind == kGateSilu ? silu_f(z) : sigmoid_f(z); };
   float ss = 0.f;
+  if (((a.vdim | (int)a.gate_ld | (int)a.out_ld) & 3) == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 15) == 0) {
+    constexpr int KEEP = 4;                    // pieces of a head that stay in registers between the two passes
+    float4 keep[KEEP], z[KEEP];
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int c = (lane + 32 * i) * 4;
+      keep[i] = z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < a.vdim) {
+        keep[i] = __ldg(reinterpret_cast<const float4*>(o + c));
+        z[i] = __ldg(reinterpret_cast<const float4*>(g + c));
+      }
+    }
+    auto sq = [&](const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+    auto put = [&](int c, const float4& v, const float4& zz, float rs) {
+      const float4 n = bf4(w + c);
+      store_act4(a.out, at + c, make_float4(v.x * rs * n.x * gated(zz.x), v.y * rs * n.y * gated(zz.y), v.z * rs * n.z * gated(zz.z), v.w * rs * n.w * gated(zz.w)), a.f32);
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) ss += sq(keep[i]);
+    for (int c = (lane + 32 * KEEP) * 4; c < a.vdim; c += 128) ss += sq(__ldg(reinterpret_cast<const float4*>(o + c)));
+    const float rs = inv / sqrtf(lane_sum(ss) * inv * inv / (float)a.vdim + a.eps);
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+      if ((lane + 32 * i) * 4 < a.vdim) put((lane + 32 * i) * 4, keep[i], z[i], rs);
+    for (int c = (lane + 32 * KEEP) * 4; c < a.vdim; c += 128) put(c, __ldg(reinterpret_cast<const float4*>(o + c)), __ldg(reinterpret_cast<const float4*>(g + c)), rs);
+    return;
+  }
   for (int c = lane; c < a.vdim; c += 32) {
     const float v = __ldg(o + c) * inv;
     ss = fmaf(v, v, ss);
   }
   const float rs = inv / sqrtf(lane_sum(ss) / (float)a.vdim + a.eps);
-  const float* g = a.gate + (long long)r * a.gate_ld + (long long)h * a.vdim;
-  const __nv_bfloat16* w = a.norm + (a.norm_per_head ? (long long)h * a.vdim : 0);
-  for (int c = lane; c < a.vdim; c += 32) {
-    const float z = __ldg(g + c), gate = a.gate_kind == kGateSilu ? silu_f(z) : sigmoid_f(z);
-    store_act(a.out, (long long)r * a.out_ld + (long long)h * a.vdim + c, __ldg(o + c) * rs * bf(w + c) * gate, a.f32);
-  }
+  for (int c = lane; c < a.vdim; c += 32) store_act(a.out, at + c, __ldg(o + c) * rs * bf(w + c) * gated(__ldg(g + c)), a.f32);
 }
 
 // ------------------------------------------------------------------------------------ one token
-// One CTA per head.  The state is requested before the wait for the predecessor: it was written a whole step ago.
-constexpr int kStepT = 512, kStepCols = kStepT / kLanes;
+// grid (share of the value columns, heads); the CTAs of a head are a cluster that meets once, for the read-out norm.  The state (written
+// a whole step ago) and the low-rank weights are requested before the wait for the predecessor.
+constexpr int kStepT = 256, kStepCols = kStepT / kLanes;
 
 // rows of a low-rank product: out[row] = W[row] . in, one warp per row
-template <class F>
-__device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, long long ld, int rows, const float* in, int warp, int lane, F store) {
+template <bool STAGED, class F>
+__device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, int ld, int rows, const float* in, int warp, int lane, F store) {
 #pragma unroll 4
   for (int r = warp; r < rows; r += kStepT / 32) {
     float acc = 0.f;
-    for (int c = lane * 4; c < (int)ld; c += 128) {
-      const uint2 p = __ldg(reinterpret_cast<const uint2*>(w + r * ld + c));
+    for (int c = lane * 4; c < ld; c += 128) {
+      const uint2* src = reinterpret_cast<const uint2*>(w + (long long)r * ld + c);
+      const uint2 p = STAGED ? *src : __ldg(src);
       const float4 x = *reinterpret_cast<const float4*>(in + c);
       acc = fmaf(bf16_lo(p.x), x.x, fmaf(bf16_hi(p.x), x.y, fmaf(bf16_lo(p.y), x.z, fmaf(bf16_hi(p.y), x.w, acc))));
     }
@@ -392,139 +645,182 @@ __device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, long long 
     if (lane == 0) store(r, acc);
   }
 }
-__host__ __device__ inline int step_floats(int dp, int vdim, int decay_ld, int gate_ld) {
-  return 3 * dp + 2 * pad4(vdim + 1) + decay_ld + gate_ld;
+__device__ __forceinline__ void stage_weights(void* dst, const __nv_bfloat16* src, int n) {        // n a multiple of 8
+  for (int i = threadIdx.x * 8; i < n; i += kStepT * 8)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(reinterpret_cast<__nv_bfloat16*>(dst) + i)), "l"(src + i) : "memory");
 }
+__host__ __device__ inline int step_floats(int dp, int per, int decay_ld, int gate_ld) { return 3 * dp + 3 * pad4(per + 1) + decay_ld + gate_ld; }
 
 template <int KIND, int NV>
-__global__ void __launch_bounds__(kStepT) state_step_kernel(const StateStepArgs a) {
+__global__ void __launch_bounds__(kStepT, 1) state_step_kernel(const StateStepArgs a, const int per, const int staged) {
   constexpr int DP = NV * 4 * kLanes, AHEAD = NV <= 4 ? 2 : 1;
   extern __shared__ __align__(16) float sh[];
-  __shared__ float red[33];
+  __shared__ float red[33], part;
+  const int rank = blockIdx.x, h = blockIdx.y, hk = h / (a.heads / a.kv_heads);
+  const int c_lo = min(a.vdim, rank * per), own = min(a.vdim, c_lo + per) - c_lo, cols = own + extra_columns<KIND>();
+  const int decay_ld = (int)a.decay_ld, gate_ld = (int)a.gate_ld;
   float* sk = sh;
   float* sq = sk + DP;
   float* sg = sq + DP;
   float* so = sg + DP;
-  float* sgate = so + pad4(a.vdim + 1);
-  float* slow = sgate + pad4(a.vdim + 1);
-  float* sgin = slow + a.decay_ld;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane & (kLanes - 1);
-  const int C = a.vdim + extra_columns<KIND>(), d4 = pad4(a.dim), h = blockIdx.x, hk = h / (a.heads / a.kv_heads);
+  float* sgate = so + pad4(per + 1);
+  float* sv = sgate + pad4(per + 1);
+  float* slow = sv + pad4(per + 1);
+  float* sgin = slow + decay_ld;
+  __nv_bfloat16* wdecay = reinterpret_cast<__nv_bfloat16*>(sgin + gate_ld);
+  __nv_bfloat16* wgate = wdecay + (KIND == kStateNormalized ? 0 : a.dim * decay_ld);
+  const __nv_bfloat16* gdecay = KIND == kStateNormalized ? nullptr : a.decay_w + (long long)h * a.dim * decay_ld;
+  const __nv_bfloat16* ggate = a.gate_w ? a.gate_w + ((long long)h * a.vdim + c_lo) * gate_ld : nullptr;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & (kLanes - 1);
+  const int C = a.vdim + extra_columns<KIND>(), d4 = pad4(a.dim);
+  if (staged) {
+    if (KIND != kStateNormalized) stage_weights(wdecay, gdecay, a.dim * decay_ld);
+    if (a.gate_w) stage_weights(wgate, ggate, own * gate_ld);
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
   const int pos = *reinterpret_cast<const volatile int*>(a.pos0);
   const int slot = state_slot(a.tags, pos, a.status);
   const float* old = a.state + max(slot, 0) * a.state_stride + (long long)h * C * d4;
   float* now = a.state + (1 - max(slot, 0)) * a.state_stride + (long long)h * C * d4;
-  auto load = [&](int c, u64 (&s)[2 * NV]) {
+  // local column j: value column c_lo + j, then the normaliser
+  auto load = [&](int j, u64 (&s)[2 * NV]) {
+    const long long at = (long long)(j < own ? c_lo + j : a.vdim) * d4;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int e = (l + kLanes * i) * 4;
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (c < C && pos > 0 && e < d4) v = __ldcg(reinterpret_cast<const float4*>(old + (long long)c * d4 + e));
+      if (j < cols && pos > 0 && e < d4) v = __ldcg(reinterpret_cast<const float4*>(old + at + e));
       s[2 * i] = pack2(v.x, v.y);
       s[2 * i + 1] = pack2(v.z, v.w);
     }
   };
   u64 first[AHEAD][2 * NV];
 #pragma unroll
-  for (int j = 0; j < AHEAD; ++j) load(threadIdx.x / kLanes + j * kStepCols, first[j]);
+  for (int j = 0; j < AHEAD; ++j) load(tid / kLanes + j * kStepCols, first[j]);
+  float d_bias = 0.f, d_rate = 0.f;            // of this thread's first decay
+  if (KIND != kStateNormalized && tid < a.dim) {
+    d_bias = bf(a.decay_b + (long long)h * a.dim + tid);
+    if (a.rate) d_rate = __ldg(a.rate + (long long)h * a.dim + tid);
+  }
   griddep_wait();
   griddep_launch();
-  if (slot < 0) return;
-  const float* p = a.proj;
-  for (int i = threadIdx.x; i < DP; i += kStepT) {
-    const bool in = i < a.dim;
-    sk[i] = in ? __ldcg(p + a.k_off + hk * a.dim + i) : 0.f;
-    sq[i] = in ? __ldcg(p + a.q_off + hk * a.dim + i) : 0.f;
-    sg[i] = 0.f;
-  }
-  if (KIND != kStateNormalized)
-    for (int i = threadIdx.x; i < a.decay_ld; i += kStepT) {
-      const float z = i < a.low_rank ? __ldcg(p + a.low_off + i) : 0.f;
-      slow[i] = a.low_tanh ? tanhf(z) : z;
+  if (slot >= 0) {                                                       // (the same for every CTA of the cluster)
+    const float* p = a.proj;
+    for (int i = tid; i < DP; i += kStepT) {
+      const bool in = i < a.dim;
+      sk[i] = in ? __ldcg(p + a.k_off + hk * a.dim + i) : 0.f;
+      sq[i] = in ? __ldcg(p + a.q_off + hk * a.dim + i) : 0.f;
+      sg[i] = 0.f;
     }
-  if (a.gate_w)
-    for (int i = threadIdx.x; i < a.gate_ld; i += kStepT) sgin[i] = i < a.gate_rank ? __ldcg(p + a.gate_off + i) : 0.f;
-  __syncthreads();
-  if (KIND != kStateNormalized) {
-    const __nv_bfloat16* b = a.decay_b + (long long)h * a.dim;
-    const float* rate = a.rate ? a.rate + (long long)h * a.dim : nullptr;
-    low_rank_rows(a.decay_w + (long long)h * a.dim * a.decay_ld, a.decay_ld, a.dim, slow, warp, lane, [&](int d, float z) {
-      z += bf(b + d);
-      sg[d] = rate ? decay_soft(z, rate[d]) : decay_exp(z);
-    });
-  }
-  if (a.gate_w)
-    low_rank_rows(a.gate_w + (long long)h * a.vdim * a.gate_ld, a.gate_ld, a.vdim, sgin, warp, lane, [&](int j, float z) { sgate[j] = z; });
-  else
-    for (int j = threadIdx.x; j < a.vdim; j += kStepT) sgate[j] = __ldcg(p + a.gate_off + (long long)h * a.vdim + j);
-  float q_scale = a.q_scale;
-  if (a.unit) {
-    float qq = 0.f, kk = 0.f;
-    for (int i = lane; i < a.dim; i += 32) {
-      qq = fmaf(sq[i], sq[i], qq);
-      kk = fmaf(sk[i], sk[i], kk);
+    for (int j = tid; j < cols; j += kStepT) {
+      sv[j] = j < own ? __ldcg(p + a.v_off + (long long)h * a.vdim + c_lo + j) : 1.f;
+      if (!a.gate_w && j < own) sgate[j] = __ldcg(p + a.gate_off + (long long)h * a.vdim + c_lo + j);
     }
-    q_scale /= sqrtf(lane_sum(qq) + kUnitEps);
-    const float ks = 1.0f / sqrtf(lane_sum(kk) + kUnitEps);
-    __syncthreads();
-    for (int i = threadIdx.x; i < a.dim; i += kStepT) sk[i] *= ks;
-  }
-  float s0 = 0.f, s1 = 0.f, floor_n = 0.f, m_new = 0.f;
-  if (KIND == kStateDelta) s0 = sigmoid_f(__ldcg(p + a.beta_off + h));
-  if (KIND == kStateNormalized) {
-    const float zi = log_input(__ldcg(p + a.gi_off + h), a.cap), zf = log_forget(__ldcg(p + a.gf_off + h), a.cap);
-    const long long m_at = (long long)(a.heads - h) * C * d4 + h;        // the maxima follow the last head's state
-    const float m = pos > 0 ? __ldcg(old + m_at) : 0.f;
-    m_new = fmaxf(zf + m, zi);
-    s0 = expf(zf + m - m_new);
-    s1 = expf(zi - m_new);
-    floor_n = expf(-m_new);
-    if (threadIdx.x == 0) now[m_at] = m_new;
-  }
-  if (KIND == kStateBonus) {
-    for (int i = lane; i < a.dim; i += 32) s0 = fmaf(sq[i] * bf(a.u + (long long)h * a.dim + i), sk[i], s0);
-    s0 = lane_sum(s0);
-  }
-  __syncthreads();
-  const ulonglong2* q = reinterpret_cast<const ulonglong2*>(sq) + l;
-  const ulonglong2* k = reinterpret_cast<const ulonglong2*>(sk) + l;
-  const ulonglong2* g = reinterpret_cast<const ulonglong2*>(sg) + l;
-  auto column = [&](int c, u64 (&s)[2 * NV]) {
-    const float v = c < a.vdim ? __ldcg(p + a.v_off + (long long)h * a.vdim + c) : c < C ? 1.f : 0.f;
-    float r = column_sum(column_step<KIND, NV>(s, q, k, g, v, s0, s1));
-    if (KIND == kStateBonus) r = fmaf(s0, v, r);
-    if (c < C) {
-#pragma unroll
-      for (int i = 0; i < NV; ++i) {
-        const int e = (l + kLanes * i) * 4;
-        if (e < d4) *reinterpret_cast<ulonglong2*>(now + (long long)c * d4 + e) = make_ulonglong2(s[2 * i], s[2 * i + 1]);
+    if (KIND != kStateNormalized)
+      for (int i = tid; i < decay_ld; i += kStepT) {
+        const float z = i < a.low_rank ? __ldcg(p + a.low_off + i) : 0.f;
+        slow[i] = a.low_tanh ? tanhf(z) : z;
       }
-      if (l == 0) so[c] = r * q_scale;
+    if (a.gate_w)
+      for (int i = tid; i < gate_ld; i += kStepT) sgin[i] = i < a.gate_rank ? __ldcg(p + a.gate_off + i) : 0.f;
+    float s0 = 0.f, s1 = 0.f, floor_n = 0.f;
+    if (KIND == kStateDelta) s0 = sigmoid_f(__ldcg(p + a.beta_off + h));
+    if (KIND == kStateNormalized) {
+      const float zi = log_input(__ldcg(p + a.gi_off + h), a.cap), zf = log_forget(__ldcg(p + a.gf_off + h), a.cap);
+      const long long m_at = (long long)(a.heads - h) * C * d4 + h;      // the maxima follow the last head's state
+      const float m = pos > 0 ? __ldcg(old + m_at) : 0.f, m_new = fmaxf(zf + m, zi);
+      s0 = expf(zf + m - m_new);
+      s1 = expf(zi - m_new);
+      floor_n = expf(-m_new);
+      if (rank == 0 && tid == 0) now[m_at] = m_new;
     }
-  };
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (KIND != kStateNormalized) {
+      auto store = [&](int d, float z) { sg[d] = z; };
+      if (staged) low_rank_rows<true>(wdecay, decay_ld, a.dim, slow, warp, lane, store);
+      else low_rank_rows<false>(gdecay, decay_ld, a.dim, slow, warp, lane, store);
+    }
+    if (a.gate_w) {
+      auto store = [&](int j, float z) { sgate[j] = z; };
+      if (staged) low_rank_rows<true>(wgate, gate_ld, own, sgin, warp, lane, store);
+      else low_rank_rows<false>(ggate, gate_ld, own, sgin, warp, lane, store);
+    }
+    float q_scale = a.q_scale;
+    if (a.unit) {
+      float qq = 0.f, kk = 0.f;
+      for (int i = lane; i < a.dim; i += 32) {
+        qq = fmaf(sq[i], sq[i], qq);
+        kk = fmaf(sk[i], sk[i], kk);
+      }
+      q_scale /= sqrtf(lane_sum(qq) + kUnitEps);
+      const float ks = 1.0f / sqrtf(lane_sum(kk) + kUnitEps);
+      __syncthreads();
+      for (int i = tid; i < a.dim; i += kStepT) sk[i] *= ks;
+    } else if (KIND != kStateNormalized) {
+      __syncthreads();
+    }
+    if (KIND != kStateNormalized)
+      for (int d = tid, e = 0; d < a.dim; d += kStepT, ++e) {
+        const float z = sg[d] + (e == 0 ? d_bias : bf(a.decay_b + (long long)h * a.dim + d));
+        sg[d] = a.rate ? decay_soft(z, e == 0 ? d_rate : a.rate[(long long)h * a.dim + d]) : decay_exp(z);
+      }
+    if (KIND == kStateBonus) {
+      for (int i = lane; i < a.dim; i += 32) s0 = fmaf(sq[i] * bf(a.u + (long long)h * a.dim + i), sk[i], s0);
+      s0 = lane_sum(s0);
+    }
+    __syncthreads();
+    const ulonglong2* q = reinterpret_cast<const ulonglong2*>(sq) + l;
+    const ulonglong2* k = reinterpret_cast<const ulonglong2*>(sk) + l;
+    const ulonglong2* g = reinterpret_cast<const ulonglong2*>(sg) + l;
+    auto column = [&](int j, u64 (&s)[2 * NV]) {
+      const float v = j < cols ? sv[j] : 0.f;
+      float r = column_sum(column_step<KIND, NV>(s, q, k, g, v, s0, s1));
+      if (KIND == kStateBonus) r = fmaf(s0, v, r);
+      if (j < cols) {
+        if (j < own || rank == 0) {
+          const long long at = (long long)(j < own ? c_lo + j : a.vdim) * d4;
 #pragma unroll
-  for (int j = 0; j < AHEAD; ++j) column(threadIdx.x / kLanes + j * kStepCols, first[j]);
-  for (int cb = AHEAD * kStepCols; cb < C; cb += kStepCols) {            // (the same trip count for every lane of a warp)
-    u64 s[2 * NV];
-    load(cb + threadIdx.x / kLanes, s);
-    column(cb + threadIdx.x / kLanes, s);
+          for (int i = 0; i < NV; ++i) {
+            const int e = (l + kLanes * i) * 4;
+            if (e < d4) *reinterpret_cast<ulonglong2*>(now + at + e) = make_ulonglong2(s[2 * i], s[2 * i + 1]);
+          }
+        }
+        if (l == 0) so[j] = r * q_scale;
+      }
+    };
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j) column(tid / kLanes + j * kStepCols, first[j]);
+    for (int jb = AHEAD * kStepCols; jb < cols; jb += kStepCols) {       // (the same trip count for every lane of a warp)
+      u64 s[2 * NV];
+      load(jb + tid / kLanes, s);
+      column(jb + tid / kLanes, s);
+    }
+    __syncthreads();
+    const float inv = KIND == kStateNormalized ? 1.0f / (fmaxf(fabsf(so[own]), floor_n) + 1e-6f) : 1.f;
+    float ss = 0.f;
+    for (int j = tid; j < own; j += kStepT) {
+      so[j] *= inv;
+      ss = fmaf(so[j], so[j], ss);
+    }
+    ss = block_sum_f(ss, red);
+    if (tid == 0) part = ss;
   }
-  __syncthreads();
-  const float inv = KIND == kStateNormalized ? 1.0f / (fmaxf(fabsf(so[a.vdim]), floor_n) + 1e-6f) : 1.f;
-  float ss = 0.f;
-  for (int j = threadIdx.x; j < a.vdim; j += kStepT) {
-    const float v = so[j] * inv;
-    ss = fmaf(v, v, ss);
+  cluster_sync_all();
+  if (slot >= 0) {
+    float ss = 0.f;
+    for (int i = 0; i < (int)gridDim.x; ++i) ss += ld_cluster_f32(&part, i);
+    const float rs = 1.0f / sqrtf(ss / (float)a.vdim + a.eps);
+    const __nv_bfloat16* w = a.norm + (a.norm_per_head ? (long long)h * a.vdim : 0) + c_lo;
+    for (int j = tid; j < own; j += kStepT)
+      a.out[(long long)h * a.vdim + c_lo + j] = so[j] * rs * bf(w + j) * (a.gate_kind == kGateSilu ? silu_f(sgate[j]) : sigmoid_f(sgate[j]));
+    // A CTA that starts after this store still finds `pos` in its own slot: only the other slot's tag changes.
+    if (rank == 0 && h == 0 && tid == 0) {
+      a.tags[1 - slot] = pos + 1;
+      if (pos == 0) a.tags[1] = -1;
+    }
   }
-  const float rs = inv / sqrtf(block_sum_f(ss, red) / (float)a.vdim + a.eps);
-  const __nv_bfloat16* w = a.norm + (a.norm_per_head ? (long long)h * a.vdim : 0);
-  for (int j = threadIdx.x; j < a.vdim; j += kStepT)
-    a.out[(long long)h * a.vdim + j] = so[j] * rs * bf(w + j) * (a.gate_kind == kGateSilu ? silu_f(sgate[j]) : sigmoid_f(sgate[j]));
-  // A CTA that starts after this store still finds `pos` in its own slot: only the other slot's tag changes.
-  if (blockIdx.x == 0 && threadIdx.x == 0) {
-    a.tags[1 - slot] = pos + 1;
-    if (pos == 0) a.tags[1] = -1;
-  }
+  cluster_sync_all();                                                    // nobody leaves while its sum is read
 }
 
 constexpr int kMaxSmem = 220 * 1024;
@@ -537,26 +833,44 @@ int allow_smem(K kern, bool& done) {
   return (int)e;
 }
 
-template <int KIND, int NV>
+template <int KIND, int L, int NV>
 int launch_chunk(const StateChunkArgs& a, cudaStream_t stream) {
   static bool configured = false;
-  if (const int rc = allow_smem(state_chunk_kernel<KIND, NV>, configured)) return rc;
+  if (const int rc = allow_smem(state_chunk_kernel<KIND, L, NV>, configured)) return rc;
+  constexpr int PER_WARP = 32 / L * kQuad;
   const int C = a.vdim + extra_columns<KIND>();
-  int warps = 8;
-  while (warps > 2 && a.heads * ((C + warps * 4 - 1) / (warps * 4)) < 100) warps /= 2;
-  const int cols = warps * 4;
-  int tokens = 32;
-  while (tokens > 4 && 8 * chunk_stage_floats(KIND, NV * 4 * kLanes, cols, tokens) > 110 * 1024) tokens /= 2;
-  const int smem = 8 * chunk_stage_floats(KIND, NV * 4 * kLanes, cols, tokens);
-  return launch_pdl(state_chunk_kernel<KIND, NV>, dim3((C + cols - 1) / cols, a.heads), dim3(warps * 32), smem, stream, false, a, tokens);
+  int warps = 8;                               // as few as it takes to give most SMs a CTA
+  while (warps > 1 && a.heads * ((C + warps * PER_WARP - 1) / (warps * PER_WARP)) < 100) warps /= 2;
+  const int cols = warps * PER_WARP, blocks = (a.rows + kStateBlock - 1) / kStateBlock;
+  if (KIND == kStateNormalized) {
+    if (const int rc = launch_pdl(gate_scan_kernel, dim3(a.heads), dim3(kScanT), 0, stream, false, a)) return rc;
+  }
+  constexpr int NC = NV * 4 * L / 32 < 4 ? NV * 4 * L / 32 : 4;
+  if (const int rc = launch_pdl(state_blocks_kernel<KIND, NC>, dim3(blocks, (a.heads + 3) / 4), dim3(128), 0, stream, false, a)) return rc;
+  const int smem = 4 * (kStages * (state_record(KIND, a.dim) + kStateBlock * cols) + warps * (32 / L) * 2 * kStateBlock * kQuad);
+  if (smem > kMaxSmem) return -7;
+  return launch_pdl(state_chunk_kernel<KIND, L, NV>, dim3((C + cols - 1) / cols, a.heads), dim3(warps * 32), smem, stream, false, a);
+}
+template <int KIND>
+int chunk_by_dim(const StateChunkArgs& a, cudaStream_t stream) {         // L * NV * 4 = state_row(dim)
+  if (a.dim <= 32) return launch_chunk<KIND, 8, 1>(a, stream);
+  if (a.dim <= 64) return launch_chunk<KIND, 16, 1>(a, stream);
+  if (a.dim <= 128) return launch_chunk<KIND, 16, 2>(a, stream);
+  if (a.dim <= 256) return launch_chunk<KIND, 16, 4>(a, stream);
+  return launch_chunk<KIND, 32, 4>(a, stream);
 }
 template <int KIND, int NV>
 int launch_state_step(const StateStepArgs& a, cudaStream_t stream, bool pdl) {
   static bool configured = false;
   if (const int rc = allow_smem(state_step_kernel<KIND, NV>, configured)) return rc;
-  const int smem = 4 * step_floats(NV * 4 * kLanes, a.vdim, (int)a.decay_ld, (int)a.gate_ld);
-  if (smem > kMaxSmem) return -7;
-  return launch_pdl(state_step_kernel<KIND, NV>, dim3(a.heads), dim3(kStepT), smem, stream, pdl, a);
+  int ctas = 1;                                // per head: a cluster, while that fits the SMs and leaves 16 columns each
+  while (ctas < 8 && a.heads * ctas * 2 <= 148 && a.vdim >= 32 * ctas) ctas *= 2;
+  const int per = (a.vdim + ctas - 1) / ctas;
+  const int base = 4 * step_floats(NV * 4 * kLanes, per, (int)a.decay_ld, (int)a.gate_ld);
+  const int weights = 2 * (int)((KIND == kStateNormalized ? 0 : a.dim * a.decay_ld) + (a.gate_w ? per * a.gate_ld : 0));
+  const bool staged = base + weights <= kMaxSmem;
+  if (base > kMaxSmem) return -7;
+  return launch_cluster(state_step_kernel<KIND, NV>, dim3(ctas, a.heads), dim3(kStepT), dim3(ctas, 1, 1), base + (staged ? weights : 0), stream, pdl, a, per, (int)staged);
 }
 
 bool sizes_ok(int heads, int kv_heads, int dim, int vdim) {
@@ -578,17 +892,18 @@ extern "C" int nrt_state_chunk_args_size() { return (int)sizeof(StateChunkArgs);
 extern "C" int nrt_short_conv_args_size() { return (int)sizeof(ShortConvArgs); }
 extern "C" int nrt_token_mix_args_size() { return (int)sizeof(TokenMixArgs); }
 extern "C" int nrt_head_gate_args_size() { return (int)sizeof(HeadGateArgs); }
+extern "C" int nrt_state_block_floats(int kind, int dim) { return state_record(kind, dim); }       // per (block, head)
 extern "C" int nrt_state_step_args_size() { return (int)sizeof(StateStepArgs); }
 
 extern "C" int nrt_state_chunk(int kind, const void* args, void* stream) {
   StateChunkArgs a;
   memcpy(&a, args, sizeof(a));
-  if (a.rows < 1 || !sizes_ok(a.heads, a.kv_heads, a.dim, a.vdim) || a.state_stride % 4) return -3;
+  if (a.rows < 1 || !sizes_ok(a.heads, a.kv_heads, a.dim, a.vdim) || a.state_stride % 4 || !a.blocks) return -3;
   if (a.history && (a.hist_rows < 1 || a.hist_rows < 2 * (a.taps - 1))) return -3;
-  if ((kind != kStateNormalized && !a.g) || (kind == kStateNormalized && (!a.gi || !a.gf || !a.den)) || (kind == kStateDelta && !a.beta) || (kind == kStateBonus && !a.u)) return -3;
-  if (kind == kStateDelta) { NRT_BY_DIM(launch_chunk, kStateDelta, a.dim, a, S(stream)) }
-  if (kind == kStateBonus) { NRT_BY_DIM(launch_chunk, kStateBonus, a.dim, a, S(stream)) }
-  if (kind == kStateNormalized) { NRT_BY_DIM(launch_chunk, kStateNormalized, a.dim, a, S(stream)) }
+  if ((kind != kStateNormalized && !a.g) || (kind == kStateNormalized && (!a.gi || !a.gf || !a.den || !a.keep)) || (kind == kStateDelta && !a.beta) || (kind == kStateBonus && !a.u)) return -3;
+  if (kind == kStateDelta) return chunk_by_dim<kStateDelta>(a, S(stream));
+  if (kind == kStateBonus) return chunk_by_dim<kStateBonus>(a, S(stream));
+  if (kind == kStateNormalized) return chunk_by_dim<kStateNormalized>(a, S(stream));
   return -2;
 }
 

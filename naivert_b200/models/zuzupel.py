@@ -199,7 +199,7 @@ def bench_spec(layers: int = 6) -> StackSpec:
     """Layers of a real model's size (random weights): the three mixers in turn at width 4096."""
     delta = DeltaStateSpec(heads=32, kv_heads=32, dim=128, vdim=128, taps=4, decay_rank=128, gate_rank=128)
     wkv = BonusStateSpec(heads=64, dim=64, decay_rank=128)
-    both = ParallelSpec(GroupedAttentionSpec(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, rotary=RotarySpec(128, 500000.0, 8.0), window=8192),
+    both = ParallelSpec(GroupedAttentionSpec(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, rotary=RotarySpec(128, 500000.0, 8.0), window=16384),
                         NormalizedStateSpec(heads=16, dim=128, vdim=256, cap=15.0))
     ff = SquaredReluSpec(ff=16384)
     return StackSpec(name=f"zuzupel-bench-L{layers}", architecture=ARCHITECTURE, hidden=4096, vocab=152576,

@@ -153,6 +153,14 @@ def state_chunk(kind: int, args: StateChunkArgs) -> None:
     K.check(lib().nrt_state_chunk(kind, C.byref(args), _stream()), "matrix-state recurrence (chunk)")
 
 
+STATE_BLOCK = 8                                       # tokens per block record of the chunk recurrence
+
+
+def state_block_floats(kind: int, dim: int) -> int:
+    """Scratch floats of the chunk recurrence per (block of tokens, head)."""
+    return lib().nrt_state_block_floats(kind, dim)
+
+
 def state_step(args: StateStepArgs, pdl: bool) -> None:
     K.check(lib().nrt_state_step(C.byref(args), _stream(), int(pdl)), "matrix-state recurrence (step)")
 
