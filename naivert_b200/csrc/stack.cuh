@@ -213,6 +213,7 @@ enum GateKind : int { kGateSigmoid = 0, kGateSilu = 1 };
 // padded with zeros to state_row(dim).  Then 64 pair coefficients, element [t][s]: s <= t: weight of token s's update in the
 // read-out of token t; s > t: what token t's update adds to S^T k at token s (delta).  Then the step sizes (delta).
 constexpr int kStateBlock = 8;
+constexpr int kStatePieces = 8;      // parts of a chunk that the recurrences without S^T k work off side by side
 __host__ __device__ inline int state_row(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : dim <= 256 ? 256 : 512; }
 __host__ __device__ inline int state_record(int kind, int dim) {
   return ((kind == kStateDelta ? 3 : 2) * kStateBlock + 1) * state_row(dim) + kStateBlock * kStateBlock + kStateBlock;
@@ -235,6 +236,8 @@ struct StateChunkArgs {
   float cap;
   float* keep;                  // normalized, scratch: [rows][heads][2] = factor on the state, factor on the new term
   float* blocks;                // scratch: [blocks][heads][state_record]
+  float* sums;                  // bonus, normalized, scratch: [kStatePieces - 1][heads][columns][dim4] states of a piece from zero, then
+                                // [kStatePieces - 1][heads][dim4] decays of a piece
   float* o;                     // [rows][heads * vdim]
   float* den;                   // normalized: [rows][heads][2] = n . q, exp(-m)
   float* state;                 // [2][state_stride]: heads x columns x dim4, then (normalized) the running maxima

@@ -170,7 +170,7 @@ __device__ __forceinline__ void scatter_sum(float (&v)[N], int l) {
 
 // One warp per (block, head); lane = key channels lane, lane + 32, ... of a slice.
 template <int KIND, int NC>
-__global__ void __launch_bounds__(128) state_blocks_kernel(const StateChunkArgs a) {
+__global__ void __launch_bounds__(128, 3) state_blocks_kernel(const StateChunkArgs a) {
   griddep_wait();
   griddep_launch();
   constexpr int B = kStateBlock;
@@ -198,15 +198,25 @@ __global__ void __launch_bounds__(128) state_blocks_kernel(const StateChunkArgs 
   for (int i = 0; i < B * B; ++i) w[i] = 0.f;
   for (int d0 = 0; d0 < dp; d0 += 32 * NC) {
     float q[B][NC], k[B][NC], g[B][NC];
+    // loads without conditions (clamped addresses), so that all of them are in flight together
 #pragma unroll
     for (int t = 0; t < B; ++t)
 #pragma unroll
       for (int i = 0; i < NC; ++i) {
-        const int d = d0 + lane + 32 * i;
-        const bool in = t < n && d < a.dim;
-        q[t][i] = in ? __ldg(a.q + (r0 + t) * a.q_ld + hk * a.dim + d) * a.q_scale : 0.f;
-        k[t][i] = in ? __ldg(a.k + (r0 + t) * a.k_ld + hk * a.dim + d) : 0.f;
-        g[t][i] = KIND == kStateNormalized ? keep[t] : in ? __ldg(a.g + (r0 + t) * a.g_ld + h * a.dim + d) : 1.f;
+        const int d = min(d0 + lane + 32 * i, a.dim - 1);
+        const long long r = min(r0 + t, a.rows - 1);
+        q[t][i] = __ldg(a.q + r * a.q_ld + hk * a.dim + d);
+        k[t][i] = __ldg(a.k + r * a.k_ld + hk * a.dim + d);
+        g[t][i] = KIND == kStateNormalized ? keep[t] : __ldg(a.g + r * a.g_ld + h * a.dim + d);
+      }
+#pragma unroll
+    for (int t = 0; t < B; ++t)
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+        const bool in = t < n && d0 + lane + 32 * i < a.dim;
+        q[t][i] = in ? q[t][i] * a.q_scale : 0.f;
+        k[t][i] = in ? k[t][i] : 0.f;
+        if (KIND != kStateNormalized && !in) g[t][i] = 1.f;
       }
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
@@ -247,7 +257,9 @@ __global__ void __launch_bounds__(128) state_blocks_kernel(const StateChunkArgs 
 }
 
 // ------------------------------------------------------------------------------------ chunk path: the recurrence
-// grid (column tiles, heads); a warp holds 4 * 32 / L columns; records and values arrive three stages deep, the records as one bulk copy.
+// grid (column tiles, heads, pieces); a warp holds 4 * 32 / L columns; records and values arrive three stages deep, the records as one
+// bulk copy.  Recurrences that are linear in the state are cut into pieces of the chunk: a first launch (SUMS) leaves each piece's end
+// state from zero and its decay, the second starts every piece from the carried state and the earlier pieces' sums.
 constexpr int kQuad = 4, kStages = 3;
 
 template <int L, int NV>
@@ -256,23 +268,29 @@ __device__ __forceinline__ void state_products(const u64 (&s)[kQuad][2 * NV], co
   constexpr int VPL = 32 / L;
   u64 acc[kStateBlock][kQuad];
 #pragma unroll
-  for (int t = 0; t < kStateBlock; ++t)
+  for (int i = 0; i < NV; ++i) {
+    ulonglong2 x[kStateBlock];
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      const ulonglong2 x = vec[t * (NV * L) + i * L];
+    for (int t = 0; t < kStateBlock; ++t) x[t] = vec[t * (NV * L) + i * L];
 #pragma unroll
-      for (int j = 0; j < kQuad; ++j) acc[t][j] = i == 0 ? mul2(s[j][0], x.x) : fma2(s[j][2 * i], x.x, acc[t][j]);
+    for (int t = 0; t < kStateBlock; ++t)
 #pragma unroll
-      for (int j = 0; j < kQuad; ++j) acc[t][j] = fma2(s[j][2 * i + 1], x.y, acc[t][j]);
-    }
+      for (int j = 0; j < kQuad; ++j) acc[t][j] = i == 0 ? mul2(s[j][0], x[t].x) : fma2(s[j][2 * i], x[t].x, acc[t][j]);
+#pragma unroll
+    for (int t = 0; t < kStateBlock; ++t)
+#pragma unroll
+      for (int j = 0; j < kQuad; ++j) acc[t][j] = fma2(s[j][2 * i + 1], x[t].y, acc[t][j]);
+  }
 #pragma unroll
   for (int v = 0; v < 32; ++v) out[v] = both(acc[(v / VPL >> 2) + L / 4 * (v % VPL)][v / VPL & 3]);
 }
 
-template <int KIND, int L, int NV>
-__global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArgs a) {
+template <int KIND, int L, int NV, bool SUMS>
+__global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArgs a, const int piece_blocks) {
   constexpr int B = kStateBlock, DP = NV * 4 * L, PER_WARP = 32 / L * kQuad, VPL = 32 / L;
-  constexpr int ROWS = (KIND == kStateDelta ? 3 : 2) * B, REC = (ROWS + 1) * DP + B * B + B;
+  constexpr int ROWS = (KIND == kStateDelta ? 3 : 2) * B, RECORD = (ROWS + 1) * DP + B * B + B;
+  constexpr int SKIP = SUMS ? (ROWS - B) * DP : 0, REC = SUMS ? (B + 1) * DP : RECORD;      // the part of a record that is read
+  constexpr int K2 = SUMS ? 0 : (ROWS - B) * DP, WHOLE = K2 + B * DP;
   extern __shared__ __align__(16) float sh[];
   __shared__ uint64_t full[kStages];
   griddep_wait();
@@ -294,9 +312,30 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
     for (int i = 0; i < NV; ++i) {
       ulonglong2 v = make_ulonglong2(0ull, 0ull);
       const int e = (l + L * i) * 4;
-      if (c + j < C && pos0 > 0 && e < d4) v = *reinterpret_cast<const ulonglong2*>(old + at + (long long)j * d4 + e);
+      if (!SUMS && c + j < C && pos0 > 0 && e < d4) v = *reinterpret_cast<const ulonglong2*>(old + at + (long long)j * d4 + e);
       s[j][2 * i] = v.x;
       s[j][2 * i + 1] = v.y;
+    }
+  const int piece = blockIdx.z;
+  float* decays = a.sums + (long long)(kStatePieces - 1) * a.heads * C * d4;
+  u64 kept[2 * NV];                            // SUMS: the piece's decay so far
+#pragma unroll
+  for (int i = 0; i < 2 * NV; ++i) kept[i] = pack2(1.f, 1.f);
+  if (!SUMS && KIND != kStateDelta)
+    for (int z = 0; z < piece; ++z) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int e = (l + L * i) * 4;
+        if (e >= d4) continue;
+        const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(decays + ((long long)z * a.heads + h) * d4 + e);
+#pragma unroll
+        for (int j = 0; j < kQuad; ++j)
+          if (c + j < C) {
+            const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(a.sums + (((long long)z * a.heads + h) * C + c + j) * d4 + e);
+            s[j][2 * i] = fma2(s[j][2 * i], g.x, v.x);
+            s[j][2 * i + 1] = fma2(s[j][2 * i + 1], g.y, v.y);
+          }
+      }
     }
 
   float* sv = sh + kStages * REC;                                        // [stages][B][cols]
@@ -310,7 +349,7 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
     mbar_fence_init();
   }
   __syncthreads();
-  const int blocks = (a.rows + B - 1) / B;
+  const int b0 = piece * piece_blocks, blocks = min((a.rows + B - 1) / B, b0 + piece_blocks);
   const float* v0 = a.v + (long long)h * a.vdim + c0;
   const int vcols = min(cols, a.vdim - c0);                              // (none in a tile that holds only the normaliser)
   const bool quads = vcols > 0 && ((reinterpret_cast<uintptr_t>(v0) & 15) | (uintptr_t)((a.v_ld | vcols) & 3)) == 0;
@@ -319,7 +358,7 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
     if (threadIdx.x == 0) {
       mbar_expect_tx(&full[st], REC * 4);
       asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                   ::"r"(smem_u32(sh + st * REC)), "l"(a.blocks + ((long long)b * a.heads + h) * REC), "r"(REC * 4), "r"(smem_u32(&full[st]))
+                   ::"r"(smem_u32(sh + st * REC)), "l"(a.blocks + ((long long)b * a.heads + h) * RECORD + SKIP), "r"(REC * 4), "r"(smem_u32(&full[st]))
                    : "memory");
     }
     const int n = min(B, a.rows - b * B);
@@ -331,15 +370,15 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
       else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory");
     }
   };
-  request(0, 0);
+  if (b0 < blocks) request(b0, 0);
   asm volatile("cp.async.commit_group;" ::: "memory");
-  if (blocks > 1) request(1, 1);
+  if (b0 + 1 < blocks) request(b0 + 1, 1);
   asm volatile("cp.async.commit_group;" ::: "memory");
   const int col = l & 3, tq = l >> 2;                                    // this lane's column and first token among the reduced values
   bool ok = true;
-  for (int b = 0, st = 0; b < blocks; ++b, st = st + 1 == kStages ? 0 : st + 1) {
+  for (int b = b0, st = 0; b < blocks; ++b, st = st + 1 == kStages ? 0 : st + 1) {
     asm volatile("cp.async.wait_group 1;" ::: "memory");
-    ok = __syncthreads_and(mbar_wait(&full[st], (b / kStages) & 1, a.status, kSiteTmaFull | st));
+    ok = __syncthreads_and(mbar_wait(&full[st], ((b - b0) / kStages) & 1, a.status, kSiteTmaFull | st));
     if (!ok) break;
     if (b + 2 < blocks) request(b + 2, st + 2 >= kStages ? st + 2 - kStages : st + 2);       // (its last reader has passed the barrier)
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -354,8 +393,10 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
 #pragma unroll
       for (int i = 0; i < VPL; ++i) work[(tq + L / 4 * i) * kQuad + col] = p[i];
     }
-    state_products<L, NV>(s, vec + (KIND == kStateDelta ? B * DP / 4 : 0), q);
-    scatter_sum<32, L>(q, l);
+    if (!SUMS) {
+      state_products<L, NV>(s, vec + (KIND == kStateDelta ? B * DP / 4 : 0), q);
+      scatter_sum<32, L>(q, l);
+    }
     const float* upd = vc;                     // the tokens' updates of the group's columns, rows of `upd_ld`
     int upd_ld = cols;
     if (KIND == kStateDelta) {
@@ -369,8 +410,10 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
         for (int t = 0; t < B; ++t) {
           const float u = pairs[B * B + t] * r[t];
           us[t * kQuad + col] = u;
+          const float4 w0 = *reinterpret_cast<const float4*>(pairs + t * B), w1 = *reinterpret_cast<const float4*>(pairs + t * B + 4);
+          const float w[B] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
 #pragma unroll
-          for (int x = t + 1; x < B; ++x) r[x] = fmaf(-pairs[t * B + x], u, r[x]);
+          for (int x = t + 1; x < B; ++x) r[x] = fmaf(-w[x], u, r[x]);
         }
       }
       __syncwarp();
@@ -380,7 +423,11 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
     // the state moves on by the whole block
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const ulonglong2 g = vec[ROWS * DP / 4 + i * L];
+      const ulonglong2 g = vec[WHOLE / 4 + i * L];
+      if (SUMS) {
+        kept[2 * i] = mul2(kept[2 * i], g.x);
+        kept[2 * i + 1] = mul2(kept[2 * i + 1], g.y);
+      }
 #pragma unroll
       for (int j = 0; j < kQuad; ++j) {
         s[j][2 * i] = mul2(s[j][2 * i], g.x);
@@ -393,7 +440,7 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
       const u64 uu[kQuad] = {pack2(u.x, u.x), pack2(u.y, u.y), pack2(u.z, u.z), pack2(u.w, u.w)};
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        const ulonglong2 k = vec[(ROWS - B + t) * DP / 4 + i * L];
+        const ulonglong2 k = vec[(K2 + t * DP) / 4 + i * L];
 #pragma unroll
         for (int j = 0; j < kQuad; ++j) {
           s[j][2 * i] = fma2(k.x, uu[j], s[j][2 * i]);
@@ -401,13 +448,23 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
         }
       }
     }
+    if (SUMS) continue;
     // read-outs: this lane's column at its tokens
+    float uc[B];
+#pragma unroll
+    for (int e = 0; e < B; ++e) uc[e] = upd[e * upd_ld + col];
 #pragma unroll
     for (int i = 0; i < VPL; ++i) {
       const int t = tq + L / 4 * i;
-      float x = q[i];
+      const float4 w0 = *reinterpret_cast<const float4*>(pairs + t * B), w1 = *reinterpret_cast<const float4*>(pairs + t * B + 4);
+      const float w[B] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+      float x = q[i], x1 = 0.f;
 #pragma unroll
-      for (int e = 0; e < B; ++e) x = fmaf(e <= t ? pairs[t * B + e] : 0.f, upd[e * upd_ld + col], x);
+      for (int e = 0; e < B; e += 2) {
+        x = fmaf(e <= t ? w[e] : 0.f, uc[e], x);
+        x1 = fmaf(e + 1 <= t ? w[e + 1] : 0.f, uc[e + 1], x1);
+      }
+      x += x1;
       const int r = b * B + t;
       if (r < a.rows) {
         if (c + col < a.vdim) a.o[((long long)r * a.heads + h) * a.vdim + c + col] = x;
@@ -421,13 +478,19 @@ __global__ void __launch_bounds__(256, 1) state_chunk_kernel(const StateChunkArg
     drain_on_error(a.status);
     return;
   }
+  if (!SUMS && piece != (int)gridDim.z - 1) return;
+  float* end = SUMS ? a.sums + ((long long)piece * a.heads + h) * C * d4 + (long long)c * d4 : now + at;
 #pragma unroll
-  for (int j = 0; j < kQuad; ++j)
+  for (int i = 0; i < NV; ++i) {
+    const int e = (l + L * i) * 4;
+    if (e >= d4) continue;
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      const int e = (l + L * i) * 4;
-      if (c + j < C && e < d4) *reinterpret_cast<ulonglong2*>(now + at + (long long)j * d4 + e) = make_ulonglong2(s[j][2 * i], s[j][2 * i + 1]);
-    }
+    for (int j = 0; j < kQuad; ++j)
+      if (c + j < C) *reinterpret_cast<ulonglong2*>(end + (long long)j * d4 + e) = make_ulonglong2(s[j][2 * i], s[j][2 * i + 1]);
+    if (SUMS && blockIdx.x == 0 && threadIdx.x < L)
+      *reinterpret_cast<ulonglong2*>(decays + ((long long)piece * a.heads + h) * d4 + e) = make_ulonglong2(kept[2 * i], kept[2 * i + 1]);
+  }
+  if (SUMS) return;
   if (a.history) {
     const int keep = min(a.taps - 1, a.rows), ctas = gridDim.x * gridDim.y, cta = blockIdx.y * gridDim.x + blockIdx.x;
     for (int i = cta * blockDim.x + threadIdx.x; i < keep * a.hist_cols; i += ctas * blockDim.x) {
@@ -836,26 +899,45 @@ int allow_smem(K kern, bool& done) {
 template <int KIND, int L, int NV>
 int launch_chunk(const StateChunkArgs& a, cudaStream_t stream) {
   static bool configured = false;
-  if (const int rc = allow_smem(state_chunk_kernel<KIND, L, NV>, configured)) return rc;
+  if (const int rc = allow_smem(state_chunk_kernel<KIND, L, NV, false>, configured)) return rc;
   constexpr int PER_WARP = 32 / L * kQuad;
   const int C = a.vdim + extra_columns<KIND>();
   int warps = 8;                               // as few as it takes to give most SMs a CTA
   while (warps > 1 && a.heads * ((C + warps * PER_WARP - 1) / (warps * PER_WARP)) < 100) warps /= 2;
   const int cols = warps * PER_WARP, blocks = (a.rows + kStateBlock - 1) / kStateBlock;
+  int pieces = KIND == kStateDelta || blocks < 16 ? 1 : blocks / 8 < kStatePieces ? blocks / 8 : kStatePieces;
+  const int per = (blocks + pieces - 1) / pieces;
+  pieces = (blocks + per - 1) / per;
   if (KIND == kStateNormalized) {
     if (const int rc = launch_pdl(gate_scan_kernel, dim3(a.heads), dim3(kScanT), 0, stream, false, a)) return rc;
   }
-  constexpr int NC = NV * 4 * L / 32 < 4 ? NV * 4 * L / 32 : 4;
+  constexpr int NC = NV * 4 * L / 32 < 2 ? 1 : 2;                        // wider slices cost occupancy
   if (const int rc = launch_pdl(state_blocks_kernel<KIND, NC>, dim3(blocks, (a.heads + 3) / 4), dim3(128), 0, stream, false, a)) return rc;
+  const dim3 grid((C + cols - 1) / cols, a.heads, pieces);
   const int smem = 4 * (kStages * (state_record(KIND, a.dim) + kStateBlock * cols) + warps * (32 / L) * 2 * kStateBlock * kQuad);
   if (smem > kMaxSmem) return -7;
-  return launch_pdl(state_chunk_kernel<KIND, L, NV>, dim3((C + cols - 1) / cols, a.heads), dim3(warps * 32), smem, stream, false, a);
+  if constexpr (KIND != kStateDelta) {
+    if (pieces > 1) {
+      static bool sums_configured = false;
+      if (const int rc = allow_smem(state_chunk_kernel<KIND, L, NV, true>, sums_configured)) return rc;
+      const int rc = launch_pdl(state_chunk_kernel<KIND, L, NV, true>, dim3(grid.x, grid.y, pieces - 1), dim3(warps * 32), smem, stream, false, a, per);
+      if (rc) return rc;
+    }
+  }
+  return launch_pdl(state_chunk_kernel<KIND, L, NV, false>, grid, dim3(warps * 32), smem, stream, false, a, per);
 }
+// L * NV * 4 = state_row(dim).  Fewer lanes per column mean fewer reductions but also fewer warps: the delta rule, which has no pieces
+// to spread, takes more lanes.
 template <int KIND>
-int chunk_by_dim(const StateChunkArgs& a, cudaStream_t stream) {         // L * NV * 4 = state_row(dim)
+int chunk_by_dim(const StateChunkArgs& a, cudaStream_t stream) {
   if (a.dim <= 32) return launch_chunk<KIND, 8, 1>(a, stream);
-  if (a.dim <= 64) return launch_chunk<KIND, 16, 1>(a, stream);
-  if (a.dim <= 128) return launch_chunk<KIND, 16, 2>(a, stream);
+  if constexpr (KIND == kStateDelta) {
+    if (a.dim <= 64) return launch_chunk<KIND, 16, 1>(a, stream);
+    if (a.dim <= 128) return launch_chunk<KIND, 16, 2>(a, stream);
+  } else {
+    if (a.dim <= 64) return launch_chunk<KIND, 8, 2>(a, stream);
+    if (a.dim <= 128) return launch_chunk<KIND, 8, 4>(a, stream);
+  }
   if (a.dim <= 256) return launch_chunk<KIND, 16, 4>(a, stream);
   return launch_chunk<KIND, 32, 4>(a, stream);
 }
@@ -893,12 +975,15 @@ extern "C" int nrt_short_conv_args_size() { return (int)sizeof(ShortConvArgs); }
 extern "C" int nrt_token_mix_args_size() { return (int)sizeof(TokenMixArgs); }
 extern "C" int nrt_head_gate_args_size() { return (int)sizeof(HeadGateArgs); }
 extern "C" int nrt_state_block_floats(int kind, int dim) { return state_record(kind, dim); }       // per (block, head)
+extern "C" long long nrt_state_sum_floats(int kind, int heads, int dim, int vdim) {
+  return kind == kStateDelta ? 0 : (long long)(kStatePieces - 1) * heads * (vdim + (kind == kStateNormalized) + 1) * pad4(dim);
+}
 extern "C" int nrt_state_step_args_size() { return (int)sizeof(StateStepArgs); }
 
 extern "C" int nrt_state_chunk(int kind, const void* args, void* stream) {
   StateChunkArgs a;
   memcpy(&a, args, sizeof(a));
-  if (a.rows < 1 || !sizes_ok(a.heads, a.kv_heads, a.dim, a.vdim) || a.state_stride % 4 || !a.blocks) return -3;
+  if (a.rows < 1 || !sizes_ok(a.heads, a.kv_heads, a.dim, a.vdim) || a.state_stride % 4 || !a.blocks || (kind != kStateDelta && !a.sums)) return -3;
   if (a.history && (a.hist_rows < 1 || a.hist_rows < 2 * (a.taps - 1))) return -3;
   if ((kind != kStateNormalized && !a.g) || (kind == kStateNormalized && (!a.gi || !a.gf || !a.den || !a.keep)) || (kind == kStateDelta && !a.beta) || (kind == kStateBonus && !a.u)) return -3;
   if (kind == kStateDelta) return chunk_by_dim<kStateDelta>(a, S(stream));

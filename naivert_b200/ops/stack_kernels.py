@@ -161,6 +161,13 @@ def state_block_floats(kind: int, dim: int) -> int:
     return lib().nrt_state_block_floats(kind, dim)
 
 
+def state_sum_floats(kind: int, heads: int, dim: int, vdim: int) -> int:
+    """Scratch floats of the chunk recurrence for the pieces' sums."""
+    f = lib().nrt_state_sum_floats
+    f.restype = C.c_longlong
+    return f(kind, heads, dim, vdim)
+
+
 def state_step(args: StateStepArgs, pdl: bool) -> None:
     K.check(lib().nrt_state_step(C.byref(args), _stream(), int(pdl)), "matrix-state recurrence (step)")
 

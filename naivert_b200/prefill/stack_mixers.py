@@ -150,13 +150,14 @@ class GatedRecurrence:
 
 
 # --------------------------------------------------------------------------- matrix states
-def blocks(pf, m, kind: int) -> Tuple[int, torch.dtype]:
-    return -(-pf.C // S.STATE_BLOCK) * m.heads * S.state_block_floats(kind, m.dim), F32
+def state_scratch(pf, m, kind: int) -> Scratch:
+    return {"blocks": (-(-pf.C // S.STATE_BLOCK) * m.heads * S.state_block_floats(kind, m.dim), F32),
+            "sums": (S.state_sum_floats(kind, m.heads, m.dim, m.vdim), F32)}
 
 
 def state_args(pf, r: dict, m, R: int, o: torch.Tensor) -> "S.StateChunkArgs":
     a = S.StateChunkArgs()
-    a.blocks = pf.buf["blocks"].data_ptr()
+    a.blocks, a.sums = pf.buf["blocks"].data_ptr(), pf.buf["sums"].data_ptr()
     a.rows, a.heads, a.kv_heads, a.dim, a.vdim, a.q_scale = R, m.heads, getattr(m, "kv_heads", m.heads), m.dim, m.vdim, 1.0
     a.o, a.state, a.state_stride, a.tags = o.data_ptr(), r["state"].data_ptr(), r["state"].shape[1], r["tags"].data_ptr()
     a.pos0, a.status = pf.pos.data_ptr(), pf.t.fab.status.data_ptr()
@@ -189,7 +190,7 @@ class DeltaState:
         C, qk, hd, hv = pf.C, m.kv_heads * m.dim, m.heads * m.dim, m.heads * m.vdim
         return {"proj": (C * pad(d["in"].n, 4), F32), "sq": (C * qk, F32), "sk": (C * qk, F32), "sv": (C * hv, F32), "low": (C * DeltaState.low_ld(m), pf.act),
                 "decay": (C * hd, F32), "sgate": (C * hv, F32), "so": (C * hv, F32), "o": (C * pad(hv, 8), pf.act),
-                "blocks": blocks(pf, m, S.STATE_DELTA)}
+                **state_scratch(pf, m, S.STATE_DELTA)}
 
     @staticmethod
     def low_ld(m) -> int:
@@ -242,7 +243,7 @@ class BonusState:
     def scratch(pf, m, d) -> Scratch:
         C, n = pf.C, m.heads * m.dim
         return {"mixes": (C * 5 * pf.h_ld, pf.act), "proj": (C * 4 * pad(d["part"], 4), F32), "low": (C * pad(m.decay_rank, 8), pf.act),
-                "decay": (C * n, F32), "so": (C * n, F32), "o": (C * pad(n, 8), pf.act), "blocks": blocks(pf, m, S.STATE_BONUS)}
+                "decay": (C * n, F32), "so": (C * n, F32), "o": (C * pad(n, 8), pf.act), **state_scratch(pf, m, S.STATE_BONUS)}
 
     @staticmethod
     def run(pf, r: dict, R: int, pos0: int) -> None:
@@ -298,7 +299,7 @@ class Parallel:
         C, a, s = pf.C, m.left, m.right
         hv = s.heads * s.vdim
         return {"proj": (C * pad(d["in"].n, 4), F32), "q": (C * a.heads * d["dp"], pf.act), "vx": (Parallel.keys(pf, a) * a.kv_heads * d["vp"], pf.act),
-                "o": (C * max(a.heads * d["vp"], pad(hv, 8)), pf.act), "so": (C * hv, F32), "den": (C * s.heads * 2, F32), "keep": (C * s.heads * 2, F32), "blocks": blocks(pf, s, S.STATE_NORMALIZED)}
+                "o": (C * max(a.heads * d["vp"], pad(hv, 8)), pf.act), "so": (C * hv, F32), "den": (C * s.heads * 2, F32), "keep": (C * s.heads * 2, F32), **state_scratch(pf, s, S.STATE_NORMALIZED)}
 
     @staticmethod
     def maps(pf, r: dict):
