@@ -255,26 +255,26 @@ __global__ void __launch_bounds__(kDecThreads) group_decode_kernel(const GroupDe
 }
 
 // Tensor-core form: grid (splits, key heads, tiles of 16 or 32 query heads).  The query heads of a key head are the M side of bf16
-// m16n8k16 MMAs; keys and values come 64 at a time through two cp.async stages, the first requested before the wait for the
+// m16n8k16 MMAs; keys and values come 64 at a time through two to four cp.async stages, the first requested before the wait for the
 // predecessor (older rows do not depend on it; the token's own row is put into its tile by hand).  tcgen05 is not used: the kernel
 // streams the cache once, and most of its M = 128 rows would idle.
 constexpr int kTcHead = 256;
 __host__ __device__ inline int tc_pitch(int n) { return (n + 15) / 16 * 16 + 8; }              // bf16 elements; rows fall into distinct banks
-__host__ __device__ inline int group_tc_smem(int dp, int vp, int ht) {
-  return 2 * (ht + 2 * kTile) * tc_pitch(dp) + 2 * 2 * kTile * tc_pitch(vp) + 4 * ht * (kTile + 4) + 2 * ht * (kTile + 8) + 4 * 3 * ht + 4 * ht * vp +
+__host__ __device__ inline int group_tc_smem(int dp, int vp, int ht, int stages) {
+  return 2 * (ht + stages * kTile) * tc_pitch(dp) + 2 * stages * kTile * tc_pitch(vp) + 4 * ht * (kTile + 4) + 2 * ht * (kTile + 8) + 4 * 3 * ht + 4 * ht * vp +
          4 * (8 * kTcHead + kTcHead) + 2 * (dp + vp);
 }
 
 template <int MT>
-__global__ void __launch_bounds__(kDecThreads, 1) group_decode_tc_kernel(const GroupDecodeArgs a) {
+__global__ void __launch_bounds__(kDecThreads, 1) group_decode_tc_kernel(const GroupDecodeArgs a, const int stages) {
   extern __shared__ __align__(16) uint8_t raw[];
   constexpr int HT = MT * 16, kSP = kTile + 4, kPP = kTile + 8, kNT = kTcHead / 64;
   const GroupPrepArgs& p = a.p;
   const int kp = tc_pitch(p.dp), vpitch = tc_pitch(p.vp), rp = (p.dp + 15) / 16 * 16;
   __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(raw);             // [HT][kp]
-  __nv_bfloat16* sk = sq + HT * kp;                                      // [2][64][kp]
-  __nv_bfloat16* sv = sk + 2 * kTile * kp;                               // [2][64][vpitch]
-  __nv_bfloat16* sp = sv + 2 * kTile * vpitch;                           // [HT][kPP]
+  __nv_bfloat16* sk = sq + HT * kp;                                      // [stages][64][kp]
+  __nv_bfloat16* sv = sk + stages * kTile * kp;                          // [stages][64][vpitch]
+  __nv_bfloat16* sp = sv + stages * kTile * vpitch;                           // [HT][kPP]
   float* ss = reinterpret_cast<float*>(sp + HT * kPP);                   // [HT][kSP]
   float* sm = ss + HT * kSP;
   float* sl = sm + HT;
@@ -296,7 +296,7 @@ __global__ void __launch_bounds__(kDecThreads, 1) group_decode_tc_kernel(const G
   const bool owner = j_hi == n && j_lo < j_hi;
   {
     uint4* z = reinterpret_cast<uint4*>(raw);                            // columns beyond a head stay zero
-    const int words = ((HT + 2 * kTile) * kp + 2 * kTile * vpitch) / 8;
+    const int words = ((HT + stages * kTile) * kp + stages * kTile * vpitch) / 8;
     for (int i = tid; i < words; i += kDecThreads) z[i] = make_uint4(0u, 0u, 0u, 0u);
   }
   for (int i = tid; i < HT * p.vp; i += kDecThreads) so[i] = 0.f;
@@ -304,18 +304,22 @@ __global__ void __launch_bounds__(kDecThreads, 1) group_decode_tc_kernel(const G
   __syncthreads();
   const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(p.k_cache) + (long long)hk * p.dp;
   const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(p.v_cache) + (long long)hk * p.vp;
-  auto request = [&](int j0, int st) {
-    const int kpieces = p.dp / 8, pieces = kpieces + p.vp / 8;
-    for (int i = tid; i < kTile * pieces; i += kDecThreads) {
-      const int t = i / pieces, c = i - t * pieces;
-      const bool in = j0 + t < j_hi && j0 + t != n - 1;                  // the token's own row is not in the cache yet
-      const long long row = start + (in ? j0 + t : j_lo);
-      if (c < kpieces) cp16(sk + (st * kTile + t) * kp + c * 8, kc + row * p.kv_heads * p.dp + c * 8, in);
-      else cp16(sv + (st * kTile + t) * vpitch + (c - kpieces) * 8, vc + row * p.kv_heads * p.vp + (c - kpieces) * 8, in);
-    }
+  const int kpieces = p.dp / 8, pieces = kpieces + p.vp / 8, t_first = tid / pieces, c_first = tid - t_first * pieces;
+  const int t_step = kDecThreads / pieces, c_step = kDecThreads - t_step * pieces;
+  auto request = [&](int j0, int st) {         // the 64 rows from j0 on (none beyond the split: an empty group keeps the count)
+    if (j0 < j_hi)
+      for (int t = t_first, c = c_first; t < kTile;) {
+        const bool in = j0 + t < j_hi && j0 + t != n - 1;                // the token's own row is not in the cache yet
+        const long long row = start + (in ? j0 + t : j_lo);
+        if (c < kpieces) cp16(sk + (st * kTile + t) * kp + c * 8, kc + row * p.kv_heads * p.dp + c * 8, in);
+        else cp16(sv + (st * kTile + t) * vpitch + (c - kpieces) * 8, vc + row * p.kv_heads * p.vp + (c - kpieces) * 8, in);
+        c += c_step;
+        t += t_step;
+        if (c >= pieces) { c -= pieces; ++t; }
+      }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (j_lo < j_hi) request(j_lo, 0);
+  for (int i = 0; i + 1 < stages; ++i) request(j_lo + i * kTile, i);
   griddep_wait();
   griddep_launch();
   if (j_lo < j_hi) {
@@ -352,13 +356,11 @@ __global__ void __launch_bounds__(kDecThreads, 1) group_decode_tc_kernel(const G
     const int ntiles = p.vp / 8, fr = lane >> 2, fc = (lane & 3) * 2;
     const float c2 = 1.4426950408889634f;                                // scores in powers of two
     int st = 0;
-    for (int j0 = j_lo; j0 < j_hi; j0 += kTile, st ^= 1) {
-      if (j0 + kTile < j_hi) {
-        request(j0 + kTile, st ^ 1);
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-      } else {
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-      }
+    for (int j0 = j_lo; j0 < j_hi; j0 += kTile, st = st + 1 == stages ? 0 : st + 1) {
+      request(j0 + (stages - 1) * kTile, st == 0 ? stages - 1 : st - 1);
+      if (stages == 4) asm volatile("cp.async.wait_group 3;" ::: "memory");
+      else if (stages == 3) asm volatile("cp.async.wait_group 2;" ::: "memory");
+      else asm volatile("cp.async.wait_group 1;" ::: "memory");
       __syncthreads();
       if (owner && n - 1 < j0 + kTile) {                                 // the last tile: the token's own row
         for (int c = tid; c < p.dp; c += kDecThreads) sk[(st * kTile + n - 1 - j0) * kp + c] = new_k[c];
@@ -468,8 +470,10 @@ int launch_decode_tc(const GroupDecodeArgs& a, cudaStream_t stream, bool pdl) {
     configured = true;
   }
   const int group = a.p.heads / a.p.kv_heads;
+  int stages = 4;
+  while (stages > 2 && group_tc_smem(a.p.dp, a.p.vp, MT * 16, stages) > 220 * 1024) --stages;
   return launch_cluster(group_decode_tc_kernel<MT>, dim3(a.splits, a.p.kv_heads, (group + MT * 16 - 1) / (MT * 16)), dim3(kDecThreads), dim3(a.splits, 1, 1),
-                        group_tc_smem(a.p.dp, a.p.vp, MT * 16), stream, pdl, a);
+                        group_tc_smem(a.p.dp, a.p.vp, MT * 16, stages), stream, pdl, a, stages);
 }
 
 template <bool F32, int VC>

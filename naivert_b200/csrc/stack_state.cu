@@ -689,182 +689,194 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const HeadGateArgs a) {
 
 // ------------------------------------------------------------------------------------ one token
 // grid (share of the value columns, heads); the CTAs of a head are a cluster that meets once, for the read-out norm.  The state (written
-// a whole step ago) and the low-rank weights are requested before the wait for the predecessor.
+// a whole step ago) and the low-rank weights are requested before the wait for the predecessor.  Every instruction runs about once, so
+// the kernel is bound by latencies, instruction fetch among them: loops stay rolled and nothing is specialised twice.
 constexpr int kStepT = 256, kStepCols = kStepT / kLanes;
 
-// rows of a low-rank product: out[row] = W[row] . in, one warp per row
-template <bool STAGED, class F>
-__device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, int ld, int rows, const float* in, int warp, int lane, F store) {
-#pragma unroll 4
-  for (int r = warp; r < rows; r += kStepT / 32) {
-    float acc = 0.f;
-    for (int c = lane * 4; c < ld; c += 128) {
-      const uint2* src = reinterpret_cast<const uint2*>(w + (long long)r * ld + c);
-      const uint2 p = STAGED ? *src : __ldg(src);
-      const float4 x = *reinterpret_cast<const float4*>(in + c);
-      acc = fmaf(bf16_lo(p.x), x.x, fmaf(bf16_hi(p.x), x.y, fmaf(bf16_lo(p.y), x.z, fmaf(bf16_hi(p.y), x.w, acc))));
-    }
-    acc = lane_sum(acc);
-    if (lane == 0) store(r, acc);
-  }
-}
 __device__ __forceinline__ void stage_weights(void* dst, const __nv_bfloat16* src, int n) {        // n a multiple of 8
+#pragma unroll 1
   for (int i = threadIdx.x * 8; i < n; i += kStepT * 8)
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(reinterpret_cast<__nv_bfloat16*>(dst) + i)), "l"(src + i) : "memory");
 }
-__host__ __device__ inline int step_floats(int dp, int per, int decay_ld, int gate_ld) { return 3 * dp + 3 * pad4(per + 1) + decay_ld + gate_ld; }
+// out[row] = W[row] . in for rows of ld bf16 (a multiple of 8), eight lanes per row
+__device__ __forceinline__ void low_rank_rows(const __nv_bfloat16* w, int ld, int rows, const float* in, float* out) {
+  const int l = threadIdx.x & (kLanes - 1);
+#pragma unroll 1
+  for (int rb = 0; rb < rows; rb += kStepT / kLanes) {                   // (the same trip count for every lane of a warp)
+    const int r = rb + (threadIdx.x / kLanes);
+    float acc = 0.f;
+    if (r < rows) {
+#pragma unroll 2
+      for (int c = l * 8; c < ld; c += 8 * kLanes) {
+        const uint4 p = *reinterpret_cast<const uint4*>(w + (long long)r * ld + c);
+        const float4 x = *reinterpret_cast<const float4*>(in + c), y = *reinterpret_cast<const float4*>(in + c + 4);
+        acc = fmaf(bf16_lo(p.x), x.x, fmaf(bf16_hi(p.x), x.y, fmaf(bf16_lo(p.y), x.z, fmaf(bf16_hi(p.y), x.w, acc))));
+        acc = fmaf(bf16_lo(p.z), y.x, fmaf(bf16_hi(p.z), y.y, fmaf(bf16_lo(p.w), y.z, fmaf(bf16_hi(p.w), y.w, acc))));
+      }
+    }
+    acc = column_sum(acc);
+    if (r < rows && l == 0) out[r] = acc;
+  }
+}
+__host__ __device__ inline int step_floats(int dp, int per, int decay_ld, int gate_ld) { return 3 * dp + 3 * pad4(per) + decay_ld + gate_ld; }
 
 template <int KIND, int NV>
 __global__ void __launch_bounds__(kStepT, 1) state_step_kernel(const StateStepArgs a, const int per, const int staged) {
-  constexpr int DP = NV * 4 * kLanes, AHEAD = NV <= 4 ? 2 : 1;
+  constexpr int DP = NV * 4 * kLanes;
   extern __shared__ __align__(16) float sh[];
   __shared__ float red[33], part;
   const int rank = blockIdx.x, h = blockIdx.y, hk = h / (a.heads / a.kv_heads);
-  const int c_lo = min(a.vdim, rank * per), own = min(a.vdim, c_lo + per) - c_lo, cols = own + extra_columns<KIND>();
+  const int c_lo = min(a.vdim, rank * per), own = min(a.vdim, c_lo + per) - c_lo;
   const int decay_ld = (int)a.decay_ld, gate_ld = (int)a.gate_ld;
   float* sk = sh;
   float* sq = sk + DP;
   float* sg = sq + DP;
   float* so = sg + DP;
-  float* sgate = so + pad4(per + 1);
-  float* sv = sgate + pad4(per + 1);
-  float* slow = sv + pad4(per + 1);
+  float* sgate = so + pad4(per);
+  float* sv = sgate + pad4(per);
+  float* slow = sv + pad4(per);
   float* sgin = slow + decay_ld;
-  __nv_bfloat16* wdecay = reinterpret_cast<__nv_bfloat16*>(sgin + gate_ld);
-  __nv_bfloat16* wgate = wdecay + (KIND == kStateNormalized ? 0 : a.dim * decay_ld);
-  const __nv_bfloat16* gdecay = KIND == kStateNormalized ? nullptr : a.decay_w + (long long)h * a.dim * decay_ld;
-  const __nv_bfloat16* ggate = a.gate_w ? a.gate_w + ((long long)h * a.vdim + c_lo) * gate_ld : nullptr;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & (kLanes - 1);
+  const __nv_bfloat16* wdecay = KIND == kStateNormalized ? nullptr : a.decay_w + (long long)h * a.dim * decay_ld;
+  const __nv_bfloat16* wgate = a.gate_w ? a.gate_w + ((long long)h * a.vdim + c_lo) * gate_ld : nullptr;
+  const int tid = threadIdx.x, lane = tid & 31, l = lane & (kLanes - 1);
   const int C = a.vdim + extra_columns<KIND>(), d4 = pad4(a.dim);
   if (staged) {
-    if (KIND != kStateNormalized) stage_weights(wdecay, gdecay, a.dim * decay_ld);
-    if (a.gate_w) stage_weights(wgate, ggate, own * gate_ld);
+    __nv_bfloat16* sw = reinterpret_cast<__nv_bfloat16*>(sgin + gate_ld);
+    if (KIND != kStateNormalized) {
+      stage_weights(sw, wdecay, a.dim * decay_ld);
+      wdecay = sw;
+      sw += a.dim * decay_ld;
+    }
+    if (a.gate_w) {
+      stage_weights(sw, wgate, own * gate_ld);
+      wgate = sw;
+    }
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
   const int pos = *reinterpret_cast<const volatile int*>(a.pos0);
   const int slot = state_slot(a.tags, pos, a.status);
   const float* old = a.state + max(slot, 0) * a.state_stride + (long long)h * C * d4;
   float* now = a.state + (1 - max(slot, 0)) * a.state_stride + (long long)h * C * d4;
-  // local column j: value column c_lo + j, then the normaliser
-  auto load = [&](int j, u64 (&s)[2 * NV]) {
-    const long long at = (long long)(j < own ? c_lo + j : a.vdim) * d4;
+  u64 s[2 * NV];
+  auto load = [&](int j) {                     // local value column j
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int e = (l + kLanes * i) * 4;
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (j < cols && pos > 0 && e < d4) v = __ldcg(reinterpret_cast<const float4*>(old + at + e));
+      if (j < own && pos > 0 && e < d4) v = __ldcg(reinterpret_cast<const float4*>(old + (long long)(c_lo + j) * d4 + e));
       s[2 * i] = pack2(v.x, v.y);
       s[2 * i + 1] = pack2(v.z, v.w);
     }
   };
-  u64 first[AHEAD][2 * NV];
-#pragma unroll
-  for (int j = 0; j < AHEAD; ++j) load(tid / kLanes + j * kStepCols, first[j]);
-  float d_bias = 0.f, d_rate = 0.f;            // of this thread's first decay
+  load(tid / kLanes);
+  float d_bias = 0.f, d_rate = 0.f, norm = 0.f, n_old = 0.f;              // of this thread's first decay, column and normaliser entry
   if (KIND != kStateNormalized && tid < a.dim) {
     d_bias = bf(a.decay_b + (long long)h * a.dim + tid);
     if (a.rate) d_rate = __ldg(a.rate + (long long)h * a.dim + tid);
   }
+  const __nv_bfloat16* nw = a.norm + (a.norm_per_head ? (long long)h * a.vdim : 0) + c_lo;
+  if (tid < own) norm = bf(nw + tid);
+  if (KIND == kStateNormalized && tid < a.dim && pos > 0) n_old = __ldcg(old + (long long)a.vdim * d4 + tid);
   griddep_wait();
   griddep_launch();
   if (slot >= 0) {                                                       // (the same for every CTA of the cluster)
     const float* p = a.proj;
+    float s0 = 0.f, s1 = 0.f, floor_n = 0.f;
+    if (KIND == kStateDelta) s0 = __ldcg(p + a.beta_off + h);
+    if (KIND == kStateNormalized) { s0 = __ldcg(p + a.gi_off + h); s1 = __ldcg(p + a.gf_off + h); }
+    float qq = 0.f, kk = 0.f, bonus = 0.f;
+#pragma unroll 1
     for (int i = tid; i < DP; i += kStepT) {
       const bool in = i < a.dim;
-      sk[i] = in ? __ldcg(p + a.k_off + hk * a.dim + i) : 0.f;
-      sq[i] = in ? __ldcg(p + a.q_off + hk * a.dim + i) : 0.f;
+      const float k = in ? __ldcg(p + a.k_off + hk * a.dim + i) : 0.f, q = in ? __ldcg(p + a.q_off + hk * a.dim + i) : 0.f;
+      sk[i] = k;
+      sq[i] = q;
       sg[i] = 0.f;
+      if (KIND == kStateDelta) {
+        qq = fmaf(q, q, qq);
+        kk = fmaf(k, k, kk);
+      }
+      if (KIND == kStateBonus && in) bonus = fmaf(q * bf(a.u + (long long)h * a.dim + i), k, bonus);
     }
-    for (int j = tid; j < cols; j += kStepT) {
-      sv[j] = j < own ? __ldcg(p + a.v_off + (long long)h * a.vdim + c_lo + j) : 1.f;
-      if (!a.gate_w && j < own) sgate[j] = __ldcg(p + a.gate_off + (long long)h * a.vdim + c_lo + j);
+#pragma unroll 1
+    for (int j = tid; j < own; j += kStepT) {
+      sv[j] = __ldcg(p + a.v_off + (long long)h * a.vdim + c_lo + j);
+      if (!a.gate_w) sgate[j] = __ldcg(p + a.gate_off + (long long)h * a.vdim + c_lo + j);
     }
-    if (KIND != kStateNormalized)
+    if (KIND != kStateNormalized) {
+#pragma unroll 1
       for (int i = tid; i < decay_ld; i += kStepT) {
         const float z = i < a.low_rank ? __ldcg(p + a.low_off + i) : 0.f;
         slow[i] = a.low_tanh ? tanhf(z) : z;
       }
-    if (a.gate_w)
+    }
+    if (a.gate_w) {
+#pragma unroll 1
       for (int i = tid; i < gate_ld; i += kStepT) sgin[i] = i < a.gate_rank ? __ldcg(p + a.gate_off + i) : 0.f;
-    float s0 = 0.f, s1 = 0.f, floor_n = 0.f;
-    if (KIND == kStateDelta) s0 = sigmoid_f(__ldcg(p + a.beta_off + h));
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (KIND != kStateNormalized) low_rank_rows(wdecay, decay_ld, a.dim, slow, sg);
+    if (a.gate_w) low_rank_rows(wgate, gate_ld, own, sgin, sgate);
+    float q_scale = a.q_scale, k_scale = 1.f;
+    if (KIND == kStateDelta) {
+      s0 = sigmoid_f(s0);
+      if (a.unit) {
+        q_scale /= sqrtf(block_sum_f(qq, red) + kUnitEps);
+        k_scale = 1.0f / sqrtf(block_sum_f(kk, red) + kUnitEps);
+      }
+    }
+    if (KIND == kStateBonus) bonus = block_sum_f(bonus, red);
     if (KIND == kStateNormalized) {
-      const float zi = log_input(__ldcg(p + a.gi_off + h), a.cap), zf = log_forget(__ldcg(p + a.gf_off + h), a.cap);
+      const float zi = log_input(s0, a.cap), zf = log_forget(s1, a.cap);
       const long long m_at = (long long)(a.heads - h) * C * d4 + h;      // the maxima follow the last head's state
       const float m = pos > 0 ? __ldcg(old + m_at) : 0.f, m_new = fmaxf(zf + m, zi);
       s0 = expf(zf + m - m_new);
       s1 = expf(zi - m_new);
       floor_n = expf(-m_new);
       if (rank == 0 && tid == 0) now[m_at] = m_new;
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    if (KIND != kStateNormalized) {
-      auto store = [&](int d, float z) { sg[d] = z; };
-      if (staged) low_rank_rows<true>(wdecay, decay_ld, a.dim, slow, warp, lane, store);
-      else low_rank_rows<false>(gdecay, decay_ld, a.dim, slow, warp, lane, store);
-    }
-    if (a.gate_w) {
-      auto store = [&](int j, float z) { sgate[j] = z; };
-      if (staged) low_rank_rows<true>(wgate, gate_ld, own, sgin, warp, lane, store);
-      else low_rank_rows<false>(ggate, gate_ld, own, sgin, warp, lane, store);
-    }
-    float q_scale = a.q_scale;
-    if (a.unit) {
-      float qq = 0.f, kk = 0.f;
-      for (int i = lane; i < a.dim; i += 32) {
-        qq = fmaf(sq[i], sq[i], qq);
-        kk = fmaf(sk[i], sk[i], kk);
+      // the normaliser: every CTA needs n . q, one keeps n
+      float nq = 0.f;
+#pragma unroll 1
+      for (int d = tid; d < a.dim; d += kStepT) {
+        const float n = fmaf(s0, d == tid ? n_old : pos > 0 ? __ldcg(old + (long long)a.vdim * d4 + d) : 0.f, s1 * sk[d]);
+        nq = fmaf(n, sq[d], nq);
+        if (rank == 0) now[(long long)a.vdim * d4 + d] = n;
       }
-      q_scale /= sqrtf(lane_sum(qq) + kUnitEps);
-      const float ks = 1.0f / sqrtf(lane_sum(kk) + kUnitEps);
-      __syncthreads();
-      for (int i = tid; i < a.dim; i += kStepT) sk[i] *= ks;
-    } else if (KIND != kStateNormalized) {
+      q_scale /= fmaxf(fabsf(block_sum_f(nq, red) * q_scale), floor_n) + 1e-6f;
+    } else {
+      __syncthreads();                                                   // the low-rank results
+#pragma unroll 1
+      for (int d = tid; d < a.dim; d += kStepT) {
+        const float z = sg[d] + (d == tid ? d_bias : bf(a.decay_b + (long long)h * a.dim + d));
+        sg[d] = a.rate ? decay_soft(z, d == tid ? d_rate : a.rate[(long long)h * a.dim + d]) : decay_exp(z);
+        if (KIND == kStateDelta) sk[d] *= k_scale;
+      }
       __syncthreads();
     }
-    if (KIND != kStateNormalized)
-      for (int d = tid, e = 0; d < a.dim; d += kStepT, ++e) {
-        const float z = sg[d] + (e == 0 ? d_bias : bf(a.decay_b + (long long)h * a.dim + d));
-        sg[d] = a.rate ? decay_soft(z, e == 0 ? d_rate : a.rate[(long long)h * a.dim + d]) : decay_exp(z);
-      }
-    if (KIND == kStateBonus) {
-      for (int i = lane; i < a.dim; i += 32) s0 = fmaf(sq[i] * bf(a.u + (long long)h * a.dim + i), sk[i], s0);
-      s0 = lane_sum(s0);
-    }
-    __syncthreads();
     const ulonglong2* q = reinterpret_cast<const ulonglong2*>(sq) + l;
     const ulonglong2* k = reinterpret_cast<const ulonglong2*>(sk) + l;
     const ulonglong2* g = reinterpret_cast<const ulonglong2*>(sg) + l;
-    auto column = [&](int j, u64 (&s)[2 * NV]) {
-      const float v = j < cols ? sv[j] : 0.f;
-      float r = column_sum(column_step<KIND, NV>(s, q, k, g, v, s0, s1));
-      if (KIND == kStateBonus) r = fmaf(s0, v, r);
-      if (j < cols) {
-        if (j < own || rank == 0) {
-          const long long at = (long long)(j < own ? c_lo + j : a.vdim) * d4;
-#pragma unroll
-          for (int i = 0; i < NV; ++i) {
-            const int e = (l + kLanes * i) * 4;
-            if (e < d4) *reinterpret_cast<ulonglong2*>(now + at + e) = make_ulonglong2(s[2 * i], s[2 * i + 1]);
-          }
-        }
-        if (l == 0) so[j] = r * q_scale;
-      }
-    };
-#pragma unroll
-    for (int j = 0; j < AHEAD; ++j) column(tid / kLanes + j * kStepCols, first[j]);
-    for (int jb = AHEAD * kStepCols; jb < cols; jb += kStepCols) {       // (the same trip count for every lane of a warp)
-      u64 s[2 * NV];
-      load(jb + tid / kLanes, s);
-      column(jb + tid / kLanes, s);
-    }
-    __syncthreads();
-    const float inv = KIND == kStateNormalized ? 1.0f / (fmaxf(fabsf(so[own]), floor_n) + 1e-6f) : 1.f;
     float ss = 0.f;
-    for (int j = tid; j < own; j += kStepT) {
-      so[j] *= inv;
-      ss = fmaf(so[j], so[j], ss);
+#pragma unroll 1
+    for (int jb = 0; jb < own; jb += kStepCols) {                        // (the same trip count for every lane of a warp)
+      const int j = jb + tid / kLanes;
+      if (jb > 0) load(j);
+      const float v = j < own ? sv[j] : 0.f;
+      float r = column_sum(column_step<KIND, NV>(s, q, k, g, v, s0, s1));
+      if (KIND == kStateBonus) r = fmaf(bonus, v, r);
+      r *= q_scale;
+      if (j < own) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int e = (l + kLanes * i) * 4;
+          if (e < d4) *reinterpret_cast<ulonglong2*>(now + (long long)(c_lo + j) * d4 + e) = make_ulonglong2(s[2 * i], s[2 * i + 1]);
+        }
+        if (l == 0) {
+          so[j] = r;
+          ss = fmaf(r, r, ss);
+        }
+      }
     }
     ss = block_sum_f(ss, red);
     if (tid == 0) part = ss;
@@ -872,18 +884,21 @@ __global__ void __launch_bounds__(kStepT, 1) state_step_kernel(const StateStepAr
   cluster_sync_all();
   if (slot >= 0) {
     float ss = 0.f;
+#pragma unroll 1
     for (int i = 0; i < (int)gridDim.x; ++i) ss += ld_cluster_f32(&part, i);
     const float rs = 1.0f / sqrtf(ss / (float)a.vdim + a.eps);
-    const __nv_bfloat16* w = a.norm + (a.norm_per_head ? (long long)h * a.vdim : 0) + c_lo;
-    for (int j = tid; j < own; j += kStepT)
-      a.out[(long long)h * a.vdim + c_lo + j] = so[j] * rs * bf(w + j) * (a.gate_kind == kGateSilu ? silu_f(sgate[j]) : sigmoid_f(sgate[j]));
+#pragma unroll 1
+    for (int j = tid; j < own; j += kStepT) {
+      const float z = sgate[j], sig = sigmoid_f(z);
+      a.out[(long long)h * a.vdim + c_lo + j] = so[j] * rs * (j == tid ? norm : bf(nw + j)) * (a.gate_kind == kGateSilu ? z * sig : sig);
+    }
     // A CTA that starts after this store still finds `pos` in its own slot: only the other slot's tag changes.
     if (rank == 0 && h == 0 && tid == 0) {
       a.tags[1 - slot] = pos + 1;
       if (pos == 0) a.tags[1] = -1;
     }
   }
-  cluster_sync_all();                                                    // nobody leaves while its sum is read
+  if (gridDim.x > 1) cluster_sync_all();                                 // nobody leaves while its sum is read
 }
 
 constexpr int kMaxSmem = 220 * 1024;
