@@ -300,23 +300,32 @@ __global__ void __launch_bounds__(kDecThreads, 1) group_decode_tc_kernel(const G
     for (int i = tid; i < words; i += kDecThreads) z[i] = make_uint4(0u, 0u, 0u, 0u);
   }
   for (int i = tid; i < HT * p.vp; i += kDecThreads) so[i] = 0.f;
-  for (int i = tid; i < HT; i += kDecThreads) { sm[i] = -FLT_MAX; sl[i] = 0.f; }
+  for (int i = tid; i < HT; i += kDecThreads) { sm[i] = -FLT_MAX; sl[i] = scorr[i] = 0.f; }
+  for (int i = tid; i < HT * kPP; i += kDecThreads) sp[i] = __float2bfloat16_rn(0.f);
   __syncthreads();
   const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(p.k_cache) + (long long)hk * p.dp;
   const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(p.v_cache) + (long long)hk * p.vp;
-  const int kpieces = p.dp / 8, pieces = kpieces + p.vp / 8, t_first = tid / pieces, c_first = tid - t_first * pieces;
-  const int t_step = kDecThreads / pieces, c_step = kDecThreads - t_step * pieces;
+  // a thread copies one 16-byte piece of every so-many-th row
+  auto rows_in = [&](int j0, __nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int width) {
+    int lanes = 1;
+    while (lanes < width / 8) lanes *= 2;
+    const int c = tid & (lanes - 1), step = kDecThreads / lanes;
+    if (c >= width / 8) return;
+    const long long row_step = (long long)p.kv_heads * width;
+    int t = tid / lanes;
+    const __nv_bfloat16* s0 = src + (long long)(start + j0 + t) * row_step + c * 8;
+    __nv_bfloat16* d = dst + t * pitch + c * 8;
+#pragma unroll 4
+    for (; t < kTile; t += step, s0 += step * row_step, d += step * pitch) {
+      const bool in = j0 + t < j_hi && j0 + t != n - 1;                  // the token's own row is not in the cache yet
+      cp16(d, in ? s0 : src, in);
+    }
+  };
   auto request = [&](int j0, int st) {         // the 64 rows from j0 on (none beyond the split: an empty group keeps the count)
-    if (j0 < j_hi)
-      for (int t = t_first, c = c_first; t < kTile;) {
-        const bool in = j0 + t < j_hi && j0 + t != n - 1;                // the token's own row is not in the cache yet
-        const long long row = start + (in ? j0 + t : j_lo);
-        if (c < kpieces) cp16(sk + (st * kTile + t) * kp + c * 8, kc + row * p.kv_heads * p.dp + c * 8, in);
-        else cp16(sv + (st * kTile + t) * vpitch + (c - kpieces) * 8, vc + row * p.kv_heads * p.vp + (c - kpieces) * 8, in);
-        c += c_step;
-        t += t_step;
-        if (c >= pieces) { c -= pieces; ++t; }
-      }
+    if (j0 < j_hi) {
+      rows_in(j0, sk + st * kTile * kp, kp, kc, p.dp);
+      rows_in(j0, sv + st * kTile * vpitch, vpitch, vc, p.vp);
+    }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   for (int i = 0; i + 1 < stages; ++i) request(j_lo + i * kTile, i);
@@ -370,33 +379,42 @@ __global__ void __launch_bounds__(kDecThreads, 1) group_decode_tc_kernel(const G
       const __nv_bfloat16* kt = sk + st * kTile * kp;
       const __nv_bfloat16* vt = sv + st * kTile * vpitch;
       // scores: warp = 8 keys, all heads
-      float acc[MT][4];
+      float acc[MT][2][4];                                               // even and odd steps: two chains
 #pragma unroll
-      for (int i = 0; i < MT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-#pragma unroll 4
-      for (int k = 0; k < rp; k += 16) {
-        uint32_t b0, b1;
-        ldsm2(b0, b1, kt + (warp * 8 + (lane & 7)) * kp + k + ((lane >> 3) & 1) * 8);
+      for (int i = 0; i < MT; ++i)
 #pragma unroll
-        for (int i = 0; i < MT; ++i) {
-          uint32_t af[4];
-          ldsm4(af, sq + (i * 16 + (lane & 15)) * kp + k + (lane >> 4) * 8);
-          mma16816(acc[i], af, b0, b1);
+        for (int q = 0; q < 8; ++q) acc[i][q >> 2][q & 3] = 0.f;
+      const __nv_bfloat16* krow = kt + (warp * 8 + (lane & 7)) * kp + ((lane >> 3) & 1) * 8;
+      const __nv_bfloat16* qrow = sq + (lane & 15) * kp + (lane >> 4) * 8;
+#pragma unroll 2
+      for (int k = 0; k < rp; k += 32) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          if (e && k + 16 >= rp) break;
+          uint32_t b0, b1;
+          ldsm2(b0, b1, krow + k + 16 * e);
+#pragma unroll
+          for (int i = 0; i < MT; ++i) {
+            uint32_t af[4];
+            ldsm4(af, qrow + i * 16 * kp + k + 16 * e);
+            mma16816(acc[i][e], af, b0, b1);
+          }
         }
       }
 #pragma unroll
       for (int i = 0; i < MT; ++i) {
         float* d = ss + (i * 16 + fr) * kSP + warp * 8 + fc;
-        d[0] = acc[i][0] * c2;
-        d[1] = acc[i][1] * c2;
-        d[8 * kSP] = acc[i][2] * c2;
-        d[8 * kSP + 1] = acc[i][3] * c2;
+        d[0] = (acc[i][0][0] + acc[i][1][0]) * c2;
+        d[1] = (acc[i][0][1] + acc[i][1][1]) * c2;
+        d[8 * kSP] = (acc[i][0][2] + acc[i][1][2]) * c2;
+        d[8 * kSP + 1] = (acc[i][0][3] + acc[i][1][3]) * c2;
       }
       __syncthreads();
       const int live = j_hi - j0;
 #pragma unroll
       for (int ti = 0; ti < HT / 8; ++ti) {
         const int t = warp + 8 * ti;
+        if (t >= nh) break;                                              // (rows without a head stay zero)
         const float s0 = lane < live ? ss[t * kSP + lane] : -FLT_MAX, s1 = lane + 32 < live ? ss[t * kSP + lane + 32] : -FLT_MAX;
         float mt = fmaxf(s0, s1);
 #pragma unroll
