@@ -17,6 +17,7 @@ import pytest
 import torch
 
 import tumatar_oracle as oracle
+from stack_testing import TOL, error, feed, tokens
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
@@ -117,20 +118,6 @@ def engine(cfg, w, dtype="fp32", capacity=512, chunk=96, kv_block=16384):
                               weights=tumatar.gather_weights(spec, lambda n: w[n].cuda()), prefill_chunk=chunk, dtype=dtype, kv_block=kv_block)
 
 
-def tokens(cfg, n, seed=5):
-    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def error(got, want):
-    """Per row: root mean square of the centred difference over that of the centred reference."""
-    d = got.double().cpu() - want
-    d, w = d - d.mean(-1, keepdim=True), want - want.mean(-1, keepdim=True)
-    return d.pow(2).mean(-1).sqrt() / w.pow(2).mean().sqrt()
-
-
-TOL = {"fp32": 2e-4, "bf16": 4e-2}
-
-
 def check(got, want, cfg, dtype, what, tol=None):
     e = error(got, want)
     over = int((e > (tol or TOL[dtype])).sum())
@@ -138,17 +125,6 @@ def check(got, want, cfg, dtype, what, tol=None):
     if dtype == "bf16" and any((x.get("mlp") or {}).get("kind") == "moe" for x in cfg["layers"]):
         allowed = max(1, len(e) // 25)
     assert torch.isfinite(e).all() and over <= allowed, (what, dtype, over, int(e.argmax()), float(e.max()))
-
-
-def feed(eng, toks, sizes):
-    """Logits of every token, fed in portions of the given sizes (the last size repeats)."""
-    eng.reset()
-    out, at, i = [], 0, 0
-    while at < len(toks):
-        n = min(sizes[min(i, len(sizes) - 1)], len(toks) - at)
-        out.append(eng.extend(toks[at:at + n], list(range(n))))
-        at, i = at + n, i + 1
-    return torch.cat(out)
 
 
 # --------------------------------------------------------------------------- mechanisms, prompts, decoding, portions
