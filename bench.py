@@ -124,13 +124,17 @@ def stack_workload(a) -> int:
     if a.gpus != 1:
         raise SystemExit("layer-stack models run on one GPU")
     import torch
-    from naivert_b200.runtime.stack_bench import closest, run
+    from naivert_b200.runtime.stack_bench import closest, closest_stack, run
     torch.cuda.set_device(0)
     model = a.model if a.model != "naive-n0.5" else "tumatar-bench"
     out = run(model, a.prompt, a.steps, a.warmup, a.prefill_chunk or 2048, a.kernels, layers=a.layers, clocks=ClockSampler(0))
     if a.closest:
         torch.cuda.empty_cache()
-        out["closest"] = closest(a.prompt, a.prefill_chunk or 2048, out["config"]["layers"], 4)
+        like = closest_stack(model)                  # another layer stack of the same size, else the speculative target
+        if like:
+            out["closest"] = run(like, a.prompt, a.steps, a.warmup, a.prefill_chunk or 2048, a.kernels, layers=out["config"]["layers"])
+        else:
+            out["closest"] = closest(a.prompt, a.prefill_chunk or 2048, out["config"]["layers"], 4)
     print(json.dumps(out))
     return 0
 
@@ -159,7 +163,7 @@ def main() -> int:
     ap.add_argument("--workload", choices=("speculative", "stack"), default="speculative",
                     help="stack: prefill and decode of a layer-stack model (--model, default tumatar-bench) on one GPU")
     ap.add_argument("--kernels", action="store_true", help="stack workload: add per-kernel tables")
-    ap.add_argument("--closest", action="store_true", help="stack workload: measure the speculative target at the same depth as well")
+    ap.add_argument("--closest", action="store_true", help="stack workload: measure the closest other model at the same size and depth as well")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_arm(a)

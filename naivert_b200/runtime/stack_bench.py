@@ -156,6 +156,11 @@ def step_table(eng, pos: int, steps: int = 4) -> List[dict]:
             for k, v in sorted(agg.items(), key=lambda kv: -kv[1][0])]
 
 
+def closest_stack(model: str) -> str:
+    """The layer-stack model of equal width, feed-forward and vocabulary that a design is measured beside ("": none)."""
+    return {"zuzupel-bench": "tumatar-bench-dense"}.get(model, "")
+
+
 def closest(prompt_len: int, chunk: int, layers: int, steps: int) -> dict:
     """The speculative target (W8A8, same width, heads and experts) at equal depth: chunked prefill, its eight-row step, and the
     kernels of both with the weight bytes they must read or the FLOPs they must do."""
