@@ -182,7 +182,7 @@ struct GroupPrepArgs {
   int capacity;
 };
 
-struct TransposeArgs {
+struct TransposeArgs {          // cols and dst_ld even
   const __nv_bfloat16* src;     // [rows][cols]
   __nv_bfloat16* dst;           // [cols][dst_ld]
   long long dst_ld;
@@ -451,7 +451,18 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit, floa
 __device__ __forceinline__ float silu_glu(float g, float u) { return g * sigmoid_f(g) * u; }
 __device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
 __device__ __forceinline__ float relu2_f(float z) { z = fmaxf(z, 0.f); return z * z; }
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// log(1 + t) for 0 <= t <= 1: twice the area tangent of s = t / (2 + t) <= 1/3, as its power series (the next term is below 2e-8)
+__device__ __forceinline__ float log1p_unit(float t) {
+  const float s = __fdividef(t, 2.0f + t), q = s * s;
+  float p = fmaf(q, 1.0f / 13.0f, 1.0f / 11.0f);
+  p = fmaf(q, p, 1.0f / 9.0f);
+  p = fmaf(q, p, 1.0f / 7.0f);
+  p = fmaf(q, p, 1.0f / 5.0f);
+  p = fmaf(q, p, 1.0f / 3.0f);
+  p = fmaf(q, p, 1.0f);
+  return 2.0f * s * p;
+}
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1p_unit(expf(-fabsf(z))); }
 __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float decay_soft(float z, float rate) { return expf(-rate * softplus_f(z)); }
 __device__ __forceinline__ float decay_exp(float z) { return expf(-expf(z)); }

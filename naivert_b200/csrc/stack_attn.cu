@@ -68,17 +68,29 @@ __global__ void __launch_bounds__(256) group_prep_kernel(const GroupPrepArgs p) 
   }
 }
 
-// dst[c][r] = src[r][c], 64 x 64 tiles
+// dst[c][r] = src[r][c], 64 x 64 tiles, two values per access; rows beyond the last become zeros up to the tile's end
 __global__ void __launch_bounds__(256) transpose_kernel(const TransposeArgs a) {
   __shared__ __nv_bfloat16 tile[64][66];
   griddep_wait();
   griddep_launch();
-  const int r0 = blockIdx.x * 64, c0 = blockIdx.y * 64, tx = threadIdx.x & 63, ty = threadIdx.x >> 6;
-  for (int i = ty; i < 64; i += 4)
-    if (r0 + i < a.rows && c0 + tx < a.cols) tile[i][tx] = a.src[(long long)(r0 + i) * a.cols + c0 + tx];
+  const int r0 = blockIdx.x * 64, c0 = blockIdx.y * 64, tx = (threadIdx.x & 31) * 2, ty = threadIdx.x >> 5;
+#pragma unroll
+  for (int i = 0; i < 64; i += 8) {
+    const int r = r0 + ty + i;
+    uint32_t v = 0u;
+    if (r < a.rows && c0 + tx < a.cols) v = __ldg(reinterpret_cast<const uint32_t*>(a.src + (long long)r * a.cols + c0 + tx));
+    *reinterpret_cast<uint32_t*>(&tile[ty + i][tx]) = v;
+  }
   __syncthreads();
-  for (int i = ty; i < 64; i += 4)
-    if (c0 + i < a.cols && r0 + tx < a.rows) a.dst[(long long)(c0 + i) * a.dst_ld + r0 + tx] = tile[tx][i];
+#pragma unroll
+  for (int i = 0; i < 64; i += 8) {
+    const int c = c0 + ty + i;
+    if (c >= a.cols || r0 + tx >= a.dst_ld) continue;
+    __nv_bfloat162 v;
+    v.x = tile[tx][ty + i];
+    v.y = tile[tx + 1][ty + i];
+    *reinterpret_cast<__nv_bfloat162*>(a.dst + (long long)c * a.dst_ld + r0 + tx) = v;
+  }
 }
 
 // ------------------------------------------------------------------------------------ one token
@@ -532,7 +544,7 @@ extern "C" int nrt_group_prep(const void* args, void* stream) {
 extern "C" int nrt_transpose(const void* args, void* stream) {
   TransposeArgs a;
   memcpy(&a, args, sizeof(a));
-  if (a.rows < 1 || a.cols < 1 || a.dst_ld < a.rows) return -3;
+  if (a.rows < 1 || a.cols < 1 || a.cols % 2 || a.dst_ld % 2 || a.dst_ld < a.rows) return -3;
   return launch_pdl(transpose_kernel, dim3((a.rows + 63) / 64, (a.cols + 63) / 64), dim3(256), 0, S(stream), false, a);
 }
 
