@@ -66,7 +66,7 @@ struct StackRowArgs {
   const float* probs;           // [rows][top_k]
   int top_k;
   const __nv_bfloat16* post_w;
-  // second half of a sublayer of two mixers side by side (null: none): y becomes half the sum of both, each RMS-normed first
+  // second branch of a sublayer with two mixers (null: none): y becomes the mean of the branches, scaled to unit RMS times join_w / join_w2
   const float* y2;
   const __nv_bfloat16* join_w;
   const __nv_bfloat16* join_w2;
@@ -100,7 +100,7 @@ struct LatentPrepArgs {
 };
 
 // Attention of chunk rows over a block of keys.  Query head h uses key / value head h / group.  With `window` > 0 positions are
-// cut into chunks of that many, counted from position 0, and a query sees only keys of its own chunk.
+// cut into chunks of that many ([0, window), [window, 2 window), ...), and a query sees only keys of its own chunk.
 struct LatentAttnArgs {
   const void* q;                // [rows][heads * dim]
   const void* k;                // keys of the block [kv_rows][heads / group * dim]
@@ -200,9 +200,10 @@ struct GroupDecodeArgs {
 // ------------------------------------------------------------------------------------ matrix-state recurrences
 // Every head carries a matrix S [dim x vdim] (stored per value column: [vdim][dim4], dim4 = dim rounded up to four).
 enum StateKind : int {
-  kStateDelta = 0,     // S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q
-  kStateBonus = 1,     // o = (S + diag(u) k v^T)^T q; S <- g S + k v^T
-  kStateNormalized = 2,// S <- a S + b k v^T, n likewise with k alone, stabilised by a running maximum; o = S^T q, with n . q beside it
+  // With S' = diag(g) S ahead of the update, o = q^T S read out:
+  kStateDelta = 0,     // S' moves towards v at k by the step beta: S = S' + beta k (v - k^T S')^T; read after the update
+  kStateBonus = 1,     // S = S' + k v^T; read before decay and update, plus the token's own term (q . u k) v
+  kStateNormalized = 2,// S = a S + b k v^T with scalar a, b from a running maximum; read after; sums of k weighted alike give the normaliser
 };
 enum GateKind : int { kGateSigmoid = 0, kGateSilu = 1 };
 

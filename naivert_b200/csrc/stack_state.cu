@@ -19,7 +19,7 @@ namespace {
 
 typedef unsigned long long u64;
 constexpr int kLanes = 8;                     // lanes per value column
-constexpr float kUnitEps = 1e-6f;             // unit vectors: x / sqrt(sum(x^2) + 1e-6)
+constexpr float kUnitEps = 1e-6f;             // added to the squared length of what becomes a unit vector
 
 __device__ __forceinline__ u64 pack2(float x, float y) {
   u64 v;

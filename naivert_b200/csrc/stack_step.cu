@@ -133,7 +133,7 @@ __device__ __forceinline__ void load_input(const StepArgs& a, int g, int k8, flo
       } else {
         if (a.y) {
           if (a.y2) {
-            // two sublayers side by side: half the sum of both, each divided by its root mean square
+            // two branches: the mean of both, scaled to unit RMS
             float s1 = 0.f, s2 = 0.f;
             each([&](int e, float4& t) { t = ldcg4(a.y + e); s1 += dot4(t); s2 += dot4(ldcg4(a.y2 + e)); });
             const float r1 = 0.5f / sqrtf(block_sum_f(s1, red) / (float)K + a.eps), r2 = 0.5f / sqrtf(block_sum_f(s2, red) / (float)K + a.eps);

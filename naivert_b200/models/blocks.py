@@ -71,7 +71,7 @@ class RotarySpec:
 @dataclass(frozen=True)
 class GroupedAttentionSpec:
     """Softmax attention with shared key / value heads, norms per head, rotary positions and biases; with ``window`` > 0
-    positions fall into chunks of that many (counted from 0) and a query sees its own chunk only."""
+    positions fall into chunks [0, window), [window, 2 window), ... and a query sees its own chunk only."""
 
     heads: int
     kv_heads: int
@@ -150,7 +150,7 @@ class NormalizedStateSpec:
 
 @dataclass(frozen=True)
 class ParallelSpec:
-    """Two mixers that read the same input; the sublayer is half the sum of their outputs, each RMS-normed."""
+    """Two mixers over one input; the sublayer is the mean of the two branches after an RMS norm each."""
 
     left: GroupedAttentionSpec
     right: NormalizedStateSpec

@@ -2,8 +2,8 @@
 
 A decoder of freely ordered layers whose sublayers read the stream itself and are layer-normed on their output: a gated
 delta rule with a decay per key channel, RWKV-style time mixing, or chunked grouped-query attention beside an xLSTM matrix
-memory, each followed by a squared-ReLU feed-forward or nothing.  A layer may use another layer's tensors with a cache or
-state of its own.  Embedding and head are separate tables.
+memory, each followed by a squared-ReLU feed-forward or nothing.  Layers may share tensors, never the memory of a
+sequence.  Embedding and head are separate tables.
 
 The widths of the low-rank products stand in no configuration key; they are the row counts of their first matrices, so
 ``spec_from_config`` takes the checkpoint's tensor shapes beside ``config.json``.
