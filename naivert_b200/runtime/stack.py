@@ -21,7 +21,7 @@ import torch
 from ..models.blocks import StackSpec
 from ..ops import kernels as K
 from ..ops import stack_kernels as S
-from .packing import Packed, pack, vector
+from .packing import pack, vector
 from .stack_mixers import MIXERS, StepBuilder
 
 

@@ -18,7 +18,6 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..ops import kernels as K
 from ..ops import stack_kernels as S
 from .packing import Packed, head_columns, head_rows, pack, pad, stacked_rows, vector
 
